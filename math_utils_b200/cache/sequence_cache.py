@@ -14,7 +14,8 @@ Layers are grouped by what their mixer keeps (its ``cache_spec``):
     run), and for each slot the list of pages it holds.  All entries of a group
     share the slot's page list, so a page index means the same positions in
     every layer of the group.  A group with a window gives pages back once no
-    later query can see them.
+    later query can see them; pages with positions that the spec keeps (the first
+    ``keep`` of a sequence) stay.
     A mixer that keeps one row per position for all its heads (``RowCacheSpec``)
     gets the same kind of group with pages of ``[page_tokens, width]``.
   * a ``StateGroup`` for each distinct state size: ``[n_slots, n_values]``
@@ -140,6 +141,8 @@ class KVGroup:
                  else (n_pages, 2, spec.n_kv_heads, page_tokens, spec.head_dim))
         self.storage: Dict[int, torch.Tensor] = {
             e: torch.zeros(shape, dtype=dtype, device=device) for e in self.entries}
+        # pages with a sequence's first positions that later queries keep seeing beside their window
+        self.kept_pages = -(-getattr(spec, "keep", 0) // page_tokens) if spec.window > 0 else 0
         # page number of each page index of each slot; -1 where none is held
         self.table = np.full((n_slots, self.max_pages), -1, dtype=np.int32)
 
@@ -150,11 +153,12 @@ class KVGroup:
         return (length - self.spec.window) // self.page_tokens
 
     def reserve(self, slot: int, old_len: int, new_len: int) -> None:
-        """Pages for positions up to new_len; with a window, drops pages that
-        every query from position old_len on has left behind."""
+        """Pages for positions up to new_len; with a window, none that every query
+        from position old_len on has left behind."""
         row = self.table[slot]
         need_upto = (new_len + self.page_tokens - 1) // self.page_tokens
-        missing = [i for i in range(need_upto) if row[i] < 0 and i >= self.first_needed_page(old_len + 1)]
+        needed_from = self.first_needed_page(old_len + 1)
+        missing = [i for i in range(need_upto) if row[i] < 0 and (i >= needed_from or i < self.kept_pages)]
         if missing:
             pages = self.pool.take(len(missing))
             for i, p in zip(missing, pages):
@@ -165,11 +169,10 @@ class KVGroup:
         if self.spec.window <= 0:
             return
         row = self.table[slot]
-        upto = self.first_needed_page(length + 1)
-        drop = [int(row[i]) for i in range(min(upto, self.max_pages)) if row[i] >= 0]
+        left = range(self.kept_pages, min(self.first_needed_page(length + 1), self.max_pages))
+        drop = [int(row[i]) for i in left if row[i] >= 0]
         if drop:
-            for i in range(min(upto, self.max_pages)):
-                row[i] = -1
+            row[left.start:left.stop] = -1
             self.pool.give_back(drop)
 
     def release(self, slot: int) -> None:

@@ -101,6 +101,42 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
     return r;
 }
 
+// --- two float32 in one 64-bit register: sm_100 multiplies and adds them as one instruction (each rounded as
+// its scalar counterpart would be)
+typedef unsigned long long float2x;
+__device__ __forceinline__ float2x pair_of_floats(float lo, float hi) {
+    float2x r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 floats_of_pair(float2x v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ float2x pair_fma(float2x a, float2x b, float2x c) {
+    float2x r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ float2x pair_mul(float2x a, float2x b) {
+    float2x r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+// Asynchronous copies global -> shared of 4 or 16 bytes, grouped and waited for by the issuing thread.
+__device__ __forceinline__ void copy_async4(float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void copy_async16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+
 // --- programmatic dependent launch -------------------------------------------------------
 // Kernels of the single-token step are launched so that the next one may start while the
 // previous one drains: it runs its prologue (index arithmetic, prefetch of weights, which
@@ -143,6 +179,21 @@ inline void prefer_shared_memory(const void* kernel) {
         cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
         cudaGetLastError();
     }
+}
+
+// A kernel whose dynamic shared memory passes the default limit asks for more, once.
+inline bool allow_shared(const void* kernel, size_t bytes) {
+    static std::mutex mutex;
+    static std::unordered_set<const void*> seen;
+    if (bytes <= 48 * 1024) return true;
+    std::lock_guard<std::mutex> lock(mutex);
+    if (seen.count(kernel)) return true;
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) {
+        cudaGetLastError();
+        return false;
+    }
+    seen.insert(kernel);
+    return true;
 }
 
 template <bool EARLY = true, typename... KArgs, typename... Args>

@@ -19,17 +19,16 @@
 //                    asynchronously, the next 16 while these are worked on.
 //                    The order of every sum is fixed by the column alone: a token's result does not depend on how
 //                    the sequence was cut into steps or on the batch.
+//
+// Option: a decay per head and key channel instead of one per head (the rows of S decay each by its own number).  The
+// decays are then made by mu_low_rank (linear_scan.cu) and staged beside the keys; S decays before the two sums, which
+// are S^T k and S^T q of the decayed state, and the read-out is S^T q + u (k . q): one exchange a token again.
 #include "common.cuh"
 
 #include <math.h>
 #include <stdint.h>
 
-#include <mutex>
-#include <unordered_set>
-
 namespace mu {
-
-__device__ __forceinline__ float dl_softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 
 template <typename TE>
 __global__ void __launch_bounds__(128)
@@ -62,9 +61,10 @@ delta_prepare_kernel(float* __restrict__ qkv, int channels, const TE* __restrict
     }
     for (int h = tid; h < n_heads; h += blockDim.x) {
         const float b = to_float(b_raw[(long long)t * ldb + h]);
-        const float a = to_float(a_raw[(long long)t * lda + h]);
         beta[(long long)t * n_heads + h] = 1.0f / (1.0f + expf(-b));
-        decay[(long long)t * n_heads + h] = expf(-expf(a_log[h]) * dl_softplus(a + dt_bias[h]));
+        if (!a_raw) continue;                                // (decays per channel come from elsewhere)
+        const float a = to_float(a_raw[(long long)t * lda + h]);
+        decay[(long long)t * n_heads + h] = expf(-expf(a_log[h]) * softplus(a + dt_bias[h]));
     }
 }
 
@@ -72,18 +72,11 @@ constexpr int DL_COLS = 16;       // columns a block takes
 constexpr int DL_CHUNK = 16;      // tokens staged at a time
 constexpr int DL_MAX_DK = 256;    // the longest column
 
-// Asynchronous copies global -> shared of 4 or 16 bytes, grouped and waited for by the issuing thread.
-__device__ __forceinline__ void dl_copy4(float* dst, const float* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+// Floats of one staged chunk: keys, queries (and the channels' decays) padded to DKP entries, the block's values,
+// (beta, decay, k . q, -).
+__host__ __device__ constexpr int dl_chunk_floats(int dkp, bool per_channel) {
+    return DL_CHUNK * ((per_channel ? 3 : 2) * dkp + DL_COLS + 4);
 }
-__device__ __forceinline__ void dl_copy16(float* dst, const float* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void dl_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void dl_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-// Floats of one staged chunk: keys and queries padded to DKP entries, the block's values, (beta, decay, k . q, -).
-__host__ __device__ constexpr int dl_chunk_floats(int dkp) { return DL_CHUNK * (2 * dkp + DL_COLS + 4); }
 
 // LANES: lanes that share a column of S; R: entries of the column a lane holds (a multiple of 4); dk <= LANES * R.
 // The column is dealt to the lanes four entries at a time: lane l holds entries 4 (l + LANES i) .. 4 (l + LANES i) + 3,
@@ -91,15 +84,15 @@ __host__ __device__ constexpr int dl_chunk_floats(int dkp) { return DL_CHUNK * (
 // 8 lanes with 16 entries each beat 16 lanes with 8 and one more exchange.)  LANES and R follow from dk alone, so the
 // order of the sums does too.
 // VEC: dk, dv, the row length and the state's offset and stride are all multiples of 4, so keys, queries, values and
-// the state move 16 bytes at a time.
-template <int R, int LANES, bool VEC>
+// the state move 16 bytes at a time.  PER_CHANNEL: `decay` is [T][n_heads * dk] (else [T][n_heads]).
+template <int R, int LANES, bool VEC, bool PER_CHANNEL>
 __global__ void __launch_bounds__(LANES * DL_COLS)
 delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __restrict__ kq,
                   const float* __restrict__ beta, const float* __restrict__ decay, int n_heads, int n_kv_heads, int dk,
                   int dv, const int* __restrict__ seq_first, const int* __restrict__ seq_slots,
                   float* __restrict__ state, long long state_stride, long long state_offset, float* __restrict__ out) {
     constexpr int DL_LANES = LANES, DL_THREADS = LANES * DL_COLS;
-    constexpr int DKP = DL_LANES * R, Q = R / 4, BUF = dl_chunk_floats(DKP);
+    constexpr int DKP = DL_LANES * R, Q = R / 4, BUF = dl_chunk_floats(DKP, PER_CHANNEL);
     extern __shared__ __align__(16) float dl_smem[];
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DL_COLS;
     const int tid = threadIdx.x, c = tid / DL_LANES, l = tid % DL_LANES;
@@ -110,17 +103,21 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
     pdl_wait();
     const int first = seq_first[s], count = seq_first[s + 1] - first;
     float* mine = state + (long long)seq_slots[s] * state_stride + state_offset + ((long long)h * dv + j) * dk;
-    float S[R];
+    float2x S[2 * Q];                                        // the lane's entries in pairs
 #pragma unroll
     for (int i = 0; i < Q; ++i) {
         const int d = 4 * (l + DL_LANES * i);
+        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (VEC) {
-            const float4 x = live && d < dk ? *reinterpret_cast<const float4*>(mine + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-            S[4 * i] = x.x, S[4 * i + 1] = x.y, S[4 * i + 2] = x.z, S[4 * i + 3] = x.w;
-        } else {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) S[4 * i + e] = live && d + e < dk ? mine[d + e] : 0.0f;
+            if (live && d < dk) x = *reinterpret_cast<const float4*>(mine + d);
+        } else if (live) {
+            if (d < dk) x.x = mine[d];
+            if (d + 1 < dk) x.y = mine[d + 1];
+            if (d + 2 < dk) x.z = mine[d + 2];
+            if (d + 3 < dk) x.w = mine[d + 3];
         }
+        S[2 * i] = pair_of_floats(x.x, x.y);
+        S[2 * i + 1] = pair_of_floats(x.z, x.w);
     }
     const long long q_off = (long long)g * dk, k_off = (long long)(n_kv_heads + g) * dk;
     const long long v_off = (long long)2 * n_kv_heads * dk + (long long)h * dv + col0;
@@ -128,7 +125,8 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
     auto stage = [&](int li0, int b) {
         float* ks = dl_smem + b * BUF;
         float* qs = ks + DL_CHUNK * DKP;
-        float* vs = qs + DL_CHUNK * DKP;
+        float* gs = qs + DL_CHUNK * DKP;
+        float* vs = gs + (PER_CHANNEL ? DL_CHUNK * DKP : 0);
         float* sc = vs + DL_CHUNK * DL_COLS;
         const int n = min(DL_CHUNK, count - li0);
         if (VEC) {
@@ -136,34 +134,36 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
             for (int i = tid; i < n * per; i += DL_THREADS) {
                 const int tok = i / per, d = 4 * (i % per);
                 const float* row = qkv + (long long)(first + li0 + tok) * channels;
-                dl_copy16(ks + tok * DKP + d, row + k_off + d);
-                dl_copy16(qs + tok * DKP + d, row + q_off + d);
+                copy_async16(ks + tok * DKP + d, row + k_off + d);
+                copy_async16(qs + tok * DKP + d, row + q_off + d);
+                if (PER_CHANNEL) copy_async16(gs + tok * DKP + d, decay + ((long long)(first + li0 + tok) * n_heads + h) * dk + d);
             }
             for (int i = tid; i < n * (DL_COLS / 4); i += DL_THREADS) {
                 const int tok = i / (DL_COLS / 4), cc = 4 * (i % (DL_COLS / 4));
                 if (col0 + cc < dv)
-                    dl_copy16(vs + tok * DL_COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
+                    copy_async16(vs + tok * DL_COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
             }
         } else {
             for (int i = tid; i < n * dk; i += DL_THREADS) {
                 const int tok = i / dk, d = i % dk;
                 const float* row = qkv + (long long)(first + li0 + tok) * channels;
-                dl_copy4(ks + tok * DKP + d, row + k_off + d);
-                dl_copy4(qs + tok * DKP + d, row + q_off + d);
+                copy_async4(ks + tok * DKP + d, row + k_off + d);
+                copy_async4(qs + tok * DKP + d, row + q_off + d);
+                if (PER_CHANNEL) copy_async4(gs + tok * DKP + d, decay + ((long long)(first + li0 + tok) * n_heads + h) * dk + d);
             }
             for (int i = tid; i < n * DL_COLS; i += DL_THREADS) {
                 const int tok = i / DL_COLS, cc = i % DL_COLS;
                 if (col0 + cc < dv)
-                    dl_copy4(vs + tok * DL_COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
+                    copy_async4(vs + tok * DL_COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
             }
         }
         for (int tok = tid; tok < n; tok += DL_THREADS) {
             const long long t = first + li0 + tok;
-            dl_copy4(sc + tok * 4 + 0, beta + t * n_heads + h);
-            dl_copy4(sc + tok * 4 + 1, decay + t * n_heads + h);
-            dl_copy4(sc + tok * 4 + 2, kq + t * n_kv_heads + g);
+            copy_async4(sc + tok * 4 + 0, beta + t * n_heads + h);
+            if (!PER_CHANNEL) copy_async4(sc + tok * 4 + 1, decay + t * n_heads + h);
+            copy_async4(sc + tok * 4 + 2, kq + t * n_kv_heads + g);
         }
-        dl_commit();
+        copy_async_commit();
     };
     __syncthreads();                                         // the zeros are down before the first copies land
     if (count > 0) stage(0, 0);
@@ -172,41 +172,47 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
         const int n = min(DL_CHUNK, count - li0);
         if (li0 + DL_CHUNK < count) {
             stage(li0 + DL_CHUNK, b ^ 1);                    // the next chunk is on its way while this one is worked on
-            dl_wait<1>();
+            copy_async_wait<1>();
         } else {
-            dl_wait<0>();
+            copy_async_wait<0>();
         }
         __syncthreads();
         const float* ks = dl_smem + b * BUF;
         const float* qs = ks + DL_CHUNK * DKP;
-        const float* vs = qs + DL_CHUNK * DKP;
+        const float* gs = qs + DL_CHUNK * DKP;
+        const float* vs = gs + (PER_CHANNEL ? DL_CHUNK * DKP : 0);
         const float* sc = vs + DL_CHUNK * DL_COLS;
-        // A token's keys, queries, value and scalars are read into registers while the token before it is still
-        // waiting for its sums to come round the lanes.
-        float4 kr[Q], qr[Q];
+        // A token's keys, queries, decays, value and scalars are read into registers while the token before it is
+        // still waiting for its sums to come round the lanes.
+        ulonglong2 kr[Q], qr[Q], gr[PER_CHANNEL ? Q : 1];
         float4 par = *reinterpret_cast<const float4*>(sc);                           // beta, decay, k . q
         float v = vs[c];
 #pragma unroll
         for (int i = 0; i < Q; ++i) {
-            kr[i] = *reinterpret_cast<const float4*>(ks + 4 * (l + DL_LANES * i));
-            qr[i] = *reinterpret_cast<const float4*>(qs + 4 * (l + DL_LANES * i));
+            kr[i] = *reinterpret_cast<const ulonglong2*>(ks + 4 * (l + DL_LANES * i));
+            qr[i] = *reinterpret_cast<const ulonglong2*>(qs + 4 * (l + DL_LANES * i));
+            if (PER_CHANNEL) gr[i] = *reinterpret_cast<const ulonglong2*>(gs + 4 * (l + DL_LANES * i));
         }
         for (int tok = 0; tok < n; ++tok) {
-            float d1[4] = {0.0f, 0.0f, 0.0f, 0.0f}, d2[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            float2x k1 = 0, k2 = 0, q1 = 0, q2 = 0;                                  // (two zeros each)
 #pragma unroll
             for (int i = 0; i < Q; ++i) {
-                d1[0] = fmaf(S[4 * i], kr[i].x, d1[0]), d2[0] = fmaf(S[4 * i], qr[i].x, d2[0]);
-                d1[1] = fmaf(S[4 * i + 1], kr[i].y, d1[1]), d2[1] = fmaf(S[4 * i + 1], qr[i].y, d2[1]);
-                d1[2] = fmaf(S[4 * i + 2], kr[i].z, d1[2]), d2[2] = fmaf(S[4 * i + 2], qr[i].z, d2[2]);
-                d1[3] = fmaf(S[4 * i + 3], kr[i].w, d1[3]), d2[3] = fmaf(S[4 * i + 3], qr[i].w, d2[3]);
+                if (PER_CHANNEL) {
+                    S[2 * i] = pair_mul(gr[i].x, S[2 * i]);
+                    S[2 * i + 1] = pair_mul(gr[i].y, S[2 * i + 1]);
+                }
+                k1 = pair_fma(S[2 * i], kr[i].x, k1), q1 = pair_fma(S[2 * i], qr[i].x, q1);
+                k2 = pair_fma(S[2 * i + 1], kr[i].y, k2), q2 = pair_fma(S[2 * i + 1], qr[i].y, q2);
             }
-            float sk = (d1[0] + d1[1]) + (d1[2] + d1[3]), sq = (d2[0] + d2[1]) + (d2[2] + d2[3]);
+            const float2 ka = floats_of_pair(k1), kb = floats_of_pair(k2), qa = floats_of_pair(q1), qb = floats_of_pair(q2);
+            float sk = (ka.x + ka.y) + (kb.x + kb.y), sq = (qa.x + qa.y) + (qb.x + qb.y);
             const int nxt = min(tok + 1, DL_CHUNK - 1);                              // the last one reads itself again
-            float4 nk[Q];
+            ulonglong2 nk[Q];
 #pragma unroll
             for (int i = 0; i < Q; ++i) {
-                nk[i] = *reinterpret_cast<const float4*>(ks + nxt * DKP + 4 * (l + DL_LANES * i));
-                qr[i] = *reinterpret_cast<const float4*>(qs + nxt * DKP + 4 * (l + DL_LANES * i));
+                nk[i] = *reinterpret_cast<const ulonglong2*>(ks + nxt * DKP + 4 * (l + DL_LANES * i));
+                qr[i] = *reinterpret_cast<const ulonglong2*>(qs + nxt * DKP + 4 * (l + DL_LANES * i));
+                if (PER_CHANNEL) gr[i] = *reinterpret_cast<const ulonglong2*>(gs + nxt * DKP + 4 * (l + DL_LANES * i));
             }
             const float4 npar = *reinterpret_cast<const float4*>(sc + nxt * 4);
             const float nv = vs[nxt * DL_COLS + c];
@@ -215,18 +221,18 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
                 sk += __shfl_xor_sync(0xffffffffu, sk, o);
                 sq += __shfl_xor_sync(0xffffffffu, sq, o);
             }
-            // the sums are of the state before its decay: (decay S)^T k = decay (S^T k)
-            const float u = par.x * (v - par.y * sk);
+            // (one decay for the head: the sums are of the state before it, (decay S)^T k = decay (S^T k))
+            const float u = par.x * (v - (PER_CHANNEL ? sk : par.y * sk));
+            const float2x u2 = pair_of_floats(u, u), dec2 = pair_of_floats(par.y, par.y);
 #pragma unroll
             for (int i = 0; i < Q; ++i) {
-                S[4 * i] = fmaf(kr[i].x, u, par.y * S[4 * i]);
-                S[4 * i + 1] = fmaf(kr[i].y, u, par.y * S[4 * i + 1]);
-                S[4 * i + 2] = fmaf(kr[i].z, u, par.y * S[4 * i + 2]);
-                S[4 * i + 3] = fmaf(kr[i].w, u, par.y * S[4 * i + 3]);
+                S[2 * i] = pair_fma(kr[i].x, u2, PER_CHANNEL ? S[2 * i] : pair_mul(dec2, S[2 * i]));
+                S[2 * i + 1] = pair_fma(kr[i].y, u2, PER_CHANNEL ? S[2 * i + 1] : pair_mul(dec2, S[2 * i + 1]));
                 kr[i] = nk[i];
             }
             if (l == 0 && live)
-                out[(long long)(first + li0 + tok) * n_heads * dv + (long long)h * dv + j] = fmaf(u, par.z, par.y * sq);
+                out[(long long)(first + li0 + tok) * n_heads * dv + (long long)h * dv + j] =
+                    fmaf(u, par.z, PER_CHANNEL ? sq : par.y * sq);
             par = npar;
             v = nv;
         }
@@ -238,42 +244,30 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
 #pragma unroll
     for (int i = 0; i < Q; ++i) {
         const int d = 4 * (l + DL_LANES * i);
+        const float2 lo = floats_of_pair(S[2 * i]), hi = floats_of_pair(S[2 * i + 1]);
+        if (!live) continue;
         if (VEC) {
-            if (live && d < dk)
-                *reinterpret_cast<float4*>(mine + d) = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
+            if (d < dk) *reinterpret_cast<float4*>(mine + d) = make_float4(lo.x, lo.y, hi.x, hi.y);
         } else {
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-                if (live && d + e < dk) mine[d + e] = S[4 * i + e];
+            if (d < dk) mine[d] = lo.x;
+            if (d + 1 < dk) mine[d + 1] = lo.y;
+            if (d + 2 < dk) mine[d + 2] = hi.x;
+            if (d + 3 < dk) mine[d + 3] = hi.y;
         }
     }
-}
-
-// A kernel whose two buffers pass the default limit of dynamic shared memory asks for more, once.
-inline bool dl_allow_shared(const void* kernel, size_t bytes) {
-    static std::mutex mutex;
-    static std::unordered_set<const void*> seen;
-    if (bytes <= 48 * 1024) return true;
-    std::lock_guard<std::mutex> lock(mutex);
-    if (seen.count(kernel)) return true;
-    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) {
-        cudaGetLastError();
-        return false;
-    }
-    seen.insert(kernel);
-    return true;
 }
 
 }  // namespace mu
 
 // qkv: the convolution's float32 output rows [T][channels], channels = 2 * kv_heads * dk + heads * dv; q and k are
-// finished in place.  b_raw, a_raw: [T][heads] views of the projection in the compute dtype.
+// finished in place.  b_raw, a_raw: [T][heads] views of the projection, both bfloat16 or both float32; a_raw null: no
+// decay per head is made (a_log, dt_bias and decay are not touched).
 MU_EXPORT int mu_delta_prepare(float* qkv, int channels, const void* b_raw, long long ldb, const void* a_raw,
                                long long lda, const float* a_log, const float* dt_bias, int n_tokens, int n_heads,
                                int n_kv_heads, int dk, float q_scale, float* kq, float* beta, float* decay,
                                int is_bf16, void* stream) {
     if (n_tokens <= 0) return MU_OK;
-    if (!qkv || !b_raw || !a_raw || !a_log || !dt_bias || !kq || !beta || !decay || n_heads <= 0 || n_kv_heads <= 0 ||
+    if (!qkv || !b_raw || (a_raw && (!a_log || !dt_bias || !decay)) || !kq || !beta || n_heads <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || dk <= 0 || channels < 2 * n_kv_heads * dk)
         return MU_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
@@ -292,7 +286,7 @@ MU_EXPORT int mu_delta_scan_max_dk() { return mu::DL_MAX_DK; }
 MU_EXPORT int mu_delta_scan(const float* qkv, int channels, const float* kq, const float* beta, const float* decay,
                             int n_seqs, int n_heads, int n_kv_heads, int dk, int dv, const int* seq_first,
                             const int* seq_slots, float* state, long long state_stride, long long state_offset,
-                            float* out, int long_steps, void* stream) {
+                            float* out, int long_steps, void* stream, int per_channel) {
     if (n_seqs <= 0) return MU_OK;
     if (!qkv || !kq || !beta || !decay || !seq_first || !seq_slots || !state || !out || n_heads <= 0 ||
         n_kv_heads <= 0 || n_heads % n_kv_heads || dk <= 0 || dv <= 0 ||
@@ -302,29 +296,31 @@ MU_EXPORT int mu_delta_scan(const float* qkv, int channels, const float* kq, con
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid(n_seqs, n_heads, (dv + mu::DL_COLS - 1) / mu::DL_COLS);
     const bool vec = dk % 4 == 0 && dv % 4 == 0 && channels % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0 &&
-                     (reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(state)) % 16 == 0;
+                     (reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(state) |
+                      (per_channel ? reinterpret_cast<uintptr_t>(decay) : 0)) % 16 == 0;
     // long_steps: many tokens a sequence (a prompt step).  The blocks then run for a long time with one warp a
     // scheduler; they start in plain stream order, on an empty device.
     // the two staging buffers of a block are most of what it needs of an SM: with the largest share of the on-chip
     // memory as shared memory several blocks fit, and the state is read once, so the L1 is no loss
-#define MU_DELTA_SCAN_V(R, LANES, V)                                                                                  \
+#define MU_DELTA_SCAN_V(R, LANES, V, PC)                                                                              \
     do {                                                                                                              \
-        const size_t smem = 2 * sizeof(float) * mu::dl_chunk_floats(LANES * R);                                       \
-        const void* kernel = (const void*)mu::delta_scan_kernel<R, LANES, V>;                                         \
-        if (!mu::dl_allow_shared(kernel, smem)) return MU_ERR_LAUNCH;                                                 \
-        mu::prefer_shared_memory(kernel);                                                                             \
+        const size_t smem = 2 * sizeof(float) * mu::dl_chunk_floats(LANES * R, PC);                                   \
+        auto kernel = mu::delta_scan_kernel<R, LANES, V, PC>;                                                         \
+        if (!mu::allow_shared((const void*)kernel, smem)) return MU_ERR_LAUNCH;                                       \
+        mu::prefer_shared_memory((const void*)kernel);                                                                \
+        const dim3 block(LANES * mu::DL_COLS);                                                                        \
         if (long_steps)                                                                                               \
-            return mu::launch_after(mu::delta_scan_kernel<R, LANES, V>, grid, dim3(LANES * mu::DL_COLS), smem, s, qkv, \
-                                    channels, kq, beta, decay, n_heads, n_kv_heads, dk, dv, seq_first, seq_slots,     \
-                                    state, state_stride, state_offset, out);                                          \
-        return mu::launch_pdl(mu::delta_scan_kernel<R, LANES, V>, grid, dim3(LANES * mu::DL_COLS), smem, s, 1, qkv,   \
-                              channels, kq, beta, decay, n_heads, n_kv_heads, dk, dv, seq_first, seq_slots, state,    \
-                              state_stride, state_offset, out);                                                       \
+            return mu::launch_after(kernel, grid, block, smem, s, qkv, channels, kq, beta, decay, n_heads,            \
+                                    n_kv_heads, dk, dv, seq_first, seq_slots, state, state_stride, state_offset, out); \
+        return mu::launch_pdl(kernel, grid, block, smem, s, 1, qkv, channels, kq, beta, decay, n_heads, n_kv_heads,   \
+                              dk, dv, seq_first, seq_slots, state, state_stride, state_offset, out);                  \
     } while (0)
 #define MU_DELTA_SCAN(R, LANES)                                                                                       \
     do {                                                                                                              \
-        if (vec) MU_DELTA_SCAN_V(R, LANES, true);                                                                     \
-        MU_DELTA_SCAN_V(R, LANES, false);                                                                             \
+        if (vec && per_channel) MU_DELTA_SCAN_V(R, LANES, true, true);                                                \
+        if (per_channel) MU_DELTA_SCAN_V(R, LANES, false, true);                                                      \
+        if (vec) MU_DELTA_SCAN_V(R, LANES, true, false);                                                              \
+        MU_DELTA_SCAN_V(R, LANES, false, false);                                                                      \
     } while (0)
     if (dk <= 32) MU_DELTA_SCAN(4, 8);
     if (dk <= 64) MU_DELTA_SCAN(8, 8);

@@ -2,6 +2,9 @@
 //
 // embed:     x[t, :] = table[id[t], :] * scale + (pos_table ? pos_table[pos[t], :] : 0)
 //            -> float32 residual stream (include/ai/LocalModel.hpp:3686-3697).
+//            With `turns` sinusoids are added: entry 2i gets sin and entry 2i + 1 cos of 2 pi pos turns[i], a
+//            frequency in turns per position given as two floats (rounded, and what the rounding left), so that the
+//            fraction of a turn is right to float32 at every position.
 // layernorm: y = (x - mean) * rsqrt(var + eps) * gamma + beta, biased variance,
 //            two passes over the row, all in float32
 //            (include/ai/LocalModel.hpp:1355-1367); output in the compute dtype.
@@ -12,7 +15,7 @@ namespace mu {
 template <typename TW>
 __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict__ pos,
                              const TW* __restrict__ table, const TW* __restrict__ pos_table,
-                             float* __restrict__ x, int hidden, float scale) {
+                             float* __restrict__ x, int hidden, float scale, const float* __restrict__ turns) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -24,6 +27,13 @@ __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict_
     for (int d = threadIdx.x; d < hidden; d += blockDim.x) {
         float v = to_float(src[d]) * scale;
         if (psrc) v += to_float(psrc[d]);
+        if (turns) {
+            const int i = d >> 1;
+            const float p = (float)pos[t], whole = p * turns[i];
+            const float rest = fmaf(p, turns[i], -whole) + p * turns[(hidden + 1) / 2 + i];
+            const float fraction = (whole - rintf(whole)) + rest;
+            v += (d & 1) ? cospif(2.0f * fraction) : sinpif(2.0f * fraction);
+        }
         dst[d] = v;
     }
 }
@@ -190,16 +200,17 @@ layernorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows,
 
 // table_bf16: 1 if the tables hold bfloat16, 0 for float32.
 MU_EXPORT int mu_embed(const int* ids, const int* pos, const void* table, const void* pos_table,
-                       float* x, int n_tokens, int hidden, int table_bf16, float scale, void* stream) {
+                       float* x, int n_tokens, int hidden, int table_bf16, float scale, void* stream,
+                       const float* turns) {
     if (n_tokens <= 0) return MU_OK;
-    if (hidden <= 0 || !ids || !table || !x || (pos_table && !pos)) return MU_ERR_BAD_ARGUMENT;
+    if (hidden <= 0 || !ids || !table || !x || ((pos_table || turns) && !pos)) return MU_ERR_BAD_ARGUMENT;
     const int threads = hidden >= 256 ? 256 : 128;
     cudaStream_t s = (cudaStream_t)stream;
     if (table_bf16)
         return mu::launch_pdl(mu::embed_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, s, 1, ids, pos,
-                              (const __nv_bfloat16*)table, (const __nv_bfloat16*)pos_table, x, hidden, scale);
+                              (const __nv_bfloat16*)table, (const __nv_bfloat16*)pos_table, x, hidden, scale, turns);
     return mu::launch_pdl(mu::embed_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, 1, ids, pos,
-                          (const float*)table, (const float*)pos_table, x, hidden, scale);
+                          (const float*)table, (const float*)pos_table, x, hidden, scale, turns);
 }
 
 // Token rows plus hashed rows of (token before, token); single_tokens: every sequence brings one token.

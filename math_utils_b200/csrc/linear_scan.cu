@@ -1,0 +1,448 @@
+// Recurrent mixers with a matrix state S [dk][dv] per head that is written without being read first:
+//     S <- decay S + take k v^T,   o = scale * S^T q,
+// and the gates they take.  Everything float32.
+//
+// mu_linear_scan   per (sequence, head, 16 columns of S), the step's tokens in order.  The decay is one number per
+//                  head (with a `take` beside it) or one per head and key channel (gated linear attention).  With a
+//                  normalizer the state has one more column, n <- decay n + take k, whose read-out n . q goes to an
+//                  array of its own (the matrix memory of xLSTM).  State of a slot, from state_offset on:
+//                  [ S: heads x dv x dk (a head's S column after column) | n: heads x dk ].
+//                  A column lives in the registers of 8 lanes, two entries to a 64-bit register.  Nothing waits for
+//                  a token's read-out, so the lanes keep their partial sums of 8 tokens and add them crosswise: 7
+//                  exchanges for 8 tokens, after which lane i holds token i's sum.  Keys, queries, decays and values
+//                  of 16 tokens at a time are copied to shared memory asynchronously, the next 16 on their way
+//                  meanwhile.  The order of every sum is fixed by dk alone: a token's result does not depend on how
+//                  the sequence was cut into steps or on the batch.
+// mu_exp_gates     the exponential gates of such a memory: i = cap tanh((i_raw + i_bias) / cap),
+//                  f = log sigmoid(cap tanh((f_raw + f_bias) / cap)), a running maximum m <- max(f + m, i) that starts
+//                  at zero and stays with the sequence's state; per token and head (decay, take, floor) =
+//                  (exp(f + m_before - m), exp(i - m), exp(-m)).  m enters S, n and the floor alike, so which
+//                  maximum is kept changes no result; it is found for 256 tokens at a time by a scan.
+// mu_low_rank      out[t][c] = fn( sum_r W[c][r] low[t][r] + bias[c] ): the second of a projection's two matrices, for
+//                  one or two such projections in one launch, with what follows it:
+//                  fn 0: nothing;  1: sigmoid(z)^power;  2: exp(-exp(A_log[c / per_head]) softplus(z)).
+#include "common.cuh"
+
+#include <math.h>
+
+namespace mu {
+
+constexpr int LS_COLS = 16;       // columns a block takes
+constexpr int LS_LANES = 8;       // lanes a column
+constexpr int LS_CHUNK = 16;      // tokens staged at a time
+constexpr int LS_GROUP = 8;       // tokens whose read-outs are summed together (= LS_LANES)
+constexpr int LS_MAX_DK = 256;
+
+// Floats of one staged chunk: keys, queries (and the channels' decays), values, (decay, take, floor, -).
+__host__ __device__ constexpr int ls_chunk_floats(int dkp, bool per_channel) {
+    return LS_CHUNK * ((per_channel ? 3 : 2) * dkp + LS_COLS + 4);
+}
+
+// One token of a lane's R entries: S = g S + k v, and the lane's share of S . q.
+template <int R, bool PER_CHANNEL>
+__device__ __forceinline__ float ls_step(float2x (&S)[R / 2], const float* __restrict__ k, const float* __restrict__ q,
+                                         const float* __restrict__ g, float decay, float v, int l) {
+    const float2x v2 = pair_of_floats(v, v), d2 = pair_of_floats(decay, decay);
+    float2x a = 0, b = 0;                                    // (two zeros each)
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const int at = 4 * (l + LS_LANES * i);
+        const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(k + at);
+        const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(q + at);
+        ulonglong2 gg = make_ulonglong2(d2, d2);
+        if (PER_CHANNEL) gg = *reinterpret_cast<const ulonglong2*>(g + at);
+        S[2 * i] = pair_fma(kk.x, v2, pair_mul(gg.x, S[2 * i]));
+        S[2 * i + 1] = pair_fma(kk.y, v2, pair_mul(gg.y, S[2 * i + 1]));
+        a = pair_fma(S[2 * i], qq.x, a);
+        b = pair_fma(S[2 * i + 1], qq.y, b);
+    }
+    const float2 x = floats_of_pair(a), y = floats_of_pair(b);
+    return (x.x + x.y) + (y.x + y.y);
+}
+
+// R: entries of a column that a lane holds (a multiple of 4); dk <= 8 R, dealt to the lanes four entries at a time.
+// VEC: every row, slice and state column starts on a 16-byte boundary.
+template <int R, bool VEC, bool PER_CHANNEL>
+__global__ void __launch_bounds__(LS_LANES * LS_COLS)
+linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, long long ld,
+                   const float* __restrict__ decay, int n_heads, int dk, int dv, float scale,
+                   const int* __restrict__ seq_first, const int* __restrict__ seq_slots, float* __restrict__ state,
+                   long long state_stride, long long state_offset, float* __restrict__ out, long long ldo,
+                   float* __restrict__ norm_out) {
+    constexpr int DKP = LS_LANES * R, Q = R / 4, BUF = ls_chunk_floats(DKP, PER_CHANNEL), THREADS = LS_LANES * LS_COLS;
+    extern __shared__ __align__(16) float ls_smem[];
+    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * LS_COLS;
+    const int tid = threadIdx.x, c = tid / LS_LANES, l = tid % LS_LANES;
+    const int j = col0 + c;
+    const bool is_norm = norm_out != nullptr && j == dv;     // the normalizer: a column whose value is always one
+    const bool live = j < dv || is_norm;
+    for (int i = tid; i < 2 * BUF; i += THREADS) ls_smem[i] = 0.0f;      // the padding past dk and dv stays zero
+    pdl_wait();
+    const int first = seq_first[s], count = seq_first[s + 1] - first;
+    float* mine = state + (long long)seq_slots[s] * state_stride + state_offset +
+                  (is_norm ? ((long long)n_heads * dv + h) * dk : ((long long)h * dv + j) * dk);
+    float2x S[2 * Q];
+#pragma unroll
+    for (int i = 0; i < Q; ++i) {
+        const int d = 4 * (l + LS_LANES * i);
+        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (VEC) {
+            if (live && d < dk) x = *reinterpret_cast<const float4*>(mine + d);
+        } else if (live) {
+            if (d < dk) x.x = mine[d];
+            if (d + 1 < dk) x.y = mine[d + 1];
+            if (d + 2 < dk) x.z = mine[d + 2];
+            if (d + 3 < dk) x.w = mine[d + 3];
+        }
+        S[2 * i] = pair_of_floats(x.x, x.y);
+        S[2 * i + 1] = pair_of_floats(x.z, x.w);
+    }
+    // stages the chunk that starts at the sequence's li0-th token of this step into buffer `b`
+    auto stage = [&](int li0, int b) {
+        float* ks = ls_smem + b * BUF;
+        float* qs = ks + LS_CHUNK * DKP;
+        float* gs = qs + LS_CHUNK * DKP;
+        float* vs = gs + (PER_CHANNEL ? LS_CHUNK * DKP : 0);
+        float* sc = vs + LS_CHUNK * LS_COLS;
+        const int n = min(LS_CHUNK, count - li0);
+        const long long t0 = first + li0;
+        if (VEC) {
+            const int per = dk / 4;
+            for (int i = tid; i < n * per; i += THREADS) {
+                const int tok = i / per, d = 4 * (i % per);
+                const long long at = (t0 + tok) * ld + (long long)h * dk + d;
+                copy_async16(ks + tok * DKP + d, k + at);
+                copy_async16(qs + tok * DKP + d, q + at);
+                if (PER_CHANNEL) copy_async16(gs + tok * DKP + d, decay + ((t0 + tok) * n_heads + h) * dk + d);
+            }
+            for (int i = tid; i < n * (LS_COLS / 4); i += THREADS) {
+                const int tok = i / (LS_COLS / 4), cc = 4 * (i % (LS_COLS / 4));
+                if (col0 + cc < dv) copy_async16(vs + tok * LS_COLS + cc, v + (t0 + tok) * ld + (long long)h * dv + col0 + cc);
+            }
+        } else {
+            for (int i = tid; i < n * dk; i += THREADS) {
+                const int tok = i / dk, d = i % dk;
+                const long long at = (t0 + tok) * ld + (long long)h * dk + d;
+                copy_async4(ks + tok * DKP + d, k + at);
+                copy_async4(qs + tok * DKP + d, q + at);
+                if (PER_CHANNEL) copy_async4(gs + tok * DKP + d, decay + ((t0 + tok) * n_heads + h) * dk + d);
+            }
+            for (int i = tid; i < n * LS_COLS; i += THREADS) {
+                const int tok = i / LS_COLS, cc = i % LS_COLS;
+                if (col0 + cc < dv) copy_async4(vs + tok * LS_COLS + cc, v + (t0 + tok) * ld + (long long)h * dv + col0 + cc);
+            }
+        }
+        if (!PER_CHANNEL)
+            for (int tok = tid; tok < n; tok += THREADS) copy_async16(sc + tok * 4, decay + 4 * ((t0 + tok) * n_heads + h));
+        copy_async_commit();
+    };
+    __syncthreads();                                         // the zeros are down before the first copies land
+    if (count > 0) stage(0, 0);
+    int b = 0;
+    for (int li0 = 0; li0 < count; li0 += LS_CHUNK, b ^= 1) {
+        const int n = min(LS_CHUNK, count - li0);
+        if (li0 + LS_CHUNK < count) {
+            stage(li0 + LS_CHUNK, b ^ 1);
+            copy_async_wait<1>();
+        } else {
+            copy_async_wait<0>();
+        }
+        __syncthreads();
+        const float* ks = ls_smem + b * BUF;
+        const float* qs = ks + LS_CHUNK * DKP;
+        const float* gs = qs + LS_CHUNK * DKP;
+        const float* vs = gs + (PER_CHANNEL ? LS_CHUNK * DKP : 0);
+        const float* sc = vs + LS_CHUNK * LS_COLS;
+        auto step = [&](int tok) {
+            float value = is_norm ? 1.0f : vs[tok * LS_COLS + c], fade = 1.0f;
+            if (!PER_CHANNEL) {
+                const float2 gate = *reinterpret_cast<const float2*>(sc + tok * 4);      // decay, take
+                fade = gate.x;
+                value *= gate.y;
+            }
+            return ls_step<R, PER_CHANNEL>(S, ks + tok * DKP, qs + tok * DKP, gs + tok * DKP, fade, value, l);
+        };
+        for (int t0 = 0; t0 < n; t0 += LS_GROUP) {
+            float acc[LS_GROUP];
+            const int left = n - t0;
+            if (left >= LS_GROUP) {                          // a whole group: no branch between the tokens
+#pragma unroll
+                for (int i = 0; i < LS_GROUP; ++i) acc[i] = step(t0 + i);
+            } else {
+#pragma unroll
+                for (int i = 0; i < LS_GROUP; ++i) {
+                    acc[i] = 0.0f;
+                    if (i < left) acc[i] = step(t0 + i);
+                }
+            }
+#pragma unroll
+            for (int width = LS_GROUP / 2; width >= 1; width >>= 1) {
+#pragma unroll
+                for (int i = 0; i < width; ++i) {
+                    const bool upper = (l & width) != 0;
+                    const float send = upper ? acc[i] : acc[i + width];
+                    const float keep = upper ? acc[i + width] : acc[i];
+                    acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, width);
+                }
+            }
+            if (l < left && live) {
+                const long long t = first + li0 + t0 + l;
+                if (is_norm) norm_out[t * n_heads + h] = scale * acc[0];
+                else out[t * ldo + (long long)h * dv + j] = scale * acc[0];
+            }
+        }
+        __syncthreads();                                     // this buffer is free for the chunk after the next
+    }
+    pdl_trigger();                                           // (only now: see the delta scan)
+#pragma unroll
+    for (int i = 0; i < Q; ++i) {
+        const int d = 4 * (l + LS_LANES * i);
+        const float2 lo = floats_of_pair(S[2 * i]), hi = floats_of_pair(S[2 * i + 1]);
+        if (!live) continue;
+        if (VEC) {
+            if (d < dk) *reinterpret_cast<float4*>(mine + d) = make_float4(lo.x, lo.y, hi.x, hi.y);
+        } else {
+            if (d < dk) mine[d] = lo.x;
+            if (d + 1 < dk) mine[d + 1] = lo.y;
+            if (d + 2 < dk) mine[d + 2] = hi.x;
+            if (d + 3 < dk) mine[d + 3] = hi.y;
+        }
+    }
+}
+
+// One block per (sequence, head); a thread a token of the chunk.  What a run of tokens does to m is a pair (F, M):
+// m -> max(F + m, M); two runs in a row are (F1 + F2, max(M1 + F2, M2)).
+__global__ void __launch_bounds__(256)
+exp_gates_kernel(const float* __restrict__ i_raw, const float* __restrict__ f_raw, long long ld,
+                 const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap, int n_heads,
+                 const int* __restrict__ seq_first, const int* __restrict__ seq_slots, float* __restrict__ state,
+                 long long state_stride, long long m_offset, float4* __restrict__ gates) {
+    __shared__ float run_f[8], run_m[8], last_m[8];
+    pdl_trigger();
+    pdl_wait();
+    const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+    const int first = seq_first[s], count = seq_first[s + 1] - first;
+    if (count <= 0) return;
+    float* kept = state + (long long)seq_slots[s] * state_stride + m_offset + h;
+    float carry = *kept;
+    const float ib = i_bias[h], fb = f_bias[h];
+    for (int li0 = 0; li0 < count; li0 += blockDim.x) {
+        const bool in = li0 + tid < count;
+        const long long t = first + li0 + tid;
+        float i = -INFINITY, f = 0.0f;                       // a token that is not there leaves m as it is
+        if (in) {
+            i = cap * tanhf((i_raw[t * ld + h] + ib) / cap);
+            f = -softplus(-cap * tanhf((f_raw[t * ld + h] + fb) / cap));
+        }
+        float F = f, M = i;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float pf = __shfl_up_sync(0xffffffffu, F, o), pm = __shfl_up_sync(0xffffffffu, M, o);
+            if (lane >= o) {
+                M = fmaxf(pm + F, M);
+                F += pf;
+            }
+        }
+        if (lane == 31) {
+            run_f[warp] = F;
+            run_m[warp] = M;
+        }
+        __syncthreads();
+        float before = carry;                                // m as this warp's first token finds it
+        for (int w = 0; w < warp; ++w) before = fmaxf(run_f[w] + before, run_m[w]);
+        const float m = fmaxf(F + before, M);
+        float prev = __shfl_up_sync(0xffffffffu, m, 1);
+        if (lane == 0) prev = before;
+        if (in) gates[t * n_heads + h] = make_float4(expf(f + prev - m), expf(i - m), expf(-m), 0.0f);
+        if (lane == 31) last_m[warp] = m;
+        __syncthreads();
+        carry = last_m[warps - 1];
+    }
+    if (tid == 0) *kept = carry;
+}
+
+constexpr int LR_CHANNELS = 128, LR_THREADS = 64;            // a thread takes two channels
+struct LowRankPart {
+    const void* w;            // [n][ldw], the first `rank` entries of a row
+    const float* bias;        // [n] or null
+    const float* a_log;       // fn 2: one per `per_head` channels
+    float* out;               // [T][n]
+    long long ldw;
+    int col, rank, n, fn, per_head;
+    float power;
+};
+
+template <int N, typename T> __device__ __forceinline__ void load_weights(float (&x)[N], const T* p, int n) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) x[i] = i < n ? to_float(p[i]) : 0.0f;
+}
+
+// A block: TOK tokens x 128 channels of one of the parts.  The tokens' low-rank rows are staged in shared memory; a
+// thread keeps eight weights of each of its two channels and runs over the tokens.  One running sum per output over r
+// in order, whatever shares its block.
+template <typename TW, int TOK>
+__global__ void __launch_bounds__(LR_THREADS)
+low_rank_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowRankPart p0, LowRankPart p1, int blocks0) {
+    extern __shared__ __align__(16) float lr_smem[];         // [TOK][rank padded to 8]
+    pdl_trigger();
+    const bool second = (int)blockIdx.y >= blocks0;
+    const LowRankPart p = second ? p1 : p0;
+    const int c0 = ((int)blockIdx.y - (second ? blocks0 : 0)) * LR_CHANNELS + threadIdx.x, c1 = c0 + LR_THREADS;
+    const int t0 = blockIdx.x * TOK, nt = min(TOK, n_tokens - t0);
+    const int rp = (p.rank + 7) & ~7;
+    pdl_wait();
+    for (int i = threadIdx.x; i < TOK * rp; i += LR_THREADS) {
+        const int t = i / rp, r = i % rp;
+        lr_smem[i] = t < nt && r < p.rank ? low[(long long)(t0 + t) * ldl + p.col + r] : 0.0f;
+    }
+    __syncthreads();
+    const TW* w0 = reinterpret_cast<const TW*>(p.w) + (long long)min(c0, p.n - 1) * p.ldw;
+    const TW* w1 = reinterpret_cast<const TW*>(p.w) + (long long)min(c1, p.n - 1) * p.ldw;
+    float a0[TOK], a1[TOK];
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) a0[t] = a1[t] = 0.0f;
+    const bool vec = sizeof(TW) == 2 && p.ldw % 8 == 0 && ((uintptr_t)p.w & 15) == 0;
+    for (int r = 0; r < p.rank; r += 8) {
+        float x0[8], x1[8];
+        if (vec && r + 8 <= p.rank) {
+            const uint4 u0 = *reinterpret_cast<const uint4*>(w0 + r), u1 = *reinterpret_cast<const uint4*>(w1 + r);
+            const __nv_bfloat162* b0 = reinterpret_cast<const __nv_bfloat162*>(&u0);
+            const __nv_bfloat162* b1 = reinterpret_cast<const __nv_bfloat162*>(&u1);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 f0 = __bfloat1622float2(b0[i]), f1 = __bfloat1622float2(b1[i]);
+                x0[2 * i] = f0.x, x0[2 * i + 1] = f0.y, x1[2 * i] = f1.x, x1[2 * i + 1] = f1.y;
+            }
+        } else {
+            load_weights<8>(x0, w0 + r, p.rank - r);
+            load_weights<8>(x1, w1 + r, p.rank - r);
+        }
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) {
+            const float4 y = *reinterpret_cast<const float4*>(lr_smem + t * rp + r);
+            const float4 z = *reinterpret_cast<const float4*>(lr_smem + t * rp + r + 4);
+            a0[t] = fmaf(x0[0], y.x, a0[t]), a1[t] = fmaf(x1[0], y.x, a1[t]);
+            a0[t] = fmaf(x0[1], y.y, a0[t]), a1[t] = fmaf(x1[1], y.y, a1[t]);
+            a0[t] = fmaf(x0[2], y.z, a0[t]), a1[t] = fmaf(x1[2], y.z, a1[t]);
+            a0[t] = fmaf(x0[3], y.w, a0[t]), a1[t] = fmaf(x1[3], y.w, a1[t]);
+            a0[t] = fmaf(x0[4], z.x, a0[t]), a1[t] = fmaf(x1[4], z.x, a1[t]);
+            a0[t] = fmaf(x0[5], z.y, a0[t]), a1[t] = fmaf(x1[5], z.y, a1[t]);
+            a0[t] = fmaf(x0[6], z.z, a0[t]), a1[t] = fmaf(x1[6], z.z, a1[t]);
+            a0[t] = fmaf(x0[7], z.w, a0[t]), a1[t] = fmaf(x1[7], z.w, a1[t]);
+        }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int c = half ? c1 : c0;
+        if (c >= p.n) continue;
+        const float bias = p.bias ? p.bias[c] : 0.0f;
+        const float rate = p.fn == 2 ? expf(p.a_log[c / p.per_head]) : 0.0f;
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) {
+            if (t >= nt) break;
+            float z = (half ? a1[t] : a0[t]) + bias;
+            if (p.fn == 1) z = expf(-p.power * softplus(-z));
+            else if (p.fn == 2) z = expf(-rate * softplus(z));
+            p.out[(long long)(t0 + t) * p.n + c] = z;
+        }
+    }
+}
+
+}  // namespace mu
+
+// The largest key size the scan takes.
+MU_EXPORT int mu_linear_scan_max_dk() { return mu::LS_MAX_DK; }
+
+// q, k [T][heads * dk], v [T][heads * dv]: float32 slices of rows `ld` apart.  per_channel: decay is [T][heads * dk];
+// else [T][heads][4] = (decay, take, -, -).  norm_out (may be null; not with per_channel): [T][heads].  long_steps:
+// many tokens a sequence; the launch then waits for an empty device.
+MU_EXPORT int mu_linear_scan(const float* q, const float* k, const float* v, long long ld, const float* decay,
+                             int per_channel, int n_seqs, int n_heads, int dk, int dv, float scale,
+                             const int* seq_first, const int* seq_slots, float* state, long long state_stride,
+                             long long state_offset, float* out, long long ldo, float* norm_out, int long_steps,
+                             void* stream) {
+    if (n_seqs <= 0) return MU_OK;
+    if (!q || !k || !v || !decay || !seq_first || !seq_slots || !state || !out || n_heads <= 0 || dk <= 0 || dv <= 0)
+        return MU_ERR_BAD_ARGUMENT;
+    if (dk > mu::LS_MAX_DK) return MU_ERR_UNSUPPORTED_SIZE;
+    if (!per_channel && ((uintptr_t)decay & 15)) return MU_ERR_ALIGNMENT;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int cols = dv + (norm_out ? 1 : 0);
+    const dim3 grid(n_seqs, n_heads, (cols + mu::LS_COLS - 1) / mu::LS_COLS), block(mu::LS_LANES * mu::LS_COLS);
+    const bool vec = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0 &&
+                     (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)state | (per_channel ? (uintptr_t)decay : 0)) & 15) == 0;
+#define MU_LINEAR_SCAN_V(R, V, PC)                                                                                    \
+    do {                                                                                                              \
+        const size_t smem = 2 * sizeof(float) * mu::ls_chunk_floats(mu::LS_LANES * R, PC);                            \
+        auto kernel = mu::linear_scan_kernel<R, V, PC>;                                                               \
+        if (!mu::allow_shared((const void*)kernel, smem)) return MU_ERR_LAUNCH;                                       \
+        mu::prefer_shared_memory((const void*)kernel);                                                                \
+        if (long_steps)                                                                                               \
+            return mu::launch_after(kernel, grid, block, smem, s, q, k, v, ld, decay, n_heads, dk, dv, scale,         \
+                                    seq_first, seq_slots, state, state_stride, state_offset, out, ldo, norm_out);     \
+        return mu::launch_pdl(kernel, grid, block, smem, s, 1, q, k, v, ld, decay, n_heads, dk, dv, scale, seq_first, \
+                              seq_slots, state, state_stride, state_offset, out, ldo, norm_out);                      \
+    } while (0)
+#define MU_LINEAR_SCAN(R)                                                                                             \
+    do {                                                                                                              \
+        if (vec && per_channel) MU_LINEAR_SCAN_V(R, true, true);                                                      \
+        if (per_channel) MU_LINEAR_SCAN_V(R, false, true);                                                            \
+        if (vec) MU_LINEAR_SCAN_V(R, true, false);                                                                    \
+        MU_LINEAR_SCAN_V(R, false, false);                                                                            \
+    } while (0)
+    if (dk <= 32) MU_LINEAR_SCAN(4);
+    if (dk <= 64) MU_LINEAR_SCAN(8);
+    if (dk <= 128) MU_LINEAR_SCAN(16);
+    MU_LINEAR_SCAN(32);
+#undef MU_LINEAR_SCAN
+#undef MU_LINEAR_SCAN_V
+}
+
+// i_raw, f_raw: [T][heads] float32 slices of rows `ld` apart; gates: [T][heads][4] = (decay, take, floor, 0).
+MU_EXPORT int mu_exp_gates(const float* i_raw, const float* f_raw, long long ld, const float* i_bias,
+                           const float* f_bias, float cap, int n_tokens, int n_seqs, int n_heads, const int* seq_first,
+                           const int* seq_slots, float* state, long long state_stride, long long m_offset, float* gates,
+                           void* stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return MU_OK;
+    if (!i_raw || !f_raw || !i_bias || !f_bias || !(cap > 0.0f) || !seq_first || !seq_slots || !state || !gates ||
+        n_heads <= 0)
+        return MU_ERR_BAD_ARGUMENT;
+    if ((uintptr_t)gates & 15) return MU_ERR_ALIGNMENT;
+    const dim3 grid(n_seqs, n_heads), block(n_tokens <= 32 * n_seqs ? 32 : 256);
+    return mu::launch_pdl(mu::exp_gates_kernel, grid, block, 0, (cudaStream_t)stream, 1, i_raw, f_raw, ld, i_bias, f_bias,
+                          cap, n_heads, seq_first, seq_slots, state, state_stride, m_offset, (float4*)gates);
+}
+
+// One or two low-rank projections of the same rows `low` (float32, a part's entries from its `col` on): `parts` is an
+// array of n_parts.  The weights are bfloat16 or float32.
+MU_EXPORT int mu_low_rank(const float* low, long long ldl, int n_tokens, const mu::LowRankPart* parts, int n_parts,
+                          int w_bf16, void* stream) {
+    if (n_tokens <= 0) return MU_OK;
+    if (!low || !parts || n_parts < 1 || n_parts > 2) return MU_ERR_BAD_ARGUMENT;
+    int blocks[2] = {0, 0}, rank = 0;
+    for (int i = 0; i < n_parts; ++i) {
+        const mu::LowRankPart& p = parts[i];
+        if (!p.w || !p.out || p.rank <= 0 || p.n <= 0 || p.col < 0 || p.ldw < p.rank || p.fn < 0 || p.fn > 2 ||
+            (p.fn == 2 && (!p.a_log || p.per_head <= 0)))
+            return MU_ERR_BAD_ARGUMENT;
+        blocks[i] = (p.n + mu::LR_CHANNELS - 1) / mu::LR_CHANNELS;
+        rank = p.rank > rank ? p.rank : rank;
+    }
+    const int tok = n_tokens >= 256 ? 16 : n_tokens >= 8 ? 4 : 1;
+    const size_t smem = (size_t)tok * ((rank + 7) / 8 * 8) * sizeof(float);
+    if (smem > 48 * 1024) return MU_ERR_UNSUPPORTED_SIZE;
+    const dim3 grid((n_tokens + tok - 1) / tok, blocks[0] + blocks[1]), block(mu::LR_THREADS);
+    cudaStream_t s = (cudaStream_t)stream;
+    const mu::LowRankPart p0 = parts[0], p1 = n_parts > 1 ? parts[1] : parts[0];
+#define MU_LOW_RANK(T, TOK)                                                                                           \
+    return mu::launch_pdl(mu::low_rank_kernel<T, TOK>, grid, block, smem, s, 1, low, ldl, n_tokens, p0, p1, blocks[0])
+    if (w_bf16) {
+        if (tok == 16) MU_LOW_RANK(__nv_bfloat16, 16);
+        if (tok == 4) MU_LOW_RANK(__nv_bfloat16, 4);
+        MU_LOW_RANK(__nv_bfloat16, 1);
+    }
+    if (tok == 16) MU_LOW_RANK(float, 16);
+    if (tok == 4) MU_LOW_RANK(float, 4);
+    MU_LOW_RANK(float, 1);
+#undef MU_LOW_RANK
+}

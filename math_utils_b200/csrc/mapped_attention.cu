@@ -24,7 +24,9 @@
 //                      is zero and which has no value), `gate` ([T, heads] in the storage type: the head's result
 //                      is multiplied by sigmoid(gate[t][h]), computed in float32), `chunk` (c > 0: a token at
 //                      position p sees the positions p - p % c .. p only, chunks counted from position 0 of the
-//                      sequence; it replaces the window).
+//                      sequence; it replaces the window), `slopes` (one float per head: the score of a key at
+//                      distance n loses slopes[h] * n), `keep` (with a window: the sequence's first `keep`
+//                      positions stay in sight of every later token, at their true distances).
 #include "common.cuh"
 
 #include <math.h>
@@ -157,7 +159,7 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
                         int n_kv_heads, int dim, int vdim, float scale, int window, float lambda, float out_scale,
                         float eps, int unit_rms, int vec, TE* __restrict__ out, long long ldo,
                         const float* __restrict__ head_scale, int sink, const TE* __restrict__ gate, long long ldg,
-                        int chunk) {
+                        int chunk, const float* __restrict__ slopes, int keep) {
     extern __shared__ float smem[];
     float* qs = smem;                                        // [MAPS][dim]
     float* part_acc = qs + MAPS * dim;                       // [warps][MAPS][vdim]
@@ -176,6 +178,9 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
         qs[d] = to_float(q[(long long)t * ldq + (long long)h * MAPS * dim + d]);
     __syncthreads();
     const int first = chunk > 0 ? pos - pos % chunk : window > 0 ? max(0, pos - window + 1) : 0;
+    // the keys in their order: the kept ones before the window, then the window
+    const int n_kept = min(keep, first), n_keys = n_kept + pos - first + 1;
+    const float slope = slopes ? slopes[h] : 0.0f;
     float m_run[MAPS], l_run[MAPS], acc[MAPS][MA_VPL];
 #pragma unroll
     for (int a = 0; a < MAPS; ++a) {
@@ -184,8 +189,8 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
 #pragma unroll
         for (int i = 0; i < MA_VPL; ++i) acc[a][i] = 0.0f;
     }
-    for (int base = first + warp * 32; base <= pos; base += MA_WARPS * 32) {
-        const int j = base + lane;
+    for (int base = warp * 32; base < n_keys; base += MA_WARPS * 32) {
+        const int j = base + lane < n_kept ? base + lane : first + base + lane - n_kept;
         const bool live = j <= pos;
         const TE* row = nullptr;
         float s[MAPS];
@@ -194,7 +199,7 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
         if (live) {
             row = rows + ((long long)pages[j / page_tokens] * page_tokens + j % page_tokens) * width;
 #pragma unroll
-            for (int a = 0; a < MAPS; ++a) s[a] = dot_key<TE>(qs + a * dim, row + key_off + a * dim, dim, vec != 0) * scale;
+            for (int a = 0; a < MAPS; ++a) s[a] = dot_key<TE>(qs + a * dim, row + key_off + a * dim, dim, vec != 0) * scale - slope * (float)(pos - j);
         }
         float p[MAPS];
 #pragma unroll
@@ -207,7 +212,7 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
 #pragma unroll
             for (int i = 0; i < MA_VPL; ++i) acc[a][i] *= corr;
         }
-        const int n_live = min(32, pos - base + 1);
+        const int n_live = min(32, n_keys - base);
         const unsigned long long mine = (unsigned long long)(uintptr_t)row;
         for (int jj = 0; jj < n_live; ++jj) {
             const TE* vrow = reinterpret_cast<const TE*>((uintptr_t)__shfl_sync(0xffffffffu, mine, jj)) + val_off;
@@ -281,7 +286,7 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
                      const int* __restrict__ block_table, int max_pages, const int* __restrict__ tok_pos,
                      const int* __restrict__ tok_seq, int n_heads, int n_kv_heads, int dim, int vdim, float scale,
                      int window, int vec, float* __restrict__ part_acc, float* __restrict__ part_ml,
-                     const float* __restrict__ head_scale, int chunk) {
+                     const float* __restrict__ head_scale, int chunk, const float* __restrict__ slopes, int keep) {
     extern __shared__ __align__(16) unsigned char md_raw[];
     const int kw = MAPS * dim, rw = kw + vdim;                 // the kv head's entries of a row
     const int pitch = rw + (vec ? 16 / (int)sizeof(TE) : 1);   // rows start in different banks
@@ -312,8 +317,12 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
 #pragma unroll
             for (int i = 0; i < MA_VPL; ++i) acc[u][a][i] = 0.0f;
         }
-    int pg = page_lo + ((share - page_lo) % MD_SPLITS + MD_SPLITS) % MD_SPLITS;     // the first page >= page_lo of this share
-    for (; pg <= page_hi; pg += MD_SPLITS) {
+    const int kept_pages = min((keep + MD_KEYS - 1) / MD_KEYS, page_lo);            // pages before the window's that hold kept positions
+    for (int pg = share; pg <= page_hi; pg += MD_SPLITS) {
+        if (pg >= kept_pages && pg < page_lo) {                // between the two runs of pages: on to the share's first of the second
+            pg += (page_lo - pg + MD_SPLITS - 1) / MD_SPLITS * MD_SPLITS;
+            if (pg > page_hi) break;
+        }
         __syncthreads();                                       // the page before is done with (and qs is written)
         const TE* src = rows + (long long)pages[pg] * MD_KEYS * width;
         if (vec) {
@@ -337,15 +346,17 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
             const int hg = warp + u * warps;                   // the head's place in its group
             if (hg >= group) break;
             const float scale_h = head_scale ? scale * head_scale[g * group + hg] : scale;
+            const float slope = slopes ? slopes[g * group + hg] : 0.0f;
 #pragma unroll
             for (int half = 0; half < MD_KEYS / 32; ++half) {
                 const int jl = half * 32 + lane, j = key0 + jl;
-                const bool live = j >= first && j <= pos;
+                const bool live = (j >= first || j < keep) && j <= pos;
                 if (__ballot_sync(0xffffffffu, live) == 0u) continue;
                 float p[MAPS];
 #pragma unroll
                 for (int a = 0; a < MAPS; ++a) {
-                    const float sc = live ? dot_key<TE>(qs + hg * kw + a * dim, tile + jl * pitch + a * dim, dim, vec != 0) * scale_h
+                    const float sc = live ? dot_key<TE>(qs + hg * kw + a * dim, tile + jl * pitch + a * dim, dim, vec != 0) * scale_h -
+                                                slope * (float)(pos - j)
                                           : -INFINITY;
                     const float m_new = fmaxf(m_run[u][a], warp_max(sc));
                     const float corr = expf(m_run[u][a] - m_new);
@@ -482,8 +493,9 @@ MU_EXPORT int mu_mapped_attention(const void* q, long long ldq, const void* rows
                                   int n_tokens, int n_heads, int n_kv_heads, int maps, int dim, int vdim, float scale,
                                   int window, float lambda, float out_scale, float eps, int unit_rms, void* out,
                                   long long ldo, int is_bf16, void* stream, const float* head_scale, int sink,
-                                  const void* gate, long long ldg, int chunk) {
+                                  const void* gate, long long ldg, int chunk, const float* slopes, int keep) {
     if (n_tokens <= 0) return MU_OK;
+    if (keep < 0) return MU_ERR_BAD_ARGUMENT;
     if (!q || !rows || !block_table || !tok_pos || !tok_seq || !out || n_heads <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || maps < 1 || maps > 2 || dim <= 0 || vdim <= 0 || page_tokens <= 0 || window < 0 ||
         chunk < 0)
@@ -501,7 +513,7 @@ MU_EXPORT int mu_mapped_attention(const void* q, long long ldq, const void* rows
     return mu::launch_pdl(mu::mapped_attention_kernel<TE, M>, grid, block, smem, s, 1, (const TE*)q, ldq,             \
                           (const TE*)rows, block_table, max_pages, page_tokens, tok_pos, tok_seq, n_heads, n_kv_heads, \
                           dim, vdim, scale, window, lambda, out_scale, eps, unit_rms, vec, (TE*)out, ldo, head_scale,  \
-                          sink, (const TE*)gate, ldg, chunk)
+                          sink, (const TE*)gate, ldg, chunk, slopes, keep)
     if (is_bf16) {
         if (maps == 2) MU_MAPPED(bf, 2);
         MU_MAPPED(bf, 1);
@@ -531,8 +543,10 @@ MU_EXPORT int mu_mapped_attention_decode(const void* q, long long ldq, const voi
                                          int n_tokens, int n_heads, int n_kv_heads, int maps, int dim, int vdim,
                                          float scale, int window, float lambda, float out_scale, float eps, int unit_rms,
                                          float* scratch, void* out, long long ldo, int is_bf16, void* stream,
-                                         const float* head_scale, int sink, const void* gate, long long ldg, int chunk) {
+                                         const float* head_scale, int sink, const void* gate, long long ldg, int chunk,
+                                         const float* slopes, int keep) {
     if (n_tokens <= 0) return MU_OK;
+    if (keep < 0) return MU_ERR_BAD_ARGUMENT;
     if (!q || !rows || !block_table || !tok_pos || !tok_seq || !out || !scratch || n_heads <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || maps < 1 || maps > 2 || dim <= 0 || vdim <= 0 || window < 0 || chunk < 0)
         return MU_ERR_BAD_ARGUMENT;
@@ -558,7 +572,7 @@ MU_EXPORT int mu_mapped_attention_decode(const void* q, long long ldq, const voi
             return MU_ERR_LAUNCH;                                                                                      \
         const int code = mu::launch_pdl(kernel, grid, block, smem, s, 1, (const TE*)q, ldq, (const TE*)rows,           \
                                         block_table, max_pages, tok_pos, tok_seq, n_heads, n_kv_heads, dim, vdim,      \
-                                        scale, window, vec, part_acc, part_ml, head_scale, chunk);                     \
+                                        scale, window, vec, part_acc, part_ml, head_scale, chunk, slopes, keep);       \
         if (code != MU_OK) return code;                                                                                \
         return mu::launch_pdl(mu::mapped_merge_kernel<TE, M>, mgrid, mblock, (size_t)vdim * sizeof(float), s, 1,       \
                               (const float*)part_acc, (const float*)part_ml, n_heads, vdim, lambda, out_scale, eps,    \

@@ -6,7 +6,7 @@
 // P enter that product as two bfloat16 terms (the rounded weight and what the rounding left), so they act with
 // some 16 bits of mantissa instead of 8.  At the end a1 - lambda a2, the head's unit rms and the output scale, and
 // the options of mapped_attention.cu (a multiplier per head on the scores, a sink in the denominator, a gate per head,
-// chunks of positions instead of a window).
+// chunks of positions instead of a window, a distance bias per head, kept first positions beside a window).
 //
 // Sizes: page of 64 positions; dim a multiple of 16 up to 256 per map; vdim a multiple of 16 up to 128; the cache
 // row a multiple of 8 entries.  Anything else takes the CUDA-core kernel.
@@ -52,7 +52,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
                             int dim, int vdim, float scale, int window, float lambda, float out_scale, float eps,
                             int unit_rms, __nv_bfloat16* __restrict__ out, long long ldo,
                             const float* __restrict__ head_scale, int sink, const __nv_bfloat16* __restrict__ gate,
-                            long long ldg, int chunk) {
+                            long long ldg, int chunk, const float* __restrict__ slopes, int keep) {
     extern __shared__ __align__(16) unsigned char raw[];
     const int kw = MAPS * dim;                               // key entries of one kv head
     const int kp = kw + MM_PAD, vp = VD + MM_PAD;            // row pitches in shared memory
@@ -73,6 +73,10 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
     // (with chunks: the first query's chunk starts first; a tile may reach into the next chunk)
     const int first_key = chunk > 0 ? pos0 - pos0 % chunk : window > 0 ? max(0, pos0 - window + 1) : 0;
     const int page_lo = first_key / MM_TILE, page_hi = last_key / MM_TILE;
+    // the pages in their order: those before the window that hold kept positions, then the window's
+    const int kept_pages = min((keep + MM_TILE - 1) / MM_TILE, page_lo), n_pages = kept_pages + page_hi - page_lo + 1;
+    auto page_at = [&](int i) { return i < kept_pages ? i : page_lo + i - kept_pages; };
+    const float slope = slopes ? slopes[h] : 0.0f;
 
     // the value columns past vdim stay zero; the queries of the tile (rows past count are zeros)
     for (int i = tid; i < 2 * MM_TILE * vp; i += blockDim.x) vs[i] = __float2bfloat16_rn(0.0f);
@@ -111,11 +115,11 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
     const int qpos[2] = {pos0 + row0, pos0 + row0 + 8};
     const bool real[2] = {row0 < count, row0 + 8 < count};
 
-    load_page(page_lo, 0);
-    for (int pg = page_lo; pg <= page_hi; ++pg) {
-        const int stage = (pg - page_lo) & 1;
-        if (pg < page_hi) {
-            load_page(pg + 1, stage ^ 1);
+    load_page(page_at(0), 0);
+    for (int turn = 0; turn < n_pages; ++turn) {
+        const int stage = turn & 1, pg = page_at(turn);
+        if (turn + 1 < n_pages) {
+            load_page(page_at(turn + 1), stage ^ 1);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -128,7 +132,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
         const int w_first = pos0 + warp * 16, w_last = min(pos0 + warp * 16 + 15, last_key);
         const bool skip = key0 > w_last || warp * 16 >= count ||
                           (chunk > 0 ? key0 + MM_TILE - 1 < w_first - w_first % chunk
-                                     : window > 0 && key0 + MM_TILE - 1 < w_first - window + 1);
+                                     : window > 0 && key0 >= keep && key0 + MM_TILE - 1 < w_first - window + 1);
         if (!skip) {
 #pragma unroll
             for (int a = 0; a < MAPS; ++a) {
@@ -154,8 +158,9 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
                     for (int e = 0; e < 4; ++e) {
                         const int r = e >> 1, kj = key0 + j * 8 + tig * 2 + (e & 1);
                         const bool seen = real[r] && kj <= qpos[r] &&
-                                          (chunk > 0 ? kj >= qpos[r] - qpos[r] % chunk : window == 0 || qpos[r] - kj < window);
-                        s[j][e] = seen ? s[j][e] * scale : -INFINITY;
+                                          (chunk > 0 ? kj >= qpos[r] - qpos[r] % chunk
+                                                     : window == 0 || qpos[r] - kj < window || kj < keep);
+                        s[j][e] = seen ? s[j][e] * scale - slope * (float)(qpos[r] - kj) : -INFINITY;
                         top[r] = fmaxf(top[r], s[j][e]);
                     }
                 float corr[2];
@@ -280,8 +285,9 @@ MU_EXPORT int mu_mapped_attention_mma(const void* q, long long ldq, const void* 
                                       const int* tiles, int n_tiles, int n_heads, int n_kv_heads, int maps, int dim,
                                       int vdim, float scale, int window, float lambda, float out_scale, float eps,
                                       int unit_rms, void* out, long long ldo, void* stream, const float* head_scale,
-                                      int sink, const void* gate, long long ldg, int chunk) {
+                                      int sink, const void* gate, long long ldg, int chunk, const float* slopes, int keep) {
     if (n_tiles <= 0) return MU_OK;
+    if (keep < 0) return MU_ERR_BAD_ARGUMENT;
     if (!q || !rows || !block_table || !tok_pos || !tok_seq || !tiles || !out || n_heads <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || window < 0 || chunk < 0)
         return MU_ERR_BAD_ARGUMENT;
@@ -304,7 +310,7 @@ MU_EXPORT int mu_mapped_attention_mma(const void* q, long long ldq, const void* 
         return mu::launch_pdl(kernel, grid, block, smem, s, 1, (const bf*)q, ldq, (const bf*)rows, block_table,        \
                               max_pages, tok_pos, tok_seq, tiles, n_heads, n_kv_heads, dim, vdim, scale, window,       \
                               lambda, out_scale, eps, unit_rms, (bf*)out, ldo, head_scale, sink, (const bf*)gate, ldg, \
-                              chunk);                                                                                  \
+                              chunk, slopes, keep);                                                                    \
     } while (0)
     if (maps == 2) {
         if (vd == 32) MU_MAPPED_MMA(2, 32);

@@ -19,7 +19,9 @@
 // router can divide the chosen weights by (their sum + renorm_eps), and compute one more number per token,
 // sigmoid(gate_w . h), which the combine multiplies a shared expert's row by before adding it.  The experts'
 // product takes an activation code (mu::ACT_*) for experts of the form W2 act(W1 x).  The combine can add its
-// result to what `out` holds.
+// result to what `out` holds.  A design whose weights act on the experts' INPUT gives them to the first product
+// (`row_weight`, one per pair: a row's products are multiplied by it before the activation, which is the product of
+// the weighted row), and none to the combine.
 #include "common.cuh"
 
 #include <math.h>
@@ -216,7 +218,7 @@ __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ pair_of, int top,
                 const T* __restrict__ w1, const T* __restrict__ w2, long long expert_stride, long long ldw,
                 const int* __restrict__ tile_info, const int* __restrict__ n_tiles, int n, int k,
-                TO* __restrict__ out, long long ldo, int act) {
+                TO* __restrict__ out, long long ldo, int act, const float* __restrict__ row_weight) {
     __shared__ float sa[MOE_TM][MOE_TK + 1];
     __shared__ float sw1[MOE_TN][MOE_TK + 1];
     __shared__ float sw2[GATED ? MOE_TN : 1][MOE_TK + 1];
@@ -270,6 +272,14 @@ moe_gemm_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ 
     for (int i = 0; i < 2; ++i) {
         const int r = 2 * ty + i;
         if (r >= rows) continue;
+        if (row_weight) {
+            const float f = row_weight[pair_of ? pair_of[slot0 + r] : slot0 + r];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                a1[i][j] *= f;
+                a2[i][j] *= f;
+            }
+        }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int col = n0 + tx + 16 * j;
@@ -296,7 +306,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, long long ldy, c
         for (int k = 0; k < top; ++k) {
             const int slot = slot_of[(long long)t * top + k];
             const float row = slot >= 0 ? y[(long long)slot * ldy + d] : to_float(x[(long long)t * ldx + d]);
-            v += weight_of[(long long)t * top + k] * row;
+            v += (weight_of ? weight_of[(long long)t * top + k] : 1.0f) * row;
         }
         if (shared) v += (shared_gate ? shared_gate[t] : 1.0f) * shared[(long long)t * lds + d];
         if (add) v += out[(long long)t * ldo + d];
@@ -332,7 +342,7 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ y, long long ld
 #pragma unroll
             for (int k = 0; k < TOP; ++k) {
                 const int slot = slot_of[(long long)t * TOP + k];
-                w[k] = weight_of[(long long)t * TOP + k];
+                w[k] = weight_of ? weight_of[(long long)t * TOP + k] : 1.0f;
                 row[k] = slot >= 0 ? load4(y + (long long)slot * ldy + d) : load4(x + (long long)t * ldx + d);
             }
 #pragma unroll
@@ -342,7 +352,7 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ y, long long ld
         } else {
             for (int k = 0; k < top; ++k) {
                 const int slot = slot_of[(long long)t * top + k];
-                const float w = weight_of[(long long)t * top + k];
+                const float w = weight_of ? weight_of[(long long)t * top + k] : 1.0f;
                 const float4 row = slot >= 0 ? load4(y + (long long)slot * ldy + d) : load4(x + (long long)t * ldx + d);
                 v.x += w * row.x; v.y += w * row.y; v.z += w * row.z; v.w += w * row.w;
             }
@@ -444,7 +454,7 @@ MU_EXPORT int mu_moe_group(const int* expert_of, int n_pairs, int n_experts, int
 MU_EXPORT int mu_moe_gemm(const void* x, long long ldx, const int* pair_of, int top, const void* w1, const void* w2,
                           long long expert_stride, long long ldw, const int* tile_info, const int* n_tiles,
                           int max_tiles, int n, int k, void* out, long long ldo, int is_bf16, int out_bf16,
-                          void* stream, int act) {
+                          void* stream, int act, const float* row_weight) {
     if (max_tiles <= 0) return MU_OK;
     if (!x || !w1 || !tile_info || !n_tiles || !out || n <= 0 || k <= 0 || (pair_of && top <= 0))
         return MU_ERR_BAD_ARGUMENT;
@@ -454,7 +464,7 @@ MU_EXPORT int mu_moe_gemm(const void* x, long long ldx, const int* pair_of, int 
     typedef __nv_bfloat16 bf;
 #define MU_MOE(T, TO, G)                                                                                             \
     return mu::launch_pdl(mu::moe_gemm_kernel<T, TO, G>, grid, block, 0, s, 1, (const T*)x, ldx, pair_of, top,        \
-                          (const T*)w1, (const T*)w2, expert_stride, ldw, tile_info, n_tiles, n, k, (TO*)out, ldo, act)
+                          (const T*)w1, (const T*)w2, expert_stride, ldw, tile_info, n_tiles, n, k, (TO*)out, ldo, act, row_weight)
     if (w2) {
         if (is_bf16 && out_bf16) MU_MOE(bf, bf, true);
         if (is_bf16) MU_MOE(bf, float, true);
@@ -466,12 +476,13 @@ MU_EXPORT int mu_moe_gemm(const void* x, long long ldx, const int* pair_of, int 
 #undef MU_MOE
 }
 
-// x (the experts' input rows, bfloat16 if x_bf16 else float32) is needed when a pair may have no slot.
+// x (the experts' input rows, bfloat16 if x_bf16 else float32) is needed when a pair may have no slot; weight_of null:
+// every choice counts once.
 MU_EXPORT int mu_moe_combine(const float* y, long long ldy, const int* slot_of, const float* weight_of, int n_tokens,
                              int top, int width, float* out, long long ldo, void* stream, const void* x, long long ldx,
                              int x_bf16, const float* shared, long long lds, const float* shared_gate, int add) {
     if (n_tokens <= 0) return MU_OK;
-    if (!y || !slot_of || !weight_of || !out || top <= 0 || width <= 0) return MU_ERR_BAD_ARGUMENT;
+    if (!y || !slot_of || !out || top <= 0 || width <= 0) return MU_ERR_BAD_ARGUMENT;
     const dim3 grid(n_tokens), block(width >= 1024 ? 256 : 128);
     const bool vec = width % 4 == 0 && ldy % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)out & 15) == 0 &&
                      (!x || (ldx % 4 == 0 && ((uintptr_t)x & (x_bf16 ? 7 : 15)) == 0)) &&
@@ -482,12 +493,14 @@ MU_EXPORT int mu_moe_combine(const float* y, long long ldy, const int* slot_of, 
     return mu::launch_pdl(mu::moe_combine_vec_kernel<TX, TOP>, grid, vblock, 0, (cudaStream_t)stream, 1, y, ldy, slot_of, \
                           weight_of, top, width, out, ldo, (const TX*)x, ldx, shared, lds, shared_gate, add)
         if (x_bf16) {
+            if (top == 1) MU_COMBINE(__nv_bfloat16, 1);
             if (top == 2) MU_COMBINE(__nv_bfloat16, 2);
             if (top == 4) MU_COMBINE(__nv_bfloat16, 4);
             if (top == 6) MU_COMBINE(__nv_bfloat16, 6);
             if (top == 8) MU_COMBINE(__nv_bfloat16, 8);
             MU_COMBINE(__nv_bfloat16, 0);
         }
+        if (top == 1) MU_COMBINE(float, 1);
         if (top == 2) MU_COMBINE(float, 2);
         if (top == 4) MU_COMBINE(float, 4);
         if (top == 6) MU_COMBINE(float, 6);

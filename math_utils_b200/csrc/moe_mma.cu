@@ -6,6 +6,8 @@
 // read as fragments with ldmatrix.  GATED: two weight stacks, out = silu(W1 x) * (W2 x).  Every output is one
 // running sum over k in order, whatever shares its tile.
 //
+// row_weight (null: none): a weight per pair that multiplies the row's products before the activation.
+//
 // The same kernel serves products PER HEAD (mu_heads_gemm): out[t, h, :] = W[h] x[t, h, :] for every token t and head
 // h, the head taking the expert's place: tile (blockIdx.x, head blockIdx.z) covers tokens 32 blockIdx.x .. + 32, and
 // a head's slice of x and of out starts x_group_offset / out_group_offset elements after the head before.
@@ -48,12 +50,14 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const in
                     const __nv_bfloat16* __restrict__ w1, const __nv_bfloat16* __restrict__ w2, long long expert_stride,
                     long long ldw, const int* __restrict__ tile_info, const int* __restrict__ n_tiles, int n, int k,
                     TO* __restrict__ out, long long ldo, int n_rows, long long x_group_offset,
-                    long long out_group_offset, const __nv_bfloat16* __restrict__ gate, long long ldg, int act) {
+                    long long out_group_offset, const __nv_bfloat16* __restrict__ gate, long long ldg, int act,
+                    const float* __restrict__ row_weight) {
     extern __shared__ __align__(16) unsigned char mm_raw[];
     constexpr int MM_ROWS = 32 * WM, NW = 2 * WM;                               // rows a block; 8-column tiles a warp
     constexpr int STAGE = (MM_ROWS + (GATED ? 2 : 1) * MM_COLS) * MM_PITCH;      // elements per stage
     __nv_bfloat16* sm = reinterpret_cast<__nv_bfloat16*>(mm_raw);
     __shared__ int src_row[64];
+    __shared__ float row_factor[64];                             // the weight of a row's pair, where weights act on the input
     pdl_trigger();
     pdl_wait();
     const int tile = blockIdx.x;
@@ -72,7 +76,9 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const in
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     if (tid < MM_ROWS) {
         const int r = min(tid, rows - 1);                        // rows past the tile's end repeat its last row
-        src_row[tid] = pair_of ? pair_of[slot0 + r] / top : slot0 + r;
+        const int pair = pair_of ? pair_of[slot0 + r] : slot0 + r;
+        src_row[tid] = pair_of ? pair / top : pair;
+        row_factor[tid] = row_weight ? row_weight[pair] : 1.0f;
     }
     __syncthreads();
     const __nv_bfloat16* w1e = w1 + (long long)e * expert_stride;
@@ -155,10 +161,11 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const in
                 const int r = row_base + m * 16 + g + half * 8;
                 const int col = n0 + col_base + j * 8 + 2 * t4;
                 if (r >= rows || col >= n) continue;
-                float v0 = acc1[m][j][2 * half], v1 = acc1[m][j][2 * half + 1];
+                const float f = row_factor[r];
+                float v0 = acc1[m][j][2 * half] * f, v1 = acc1[m][j][2 * half + 1] * f;
                 if (GATED) {
-                    v0 = v0 / (1.0f + expf(-v0)) * acc2[m][j][2 * half];
-                    v1 = v1 / (1.0f + expf(-v1)) * acc2[m][j][2 * half + 1];
+                    v0 = v0 / (1.0f + expf(-v0)) * (acc2[m][j][2 * half] * f);
+                    v1 = v1 / (1.0f + expf(-v1)) * (acc2[m][j][2 * half + 1] * f);
                 } else if (act == ACT_RELU2) {
                     v0 = relu2(v0);
                     v1 = relu2(v1);
@@ -179,7 +186,7 @@ int launch_moe_mma(dim3 grid, cudaStream_t s, const __nv_bfloat16* x, long long 
                    const __nv_bfloat16* w1, const __nv_bfloat16* w2, long long expert_stride, long long ldw,
                    const int* tile_info, const int* n_tiles, int n, int k, TO* out, long long ldo, int n_rows = 0,
                    long long x_group_offset = 0, long long out_group_offset = 0, const __nv_bfloat16* gate = nullptr,
-                   long long ldg = 0, int act = 0) {
+                   long long ldg = 0, int act = 0, const float* row_weight = nullptr) {
     constexpr size_t smem = MM_STAGES * (32 * WM + (GATED ? 2 : 1) * MM_COLS) * MM_PITCH * sizeof(__nv_bfloat16);
     static bool set = false;
     if (!set) {
@@ -190,7 +197,7 @@ int launch_moe_mma(dim3 grid, cudaStream_t s, const __nv_bfloat16* x, long long 
     }
     return launch_pdl(moe_gemm_mma_kernel<TO, GATED, WM>, grid, dim3(MM_THREADS), smem, s, 1, x, ldx, pair_of, top, w1, w2,
                       expert_stride, ldw, tile_info, n_tiles, n, k, out, ldo, n_rows, x_group_offset, out_group_offset, gate,
-                      ldg, act);
+                      ldg, act, row_weight);
 }
 
 }  // namespace mu
@@ -199,7 +206,7 @@ int launch_moe_mma(dim3 grid, cudaStream_t s, const __nv_bfloat16* x, long long 
 MU_EXPORT int mu_moe_gemm_mma(const void* x, long long ldx, const int* pair_of, int top, const void* w1, const void* w2,
                               long long expert_stride, long long ldw, const int* tile_info, const int* n_tiles,
                               int max_tiles, int tile_rows, int n, int k, void* out, long long ldo, int out_bf16,
-                              void* stream, int act) {
+                              void* stream, int act, const float* row_weight) {
     if (max_tiles <= 0) return MU_OK;
     if (!x || !w1 || !tile_info || !n_tiles || !out || n <= 0 || k <= 0 || (pair_of && top <= 0) ||
         (tile_rows != 32 && tile_rows != 64))
@@ -214,10 +221,10 @@ MU_EXPORT int mu_moe_gemm_mma(const void* x, long long ldx, const int* pair_of, 
     return tile_rows == 64                                                                                          \
                ? mu::launch_moe_mma<TO, G, 2>(grid, s, (const bf*)x, ldx, pair_of, top, (const bf*)w1, (const bf*)w2, \
                                               expert_stride, ldw, tile_info, n_tiles, n, k, (TO*)out, ldo, 0, 0, 0,  \
-                                              nullptr, 0, act)                                                      \
+                                              nullptr, 0, act, row_weight)                                          \
                : mu::launch_moe_mma<TO, G, 1>(grid, s, (const bf*)x, ldx, pair_of, top, (const bf*)w1, (const bf*)w2, \
                                               expert_stride, ldw, tile_info, n_tiles, n, k, (TO*)out, ldo, 0, 0, 0,  \
-                                              nullptr, 0, act)
+                                              nullptr, 0, act, row_weight)
     if (w2) {
         if (out_bf16) MU_MM(bf, true);
         MU_MM(float, true);

@@ -5,7 +5,9 @@
 //                float32 residual stream); input always float32, output float32 or the compute dtype.
 // rms_norm:      y = x / sqrt(mean(x^2) + eps) * w, statistics in float32.
 // sigmoid_gate:  o *= 1 / (1 + exp(-g)), element by element, in float32.
+// rms_norm_out with groups: the row in equal consecutive parts, each normed by itself (a block a part).
 // rms_norm_pair: two RMS norms of the same rows (one statistic, two weights, two outputs).
+// rms_norm_sum:  y (+)= a * rms_norm(p) * wp + b * rms_norm(q) * wq: two branches, each normed, joined in one pass.
 // softcap:       x <- cap * tanh(x / cap) on float32 rows, in place.
 #include "common.cuh"
 
@@ -62,9 +64,12 @@ __global__ void rms_norm_out_kernel(const float* __restrict__ x, long long ldx, 
     pdl_wait();
     const int r = blockIdx.x;
     const long long from = rows ? (long long)rows[r] : (long long)r;
-    const float* src = x + from * ldx;
-    const float* src2 = x2 ? x2 + from * ldx2 : nullptr;
-    TO* dst = y + (long long)r * ldy;
+    const long long part0 = (long long)blockIdx.y * n;
+    const float* src = x + from * ldx + part0;
+    const float* src2 = x2 ? x2 + from * ldx2 + part0 : nullptr;
+    TO* dst = y + (long long)r * ldy + part0;
+    w += part0;
+    if (copy) copy += part0;
     float s = 0.0f;
     for (int d = threadIdx.x; d < n; d += blockDim.x) {
         const float v = src2 ? a * src[d] + b * src2[d] : src[d];
@@ -92,8 +97,12 @@ rms_norm_out_vec_kernel(const float* __restrict__ x, long long ldx, const float*
     pdl_wait();
     const int r = blockIdx.x, n4 = n / 4;
     const long long from = rows ? (long long)rows[r] : (long long)r;
-    const float4* src = reinterpret_cast<const float4*>(x + from * ldx);
-    const float4* src2 = x2 ? reinterpret_cast<const float4*>(x2 + from * ldx2) : nullptr;
+    const long long part0 = (long long)blockIdx.y * n;
+    const float4* src = reinterpret_cast<const float4*>(x + from * ldx + part0);
+    const float4* src2 = x2 ? reinterpret_cast<const float4*>(x2 + from * ldx2 + part0) : nullptr;
+    w += part0;
+    y += part0;
+    if (copy) copy += part0;
     float4 v[4];
     float s = 0.0f;
 #pragma unroll
@@ -213,6 +222,65 @@ rms_norm_pair_kernel(const float* __restrict__ x, long long ldx, const float* __
     }
 }
 
+// y (+)= a * p / rms(p) * wp + b * q / rms(q) * wq, float32 rows.  VEC: rows of up to 4,096 values in whole, aligned
+// 16-byte pieces, read once and kept in registers between the statistics and the output.
+template <bool ADD, bool VEC>
+__global__ void __launch_bounds__(256)
+rms_norm_sum_kernel(const float* __restrict__ p, long long ldp, float a, const float* __restrict__ wp,
+                    const float* __restrict__ q, long long ldq, float b, const float* __restrict__ wq, float eps,
+                    float* __restrict__ y, long long ldy, int n) {
+    __shared__ float scratch[2][32];
+    pdl_trigger();
+    pdl_wait();
+    const int r = blockIdx.x, n4 = n / 4;
+    const float* ps = p + (long long)r * ldp;
+    const float* qs = q + (long long)r * ldq;
+    float* dst = y + (long long)r * ldy;
+    float sp = 0.0f, sq = 0.0f;
+    float4 u[4], v[4];
+    if (VEC) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int idx = threadIdx.x + 256 * i;
+            u[i] = v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (idx < n4) {
+                u[i] = reinterpret_cast<const float4*>(ps)[idx];
+                v[i] = reinterpret_cast<const float4*>(qs)[idx];
+            }
+            sp += (u[i].x * u[i].x + u[i].y * u[i].y) + (u[i].z * u[i].z + u[i].w * u[i].w);
+            sq += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+        }
+    } else {
+        for (int d = threadIdx.x; d < n; d += blockDim.x) {
+            sp += ps[d] * ps[d];
+            sq += qs[d] * qs[d];
+        }
+    }
+    const float fp = a / sqrtf(block_sum(sp, scratch[0]) / (float)n + eps);
+    const float fq = b / sqrtf(block_sum(sq, scratch[1]) / (float)n + eps);
+    if (VEC) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int idx = threadIdx.x + 256 * i;
+            if (idx >= n4) continue;
+            const float4 g = reinterpret_cast<const float4*>(wp)[idx], h = reinterpret_cast<const float4*>(wq)[idx];
+            float4 o = make_float4(u[i].x * fp * g.x + v[i].x * fq * h.x, u[i].y * fp * g.y + v[i].y * fq * h.y,
+                                   u[i].z * fp * g.z + v[i].z * fq * h.z, u[i].w * fp * g.w + v[i].w * fq * h.w);
+            if (ADD) {
+                const float4 old = reinterpret_cast<const float4*>(dst)[idx];
+                o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w;
+            }
+            reinterpret_cast<float4*>(dst)[idx] = o;
+        }
+    } else {
+        for (int d = threadIdx.x; d < n; d += blockDim.x) {
+            float o = ps[d] * fp * wp[d] + qs[d] * fq * wq[d];
+            if (ADD) o += dst[d];
+            dst[d] = o;
+        }
+    }
+}
+
 // x <- cap * tanh(x / cap), float32 rows in place.
 __global__ void softcap_kernel(float* __restrict__ x, long long ldx, int n_rows, int width, float cap) {
     pdl_trigger();
@@ -273,15 +341,16 @@ MU_EXPORT int mu_rms_norm(const void* x, long long ldx, int x_bf16, const float*
 MU_EXPORT int mu_rms_norm_out(const float* x, long long ldx, const float* x2, long long ldx2, float a, float b,
                               const int* rows, const float* w, float offset, float scale, float eps, void* y,
                               long long ldy, int y_bf16, int add, void* copy, long long ldc, int n_rows, int n,
-                              void* stream) {
+                              void* stream, int groups) {
     if (n_rows <= 0) return MU_OK;
-    if (n <= 0 || !x || !w || !y || (add && y_bf16)) return MU_ERR_BAD_ARGUMENT;
+    if (n <= 0 || !x || !w || !y || (add && y_bf16) || groups < 1 || groups > 65535 || n % groups) return MU_ERR_BAD_ARGUMENT;
+    n /= groups;                                             // a block takes one part of a row
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
     const bool vec = n % 4 == 0 && n <= 4096 && ldx % 4 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0 &&
                      (!x2 || (ldx2 % 4 == 0 && ((uintptr_t)x2 & 15) == 0)) && ldy % 4 == 0 &&
                      ((uintptr_t)y & 15) == 0 && (!copy || (ldc % 4 == 0 && ((uintptr_t)copy & 7) == 0));
-    const dim3 grid(n_rows), block(vec ? 256 : (n >= 1024 ? 256 : 128));
+    const dim3 grid(n_rows, groups), block(vec ? 256 : (n >= 1024 ? 256 : 128));
 #define MU_RMS_OUT(KERNEL, TO, ADD)                                                                                    \
     return mu::launch_pdl(mu::KERNEL<TO, ADD>, grid, block, 0, s, 1, x, ldx, x2, ldx2, a, b, rows, w, offset, scale,   \
                           eps, (TO*)y, ldy, (bf*)copy, ldc, n)
@@ -326,6 +395,26 @@ MU_EXPORT int mu_rms_norm_pair(const float* x, long long ldx, const float* w1, c
                               (__nv_bfloat16*)y1, ldy1, (__nv_bfloat16*)y2, ldy2, n, vec);
     return mu::launch_pdl(mu::rms_norm_pair_kernel<float>, grid, block, 0, s, 1, x, ldx, w1, w2, eps, (float*)y1, ldy1,
                           (float*)y2, ldy2, n, vec);
+}
+
+// y (+)= a * rms_norm(p) * wp + b * rms_norm(q) * wq, all float32 rows of n values, one eps.
+MU_EXPORT int mu_rms_norm_sum(const float* p, long long ldp, float a, const float* wp, const float* q, long long ldq,
+                              float b, const float* wq, float eps, float* y, long long ldy, int n_rows, int n, int add,
+                              void* stream) {
+    if (n_rows <= 0) return MU_OK;
+    if (n <= 0 || !p || !q || !wp || !wq || !y) return MU_ERR_BAD_ARGUMENT;
+    const bool vec = n % 4 == 0 && n <= 4096 && ldp % 4 == 0 && ldq % 4 == 0 && ldy % 4 == 0 &&
+                     (((uintptr_t)p | (uintptr_t)q | (uintptr_t)wp | (uintptr_t)wq | (uintptr_t)y) & 15) == 0;
+#define MU_RMS_SUM(ADD, VEC)                                                                                           \
+    return mu::launch_pdl(mu::rms_norm_sum_kernel<ADD, VEC>, dim3(n_rows), dim3(256), 0, (cudaStream_t)stream, 1, p,   \
+                          ldp, a, wp, q, ldq, b, wq, eps, y, ldy, n)
+    if (vec) {
+        if (add) MU_RMS_SUM(true, true);
+        MU_RMS_SUM(false, true);
+    }
+    if (add) MU_RMS_SUM(true, false);
+    MU_RMS_SUM(false, false);
+#undef MU_RMS_SUM
 }
 
 // x <- cap * tanh(x / cap) on float32 rows, in place.

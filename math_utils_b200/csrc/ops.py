@@ -53,7 +53,7 @@ _c_int, _c_ll, _c_f, _c_p, _c_ull = ctypes.c_int, ctypes.c_longlong, ctypes.c_fl
 
 _SIGNATURES = {
     "mu_copy_async": [_c_p, _c_p, _c_ll, _c_p],
-    "mu_embed": [_c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p],
+    "mu_embed": [_c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p, _c_p],
     "mu_layernorm": [_c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_f, _c_int, _c_p],
     "mu_gemm_simt": [_c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_ll, _c_ll, _c_ll, _c_ll,
                      _c_int, _c_int, _c_int, _c_p],
@@ -88,7 +88,8 @@ _SIGNATURES = {
     "mu_embed_pair": [_c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_ll,
                       _c_ll, _c_int, _c_int, _c_p],
     "mu_rms_norm_out": [_c_p, _c_ll, _c_p, _c_ll, _c_f, _c_f, _c_p, _c_p, _c_f, _c_f, _c_f, _c_p, _c_ll, _c_int, _c_int,
-                        _c_p, _c_ll, _c_int, _c_int, _c_p],
+                        _c_p, _c_ll, _c_int, _c_int, _c_p, _c_int],
+    "mu_rms_norm_sum": [_c_p, _c_ll, _c_f, _c_p, _c_p, _c_ll, _c_f, _c_p, _c_f, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p],
     "mu_gated_act": [_c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_p],
     "mu_scaled_sum": [_c_p, _c_ll, _c_f, _c_p, _c_ll, _c_f, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p],
     "mu_cast_rows": [_c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_p],
@@ -96,16 +97,16 @@ _SIGNATURES = {
                       _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_p, _c_int],
     "mu_mapped_attention": [_c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                             _c_int, _c_f, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_ll, _c_int, _c_p,
-                            _c_p, _c_int, _c_p, _c_ll, _c_int],
+                            _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
     "mu_mapped_decode_fits": [_c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int],
     "mu_mapped_decode_scratch": [_c_int, _c_int, _c_int, _c_int],
     "mu_mapped_attention_decode": [_c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                                    _c_int, _c_f, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_p, _c_ll, _c_int, _c_p,
-                                   _c_p, _c_int, _c_p, _c_ll, _c_int],
+                                   _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
     "mu_mapped_attention_mma_fits": [_c_int, _c_int, _c_int, _c_int, _c_int],
     "mu_mapped_attention_mma": [_c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
                                 _c_int, _c_int, _c_f, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_ll, _c_p,
-                                _c_p, _c_int, _c_p, _c_ll, _c_int],
+                                _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
     "mu_qkv_norm_rows": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_f, _c_int, _c_int, _c_int, _c_int, _c_int,
                          _c_int, _c_p, _c_int, _c_f, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_p],
     "mu_residual_add_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_f, _c_p, _c_f, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p],
@@ -113,13 +114,19 @@ _SIGNATURES = {
                          _c_p, _c_p, _c_p, _c_int, _c_p],
     "mu_delta_scan_max_dk": [],
     "mu_delta_scan": [_c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_ll,
-                      _c_ll, _c_p, _c_int, _c_p],
+                      _c_ll, _c_p, _c_int, _c_p, _c_int],
+    "mu_linear_scan_max_dk": [],
+    "mu_linear_scan": [_c_p, _c_p, _c_p, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_p, _c_p, _c_p,
+                       _c_ll, _c_ll, _c_p, _c_ll, _c_p, _c_int, _c_p],
+    "mu_exp_gates": [_c_p, _c_p, _c_ll, _c_p, _c_p, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_ll, _c_ll, _c_p,
+                     _c_p],
+    "mu_low_rank": [_c_p, _c_ll, _c_int, _c_p, _c_int, _c_int, _c_p],
     "mu_xielu": [_c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p],
     "mu_ssd_conv": [_c_p, _c_ll, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_p, _c_ll,
                     _c_int, _c_p, _c_p],
     "mu_ssd_scan": [_c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p,
                     _c_p, _c_p, _c_ll, _c_ll, _c_p, _c_int, _c_p],
-    "mu_gated_group_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p, _c_ll, _c_int, _c_p, _c_int],
+    "mu_gated_group_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p, _c_ll, _c_int, _c_p, _c_int, _c_int, _c_p, _c_p, _c_int],
     "mu_dynamic_tanh": [_c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_p],
     "mu_rms_norm": [_c_p, _c_ll, _c_int, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_f, _c_p],
     "mu_sigmoid_gate": [_c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p],
@@ -138,9 +145,9 @@ _SIGNATURES = {
                      _c_p, _c_f, _c_p, _c_p],
     "mu_moe_group": [_c_p, _c_int, _c_int, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_int],
     "mu_moe_gemm": [_c_p, _c_ll, _c_p, _c_int, _c_p, _c_p, _c_ll, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_int, _c_p, _c_ll,
-                    _c_int, _c_int, _c_p, _c_int],
+                    _c_int, _c_int, _c_p, _c_int, _c_p],
     "mu_moe_gemm_mma": [_c_p, _c_ll, _c_p, _c_int, _c_p, _c_p, _c_ll, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p,
-                        _c_ll, _c_int, _c_p, _c_int],
+                        _c_ll, _c_int, _c_p, _c_int, _c_p],
     "mu_heads_gemm": [_c_p, _c_ll, _c_ll, _c_p, _c_ll, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_p, _c_ll, _c_ll, _c_int,
                       _c_p, _c_ll, _c_p],
     "mu_moe_combine": [_c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_int, _c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, _c_p,
@@ -272,9 +279,15 @@ def zeroed_workspace(name: str, device, n_bytes: int) -> torch.Tensor:
 
 # ------------------------------------------------------------------ elementwise
 def embed(ids: torch.Tensor, positions: Optional[torch.Tensor], table: torch.Tensor,
-          pos_table: Optional[torch.Tensor], out: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
-    """out[t] = table[ids[t]] * scale + pos_table[positions[t]] as float32 [T, hidden]."""
-    _need_cuda(ids, positions, table, pos_table)
+          pos_table: Optional[torch.Tensor], out: Optional[torch.Tensor] = None, scale: float = 1.0,
+          turns: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t] = table[ids[t]] * scale + pos_table[positions[t]] as float32 [T, hidden].  ``turns`` (float32
+    [2, (hidden + 1) // 2]: frequencies in turns per position, rounded, and what the rounding left) adds sinusoids:
+    entry 2i the sine and entry 2i + 1 the cosine of 2 pi * position * turns[:, i].sum()."""
+    _need_cuda(ids, positions, table, pos_table, turns)
+    if turns is not None and (turns.dtype != torch.float32 or not turns.is_contiguous() or positions is None
+                              or tuple(turns.shape) != (2, (table.shape[1] + 1) // 2)):
+        raise KernelError("embed: the sinusoids' frequencies are contiguous float32 [2, (hidden + 1) // 2]")
     _i32(ids, "ids"); _i32(positions, "positions")
     n, hidden = ids.numel(), table.shape[1]
     if pos_table is not None and (pos_table.dtype != table.dtype or pos_table.shape[1] != hidden):
@@ -285,7 +298,7 @@ def embed(ids: torch.Tensor, positions: Optional[torch.Tensor], table: torch.Ten
         out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
     _check(library().mu_embed(_ptr(ids), _ptr(positions),
                               _ptr(table), _ptr(pos_table), _ptr(out), n, hidden, _is_bf16(table), float(scale),
-                              _stream()),
+                              _stream(), _ptr(turns)),
            "embed")
     return out
 
@@ -354,10 +367,11 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: Optio
 def rms_norm_out(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float = 0.0, scale: float = 1.0,
                  out_dtype: Optional[torch.dtype] = None, rows: Optional[torch.Tensor] = None,
                  out: Optional[torch.Tensor] = None, add: bool = False,
-                 copy: Optional[torch.Tensor] = None, second=None) -> torch.Tensor:
+                 copy: Optional[torch.Tensor] = None, second=None, groups: int = 1) -> torch.Tensor:
     """scale * v / sqrt(mean(v^2) + eps) * (offset + weight) of float32 rows v = x (optionally the rows that ``rows``
     picks), written to ``out`` or, with ``add``, added to the float32 ``out``.  ``copy`` (bfloat16, shaped like
-    ``out``) receives what ``out`` then holds.  ``second`` = (a, x2, b): the rows are v = a * x + b * x2."""
+    ``out``) receives what ``out`` then holds.  ``second`` = (a, x2, b): the rows are v = a * x + b * x2.  ``groups``:
+    the row in that many consecutive equal parts, each normed by itself."""
     a, x2, b = second if second is not None else (1.0, None, 0.0)
     _need_cuda(x, weight, rows, out, copy, x2)
     if x2 is not None and (x2.dtype != torch.float32 or x2.shape != x.shape or x2.stride(1) != 1):
@@ -380,8 +394,25 @@ def rms_norm_out(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: floa
     _check(library().mu_rms_norm_out(_ptr(x), x.stride(0), _ptr(x2), x2.stride(0) if x2 is not None else 0, float(a),
                                      float(b), _ptr(rows), _ptr(weight), float(offset), float(scale),
                                      float(eps), _ptr(out), out.stride(0), _is_bf16(out), int(add), _ptr(copy),
-                                     copy.stride(0) if copy is not None else 0, n_rows, n, _stream()),
-           ("rms_norm_out(n={})", n))
+                                     copy.stride(0) if copy is not None else 0, n_rows, n, _stream(), int(groups)),
+           ("rms_norm_out(n={}, groups={})", n, groups))
+    return out
+
+
+def rms_norm_sum(p: torch.Tensor, a: float, wp: torch.Tensor, q: torch.Tensor, b: float, wq: torch.Tensor, eps: float,
+                 out: torch.Tensor, add: bool = False) -> torch.Tensor:
+    """out (+)= a * p / rms(p) * wp + b * q / rms(q) * wq: two float32 branches, each normed over its row, joined."""
+    _need_cuda(p, wp, q, wq, out)
+    n = p.shape[1]
+    for t in (p, q, out):
+        if t.dtype != torch.float32 or t.dim() != 2 or t.shape != p.shape or t.stride(1) != 1:
+            raise KernelError("rms_norm_sum works on float32 [rows, n] of one shape with unit inner stride")
+    for w in (wp, wq):
+        if w.dtype != torch.float32 or not w.is_contiguous() or w.numel() != n:
+            raise KernelError("rms_norm_sum takes contiguous float32 weights of n values")
+    _check(library().mu_rms_norm_sum(_ptr(p), p.stride(0), float(a), _ptr(wp), _ptr(q), q.stride(0), float(b), _ptr(wq),
+                                     float(eps), _ptr(out), out.stride(0), p.shape[0], n, int(add), _stream()),
+           ("rms_norm_sum(n={})", n))
     return out
 
 
@@ -489,7 +520,8 @@ def mapped_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
                      unit_rms: bool = False, tiles: Optional[torch.Tensor] = None,
                      tensor_cores: Optional[bool] = None, single_tokens: bool = False,
                      head_scale: Optional[torch.Tensor] = None, sink: bool = False,
-                     gate: Optional[torch.Tensor] = None, chunk: int = 0) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, chunk: int = 0, slopes: Optional[torch.Tensor] = None,
+                     keep: int = 0) -> torch.Tensor:
     """Softmax attention of every (token, head) over the cached rows it sees (``window`` 0: all up to its own
     position), one result per score map over the same values; with two maps a1 - lam * a2.  ``unit_rms`` brings
     each head's result to unit rms (eps inside the root); ``out_scale`` multiplies it.
@@ -502,15 +534,21 @@ def mapped_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
     ``head_scale`` (float32, one per head) multiplies the head's scores besides ``scale``; ``sink`` adds to the
     softmax's denominator one key of score zero that has no value; ``gate`` ([T, heads] view in the compute dtype)
     multiplies each head's result by sigmoid(gate[t, h]); ``chunk`` c > 0 replaces the window: position p sees
-    p - p % c .. p."""
-    _need_cuda(q, rows, block_table, tok_pos, tok_seq, out, head_scale, gate)
+    p - p % c .. p; ``slopes`` (float32, one per head): a key at distance n loses slopes[h] * n of its score;
+    ``keep`` (with a window): the sequence's first ``keep`` positions stay in sight."""
+    _need_cuda(q, rows, block_table, tok_pos, tok_seq, out, head_scale, gate, slopes)
+    if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != n_heads or not slopes.is_contiguous()):
+        raise KernelError("mapped_attention: slopes are one contiguous float32 per head")
+    if keep < 0 or (keep and chunk):
+        raise KernelError("mapped_attention: kept positions go with a window, not with chunks")
     if head_scale is not None and (head_scale.dtype != torch.float32 or head_scale.numel() != n_heads
                                    or not head_scale.is_contiguous()):
         raise KernelError("mapped_attention: head_scale is one contiguous float32 per head")
     if gate is not None and (gate.dtype != rows.dtype or gate.dim() != 2 or gate.shape != (q.shape[0], n_heads)
                              or gate.stride(1) != 1):
         raise KernelError("mapped_attention: the gate is [T, heads] in the compute dtype with unit inner stride")
-    extras = (_ptr(head_scale), int(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, int(chunk))
+    extras = (_ptr(head_scale), int(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, int(chunk),
+              _ptr(slopes), int(keep))
     for t, name in ((tok_pos, "tok_pos"), (tok_seq, "tok_seq"), (block_table, "block_table")):
         _i32(t, name)
     if (q.dtype != rows.dtype or out.dtype != rows.dtype or q.stride(1) != 1 or out.stride(1) != 1
@@ -595,18 +633,26 @@ def ssd_scan(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias, a_log, skip, n_he
 
 
 def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float,
-                     out: torch.Tensor, gate_after: bool = False) -> torch.Tensor:
+                     out: torch.Tensor, gate_after: bool = False, sigmoid: bool = False,
+                     den: Optional[torch.Tensor] = None, den_floor: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out = unit_rms_per_part(y * silu(z)) * weight, or with ``gate_after`` unit_rms_per_part(y) * weight * silu(z):
-    ``y`` float32, ``z`` and ``out`` in the compute dtype."""
-    _need_cuda(y, z, weight, out)
+    ``y`` float32, ``out`` in the compute dtype, ``z`` in that or float32.  ``sigmoid``: sigmoid(z) is the gate.
+    ``den`` (float32 [T, parts]) with ``den_floor`` ([T, parts] view of one stride): y is first divided by
+    max(|den|, den_floor) + 1e-6."""
+    _need_cuda(y, z, weight, out, den, den_floor)
     inner = y.shape[1]
-    if (y.dtype != torch.float32 or y.stride(1) != 1 or z.stride(1) != 1 or out.stride(1) != 1 or z.dtype != out.dtype
-            or z.shape != y.shape or out.shape != y.shape or weight.dtype != torch.float32 or weight.numel() != inner
-            or inner % parts):
+    if (y.dtype != torch.float32 or y.stride(1) != 1 or z.stride(1) != 1 or out.stride(1) != 1
+            or z.dtype not in (out.dtype, torch.float32) or z.shape != y.shape or out.shape != y.shape
+            or weight.dtype != torch.float32 or weight.numel() != inner or inner % parts):
         raise KernelError("gated_group_norm: inputs do not fit")
+    if den is not None and (den.dtype != torch.float32 or tuple(den.shape) != (y.shape[0], parts) or not den.is_contiguous()
+                            or den_floor is None or den_floor.dtype != torch.float32 or den_floor.shape != den.shape
+                            or (parts > 1 and y.shape[0] > 1 and den_floor.stride(0) != parts * den_floor.stride(1))):
+        raise KernelError("gated_group_norm: the divisor is contiguous float32 [T, parts], its floor a view of one stride")
     _check(library().mu_gated_group_norm(_ptr(y), y.stride(0), _ptr(z), z.stride(0), _ptr(weight), y.shape[0], inner,
                                          int(parts), float(eps), _ptr(out), out.stride(0), _is_bf16(out), _stream(),
-                                         int(gate_after)),
+                                         int(gate_after) | 2 * int(sigmoid), _is_bf16(z), _ptr(den), _ptr(den_floor),
+                                         den_floor.stride(1) if den_floor is not None else 0),
            "gated_group_norm")
     return out
 
@@ -683,23 +729,27 @@ def delta_scan_max_dk() -> int:
     return int(library().mu_delta_scan_max_dk())
 
 
-def delta_prepare(qkv: torch.Tensor, b_raw: torch.Tensor, a_raw: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
-                  n_heads: int, n_kv_heads: int, dk: int, q_scale: float, kq: torch.Tensor, beta: torch.Tensor,
-                  decay: torch.Tensor) -> None:
+def delta_prepare(qkv: torch.Tensor, b_raw: torch.Tensor, a_raw: Optional[torch.Tensor], a_log: Optional[torch.Tensor],
+                  dt_bias: Optional[torch.Tensor], n_heads: int, n_kv_heads: int, dk: int, q_scale: float,
+                  kq: torch.Tensor, beta: torch.Tensor, decay: Optional[torch.Tensor]) -> None:
     """Finishes the convolved rows ``qkv`` (float32 [T, 2 * kv heads * dk + ...]) in place: q and k of every kv head to
     unit vectors (eps 1e-6 under the root), q times ``q_scale``; ``kq`` [T, kv heads] their product; per head
-    ``beta`` = sigmoid(b_raw) and ``decay`` = exp(-exp(A_log) softplus(a_raw + dt_bias)), float32 [T, heads]."""
+    ``beta`` = sigmoid(b_raw) and, with ``a_raw``, ``decay`` = exp(-exp(A_log) softplus(a_raw + dt_bias)), float32
+    [T, heads] (None: the decays are made elsewhere)."""
     _need_cuda(qkv, b_raw, a_raw, a_log, dt_bias, kq, beta, decay)
     T = qkv.shape[0]
-    if (qkv.dtype != torch.float32 or not qkv.is_contiguous() or b_raw.dtype != a_raw.dtype or b_raw.stride(1) != 1
-            or a_raw.stride(1) != 1 or tuple(b_raw.shape) != (T, n_heads) or tuple(a_raw.shape) != (T, n_heads)):
+    if (qkv.dtype != torch.float32 or not qkv.is_contiguous() or b_raw.stride(1) != 1 or tuple(b_raw.shape) != (T, n_heads)
+            or (a_raw is not None and (b_raw.dtype != a_raw.dtype or a_raw.stride(1) != 1
+                                       or tuple(a_raw.shape) != (T, n_heads)))):
         raise KernelError("delta_prepare: rows or raw gates do not fit")
-    for t, n in ((a_log, n_heads), (dt_bias, n_heads), (kq, T * n_kv_heads), (beta, T * n_heads), (decay, T * n_heads)):
+    heads = ((a_log, n_heads), (dt_bias, n_heads), (decay, T * n_heads)) if a_raw is not None else ()
+    for t, n in ((kq, T * n_kv_heads), (beta, T * n_heads)) + heads:
         if t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous():
             raise KernelError("delta_prepare: float32 per-head parameters and outputs of the sizes given")
-    _check(library().mu_delta_prepare(_ptr(qkv), qkv.shape[1], _ptr(b_raw), b_raw.stride(0), _ptr(a_raw), a_raw.stride(0),
-                                      _ptr(a_log), _ptr(dt_bias), T, int(n_heads), int(n_kv_heads), int(dk),
-                                      float(q_scale), _ptr(kq), _ptr(beta), _ptr(decay), _is_bf16(b_raw), _stream()),
+    _check(library().mu_delta_prepare(_ptr(qkv), qkv.shape[1], _ptr(b_raw), b_raw.stride(0), _ptr(a_raw),
+                                      a_raw.stride(0) if a_raw is not None else 0, _ptr(a_log), _ptr(dt_bias), T,
+                                      int(n_heads), int(n_kv_heads), int(dk), float(q_scale), _ptr(kq), _ptr(beta),
+                                      _ptr(decay), _is_bf16(b_raw), _stream()),
            "delta_prepare")
 
 
@@ -707,21 +757,121 @@ def delta_scan(qkv: torch.Tensor, kq: torch.Tensor, beta: torch.Tensor, decay: t
                n_kv_heads: int, dk: int, dv: int, seq_first, seq_slots, state: torch.Tensor, state_offset: int,
                out: torch.Tensor) -> torch.Tensor:
     """The recurrence S = decay S; u = beta (v - S^T k); S += k u^T; o = S^T q per (sequence, head) over the step's
-    tokens, from and to ``state[slot][state_offset:]`` (heads x dv x dk float32); ``out`` float32 [T, heads * dv]."""
+    tokens, from and to ``state[slot][state_offset:]`` (heads x dv x dk float32); ``out`` float32 [T, heads * dv].
+    ``decay`` [T, heads] (one number per head) or [T, heads * dk] (one per head and key channel, acting on S's rows)."""
     _need_cuda(qkv, kq, beta, decay, seq_first, seq_slots, state, out)
     _i32(seq_first, "seq_first"); _i32(seq_slots, "seq_slots")
     T = qkv.shape[0]
+    per_channel = decay.numel() != T * n_heads or decay.shape[-1] == n_heads * dk
     if (qkv.dtype != torch.float32 or not qkv.is_contiguous() or qkv.shape[1] != 2 * n_kv_heads * dk + n_heads * dv
             or out.dtype != torch.float32 or not out.is_contiguous() or tuple(out.shape) != (T, n_heads * dv)
             or state.dtype != torch.float32 or state.stride(1) != 1
-            or state.shape[1] < state_offset + n_heads * dv * dk):
-        raise KernelError("delta_scan: rows, state or output do not fit")
+            or state.shape[1] < state_offset + n_heads * dv * dk or decay.dtype != torch.float32
+            or not decay.is_contiguous() or decay.numel() != T * n_heads * (dk if per_channel else 1)):
+        raise KernelError("delta_scan: rows, decays, state or output do not fit")
     _check(library().mu_delta_scan(_ptr(qkv), qkv.shape[1], _ptr(kq), _ptr(beta), _ptr(decay), seq_slots.numel(),
                                    int(n_heads), int(n_kv_heads), int(dk), int(dv), _ptr(seq_first), _ptr(seq_slots),
                                    _ptr(state), state.stride(0), int(state_offset), _ptr(out),
-                                   int(T > 4 * seq_slots.numel()), _stream()),
+                                   int(T > 4 * seq_slots.numel()), _stream(), int(per_channel)),
            ("delta_scan(heads={}, dk={}, dv={})", n_heads, dk, dv))
     return out
+
+
+# ------------------------------------------------------------------ linear recurrences, their gates
+def linear_scan_max_dk() -> int:
+    return int(library().mu_linear_scan_max_dk())
+
+
+def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, n_heads: int, dk: int, dv: int,
+                scale: float, seq_first, seq_slots, state: torch.Tensor, state_offset: int, out: torch.Tensor,
+                norm_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The recurrence S = decay S + take k v^T, o = scale S^T q per (sequence, head) over the step's tokens, from and
+    to ``state[slot][state_offset:]`` (heads x dv x dk float32).  ``q``, ``k``, ``v``: float32 column blocks of one
+    buffer.  ``decay`` [T, heads * dk]: one per key channel, take 1; [T, heads, 4]: (decay, take, -, -) per head.
+    ``norm_out`` [T, heads] (with [T, heads, 4] gates): the read-out of a normalizer n = decay n + take k, whose
+    heads x dk values follow S in the state."""
+    _need_cuda(q, k, v, decay, seq_first, seq_slots, state, out, norm_out)
+    _i32(seq_first, "seq_first"); _i32(seq_slots, "seq_slots")
+    T = q.shape[0]
+    per_channel = decay.dim() == 2
+    for t, n in ((q, n_heads * dk), (k, n_heads * dk), (v, n_heads * dv)):
+        if t.dtype != torch.float32 or tuple(t.shape) != (T, n) or t.stride(1) != 1 or t.stride(0) != q.stride(0):
+            raise KernelError("linear_scan: queries, keys and values are float32 column blocks of one buffer")
+    wanted = (T, n_heads * dk) if per_channel else (T, n_heads, 4)
+    values = n_heads * dk * (dv + (1 if norm_out is not None else 0))
+    if (tuple(decay.shape) != wanted or decay.dtype != torch.float32 or not decay.is_contiguous()
+            or out.dtype != torch.float32 or out.stride(1) != 1 or tuple(out.shape) != (T, n_heads * dv)
+            or state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < state_offset + values):
+        raise KernelError("linear_scan: decays, state or output do not fit")
+    if norm_out is not None and (per_channel or norm_out.dtype != torch.float32 or not norm_out.is_contiguous()
+                                 or tuple(norm_out.shape) != (T, n_heads)):
+        raise KernelError("linear_scan: the normalizer's read-out is contiguous float32 [T, heads], with gates per head")
+    _check(library().mu_linear_scan(_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), int(per_channel),
+                                    seq_slots.numel(), int(n_heads), int(dk), int(dv), float(scale), _ptr(seq_first),
+                                    _ptr(seq_slots), _ptr(state), state.stride(0), int(state_offset), _ptr(out),
+                                    out.stride(0), _ptr(norm_out), int(T > 4 * seq_slots.numel()), _stream()),
+           ("linear_scan(heads={}, dk={}, dv={})", n_heads, dk, dv))
+    return out
+
+
+def exp_gates(i_raw: torch.Tensor, f_raw: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, seq_first,
+              seq_slots, state: torch.Tensor, m_offset: int, gates: torch.Tensor) -> torch.Tensor:
+    """Exponential gates with a running maximum m (``state[slot][m_offset + h]``, starting at zero): from
+    i = cap tanh((i_raw + i_bias) / cap) and f = log sigmoid(cap tanh((f_raw + f_bias) / cap)), m = max(f + m, i), per
+    token and head ``gates`` [T, heads, 4] = (exp(f + m_before - m), exp(i - m), exp(-m), 0)."""
+    _need_cuda(i_raw, f_raw, i_bias, f_bias, seq_first, seq_slots, state, gates)
+    _i32(seq_first, "seq_first"); _i32(seq_slots, "seq_slots")
+    T, H = i_raw.shape
+    for t in (i_raw, f_raw):
+        if t.dtype != torch.float32 or tuple(t.shape) != (T, H) or t.stride(1) != 1 or t.stride(0) != i_raw.stride(0):
+            raise KernelError("exp_gates: the raw gates are float32 column blocks of one buffer")
+    if (i_bias.dtype != torch.float32 or f_bias.dtype != torch.float32 or i_bias.numel() != H or f_bias.numel() != H
+            or gates.dtype != torch.float32 or not gates.is_contiguous() or tuple(gates.shape) != (T, H, 4)
+            or state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < m_offset + H or not cap > 0.0):
+        raise KernelError("exp_gates: biases, state or output do not fit")
+    _check(library().mu_exp_gates(_ptr(i_raw), _ptr(f_raw), i_raw.stride(0), _ptr(i_bias), _ptr(f_bias), float(cap), T,
+                                  seq_slots.numel(), H, _ptr(seq_first), _ptr(seq_slots), _ptr(state), state.stride(0),
+                                  int(m_offset), _ptr(gates), _stream()), ("exp_gates(heads={})", H))
+    return gates
+
+
+class LowRankPart(ctypes.Structure):
+    """One projection of ``low_rank``; the fields are the kernel's ``LowRankPart``, in its order."""
+    _fields_ = [("w", _c_p), ("bias", _c_p), ("a_log", _c_p), ("out", _c_p), ("ldw", _c_ll), ("col", _c_int),
+                ("rank", _c_int), ("n", _c_int), ("fn", _c_int), ("per_head", _c_int), ("power", _c_f)]
+
+
+LOW_RANK_FNS = {None: 0, "sigmoid_power": 1, "exp_softplus": 2}
+
+
+def low_rank_part(weight: torch.Tensor, col: int, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                  fn: Optional[str] = None, power: float = 1.0, a_log: Optional[torch.Tensor] = None) -> LowRankPart:
+    """``out`` [T, n] float32 = fn(weight [n, rank] @ low[:, col: col + rank] + bias); ``fn``: None, ``sigmoid_power``
+    (sigmoid(z)^power) or ``exp_softplus`` (exp(-exp(a_log[head]) softplus(z)), n / heads channels a head)."""
+    _need_cuda(weight, out, bias, a_log)
+    n, rank = weight.shape
+    if weight.stride(1) != 1 or out.dtype != torch.float32 or not out.is_contiguous() or out.shape[1] != n:
+        raise KernelError("low_rank: a weight [n, rank] with unit inner stride and a contiguous float32 output [T, n]")
+    for t in (bias, a_log):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+            raise KernelError("low_rank: bias and A_log are contiguous float32")
+    if (bias is not None and bias.numel() != n) or (fn == "exp_softplus" and (a_log is None or n % a_log.numel())):
+        raise KernelError("low_rank: the bias has n values, A_log one per head")
+    return LowRankPart(_ptr(weight), _ptr(bias), _ptr(a_log), _ptr(out), weight.stride(0), int(col), int(rank), int(n),
+                       LOW_RANK_FNS[fn], n // a_log.numel() if a_log is not None else 1, float(power))
+
+
+def low_rank(low: torch.Tensor, weights_dtype: torch.dtype, *parts: LowRankPart) -> None:
+    """The second matrix of one or two projections through two matrices, with what follows it, in one launch:
+    ``low`` float32 [T, *] holds the first matrices' results, each part's from its ``col`` on."""
+    _need_cuda(low)
+    if low.dtype != torch.float32 or low.dim() != 2 or low.stride(1) != 1 or weights_dtype not in (torch.float32, torch.bfloat16):
+        raise KernelError("low_rank takes float32 rows with unit inner stride and bfloat16 or float32 weights")
+    if any(p.col + p.rank > low.shape[1] for p in parts):
+        raise KernelError("low_rank: a part's columns lie past the rows' end")
+    array = (LowRankPart * len(parts))(*parts)
+    _check(library().mu_low_rank(_ptr(low), low.stride(0), low.shape[0], ctypes.addressof(array), len(parts),
+                                 int(weights_dtype == torch.bfloat16), _stream()), ("low_rank(rank={})", parts[0].rank))
 
 
 def sigmoid_gate(o: torch.Tensor, g: torch.Tensor) -> torch.Tensor:
@@ -900,13 +1050,17 @@ def moe_group(expert_of: torch.Tensor, n_experts: int, slot_of: torch.Tensor, pa
 
 def moe_gemm(x: torch.Tensor, pair_of: Optional[torch.Tensor], top: int, w1: torch.Tensor, w2: Optional[torch.Tensor],
              tile_info: torch.Tensor, n_tiles: torch.Tensor, max_tiles: int, out: torch.Tensor,
-             tensor_cores: Optional[bool] = None, tile_rows: int = 0, act: Optional[str] = None) -> torch.Tensor:
+             tensor_cores: Optional[bool] = None, tile_rows: int = 0, act: Optional[str] = None,
+             row_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[slot] = act(W1[e] x[row]) (or silu(W1[e] x[row]) * W2[e] x[row] with ``w2``) for every slot of every expert e
     (``act``: None or ``relu2``);
     ``w1``/``w2`` [experts, n, k]; rows of ``x`` by the slot's token (``pair_of``) or by slot.  bfloat16 operands
     with 16-byte aligned rows go to the tensor cores unless ``tensor_cores`` is false.  ``tile_rows``: what
-    ``moe_group`` was given (the CUDA-core product takes its own tile only)."""
-    _need_cuda(x, pair_of, w1, w2, tile_info, n_tiles, out)
+    ``moe_group`` was given (the CUDA-core product takes its own tile only).  ``row_weight`` (float32, one per pair, or
+    per slot without ``pair_of``): the row of x is taken times it (the products are, before the activation)."""
+    _need_cuda(x, pair_of, w1, w2, tile_info, n_tiles, out, row_weight)
+    if row_weight is not None and (row_weight.dtype != torch.float32 or not row_weight.is_contiguous()):
+        raise KernelError("moe_gemm: the row weights are contiguous float32")
     if w1.dim() != 3 or not w1.is_contiguous() or w1.dtype != x.dtype or x.stride(1) != 1 or x.shape[1] != w1.shape[2]:
         raise KernelError("moe_gemm takes rows [*, k] and contiguous weights [experts, n, k] of one dtype")
     if w2 is not None and (w2.shape != w1.shape or w2.dtype != w1.dtype or not w2.is_contiguous()):
@@ -924,14 +1078,14 @@ def moe_gemm(x: torch.Tensor, pair_of: Optional[torch.Tensor], top: int, w1: tor
         _check(library().mu_moe_gemm_mma(_ptr(x), x.stride(0), _ptr(pair_of), int(top), _ptr(w1), _ptr(w2),
                                          w1.stride(0), w1.stride(1), _ptr(tile_info), _ptr(n_tiles), int(max_tiles),
                                          tile_rows, w1.shape[1], w1.shape[2], _ptr(out), out.stride(0), _is_bf16(out),
-                                         _stream(), code), ("moe_gemm_mma(n={}, k={})", w1.shape[1], w1.shape[2]))
+                                         _stream(), code, _ptr(row_weight)), ("moe_gemm_mma(n={}, k={})", w1.shape[1], w1.shape[2]))
         return out
     if tile_rows != moe_tile_rows():
         raise KernelError(f"the CUDA-core experts' product takes tiles of {moe_tile_rows()} slots, got {tile_rows}")
     _check(library().mu_moe_gemm(_ptr(x), x.stride(0), _ptr(pair_of), int(top), _ptr(w1), _ptr(w2),
                                  w1.stride(0), w1.stride(1), _ptr(tile_info), _ptr(n_tiles), int(max_tiles),
                                  w1.shape[1], w1.shape[2], _ptr(out), out.stride(0), _is_bf16(x), _is_bf16(out),
-                                 _stream(), code), ("moe_gemm(n={}, k={})", w1.shape[1], w1.shape[2]))
+                                 _stream(), code, _ptr(row_weight)), ("moe_gemm(n={}, k={})", w1.shape[1], w1.shape[2]))
     return out
 
 
@@ -962,13 +1116,13 @@ def heads_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_strid
     return out
 
 
-def moe_combine(y: torch.Tensor, slot_of: torch.Tensor, weight_of: torch.Tensor, top: int, out: torch.Tensor,
+def moe_combine(y: torch.Tensor, slot_of: torch.Tensor, weight_of: Optional[torch.Tensor], top: int, out: torch.Tensor,
                 identity_rows: Optional[torch.Tensor] = None, shared: Optional[torch.Tensor] = None,
                 shared_gate: Optional[torch.Tensor] = None, add: bool = False) -> torch.Tensor:
     """out[t] (+)= sum over the token's choices, in their order, of weight * y[slot]; float32.  A choice without a
     slot (an identity expert, slot -1) contributes weight * ``identity_rows[t]`` (the experts' input rows, compute
     dtype).  ``shared`` (float32 [T, width]) is added to every token, times ``shared_gate[t]`` if given.  ``add``:
-    the result is added to what ``out`` holds."""
+    the result is added to what ``out`` holds.  ``weight_of`` None: every choice counts once."""
     _need_cuda(y, slot_of, weight_of, out, identity_rows, shared, shared_gate)
     if y.dtype != torch.float32 or out.dtype != torch.float32 or y.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError("moe_combine works on float32 rows with unit inner stride")

@@ -13,7 +13,9 @@
 //               everything float32; head h reads B and C of group h / (heads / groups).
 // mu_gated_group_norm   y * silu(z), unit rms over each of `parts` equal parts of the row (eps inside the
 //               root), times a weight; output in the compute dtype.  With `gate_after` the order is the other
-//               one: y to unit rms per part, times the weight, times silu(z).
+//               one: y to unit rms per part, times the weight, times silu(z).  Options: sigmoid(z) as the gate;
+//               z float32 where the output is bfloat16; a divisor per token and part, applied to y first:
+//               max(|den|, floor) + 1e-6.
 #include "common.cuh"
 
 #include <math.h>
@@ -310,28 +312,40 @@ ssd_scan_cols_kernel(const float* __restrict__ xbc, int channels, const TE* __re
 }
 
 constexpr int GN_KEEP = 8;       // gated values a thread keeps between the statistics and the output
+constexpr int GN_AFTER = 1, GN_SIGMOID = 2;                  // flags of mu_gated_group_norm
 
-template <typename TE>
+__device__ __forceinline__ float gn_gate(float z, int flags) {
+    const float s = 1.0f / (1.0f + expf(-z));
+    return (flags & GN_SIGMOID) ? s : z * s;
+}
+// What y of (token, part) is multiplied by before anything else: one over the divisor, if there is one.
+__device__ __forceinline__ float gn_factor(const float* den, const float* den_floor, int floor_stride, long long item) {
+    return den ? 1.0f / (fmaxf(fabsf(den[item]), den_floor[item * floor_stride]) + 1e-6f) : 1.0f;
+}
+
+template <typename TE, typename TZ>
 __global__ void __launch_bounds__(256)
-gated_group_norm_kernel(const float* __restrict__ y, long long ldy, const TE* __restrict__ z, long long ldz,
+gated_group_norm_kernel(const float* __restrict__ y, long long ldy, const TZ* __restrict__ z, long long ldz,
                         const float* __restrict__ weight, int width, float eps, TE* __restrict__ out, long long ldo,
-                        int gate_after) {
+                        int flags, const float* __restrict__ den, const float* __restrict__ den_floor, int floor_stride) {
     __shared__ float scratch[32];
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x, part = blockIdx.y;
+    const bool gate_after = flags & GN_AFTER;
     const float* ys = y + (long long)t * ldy + (long long)part * width;
-    const TE* zs = z + (long long)t * ldz + (long long)part * width;
+    const TZ* zs = z + (long long)t * ldz + (long long)part * width;
+    const float factor = gn_factor(den, den_floor, floor_stride, (long long)t * gridDim.y + part);
     float kept[GN_KEEP];
     float sq = 0.0f;
 #pragma unroll
     for (int i = 0; i < GN_KEEP; ++i) {
         const int d = threadIdx.x + i * blockDim.x;
-        kept[i] = d < width ? (gate_after ? ys[d] : ys[d] * silu_f(to_float(zs[d]))) : 0.0f;
+        kept[i] = d < width ? factor * (gate_after ? ys[d] : ys[d] * gn_gate(to_float(zs[d]), flags)) : 0.0f;
         sq += kept[i] * kept[i];
     }
     for (int d = threadIdx.x + GN_KEEP * blockDim.x; d < width; d += blockDim.x) {
-        const float v = gate_after ? ys[d] : ys[d] * silu_f(to_float(zs[d]));
+        const float v = factor * (gate_after ? ys[d] : ys[d] * gn_gate(to_float(zs[d]), flags));
         sq += v * v;
     }
     const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)width + eps);
@@ -340,19 +354,20 @@ gated_group_norm_kernel(const float* __restrict__ y, long long ldy, const TE* __
 #pragma unroll
     for (int i = 0; i < GN_KEEP; ++i) {
         const int d = threadIdx.x + i * blockDim.x;
-        if (d < width) dst[d] = from_float<TE>(gate_after ? kept[i] * inv * w[d] * silu_f(to_float(zs[d])) : kept[i] * inv * w[d]);
+        if (d < width) dst[d] = from_float<TE>(gate_after ? kept[i] * inv * w[d] * gn_gate(to_float(zs[d]), flags) : kept[i] * inv * w[d]);
     }
     for (int d = threadIdx.x + GN_KEEP * blockDim.x; d < width; d += blockDim.x)
-        dst[d] = from_float<TE>(ys[d] * silu_f(to_float(zs[d])) * inv * w[d]);
+        dst[d] = from_float<TE>(factor * ys[d] * gn_gate(to_float(zs[d]), flags) * inv * w[d]);
 }
 
 // The same for parts of up to 32 * GN_KEEP entries (a head's values, as a rule): a warp a part, one or four parts a
 // block, no barrier; the gate and the weight are on their way before the statistics are known.
-template <typename TE>
+template <typename TE, typename TZ>
 __global__ void __launch_bounds__(128)
-gated_group_norm_warp_kernel(const float* __restrict__ y, long long ldy, const TE* __restrict__ z, long long ldz,
+gated_group_norm_warp_kernel(const float* __restrict__ y, long long ldy, const TZ* __restrict__ z, long long ldz,
                              const float* __restrict__ weight, int width, int parts, long long n_parts, float eps,
-                             TE* __restrict__ out, long long ldo, int gate_after) {
+                             TE* __restrict__ out, long long ldo, int flags, const float* __restrict__ den,
+                             const float* __restrict__ den_floor, int floor_stride) {
     pdl_trigger();
     pdl_wait();
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -360,18 +375,20 @@ gated_group_norm_warp_kernel(const float* __restrict__ y, long long ldy, const T
     const int lane = threadIdx.x & 31;
     const long long t = item / parts;
     const int part = (int)(item % parts);
+    const bool gate_after = flags & GN_AFTER;
     const float* ys = y + t * ldy + (long long)part * width;
-    const TE* zs = z + t * ldz + (long long)part * width;
+    const TZ* zs = z + t * ldz + (long long)part * width;
     const float* w = weight + (long long)part * width;
+    const float factor = gn_factor(den, den_floor, floor_stride, item);
     float kept[GN_KEEP], gate[GN_KEEP], wk[GN_KEEP];
     float sq = 0.0f;
 #pragma unroll
     for (int i = 0; i < GN_KEEP; ++i) {
         const int d = lane + 32 * i;
         const bool in = d < width;
-        gate[i] = in ? silu_f(to_float(zs[d])) : 0.0f;
+        gate[i] = in ? gn_gate(to_float(zs[d]), flags) : 0.0f;
         wk[i] = in ? w[d] : 0.0f;
-        kept[i] = in ? (gate_after ? ys[d] : ys[d] * gate[i]) : 0.0f;
+        kept[i] = in ? factor * (gate_after ? ys[d] : ys[d] * gate[i]) : 0.0f;
         sq = fmaf(kept[i], kept[i], sq);
     }
     const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)width + eps);
@@ -461,11 +478,17 @@ MU_EXPORT int mu_ssd_scan(const float* xbc, int channels, const void* dt_raw, lo
                                     seq_first, seq_slots, state, state_stride, state_offset, y);
 }
 
+// flags: 1 the gate after the norm, 2 sigmoid(z) instead of silu(z).  out is bfloat16 or float32; z is bfloat16 (with
+// a bfloat16 output only) or float32.  den (may be null) [tokens][parts], den_floor [tokens][parts] entries apart by
+// floor_stride: y is first divided by max(|den|, floor) + 1e-6.
 MU_EXPORT int mu_gated_group_norm(const float* y, long long ldy, const void* z, long long ldz, const float* weight,
                                   int n_tokens, int inner, int parts, float eps, void* out, long long ldo, int is_bf16,
-                                  void* stream, int gate_after) {
+                                  void* stream, int flags, int z_bf16, const float* den, const float* den_floor,
+                                  int floor_stride) {
     if (n_tokens <= 0) return MU_OK;
-    if (!y || !z || !weight || !out || inner <= 0 || parts <= 0 || inner % parts) return MU_ERR_BAD_ARGUMENT;
+    if (!y || !z || !weight || !out || inner <= 0 || parts <= 0 || inner % parts || (z_bf16 && !is_bf16) ||
+        (den && (!den_floor || floor_stride <= 0)))
+        return MU_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     const int width = inner / parts;
     typedef __nv_bfloat16 bf;
@@ -473,15 +496,20 @@ MU_EXPORT int mu_gated_group_norm(const float* y, long long ldy, const void* z, 
         const long long n_parts = (long long)n_tokens * parts;
         const int warps = n_parts >= 4096 ? 4 : 1;            // a few parts: a block each, spread over the SMs
         const dim3 grid((unsigned)((n_parts + warps - 1) / warps)), block(32 * warps);
-        return is_bf16 ? mu::launch_pdl(mu::gated_group_norm_warp_kernel<bf>, grid, block, 0, s, 1, y, ldy, (const bf*)z,
-                                        ldz, weight, width, parts, n_parts, eps, (bf*)out, ldo, gate_after)
-                       : mu::launch_pdl(mu::gated_group_norm_warp_kernel<float>, grid, block, 0, s, 1, y, ldy,
-                                        (const float*)z, ldz, weight, width, parts, n_parts, eps, (float*)out, ldo,
-                                        gate_after);
+#define MU_GATED_WARP(TE, TZ)                                                                                          \
+    return mu::launch_pdl(mu::gated_group_norm_warp_kernel<TE, TZ>, grid, block, 0, s, 1, y, ldy, (const TZ*)z, ldz,   \
+                          weight, width, parts, n_parts, eps, (TE*)out, ldo, flags, den, den_floor, floor_stride)
+        if (z_bf16) MU_GATED_WARP(bf, bf);
+        if (is_bf16) MU_GATED_WARP(bf, float);
+        MU_GATED_WARP(float, float);
+#undef MU_GATED_WARP
     }
     const dim3 grid(n_tokens, parts), block(width >= 1024 ? 256 : 128);
-    return is_bf16 ? mu::launch_pdl(mu::gated_group_norm_kernel<bf>, grid, block, 0, s, 1, y, ldy, (const bf*)z, ldz, weight,
-                                    width, eps, (bf*)out, ldo, gate_after)
-                   : mu::launch_pdl(mu::gated_group_norm_kernel<float>, grid, block, 0, s, 1, y, ldy, (const float*)z, ldz,
-                                    weight, width, eps, (float*)out, ldo, gate_after);
+#define MU_GATED(TE, TZ)                                                                                               \
+    return mu::launch_pdl(mu::gated_group_norm_kernel<TE, TZ>, grid, block, 0, s, 1, y, ldy, (const TZ*)z, ldz, weight, \
+                          width, eps, (TE*)out, ldo, flags, den, den_floor, floor_stride)
+    if (z_bf16) MU_GATED(bf, bf);
+    if (is_bf16) MU_GATED(bf, float);
+    MU_GATED(float, float);
+#undef MU_GATED
 }

@@ -29,10 +29,35 @@ PART_ROLES = ("embedding", "position", "norm", "mixer", "feed_forward", "head", 
 
 
 @dataclass(frozen=True)
+class FreeSize:
+    """A size that the weight file alone gives (the inner size of a projection through two matrices, say): in a
+    tensor's shape it stands for any size, the same one wherever ``name`` occurs.  ``default`` is what the
+    random-weights mode takes."""
+    name: str
+    default: int
+
+
+def shape_fits(found: Sequence[int], shape: Sequence[Any], free: Dict[str, int]) -> bool:
+    """Whether a tensor of shape ``found`` is what ``shape`` asks for; ``free`` collects the free sizes by name."""
+    if len(found) != len(shape):
+        return False
+    for n, want in zip(found, shape):
+        if isinstance(want, FreeSize):
+            want = free.setdefault(want.name, max(int(n), 1))
+        if int(n) != want:
+            return False
+    return True
+
+
+def default_shape(shape: Sequence[Any]) -> Tuple[int, ...]:
+    return tuple(n.default if isinstance(n, FreeSize) else n for n in shape)
+
+
+@dataclass(frozen=True)
 class TensorSpec:
     """One tensor a part reads from the weight file.
 
-    ``shape`` is the shape on disk.  ``role`` is ``"matrix"`` (a GEMM operand,
+    ``shape`` is the shape on disk (a size may be a ``FreeSize``).  ``role`` is ``"matrix"`` (a GEMM operand,
     kept in the compute dtype), ``"table"`` (rows gathered by an index, kept in
     the compute dtype), ``"vector"`` (bias or norm parameter, kept in 32-bit),
     ``"matrix32"`` (a small matrix whose product is always 32-bit: a router)
@@ -44,7 +69,7 @@ class TensorSpec:
     ``norm_bias``.
     """
     name: str
-    shape: Tuple[int, ...]
+    shape: Tuple[Any, ...]
     role: str = "matrix"
     transpose: bool = False
     init: str = "normal"
@@ -63,9 +88,11 @@ class KVCacheSpec:
 @dataclass(frozen=True)
 class RowCacheSpec:
     """A mixer that keeps ONE row of ``width`` values per earlier position, whatever its number of heads (a
-    compressed latent that every head reads); paged and windowed like keys and values."""
+    compressed latent that every head reads); paged and windowed like keys and values.  ``keep``: with a window, the
+    sequence's first ``keep`` positions stay as long as the sequence does."""
     width: int
     window: int = 0
+    keep: int = 0
 
 
 @dataclass(frozen=True)
@@ -198,12 +225,17 @@ class Norm(Part):
 
 
 class PositionEncoding(Part):
-    """Two hooks, either may do nothing: ``embedding_table()`` is a
+    """Three hooks, each may do nothing: ``embedding_table()`` is a
     ``[max_positions, hidden]`` table added to the token embedding by absolute
-    position, or ``None``; ``rotate(q, k, ctx)`` changes queries and keys in
-    place before keys reach the cache."""
+    position, or ``None``; ``embedding_turns()`` the frequencies of sinusoids
+    that the embedding's launch computes and adds (``ops.embed``), or ``None``;
+    ``rotate(q, k, ctx)`` changes queries and keys in place before keys reach
+    the cache."""
 
     def embedding_table(self):
+        return None
+
+    def embedding_turns(self):
         return None
 
     def rotate(self, q, k, ctx) -> None:

@@ -25,7 +25,8 @@ read and written once per sublayer.
 ``parallel_pre_norm``: x += mixer(norm1(x)) + feed_forward(norm2(x)), both sublayers reading the SAME x through a
 norm of their own.  Both norms are made before either sublayer adds into the stream (two RMS norms with one eps
 by one launch: one pass over x, one statistic, two weights); then the mixer and the feed-forward add into the
-float32 stream in their last launches.  A layer without a feed-forward is x += mixer(norm1(x)).
+float32 stream in their last launches.  A layer without a feed-forward is x += mixer(norm1(x)).  With the parameter
+``shared_norm`` there is one norm, and both sublayers read its output: x += mixer(norm1(x)) + feed_forward(norm1(x)).
 """
 from __future__ import annotations
 
@@ -200,7 +201,7 @@ class ScaledPreNormBlock(Arrangement):
     @staticmethod
     def _norm(norm, x, ctx):
         """The normed stream, with what is still to be added to the stream added by the same launch."""
-        if isinstance(norm, RmsNorm) and norm.offset == 0.0 and norm.scale == 1.0 and x.stride(1) == 1:
+        if isinstance(norm, RmsNorm) and norm.offset == 0.0 and norm.scale == 1.0 and norm.groups == 1 and x.stride(1) == 1:
             pending, ctx.pending_join = ctx.pending_join, None
             if pending is not None and pending[0] is not x:
                 ctx.pending_join = pending
@@ -214,11 +215,21 @@ class ScaledPreNormBlock(Arrangement):
 
 
 class ParallelPreNormBlock(Arrangement):
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.shared_norm = bool(self.param("shared_norm", False))
+
     def forward(self, x, layer, ctx, cache, owns_cache: bool) -> None:
         n1, n2 = layer.norm1, layer.norm2
         alone = isinstance(layer.feed_forward, NoFeedForward)
-        if (not alone and type(n1) is RmsNorm and type(n2) is RmsNorm and n1.eps == n2.eps and x.stride(1) == 1
-                and n1.offset == n2.offset == 0.0 and n1.scale == n2.scale == 1.0):
+        if self.shared_norm:
+            if type(n1) is RmsNorm:
+                h1 = n1.forward(x, out=ctx.buffer("stream.normed", tuple(x.shape), n1.runtime.dtype))
+            else:
+                h1 = n1.forward(x)
+            h2 = h1
+        elif (not alone and type(n1) is RmsNorm and type(n2) is RmsNorm and n1.eps == n2.eps and x.stride(1) == 1
+                and n1.offset == n2.offset == 0.0 and n1.scale == n2.scale == 1.0 and n1.groups == n2.groups == 1):
             dt = n1.runtime.dtype
             h1 = ctx.buffer("stream.normed", tuple(x.shape), dt)
             h2 = ctx.buffer("stream.normed2", tuple(x.shape), dt)

@@ -14,6 +14,12 @@ o is brought to unit rms over vdim, multiplied by a weight of vdim entries (the 
 silu(G x), and goes through the output matrix.  A sequence's state (the convolution's last taps - 1 inputs and every
 head's S) is float32 and lives in the sequence's cache slot; gates, decays and the recurrence are float32 whatever
 the compute dtype.
+
+Switches for other designs: ``channel_decay`` gives every head and key channel a decay of its own,
+exp(-exp(A_log_h) softplus(A2 (A1 x) + dt_bias)) with dt_bias of n_heads x dim entries, acting on the rows of S (tensors
+``decay_down``, ``decay_up`` instead of ``decay``); ``low_rank_gate`` makes the output gate's input G2 (G1 x) (tensors
+``gate_down``, ``gate_up`` instead of ``gate``); ``gate_act`` ``"sigmoid"`` gates with sigmoid instead of silu.  With
+``channel_decay`` the input product leaves float32 rows.
 """
 from __future__ import annotations
 
@@ -22,6 +28,7 @@ import torch
 from ..config.base import ConfigError, PartSpec
 from .base import Mixer, StateCacheSpec, TensorSpec, register_part
 from .linear import Linear
+from .low_rank import LowRank
 
 
 class GatedDeltaMixer(Mixer):
@@ -34,12 +41,23 @@ class GatedDeltaMixer(Mixer):
         self.n_kv_heads = int(p("n_kv_heads", self.n_heads))
         self.dim, self.vdim, self.taps = int(p("dim")), int(p("vdim")), int(p("conv"))
         self.eps = float(p("eps"))
+        self.channel_decay, self.low_rank_gate = bool(p("channel_decay", False)), bool(p("low_rank_gate", False))
+        self.gate_act = p("gate_act", "silu")
+        if self.gate_act not in ("silu", "sigmoid"):
+            raise ConfigError(f"gated delta mixer: gate_act '{self.gate_act}' is not silu or sigmoid")
+        if self.low_rank_gate and not self.channel_decay:
+            raise ConfigError("gated delta mixer: a gate through two matrices goes with decays per channel")
         if self.n_heads % self.n_kv_heads:
             raise ConfigError(f"gated delta mixer: {self.n_heads} heads do not split over {self.n_kv_heads} key heads")
         self.qk_width = self.n_kv_heads * self.dim
         self.inner = self.n_heads * self.vdim
         self.channels = 2 * self.qk_width + self.inner                        # what the convolution sees: q | k | v
         self.tail_values = (self.taps - 1) * self.channels
+        self.decays = self.n_heads * (self.dim if self.channel_decay else 1)
+        self.decay_pair = (LowRank(self, "decay_down", "decay_up", self.decays, self.hidden_size, self.dim)
+                           if self.channel_decay else None)
+        self.gate_pair = (LowRank(self, "gate_down", "gate_up", self.inner, self.hidden_size, self.vdim)
+                          if self.low_rank_gate else None)
 
     def tensor_specs(self):
         name, H, D = self.tensor_name, self.n_heads, self.hidden_size
@@ -48,11 +66,12 @@ class GatedDeltaMixer(Mixer):
                 TensorSpec(name("q_conv"), (self.qk_width, self.taps), role="vector", init="conv"),
                 TensorSpec(name("k_conv"), (self.qk_width, self.taps), role="vector", init="conv"),
                 TensorSpec(name("v_conv"), (self.inner, self.taps), role="vector", init="conv"),
-                TensorSpec(name("beta"), (H, D)), TensorSpec(name("decay"), (H, D)),
+                TensorSpec(name("beta"), (H, D)),
+                *(self.decay_pair.tensor_specs() if self.decay_pair else (TensorSpec(name("decay"), (H, D)),)),
                 TensorSpec(name("A_log"), (H,), role="vector", init="bias"),
-                TensorSpec(name("dt_bias"), (H,), role="vector", init="bias"),
+                TensorSpec(name("dt_bias"), (self.decays,), role="vector", init="bias"),
                 TensorSpec(name("norm"), (self.vdim,), role="vector", init="norm_weight"),
-                TensorSpec(name("gate"), (self.inner, D)),
+                *(self.gate_pair.tensor_specs() if self.gate_pair else (TensorSpec(name("gate"), (self.inner, D)),)),
                 TensorSpec(name("out"), (D, self.inner), init="residual_projection"))
 
     def cache_spec(self):
@@ -64,12 +83,20 @@ class GatedDeltaMixer(Mixer):
         if self.dim > runtime.ops.delta_scan_max_dk():
             raise ConfigError(f"gated delta mixer: keys of {self.dim} entries are more than the scan's "
                               f"{runtime.ops.delta_scan_max_dk()}")
-        mats = [t(r) for r in ("q", "k", "v", "gate", "beta", "decay")]
-        self.widths = [m.shape[0] for m in mats]
-        pad = -sum(self.widths) % 8
+        for pair in (self.decay_pair, self.gate_pair):
+            if pair is not None:
+                pair.bind(tensors)
+        # one product: q | k | v | gate (or its first matrix) | beta | decay (or its first matrix)
+        mats = [t("q"), t("k"), t("v"), self.gate_pair.down if self.gate_pair else t("gate"), t("beta"),
+                self.decay_pair.down if self.decay_pair else t("decay")]
+        widths = [m.shape[0] for m in mats]
+        pad = -sum(widths) % 8
         if pad:
             mats.append(torch.zeros((pad, self.hidden_size), dtype=mats[0].dtype, device=mats[0].device))
-        self.total = sum(self.widths) + pad
+            widths.append(pad)
+        self.columns = (self.channels,) + tuple(widths[3:])                  # what the convolution sees, then the rest
+        self.total = sum(widths)
+        self.proj_dtype = torch.float32 if self.channel_decay else runtime.dtype
         self.proj = Linear(torch.cat(mats, dim=0).contiguous(), None, runtime)
         self.out = Linear(t("out"), None, runtime)
         self.conv_weight = torch.cat([t("q_conv"), t("k_conv"), t("v_conv")], dim=0).contiguous()
@@ -81,23 +108,32 @@ class GatedDeltaMixer(Mixer):
         T, C, inner, H, G = ctx.n_tokens, self.channels, self.inner, self.n_heads, self.n_kv_heads
         if not owns_cache:
             raise ConfigError("a gated delta mixer keeps its own state: it cannot read another layer's")
-        u = ctx.buffer("delta.proj", (T, self.total), dt)
+        u, conv_in, gate, b_raw, a_raw = ctx.buffer("delta.proj", (T, self.total), self.proj_dtype, columns=self.columns)[:5]
         self.proj(h, out=u)
-        conv_in, gate = u[:, :C], u[:, C:C + inner]
-        b_raw, a_raw = u[:, C + inner:C + inner + H], u[:, C + inner + H:C + inner + 2 * H]
+        decay = ctx.buffer("delta.decay", (T, self.decays), torch.float32)
+        if self.channel_decay:
+            parts = [self.decay_pair.part(ops, C + gate.shape[1] + H, decay, bias=self.dt_bias, fn="exp_softplus",
+                                          a_log=self.a_log)]
+            if self.gate_pair is not None:
+                gate = ctx.buffer("delta.gate", (T, inner), torch.float32)
+                parts.append(self.gate_pair.part(ops, C, gate))
+            ops.low_rank(u, self.decay_pair.up.dtype, *parts)
         qkv = ctx.buffer("delta.qkv", (T, C), torch.float32)
         ops.ssd_conv(conv_in, self.conv_weight, None, ctx.tok_seq, ctx.seq_first, ctx.seq_slots, cache.values,
                      ctx.is_decode, qkv)
         kq = ctx.buffer("delta.kq", (T, G), torch.float32)
         beta = ctx.buffer("delta.beta", (T, H), torch.float32)
-        decay = ctx.buffer("delta.decay", (T, H), torch.float32)
-        ops.delta_prepare(qkv, b_raw, a_raw, self.a_log, self.dt_bias, H, G, self.dim, self.dim ** -0.5, kq, beta, decay)
+        if self.channel_decay:
+            ops.delta_prepare(qkv, b_raw, None, None, None, H, G, self.dim, self.dim ** -0.5, kq, beta, None)
+        else:
+            ops.delta_prepare(qkv, b_raw, a_raw, self.a_log, self.dt_bias, H, G, self.dim, self.dim ** -0.5, kq, beta, decay)
         o = ctx.buffer("delta.o", (T, inner), torch.float32)
         ops.delta_scan(qkv, kq, beta, decay, H, G, self.dim, self.vdim, ctx.seq_first, ctx.seq_slots, cache.values,
                        self.tail_values, o)
         ctx.note("scan", o)
         gated = ctx.buffer("delta.gated", (T, inner), dt)
-        ops.gated_group_norm(o, gate, self.norm_weight, H, self.eps, gated, gate_after=True)
+        ops.gated_group_norm(o, gate, self.norm_weight, H, self.eps, gated, gate_after=True,
+                             sigmoid=self.gate_act == "sigmoid")
         ctx.note("attn", gated)
         self.out(gated, residual=residual if accumulate else None, out=residual)
 

@@ -1,6 +1,6 @@
 """Token embedding: a row of the table per token (times the parameter
-``scale``, 1 if absent), plus the position table's row when the position
-encoding has one; the result is the float32 residual stream
+``scale``, 1 if absent), plus the position table's row or the sinusoids when the
+position encoding has them; the result is the float32 residual stream
 (include/ai/LocalModel.hpp:3686-3697).  Heads: ``tied_head`` (the token table
 itself) and ``linear_head`` (a matrix of its own, no bias)."""
 from __future__ import annotations
@@ -27,7 +27,8 @@ class TokenEmbedding(Embedding):
         return self.weight
 
     def forward(self, ctx, position_table):
-        return self.runtime.ops.embed(ctx.token_ids, ctx.tok_pos, self.weight, position_table, scale=self.scale)
+        return self.runtime.ops.embed(ctx.token_ids, ctx.tok_pos, self.weight, position_table, scale=self.scale,
+                                      turns=ctx.position.embedding_turns())
 
 
 class TokenPairEmbedding(Embedding):

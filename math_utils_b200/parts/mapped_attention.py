@@ -20,7 +20,11 @@ give them (no ``q_norm`` / ``k_norm`` tensors); ``rot_layout`` ``"pairs"`` turns
 of entry i with entry i + dims/2; ``chunk`` c > 0 replaces the window by chunks of c positions counted from the
 sequence's position 0 (position p sees p - p % c .. p; the cache keeps everything); ``head_gate`` multiplies head
 h's result by sigmoid(G x)_h, one number per head from the mixer's own input (tensor ``gate`` [heads, hidden], no
-bias), before the output projection.
+bias), before the output projection; ``qk_norm`` ``"unit"`` norms queries and keys without a weight; ``rot`` None
+rotates nothing; ``key_values`` makes the projected keys, as they are before their norm, the values too (no ``v``
+tensor; vdim equals dim); ``slopes``: ``"geometric"`` takes slope_h * distance off every score,
+slope_h = 2^(-8 (h + 1) / n_heads); ``keep`` n > 0, with a window, leaves the sequence's first n positions in sight of
+every later token (the cache keeps them).
 """
 from __future__ import annotations
 
@@ -47,7 +51,18 @@ class MappedAttention(Mixer):
         self.own_kv = bool(p("own_kv", True))
         self.bias = bool(p("bias", False))
         self.diff = float(p("diff", 0.0))
-        self.qk_norm = bool(p("qk_norm", True))
+        self.qk_norm = p("qk_norm", True)
+        self.key_values = bool(p("key_values", False))
+        self.slopes = p("slopes", None)
+        self.keep = int(p("keep", 0))
+        if self.qk_norm not in (True, False, "unit"):
+            raise ConfigError(f"mapped attention: qk_norm '{self.qk_norm}' is not true, false or 'unit'")
+        if self.key_values and (self.dim != self.vdim or self.maps != 1 or not self.own_kv):
+            raise ConfigError("mapped attention: keys that are the values too have the values' size and one score map")
+        if self.slopes not in (None, "geometric"):
+            raise ConfigError(f"mapped attention: slopes '{self.slopes}' is not 'geometric'")
+        if self.keep and (not self.window or self.cache_window != self.window):
+            raise ConfigError("mapped attention: kept positions go with a window of the layer's own")
         self.rot_layout = p("rot_layout", "half")
         self.chunk = int(p("chunk", 0))
         self.head_gate = bool(p("head_gate", False))
@@ -61,7 +76,7 @@ class MappedAttention(Mixer):
             raise ConfigError(f"mapped attention: {self.n_heads} heads do not split over {self.n_kv_heads} kv heads")
         if self.window and self.cache_window and self.cache_window < self.window:
             raise ConfigError("mapped attention: the cache keeps fewer positions than the window sees")
-        rot = p("rot")
+        rot = p("rot") or {"dims": 0, "base": 1.0}
         self.rot_dims = int(rot["dims"])
         if self.rot_dims > self.dim or self.rot_dims % 2:
             raise ConfigError(f"mapped attention: {self.rot_dims} rotated entries do not fit a map of {self.dim}")
@@ -73,14 +88,16 @@ class MappedAttention(Mixer):
     def tensor_specs(self):
         D, name = self.hidden_size, self.tensor_name
         specs = [TensorSpec(name("q"), (self.q_width, D))]
-        if self.qk_norm:
+        if self.qk_norm is True:
             specs.append(TensorSpec(name("q_norm"), (self.dim,), role="vector", init="norm_weight"))
         widths = [("q_bias", self.q_width)]
         if self.own_kv:
-            specs += [TensorSpec(name("k"), (self.k_width, D)), TensorSpec(name("v"), (self.v_width, D))]
-            if self.qk_norm:
+            specs.append(TensorSpec(name("k"), (self.k_width, D)))
+            if not self.key_values:
+                specs.append(TensorSpec(name("v"), (self.v_width, D)))
+            if self.qk_norm is True:
                 specs.append(TensorSpec(name("k_norm"), (self.dim,), role="vector", init="norm_weight"))
-            widths += [("k_bias", self.k_width), ("v_bias", self.v_width)]
+            widths += [("k_bias", self.k_width)] + ([] if self.key_values else [("v_bias", self.v_width)])
         if self.head_gate:
             specs.append(TensorSpec(name("gate"), (self.n_heads, D)))
         specs.append(TensorSpec(name("out"), (D, self.n_heads * self.vdim), init="residual_projection"))
@@ -92,12 +109,12 @@ class MappedAttention(Mixer):
         return specs
 
     def cache_spec(self):
-        return RowCacheSpec(self.k_width + self.v_width, self.cache_window)
+        return RowCacheSpec(self.k_width + self.v_width, self.cache_window, self.keep)
 
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
         t = lambda role: tensors[self.tensor_name(role)]
-        roles = ["q"] + (["k", "v"] if self.own_kv else [])
+        roles = ["q"] + ((["k"] if self.key_values else ["k", "v"]) if self.own_kv else [])
         mats = [t(r) for r in roles]
         biases = [t(r + "_bias") for r in roles] if self.bias else None
         self.gate_at = None
@@ -116,8 +133,16 @@ class MappedAttention(Mixer):
         self.widths = tuple(m.shape[0] for m in mats)
         self.proj = Linear(weight, bias, runtime)
         self.out = Linear(t("out"), t("out_bias") if self.bias else None, runtime)
-        self.q_norm = t("q_norm") if self.qk_norm else None
-        self.k_norm = t("k_norm") if self.own_kv and self.qk_norm else None
+        if self.qk_norm == "unit":
+            self.q_norm = torch.ones(self.dim, dtype=torch.float32, device=runtime.device)
+            self.k_norm = self.q_norm if self.own_kv else None
+        else:
+            self.q_norm = t("q_norm") if self.qk_norm else None
+            self.k_norm = t("k_norm") if self.own_kv and self.qk_norm else None
+        self.slope_table = None
+        if self.slopes:
+            self.slope_table = torch.tensor([2.0 ** (-8.0 * (h + 1) / self.n_heads) for h in range(self.n_heads)],
+                                            dtype=torch.float32, device=runtime.device)
         self.freq_table = torch.tensor(self.freqs or [0.0], dtype=torch.float64).to(torch.float32).to(runtime.device)
         self.lam, self.out_scale = 0.0, 1.0
         if self.maps == 2:
@@ -134,7 +159,7 @@ class MappedAttention(Mixer):
         views = ctx.buffer("mapped.proj" if self.own_kv else "mapped.proj_q", (T, sum(self.widths)), dt, columns=self.widths)
         self.proj(h, out=views[0])
         q = views[1]
-        k, v = (views[2], views[3]) if owns_cache else (None, None)
+        k, v = (views[2], views[2 if self.key_values else 3]) if owns_cache else (None, None)
         gate = views[self.gate_at] if self.gate_at is not None else None
         table = ctx.block_tables[cache.group]
         ops.qk_prepare(q, k, v, self.q_norm, self.k_norm, self.freq_table, self.magnitude, self.rot_dims, self.eps,
@@ -147,7 +172,7 @@ class MappedAttention(Mixer):
                              self.n_kv_heads, self.maps, self.dim, self.vdim, self.scale, self.window, heads,
                              lam=self.lam, out_scale=self.out_scale, eps=self.eps, unit_rms=self.maps == 2,
                              tiles=None if ctx.is_decode else ctx.q_tiles, single_tokens=ctx.is_decode,
-                             gate=gate, chunk=self.chunk)
+                             gate=gate, chunk=self.chunk, slopes=self.slope_table, keep=self.keep)
         ctx.note("attn", heads)
         self.out(heads, residual=residual if accumulate else None, out=residual)
 

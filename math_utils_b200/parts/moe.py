@@ -13,7 +13,8 @@ correction have ``n_experts + identity`` rows); ``renorm_eps`` is added to the c
 division; ``shared`` = {``inner_size``, ``gate``: bool} adds an expert of the same form that every token
 passes through (tensors ``shared_up``, ``shared_down``, with ``expert_form`` gated also ``shared_gate_proj``),
 its result multiplied, with ``gate`` true, by sigmoid(g . h), one number per token (tensor ``shared_gate``
-[1, hidden]).
+[1, hidden]); ``weight_on`` ``"input"`` lets a choice's weight w act on what the expert reads, expert(w h), instead of
+on its result.
 
 Router logits, scores and weights are float32.  The (token, expert) pairs are grouped by expert on the
 device, each expert's products run over its own rows only, and the results are summed per token in the
@@ -42,12 +43,17 @@ class RoutedExperts(FeedForward):
         self.form = p("expert_form", "gated_silu")
         self.identity = int(p("identity", 0))
         self.renorm_eps = float(p("renorm_eps", 0.0))
+        self.weight_on = p("weight_on", "output")
+        if self.weight_on not in ("input", "output"):
+            raise ConfigError(f"routed_experts: weight_on '{self.weight_on}' is not input or output")
         shared = p("shared", None)
         self.shared_inner = int(shared["inner_size"]) if shared else 0
         self.shared_gated = bool(shared.get("gate", False)) if shared else False
         self.n_outputs = self.n_experts + self.identity          # what the router chooses among
         if self.form not in ("gated_silu", "relu2"):
             raise ConfigError(f"routed_experts: expert_form '{self.form}' is not gated_silu or relu2")
+        if self.identity and self.weight_on == "input":
+            raise ConfigError("routed_experts: identity experts take their weight on the output")
         if self.identity < 0:
             raise ConfigError("routed_experts: identity counts the identity experts, 0 or more")
         if self.score not in ("sigmoid", "softmax"):
@@ -121,11 +127,15 @@ class RoutedExperts(FeedForward):
                       n_real=E if self.identity else 0)
         ctx.note("route", weight_of)
         hidden = ctx.buffer("moe.hidden", (P, self.inner_size), dt)
+        row_weight = None
+        if self.weight_on == "input":
+            row_weight, weight_of = weight_of, None              # the first product takes the weights, the sum none
         if gated:
-            ops.moe_gemm(h, pair_of, top, self.w_gate, self.w_up, tile_info, n_tiles, max_tiles, hidden, tile_rows=tile_rows)
+            ops.moe_gemm(h, pair_of, top, self.w_gate, self.w_up, tile_info, n_tiles, max_tiles, hidden, tile_rows=tile_rows,
+                         row_weight=row_weight)
         else:
             ops.moe_gemm(h, pair_of, top, self.w_up, None, tile_info, n_tiles, max_tiles, hidden, tile_rows=tile_rows,
-                         act="relu2")
+                         act="relu2", row_weight=row_weight)
         ctx.note("act", hidden)
         y = ctx.buffer("moe.out", (P, self.hidden_size), torch.float32)
         ops.moe_gemm(hidden, None, top, self.w_down, None, tile_info, n_tiles, max_tiles, y, tile_rows=tile_rows)
@@ -153,19 +163,15 @@ class RoutedExperts(FeedForward):
         if output_norm is not None:
             # residual += norm(sum of the token's experts); Dynamic Tanh in the same launch as the sum
             from .norm import DynamicTanh
-            if type(output_norm) is DynamicTanh:
+            if type(output_norm) is DynamicTanh and weight_of is not None:
                 ops.moe_combine_tanh(y, slot_of, weight_of, top, output_norm.weight, output_norm.bias, output_norm.alpha,
                                      residual)
             else:
                 mixed = ctx.buffer("moe.mixed", (T, self.hidden_size), torch.float32)
                 ops.moe_combine(y, slot_of, weight_of, top, mixed)
                 output_norm.add_into(mixed, residual)
-        elif accumulate:
-            mixed = ctx.buffer("moe.mixed", (T, self.hidden_size), torch.float32)
-            ops.moe_combine(y, slot_of, weight_of, top, mixed)
-            residual += mixed
         else:
-            ops.moe_combine(y, slot_of, weight_of, top, residual)
+            ops.moe_combine(y, slot_of, weight_of, top, residual, add=accumulate)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts, replace=True)

@@ -8,10 +8,12 @@ mean, no variance, no eps.  Tensors ``weight``, ``bias``, ``alpha`` (a scalar).
 
 ``rms_norm``: scale * x / sqrt(mean(x^2) + eps) * (weight_offset + weight), statistics in float32.
 ``weight_offset`` (0 unless given; 1 for a weight stored around zero) and ``scale`` (1 unless given:
-the multiplier with which a normed sublayer output joins the residual stream) are parameters."""
+the multiplier with which a normed sublayer output joins the residual stream) are parameters, and so is
+``groups`` (1 unless given): the row in that many consecutive equal parts, each divided by its own rms, times one
+weight for the whole row."""
 from __future__ import annotations
 
-from ..config.base import PartSpec
+from ..config.base import ConfigError, PartSpec
 from .base import Norm, TensorSpec, register_part
 
 
@@ -71,6 +73,9 @@ class RmsNorm(Norm):
         self.eps = float(self.param("eps"))
         self.offset = float(self.param("weight_offset", 0.0))
         self.scale = float(self.param("scale", 1.0))
+        self.groups = int(self.param("groups", 1))
+        if self.groups < 1 or self.size % self.groups:
+            raise ConfigError(f"rms_norm: {self.size} entries do not split into {self.groups} equal groups")
 
     def tensor_specs(self):
         return (TensorSpec(self.tensor_name("weight"), (self.size,), role="vector",
@@ -80,18 +85,18 @@ class RmsNorm(Norm):
         super().bind(tensors, runtime)
         self.weight = tensors[self.tensor_name("weight")]
 
-    def forward(self, x, rows=None):
-        return self.runtime.ops.rms_norm_out(x, self.weight, self.eps, self.offset, self.scale,
-                                             out_dtype=self.runtime.dtype, rows=rows)
+    def forward(self, x, rows=None, out=None):
+        return self.runtime.ops.rms_norm_out(x, self.weight, self.eps, self.offset, self.scale, out=out,
+                                             out_dtype=self.runtime.dtype, rows=rows, groups=self.groups)
 
     def forward_float(self, x, out=None):
-        return self.runtime.ops.rms_norm_out(x, self.weight, self.eps, self.offset, self.scale, out=out)
+        return self.runtime.ops.rms_norm_out(x, self.weight, self.eps, self.offset, self.scale, out=out, groups=self.groups)
 
     def add_into(self, y, residual, copy=None, second=None) -> None:
         """residual += norm(y); ``copy`` (bfloat16, shaped like the stream) receives the stream as it then is;
         ``second`` = (a, y2, b): the norm's input is a * y + b * y2."""
         self.runtime.ops.rms_norm_out(y, self.weight, self.eps, self.offset, self.scale, out=residual, add=True,
-                                      copy=copy, second=second)
+                                      copy=copy, second=second, groups=self.groups)
 
 
 register_part("norm", "layer_norm", LayerNorm, replace=True)

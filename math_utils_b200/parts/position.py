@@ -4,6 +4,9 @@
 token's absolute position is added to its embedding
 (include/ai/LocalModel.hpp:3694-3697); queries and keys are left as they are.
 
+``sinusoidal``: entry 2i of a token's embedding gets sin(p f_i), entry 2i + 1 cos(p f_i), f_i = base^(-2i / hidden),
+p the token's absolute position; computed by the embedding's launch, so no table bounds the positions.
+
 ``rotary_frequencies``: the frequency table of a rotary encoding, plain or
 stretched for long contexts; the mixers that rotate their own queries and keys
 hand it to ``ops.rotary``.
@@ -31,11 +34,33 @@ class LearnedAbsolutePositions(PositionEncoding):
         return self.weight
 
 
+class SinusoidalPositions(PositionEncoding):
+    """Parameters ``hidden_size`` and ``base``.  The frequencies are kept in turns per position, each as a float32 and
+    what its rounding left, so that the kernel finds the fraction of a turn at far positions too."""
+
+    def __init__(self, spec: PartSpec):
+        super().__init__(spec)
+        self.hidden_size = int(self.param("hidden_size"))
+        self.base = float(self.param("base"))
+
+    def bind(self, tensors, runtime):
+        super().bind(tensors, runtime)
+        import torch
+        i = torch.arange((self.hidden_size + 1) // 2, dtype=torch.float64)
+        turns = self.base ** (-2.0 * i / self.hidden_size) / (2.0 * torch.pi)
+        head = turns.to(torch.float32)
+        self.turns = torch.stack([head, (turns - head.double()).to(torch.float32)]).contiguous().to(runtime.device)
+
+    def embedding_turns(self):
+        return self.turns
+
+
 class NoPositions(PositionEncoding):
     """Nothing is added and nothing is rotated."""
 
 
 register_part("position", "learned_absolute", LearnedAbsolutePositions, replace=True)
+register_part("position", "sinusoidal", SinusoidalPositions, replace=True)
 register_part("position", "none", NoPositions, replace=True)
 
 

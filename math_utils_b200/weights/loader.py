@@ -19,7 +19,7 @@ from typing import Dict, Iterable, List, Mapping, Sequence
 
 import torch
 
-from ..parts.base import TensorSpec
+from ..parts.base import FreeSize, TensorSpec, shape_fits
 from .safetensors import SafetensorsError, SafetensorsFile
 
 
@@ -85,7 +85,7 @@ def load_weights(model_dir: str, specs: Sequence[TensorSpec], compute_dtype: tor
                     raise WeightError(model_dir, other=[f"tensor '{s.name}' is asked for with two shapes"])
             wanted.setdefault(s.name, s)
 
-        missing, wrong = [], []
+        missing, wrong, free = [], [], {}
         for name, s in wanted.items():
             f = where_of.get(prefix + name)
             if f is None:
@@ -93,8 +93,10 @@ def load_weights(model_dir: str, specs: Sequence[TensorSpec], compute_dtype: tor
                     missing.append(prefix + name)
                 continue
             found = f.tensors[prefix + name].shape
-            if tuple(found) != tuple(s.shape):
-                wrong.append((prefix + name, found, s.shape))
+            if not shape_fits(found, s.shape, free):
+                # (a size the file gives reads as what the tensors before said, or as '*')
+                wrong.append((prefix + name, found, tuple(free.get(n.name, "*") if isinstance(n, FreeSize) else n
+                                                          for n in s.shape)))
         unexpected = []
         for n in where_of:
             base = n[len(prefix):] if n.startswith(prefix) else None

@@ -21,6 +21,7 @@ import numpy as np
 import torch
 
 from ..config.registry import architecture_for
+from ..parts.base import default_shape
 from .safetensors import write_safetensors
 
 _MASK = (1 << 64) - 1
@@ -53,7 +54,7 @@ def random_tensors(config, plan, seed: int, store_dtype: torch.dtype) -> Dict[st
             continue
         mean, std = config.init_distribution(spec.init)
         rng = tensor_generator(seed, spec.name)
-        values = rng.standard_normal(size=spec.shape, dtype=np.float32)
+        values = rng.standard_normal(size=default_shape(spec.shape), dtype=np.float32)
         values = values * np.float32(std) + np.float32(mean)
         if spec.role == "int_table":
             raise ValueError(f"tensor '{spec.name}': no random rule for integer tables")
