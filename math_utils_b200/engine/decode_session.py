@@ -28,7 +28,9 @@ Three ways to drive it:
 """
 from __future__ import annotations
 
+import contextlib
 import dataclasses
+import gc
 from typing import List, Optional, Sequence
 
 import numpy as np
@@ -36,6 +38,19 @@ import torch
 
 from ..sampling import SamplingParams
 from .batch import StepContext
+
+
+@contextlib.contextmanager
+def _no_collection():
+    """Holds the garbage collector off while a graph is recorded: a collection in the middle could destroy another
+    model's dropped graphs, which a stream that is recording does not survive."""
+    was = gc.isenabled()
+    gc.disable()
+    try:
+        yield
+    finally:
+        if was:
+            gc.enable()
 
 
 class DecodeSession:
@@ -271,7 +286,7 @@ class DecodeSession:
             pool = torch.cuda.graph_pool_handle()
             keeper = torch.cuda.CUDAGraph()
             side.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(side):
+            with torch.cuda.stream(side), _no_collection():
                 keeper.capture_begin(pool=pool)
                 try:
                     held = torch.zeros(16, dtype=torch.int32, device=self.model.runtime.device)
@@ -280,7 +295,7 @@ class DecodeSession:
             self.model.__dict__["_graph_pool_keeper"] = (keeper, held)
             self.model.__dict__["_graph_pool"] = pool
         side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
+        with torch.cuda.stream(side), _no_collection():
             graph.capture_begin(pool=pool)
             try:
                 body()
