@@ -8,6 +8,7 @@
     python bench.py --family lusalorn [--size s|m] [--batch B] [--steps K]  # Lusalorn beside GPT-2 at equal size
     python bench.py --family seledra [--size s|m] [--batch B] [--steps K]   # Seledra beside Lusalorn at equal size
     python bench.py --family tibopel [--size s|m] [--batch B] [--steps K]   # Tibopel beside Forisun at equal size
+    python bench.py --family pelenex [--size s|m] [--batch B] [--steps K]   # Pelenex beside Seledra, Lusalorn and Tibopel
 
 A "step" is one decode step of the whole batch.  The default run has the layer
 sizes of GPT-2 small (BASELINE.json's third configuration) with seeded random
@@ -571,6 +572,35 @@ def tibopel_config(size):
     return ours, forisun_config(size)[0]
 
 
+PELENEX_SIZES = {
+    # width, delta rule (heads, key heads, dim, vdim, taps), matrix LSTM (heads, dim, vdim), attention (heads, kv heads, dim,
+    # window, kept), linear attention (heads, dim, vdim), dense ff, experts (experts, top, expert ff, shared ff)
+    "s": (1024, (8, 4, 128, 128, 4), (8, 128, 128), (8, 2, 128, 512, 16), (8, 128, 128), 4096, (16, 4, 512, 1024)),
+    "m": (2048, (16, 8, 128, 128, 4), (16, 128, 128), (16, 4, 128, 512, 16), (16, 128, 128), 8192, (64, 6, 1408, 2816)),
+}
+
+
+def pelenex_config(size):
+    """A Pelenex configuration with layer sizes of a real model's order (random weights): a layer of the delta rule
+    with a decay per channel, a matrix LSTM with routed experts, attention beside linear attention, a second matrix
+    LSTM with routed experts; and beside it the three designs its layers are like, each at its own configuration of
+    this size (equal width, layer count and vocabulary): Seledra (the delta rule), Lusalorn (windowed attention, a
+    recurrent mixer beside attention, a gated feed-forward), Tibopel (routed experts beside a shared one)."""
+    D, (H, G, d, dv, taps), (mh, md, mv), (ah, ag, ad, window, kept), (lh, ld, lv), ff, (E, top, eff, shared) = PELENEX_SIZES[size]
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}, "shared": {"ff": shared}}
+    lstm = {"type": "mlstm", "mixer": {"heads": mh, "dim": md, "vdim": mv, "gate_cap": 15.0}, "mlp": moe}
+    layers = [{"type": "channel_delta", "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": dv, "conv": taps}, "mlp": dense},
+              lstm,
+              {"type": "parallel", "mixer": {"left": {"heads": ah, "kv_heads": ag, "dim": ad, "vdim": ad, "scale": ad ** -0.5,
+                                                      "mask": {"size": window, "keep_first": kept}},
+                                             "right": {"heads": lh, "dim": ld, "vdim": lv, "tau": 8.0}}, "mlp": dense},
+              lstm]
+    ours = {"architecture": "Pelenex", "vocab": FAMILY_VOCAB, "width": D, "norm": {"eps": 1e-5, "groups": 4},
+            "logit_softcap": 30.0, "layers": layers}
+    return ours, seledra_config(size)[0], lusalorn_config(size)[0], tibopel_config(size)[0]
+
+
 def stage_times(model, prompts, single_steps=8):
     """Device milliseconds per stage of one eager prompt step and of eager single-token steps (their mean)."""
     import torch
@@ -594,19 +624,21 @@ def stage_times(model, prompts, single_steps=8):
 
 
 def run_family(args):
-    """``--family forisun | lusalorn | seledra | tibopel``: prompt and single-token throughput of that design at sizes of a real
-    model's order beside GPT-2 (Seledra: beside Lusalorn; Tibopel: beside Forisun) at equal size, the same workload shape as the default run (2 x 1,024-token prompts; a batch from
+    """``--family forisun | lusalorn | seledra | tibopel | pelenex``: prompt and single-token throughput of that design at
+    sizes of a real model's order beside GPT-2 (Seledra: beside Lusalorn; Tibopel: beside Forisun; Pelenex: beside the
+    three it is like) at equal size, the same workload shape as the default run (2 x 1,024-token prompts; a batch from
     512-token prompts towards 1,024).  Prints one JSON line; the default run and its line are not touched."""
     import numpy as np
     from math_utils_b200.sampling import SamplingParams
     pk = peaks()
     rng = np.random.default_rng(0)
     configs = {"forisun": forisun_config, "lusalorn": lusalorn_config, "seledra": seledra_config,
-               "tibopel": tibopel_config}[args.family](args.size)
-    other = {"seledra": "lusalorn_twin", "tibopel": "forisun_twin"}.get(args.family, "gpt2_twin")
+               "tibopel": tibopel_config, "pelenex": pelenex_config}[args.family](args.size)
+    others = {"seledra": ("lusalorn_twin",), "tibopel": ("forisun_twin",),
+              "pelenex": ("seledra_twin", "lusalorn_twin", "tibopel_twin")}.get(args.family, ("gpt2_twin",))
     record = {"family": args.family, "size": args.size, "batch": args.batch, "steps": args.steps, "dtype": "bfloat16",
               "data": "synthetic: random weights, random tokens", "peaks": pk, "models": {}}
-    for name, cfg in zip((args.family, other), configs):
+    for name, cfg in zip((args.family,) + others, configs):
         llm = load_random(cfg, temperature=0.0, context=CONTEXT)
         model = llm.model
         pre = [rng.integers(0, FAMILY_VOCAB, size=CONTEXT).tolist() for _ in range(PREFILL_SEQS)]
@@ -790,9 +822,9 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="with --only decode: tokens per prompt")
     ap.add_argument("--reference-dir", default="", help="with --impl reference: a checkout other than baseline/_ref")
     ap.add_argument("--tokens", type=int, default=0, help="with --config: fewer tokens per request than fill the context")
-    ap.add_argument("--family", default="", choices=["", "forisun", "lusalorn", "seledra", "tibopel"],
+    ap.add_argument("--family", default="", choices=["", "forisun", "lusalorn", "seledra", "tibopel", "pelenex"],
                     help="that design at sizes of a real model's order beside GPT-2 (seledra: beside Lusalorn; tibopel: "
-                         "beside Forisun) at equal size")
+                         "beside Forisun; pelenex: beside Seledra, Lusalorn and Tibopel) at equal size")
     ap.add_argument("--size", default="s", choices=sorted(FORISUN_SIZES), help="with --family: which sizes")
     args = ap.parse_args()
     if args.gpus != 1:

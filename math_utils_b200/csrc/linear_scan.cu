@@ -2,17 +2,18 @@
 //     S <- decay S + take k v^T,   o = scale * S^T q,
 // and the gates they take.  Everything float32.
 //
-// mu_linear_scan   per (sequence, head, 16 columns of S), the step's tokens in order.  The decay is one number per
+// mu_linear_scan   per (sequence, head, a few columns of S), the step's tokens in order.  The decay is one number per
 //                  head (with a `take` beside it) or one per head and key channel (gated linear attention).  With a
 //                  normalizer the state has one more column, n <- decay n + take k, whose read-out n . q goes to an
 //                  array of its own (the matrix memory of xLSTM).  State of a slot, from state_offset on:
 //                  [ S: heads x dv x dk (a head's S column after column) | n: heads x dk ].
-//                  A column lives in the registers of 8 lanes, two entries to a 64-bit register.  Nothing waits for
-//                  a token's read-out, so the lanes keep their partial sums of 8 tokens and add them crosswise: 7
-//                  exchanges for 8 tokens, after which lane i holds token i's sum.  Keys, queries, decays and values
-//                  of 16 tokens at a time are copied to shared memory asynchronously, the next 16 on their way
-//                  meanwhile.  The order of every sum is fixed by dk alone: a token's result does not depend on how
-//                  the sequence was cut into steps or on the batch.
+//                  Four columns live in the registers of up to 32 lanes, two entries to a 64-bit register; a key, a
+//                  query and a decay read from shared memory serve four columns.  Nothing waits for a token's
+//                  read-out, so the lanes keep their partial sums of as many (token, column) pairs as there are lanes
+//                  and add them crosswise: 31 exchanges for 8 tokens of 4 columns over 32 lanes, after which every lane
+//                  holds one finished sum.  Keys, queries, decays and values of 16 tokens at a time are copied to
+//                  shared memory asynchronously, the next 16 on their way meanwhile.  The order of every sum is fixed
+//                  by dk alone: a token's result does not depend on how the sequence was cut into steps or on the batch.
 // mu_exp_gates     the exponential gates of such a memory: i = cap tanh((i_raw + i_bias) / cap),
 //                  f = log sigmoid(cap tanh((f_raw + f_bias) / cap)), a running maximum m <- max(f + m, i) that starts
 //                  at zero and stays with the sequence's state; per token and head (decay, take, floor) =
@@ -20,6 +21,7 @@
 //                  maximum is kept changes no result; it is found for 256 tokens at a time by a scan.
 // mu_low_rank      out[t][c] = fn( sum_r W[c][r] low[t][r] + bias[c] ): the second of a projection's two matrices, for
 //                  one or two such projections in one launch, with what follows it:
+//                  (bfloat16 weights and many tokens: tensor cores, else one running sum per output over r.)
 //                  fn 0: nothing;  1: sigmoid(z)^power;  2: exp(-exp(A_log[c / per_head]) softplus(z)).
 #include "common.cuh"
 
@@ -27,113 +29,102 @@
 
 namespace mu {
 
-constexpr int LS_COLS = 16;       // columns a block takes
-constexpr int LS_LANES = 8;       // lanes a column
+constexpr int LS_THREADS = 128;
+constexpr int LS_PER = 4;         // columns of S whose entries a lane holds
 constexpr int LS_CHUNK = 16;      // tokens staged at a time
-constexpr int LS_GROUP = 8;       // tokens whose read-outs are summed together (= LS_LANES)
 constexpr int LS_MAX_DK = 256;
 
+// Columns a block takes: LANES lanes share four columns.
+__host__ __device__ constexpr int ls_columns(int lanes) { return LS_PER * LS_THREADS / lanes; }
 // Floats of one staged chunk: keys, queries (and the channels' decays), values, (decay, take, floor, -).
-__host__ __device__ constexpr int ls_chunk_floats(int dkp, bool per_channel) {
-    return LS_CHUNK * ((per_channel ? 3 : 2) * dkp + LS_COLS + 4);
+__host__ __device__ constexpr int ls_chunk_floats(int dkp, int cols, bool per_channel) {
+    return LS_CHUNK * ((per_channel ? 3 : 2) * dkp + cols + 4);
 }
 
-// One token of a lane's R entries: S = g S + k v, and the lane's share of S . q.
-template <int R, bool PER_CHANNEL>
-__device__ __forceinline__ float ls_step(float2x (&S)[R / 2], const float* __restrict__ k, const float* __restrict__ q,
-                                         const float* __restrict__ g, float decay, float v, int l) {
-    const float2x v2 = pair_of_floats(v, v), d2 = pair_of_floats(decay, decay);
-    float2x a = 0, b = 0;                                    // (two zeros each)
-#pragma unroll
-    for (int i = 0; i < R / 4; ++i) {
-        const int at = 4 * (l + LS_LANES * i);
-        const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(k + at);
-        const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(q + at);
-        ulonglong2 gg = make_ulonglong2(d2, d2);
-        if (PER_CHANNEL) gg = *reinterpret_cast<const ulonglong2*>(g + at);
-        S[2 * i] = pair_fma(kk.x, v2, pair_mul(gg.x, S[2 * i]));
-        S[2 * i + 1] = pair_fma(kk.y, v2, pair_mul(gg.y, S[2 * i + 1]));
-        a = pair_fma(S[2 * i], qq.x, a);
-        b = pair_fma(S[2 * i + 1], qq.y, b);
-    }
-    const float2 x = floats_of_pair(a), y = floats_of_pair(b);
-    return (x.x + x.y) + (y.x + y.y);
-}
-
-// R: entries of a column that a lane holds (a multiple of 4); dk <= 8 R, dealt to the lanes four entries at a time.
-// VEC: every row, slice and state column starts on a 16-byte boundary.
-template <int R, bool VEC, bool PER_CHANNEL>
-__global__ void __launch_bounds__(LS_LANES * LS_COLS)
+// LANES lanes hold four columns of S, R entries of each a lane (a multiple of 4; dk <= LANES R), dealt to the lanes
+// four entries at a time: what a lane reads of a staged key, query and decay serves its four columns.  LANES and R
+// follow from dk alone.  VEC: every row, slice and state column starts on a 16-byte boundary.
+template <int R, int LANES, bool VEC, bool PER_CHANNEL>
+__global__ void __launch_bounds__(LS_THREADS)
 linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, long long ld,
                    const float* __restrict__ decay, int n_heads, int dk, int dv, float scale,
                    const int* __restrict__ seq_first, const int* __restrict__ seq_slots, float* __restrict__ state,
                    long long state_stride, long long state_offset, float* __restrict__ out, long long ldo,
                    float* __restrict__ norm_out) {
-    constexpr int DKP = LS_LANES * R, Q = R / 4, BUF = ls_chunk_floats(DKP, PER_CHANNEL), THREADS = LS_LANES * LS_COLS;
+    constexpr int DKP = LANES * R, Q = R / 4, COLS = ls_columns(LANES), BUF = ls_chunk_floats(DKP, COLS, PER_CHANNEL);
+    constexpr int GROUP = LANES / LS_PER;                    // tokens whose read-outs are summed together
     extern __shared__ __align__(16) float ls_smem[];
-    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * LS_COLS;
-    const int tid = threadIdx.x, c = tid / LS_LANES, l = tid % LS_LANES;
-    const int j = col0 + c;
-    const bool is_norm = norm_out != nullptr && j == dv;     // the normalizer: a column whose value is always one
-    const bool live = j < dv || is_norm;
-    for (int i = tid; i < 2 * BUF; i += THREADS) ls_smem[i] = 0.0f;      // the padding past dk and dv stays zero
+    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
+    const int tid = threadIdx.x, c0 = LS_PER * (tid / LANES), l = tid % LANES;
+    for (int i = tid; i < 2 * BUF; i += LS_THREADS) ls_smem[i] = 0.0f;   // the padding past dk and dv stays zero
     pdl_wait();
     const int first = seq_first[s], count = seq_first[s + 1] - first;
-    float* mine = state + (long long)seq_slots[s] * state_stride + state_offset +
-                  (is_norm ? ((long long)n_heads * dv + h) * dk : ((long long)h * dv + j) * dk);
-    float2x S[2 * Q];
+    float* const slot = state + (long long)seq_slots[s] * state_stride + state_offset;
+    // the columns of this lane: a value entry each, or (column dv, where asked for) the normalizer, whose value is one
+    auto column = [&](int c) {
+        const int j = col0 + c0 + c;
+        return slot + (j == dv ? (long long)n_heads * dv + h : (long long)h * dv + j) * dk;
+    };
+    const int n_live = min(LS_PER, dv + (norm_out ? 1 : 0) - col0 - c0);         // (may be negative)
+    const int norm_at = norm_out ? dv - col0 - c0 : LS_PER;                      // which of the four is the normalizer
+    float2x S[LS_PER][2 * Q];
 #pragma unroll
-    for (int i = 0; i < Q; ++i) {
-        const int d = 4 * (l + LS_LANES * i);
-        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (VEC) {
-            if (live && d < dk) x = *reinterpret_cast<const float4*>(mine + d);
-        } else if (live) {
-            if (d < dk) x.x = mine[d];
-            if (d + 1 < dk) x.y = mine[d + 1];
-            if (d + 2 < dk) x.z = mine[d + 2];
-            if (d + 3 < dk) x.w = mine[d + 3];
+    for (int c = 0; c < LS_PER; ++c)
+#pragma unroll
+        for (int i = 0; i < Q; ++i) {
+            const int d = 4 * (l + LANES * i);
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (c < n_live) {
+                const float* mine = column(c);
+                if (VEC) {
+                    if (d < dk) x = *reinterpret_cast<const float4*>(mine + d);
+                } else {
+                    if (d < dk) x.x = mine[d];
+                    if (d + 1 < dk) x.y = mine[d + 1];
+                    if (d + 2 < dk) x.z = mine[d + 2];
+                    if (d + 3 < dk) x.w = mine[d + 3];
+                }
+            }
+            S[c][2 * i] = pair_of_floats(x.x, x.y);
+            S[c][2 * i + 1] = pair_of_floats(x.z, x.w);
         }
-        S[2 * i] = pair_of_floats(x.x, x.y);
-        S[2 * i + 1] = pair_of_floats(x.z, x.w);
-    }
     // stages the chunk that starts at the sequence's li0-th token of this step into buffer `b`
     auto stage = [&](int li0, int b) {
         float* ks = ls_smem + b * BUF;
         float* qs = ks + LS_CHUNK * DKP;
         float* gs = qs + LS_CHUNK * DKP;
         float* vs = gs + (PER_CHANNEL ? LS_CHUNK * DKP : 0);
-        float* sc = vs + LS_CHUNK * LS_COLS;
+        float* sc = vs + LS_CHUNK * COLS;
         const int n = min(LS_CHUNK, count - li0);
         const long long t0 = first + li0;
         if (VEC) {
             const int per = dk / 4;
-            for (int i = tid; i < n * per; i += THREADS) {
+            for (int i = tid; i < n * per; i += LS_THREADS) {
                 const int tok = i / per, d = 4 * (i % per);
                 const long long at = (t0 + tok) * ld + (long long)h * dk + d;
                 copy_async16(ks + tok * DKP + d, k + at);
                 copy_async16(qs + tok * DKP + d, q + at);
                 if (PER_CHANNEL) copy_async16(gs + tok * DKP + d, decay + ((t0 + tok) * n_heads + h) * dk + d);
             }
-            for (int i = tid; i < n * (LS_COLS / 4); i += THREADS) {
-                const int tok = i / (LS_COLS / 4), cc = 4 * (i % (LS_COLS / 4));
-                if (col0 + cc < dv) copy_async16(vs + tok * LS_COLS + cc, v + (t0 + tok) * ld + (long long)h * dv + col0 + cc);
+            for (int i = tid; i < n * (COLS / 4); i += LS_THREADS) {
+                const int tok = i / (COLS / 4), cc = 4 * (i % (COLS / 4));
+                if (col0 + cc < dv) copy_async16(vs + tok * COLS + cc, v + (t0 + tok) * ld + (long long)h * dv + col0 + cc);
             }
         } else {
-            for (int i = tid; i < n * dk; i += THREADS) {
+            for (int i = tid; i < n * dk; i += LS_THREADS) {
                 const int tok = i / dk, d = i % dk;
                 const long long at = (t0 + tok) * ld + (long long)h * dk + d;
                 copy_async4(ks + tok * DKP + d, k + at);
                 copy_async4(qs + tok * DKP + d, q + at);
                 if (PER_CHANNEL) copy_async4(gs + tok * DKP + d, decay + ((t0 + tok) * n_heads + h) * dk + d);
             }
-            for (int i = tid; i < n * LS_COLS; i += THREADS) {
-                const int tok = i / LS_COLS, cc = i % LS_COLS;
-                if (col0 + cc < dv) copy_async4(vs + tok * LS_COLS + cc, v + (t0 + tok) * ld + (long long)h * dv + col0 + cc);
+            for (int i = tid; i < n * COLS; i += LS_THREADS) {
+                const int tok = i / COLS, cc = i % COLS;
+                if (col0 + cc < dv) copy_async4(vs + tok * COLS + cc, v + (t0 + tok) * ld + (long long)h * dv + col0 + cc);
             }
         }
         if (!PER_CHANNEL)
-            for (int tok = tid; tok < n; tok += THREADS) copy_async16(sc + tok * 4, decay + 4 * ((t0 + tok) * n_heads + h));
+            for (int tok = tid; tok < n; tok += LS_THREADS) copy_async16(sc + tok * 4, decay + 4 * ((t0 + tok) * n_heads + h));
         copy_async_commit();
     };
     __syncthreads();                                         // the zeros are down before the first copies land
@@ -152,31 +143,57 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
         const float* qs = ks + LS_CHUNK * DKP;
         const float* gs = qs + LS_CHUNK * DKP;
         const float* vs = gs + (PER_CHANNEL ? LS_CHUNK * DKP : 0);
-        const float* sc = vs + LS_CHUNK * LS_COLS;
-        auto step = [&](int tok) {
-            float value = is_norm ? 1.0f : vs[tok * LS_COLS + c], fade = 1.0f;
+        const float* sc = vs + LS_CHUNK * COLS;
+        // One token: S = g S + k v for the lane's entries, and the lane's share of each column's S . q into `sum`.
+        auto step = [&](int tok, float* sum) {
+            float4 v4 = *reinterpret_cast<const float4*>(vs + tok * COLS + c0);
+            float value[LS_PER] = {v4.x, v4.y, v4.z, v4.w};
+            float2x fade = 0;
             if (!PER_CHANNEL) {
                 const float2 gate = *reinterpret_cast<const float2*>(sc + tok * 4);      // decay, take
-                fade = gate.x;
-                value *= gate.y;
+                fade = pair_of_floats(gate.x, gate.x);
+#pragma unroll
+                for (int c = 0; c < LS_PER; ++c) value[c] = (c == norm_at ? 1.0f : value[c]) * gate.y;
             }
-            return ls_step<R, PER_CHANNEL>(S, ks + tok * DKP, qs + tok * DKP, gs + tok * DKP, fade, value, l);
-        };
-        for (int t0 = 0; t0 < n; t0 += LS_GROUP) {
-            float acc[LS_GROUP];
-            const int left = n - t0;
-            if (left >= LS_GROUP) {                          // a whole group: no branch between the tokens
+            float2x a[LS_PER] = {0, 0, 0, 0};                                            // (two zeros each)
 #pragma unroll
-                for (int i = 0; i < LS_GROUP; ++i) acc[i] = step(t0 + i);
-            } else {
+            for (int i = 0; i < Q; ++i) {
+                const int at = tok * DKP + 4 * (l + LANES * i);
+                const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(ks + at);
+                const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(qs + at);
+                ulonglong2 gg = make_ulonglong2(fade, fade);
+                if (PER_CHANNEL) gg = *reinterpret_cast<const ulonglong2*>(gs + at);
 #pragma unroll
-                for (int i = 0; i < LS_GROUP; ++i) {
-                    acc[i] = 0.0f;
-                    if (i < left) acc[i] = step(t0 + i);
+                for (int c = 0; c < LS_PER; ++c) {
+                    const float2x v2 = pair_of_floats(value[c], value[c]);
+                    S[c][2 * i] = pair_fma(kk.x, v2, pair_mul(gg.x, S[c][2 * i]));
+                    S[c][2 * i + 1] = pair_fma(kk.y, v2, pair_mul(gg.y, S[c][2 * i + 1]));
+                    a[c] = pair_fma(S[c][2 * i], qq.x, a[c]);
+                    a[c] = pair_fma(S[c][2 * i + 1], qq.y, a[c]);
                 }
             }
 #pragma unroll
-            for (int width = LS_GROUP / 2; width >= 1; width >>= 1) {
+            for (int c = 0; c < LS_PER; ++c) {
+                const float2 x = floats_of_pair(a[c]);
+                sum[c] = x.x + x.y;
+            }
+        };
+        for (int t0 = 0; t0 < n; t0 += GROUP) {
+            float acc[LANES];                                // token t0 + i, column c at [4 i + c]
+            const int left = n - t0;
+            if (left >= GROUP) {                             // a whole group: no branch between the tokens
+#pragma unroll
+                for (int i = 0; i < GROUP; ++i) step(t0 + i, acc + LS_PER * i);
+            } else {
+#pragma unroll
+                for (int i = 0; i < GROUP; ++i) {
+#pragma unroll
+                    for (int c = 0; c < LS_PER; ++c) acc[LS_PER * i + c] = 0.0f;
+                    if (i < left) step(t0 + i, acc + LS_PER * i);
+                }
+            }
+#pragma unroll
+            for (int width = LANES / 2; width >= 1; width >>= 1) {
 #pragma unroll
                 for (int i = 0; i < width; ++i) {
                     const bool upper = (l & width) != 0;
@@ -185,29 +202,33 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
                     acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, width);
                 }
             }
-            if (l < left && live) {
-                const long long t = first + li0 + t0 + l;
-                if (is_norm) norm_out[t * n_heads + h] = scale * acc[0];
-                else out[t * ldo + (long long)h * dv + j] = scale * acc[0];
+            const int tok = l / LS_PER, c = l % LS_PER;      // what this lane's sum is of
+            if (tok < left && c < n_live) {
+                const long long t = first + li0 + t0 + tok;
+                if (c == norm_at) norm_out[t * n_heads + h] = scale * acc[0];
+                else out[t * ldo + (long long)h * dv + col0 + c0 + c] = scale * acc[0];
             }
         }
         __syncthreads();                                     // this buffer is free for the chunk after the next
     }
     pdl_trigger();                                           // (only now: see the delta scan)
 #pragma unroll
-    for (int i = 0; i < Q; ++i) {
-        const int d = 4 * (l + LS_LANES * i);
-        const float2 lo = floats_of_pair(S[2 * i]), hi = floats_of_pair(S[2 * i + 1]);
-        if (!live) continue;
-        if (VEC) {
-            if (d < dk) *reinterpret_cast<float4*>(mine + d) = make_float4(lo.x, lo.y, hi.x, hi.y);
-        } else {
-            if (d < dk) mine[d] = lo.x;
-            if (d + 1 < dk) mine[d + 1] = lo.y;
-            if (d + 2 < dk) mine[d + 2] = hi.x;
-            if (d + 3 < dk) mine[d + 3] = hi.y;
+    for (int c = 0; c < LS_PER; ++c)
+#pragma unroll
+        for (int i = 0; i < Q; ++i) {
+            const int d = 4 * (l + LANES * i);
+            const float2 lo = floats_of_pair(S[c][2 * i]), hi = floats_of_pair(S[c][2 * i + 1]);
+            if (c >= n_live) continue;
+            float* mine = column(c);
+            if (VEC) {
+                if (d < dk) *reinterpret_cast<float4*>(mine + d) = make_float4(lo.x, lo.y, hi.x, hi.y);
+            } else {
+                if (d < dk) mine[d] = lo.x;
+                if (d + 1 < dk) mine[d + 1] = lo.y;
+                if (d + 2 < dk) mine[d + 2] = hi.x;
+                if (d + 3 < dk) mine[d + 3] = hi.y;
+            }
         }
-    }
 }
 
 // One block per (sequence, head); a thread a token of the chunk.  What a run of tokens does to m is a pair (F, M):
@@ -271,6 +292,12 @@ struct LowRankPart {
     int col, rank, n, fn, per_head;
     float power;
 };
+
+__device__ __forceinline__ float low_rank_fn(float z, const LowRankPart& p, float rate) {
+    if (p.fn == 1) return expf(-p.power * softplus(-z));
+    if (p.fn == 2) return expf(-rate * softplus(z));
+    return z;
+}
 
 template <int N, typename T> __device__ __forceinline__ void load_weights(float (&x)[N], const T* p, int n) {
 #pragma unroll
@@ -340,12 +367,88 @@ low_rank_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowR
 #pragma unroll
         for (int t = 0; t < TOK; ++t) {
             if (t >= nt) break;
-            float z = (half ? a1[t] : a0[t]) + bias;
-            if (p.fn == 1) z = expf(-p.power * softplus(-z));
-            else if (p.fn == 2) z = expf(-rate * softplus(z));
-            p.out[(long long)(t0 + t) * p.n + c] = z;
+            p.out[(long long)(t0 + t) * p.n + c] = low_rank_fn((half ? a1[t] : a0[t]) + bias, p, rate);
         }
     }
+}
+
+// The same on tensor cores for steps of many tokens with bfloat16 weights: a block takes 64 tokens x 64 channels of one
+// part, a warp 16 tokens.  The tokens' rows enter as two bfloat16 terms (rounded, and what the rounding left), so a
+// product keeps 16 bits of the row and all of the weight; float32 accumulators.  rank: a multiple of 16.
+constexpr int LM_TOK = 64, LM_CH = 64, LM_PAD = 8;
+
+__device__ __forceinline__ void lm_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void lm_ldmatrix(uint32_t (&r)[4], const __nv_bfloat16* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+
+__global__ void __launch_bounds__(128)
+low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowRankPart p0, LowRankPart p1, int blocks0) {
+    extern __shared__ __align__(16) unsigned char lm_raw[];  // weights [64][pitch], rows' two terms [64][pitch] each
+    pdl_trigger();
+    const bool second = (int)blockIdx.y >= blocks0;
+    const LowRankPart p = second ? p1 : p0;
+    const int c0 = ((int)blockIdx.y - (second ? blocks0 : 0)) * LM_CH, t0 = blockIdx.x * LM_TOK;
+    const int pitch = p.rank + LM_PAD, pieces = p.rank / 8;
+    __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(lm_raw);
+    __nv_bfloat16* hi = ws + LM_CH * pitch;
+    __nv_bfloat16* lo = hi + LM_TOK * pitch;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
+    for (int i = tid; i < LM_CH * pieces; i += 128) {        // (the weights: nothing in flight writes them)
+        const int r = i / pieces, c = 8 * (i % pieces);
+        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.w) + (long long)min(c0 + r, p.n - 1) * p.ldw + c;
+        *reinterpret_cast<uint4*>(ws + r * pitch + c) = *reinterpret_cast<const uint4*>(src);
+    }
+    pdl_wait();
+    for (int i = tid; i < LM_TOK * (p.rank / 4); i += 128) {
+        const int r = i / (p.rank / 4), c = 4 * (i % (p.rank / 4));
+        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (t0 + r < n_tokens) {
+            const float* src = low + (long long)(t0 + r) * ldl + p.col + c;
+            x = make_float4(src[0], src[1], src[2], src[3]);
+        }
+        const __nv_bfloat162 h0 = __floats2bfloat162_rn(x.x, x.y), h1 = __floats2bfloat162_rn(x.z, x.w);
+        __nv_bfloat162* hp = reinterpret_cast<__nv_bfloat162*>(hi + r * pitch + c);
+        __nv_bfloat162* lp = reinterpret_cast<__nv_bfloat162*>(lo + r * pitch + c);
+        hp[0] = h0, hp[1] = h1;
+        lp[0] = __floats2bfloat162_rn(x.x - __low2float(h0), x.y - __high2float(h0));
+        lp[1] = __floats2bfloat162_rn(x.z - __low2float(h1), x.w - __high2float(h1));
+    }
+    __syncthreads();
+    float acc[LM_CH / 8][4] = {};
+    for (int kk = 0; kk < p.rank; kk += 16) {
+        uint32_t ah[4], al[4], bf[4];
+        const int arow = (warp * 16 + (lane & 15)) * pitch + kk + (lane >> 4) * 8;
+        lm_ldmatrix(ah, hi + arow);
+        lm_ldmatrix(al, lo + arow);
+#pragma unroll
+        for (int j = 0; j < LM_CH / 8; j += 2) {
+            lm_ldmatrix(bf, ws + (j * 8 + (lane & 7) + (lane >> 4) * 8) * pitch + kk + ((lane >> 3) & 1) * 8);
+            lm_mma(acc[j], ah, bf[0], bf[1]);
+            lm_mma(acc[j], al, bf[0], bf[1]);
+            lm_mma(acc[j + 1], ah, bf[2], bf[3]);
+            lm_mma(acc[j + 1], al, bf[2], bf[3]);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < LM_CH / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int c = c0 + j * 8 + tig * 2 + e;
+            if (c >= p.n) continue;
+            const float bias = p.bias ? p.bias[c] : 0.0f;
+            const float rate = p.fn == 2 ? expf(p.a_log[c / p.per_head]) : 0.0f;
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int t = t0 + warp * 16 + gid + 8 * half;
+                if (t < n_tokens) p.out[(long long)t * p.n + c] = low_rank_fn(acc[j][2 * half + e] + bias, p, rate);
+            }
+        }
 }
 
 }  // namespace mu
@@ -368,13 +471,14 @@ MU_EXPORT int mu_linear_scan(const float* q, const float* k, const float* v, lon
     if (!per_channel && ((uintptr_t)decay & 15)) return MU_ERR_ALIGNMENT;
     cudaStream_t s = (cudaStream_t)stream;
     const int cols = dv + (norm_out ? 1 : 0);
-    const dim3 grid(n_seqs, n_heads, (cols + mu::LS_COLS - 1) / mu::LS_COLS), block(mu::LS_LANES * mu::LS_COLS);
     const bool vec = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0 &&
                      (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)state | (per_channel ? (uintptr_t)decay : 0)) & 15) == 0;
-#define MU_LINEAR_SCAN_V(R, V, PC)                                                                                    \
+#define MU_LINEAR_SCAN_V(R, LANES, V, PC)                                                                             \
     do {                                                                                                              \
-        const size_t smem = 2 * sizeof(float) * mu::ls_chunk_floats(mu::LS_LANES * R, PC);                            \
-        auto kernel = mu::linear_scan_kernel<R, V, PC>;                                                               \
+        const size_t smem = 2 * sizeof(float) * mu::ls_chunk_floats(LANES * R, mu::ls_columns(LANES), PC);            \
+        const dim3 grid(n_seqs, n_heads, (cols + mu::ls_columns(LANES) - 1) / mu::ls_columns(LANES));                 \
+        const dim3 block(mu::LS_THREADS);                                                                             \
+        auto kernel = mu::linear_scan_kernel<R, LANES, V, PC>;                                                        \
         if (!mu::allow_shared((const void*)kernel, smem)) return MU_ERR_LAUNCH;                                       \
         mu::prefer_shared_memory((const void*)kernel);                                                                \
         if (long_steps)                                                                                               \
@@ -383,17 +487,17 @@ MU_EXPORT int mu_linear_scan(const float* q, const float* k, const float* v, lon
         return mu::launch_pdl(kernel, grid, block, smem, s, 1, q, k, v, ld, decay, n_heads, dk, dv, scale, seq_first, \
                               seq_slots, state, state_stride, state_offset, out, ldo, norm_out);                      \
     } while (0)
-#define MU_LINEAR_SCAN(R)                                                                                             \
+#define MU_LINEAR_SCAN(R, LANES)                                                                                      \
     do {                                                                                                              \
-        if (vec && per_channel) MU_LINEAR_SCAN_V(R, true, true);                                                      \
-        if (per_channel) MU_LINEAR_SCAN_V(R, false, true);                                                            \
-        if (vec) MU_LINEAR_SCAN_V(R, true, false);                                                                    \
-        MU_LINEAR_SCAN_V(R, false, false);                                                                            \
+        if (vec && per_channel) MU_LINEAR_SCAN_V(R, LANES, true, true);                                               \
+        if (per_channel) MU_LINEAR_SCAN_V(R, LANES, false, true);                                                     \
+        if (vec) MU_LINEAR_SCAN_V(R, LANES, true, false);                                                             \
+        MU_LINEAR_SCAN_V(R, LANES, false, false);                                                                     \
     } while (0)
-    if (dk <= 32) MU_LINEAR_SCAN(4);
-    if (dk <= 64) MU_LINEAR_SCAN(8);
-    if (dk <= 128) MU_LINEAR_SCAN(16);
-    MU_LINEAR_SCAN(32);
+    if (dk <= 32) MU_LINEAR_SCAN(4, 8);
+    if (dk <= 64) MU_LINEAR_SCAN(4, 16);
+    if (dk <= 128) MU_LINEAR_SCAN(4, 32);
+    MU_LINEAR_SCAN(8, 32);
 #undef MU_LINEAR_SCAN
 #undef MU_LINEAR_SCAN_V
 }
@@ -428,12 +532,24 @@ MU_EXPORT int mu_low_rank(const float* low, long long ldl, int n_tokens, const m
         blocks[i] = (p.n + mu::LR_CHANNELS - 1) / mu::LR_CHANNELS;
         rank = p.rank > rank ? p.rank : rank;
     }
+    const mu::LowRankPart p0 = parts[0], p1 = n_parts > 1 ? parts[1] : parts[0];
+    cudaStream_t s = (cudaStream_t)stream;
+    // steps of many tokens with weights in whole 16-byte pieces: tensor cores
+    bool tc = w_bf16 && n_tokens >= 64;
+    for (int i = 0; i < n_parts; ++i)
+        tc = tc && parts[i].rank % 16 == 0 && parts[i].rank <= 512 && parts[i].ldw % 8 == 0 && ((uintptr_t)parts[i].w & 15) == 0;
+    if (tc) {
+        int by[2] = {0, 0};
+        for (int i = 0; i < n_parts; ++i) by[i] = (parts[i].n + mu::LM_CH - 1) / mu::LM_CH;
+        const size_t bytes = (size_t)(mu::LM_CH + 2 * mu::LM_TOK) * (rank + mu::LM_PAD) * sizeof(__nv_bfloat16);
+        if (!mu::allow_shared((const void*)mu::low_rank_mma_kernel, 220 * 1024)) return MU_ERR_LAUNCH;
+        return mu::launch_pdl(mu::low_rank_mma_kernel, dim3((n_tokens + mu::LM_TOK - 1) / mu::LM_TOK, by[0] + by[1]), dim3(128),
+                              bytes, s, 1, low, ldl, n_tokens, p0, p1, by[0]);
+    }
     const int tok = n_tokens >= 256 ? 16 : n_tokens >= 8 ? 4 : 1;
     const size_t smem = (size_t)tok * ((rank + 7) / 8 * 8) * sizeof(float);
     if (smem > 48 * 1024) return MU_ERR_UNSUPPORTED_SIZE;
     const dim3 grid((n_tokens + tok - 1) / tok, blocks[0] + blocks[1]), block(mu::LR_THREADS);
-    cudaStream_t s = (cudaStream_t)stream;
-    const mu::LowRankPart p0 = parts[0], p1 = n_parts > 1 ? parts[1] : parts[0];
 #define MU_LOW_RANK(T, TOK)                                                                                           \
     return mu::launch_pdl(mu::low_rank_kernel<T, TOK>, grid, block, smem, s, 1, low, ldl, n_tokens, p0, p1, blocks[0])
     if (w_bf16) {

@@ -109,7 +109,7 @@ _SIGNATURES = {
                                 _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
     "mu_qkv_norm_rows": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_f, _c_int, _c_int, _c_int, _c_int, _c_int,
                          _c_int, _c_p, _c_int, _c_f, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_p],
-    "mu_residual_add_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_f, _c_p, _c_f, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p],
+    "mu_residual_add_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_f, _c_p, _c_f, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
     "mu_delta_prepare": [_c_p, _c_int, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_f,
                          _c_p, _c_p, _c_p, _c_int, _c_p],
     "mu_delta_scan_max_dk": [],
@@ -692,9 +692,10 @@ def qkv_norm_rows(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.
 
 
 def residual_add_norm(x: torch.Tensor, y: Optional[torch.Tensor], mult: float, weight: Optional[torch.Tensor],
-                      eps: float, out: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+                      eps: float, out: Optional[torch.Tensor], groups: int = 1) -> Optional[torch.Tensor]:
     """x += mult * y on the float32 stream (``y`` None: nothing is added), then out = x / rms(x) * weight in
-    ``out``'s dtype (``weight`` None: the addition only)."""
+    ``out``'s dtype (``weight`` None: the addition only).  ``groups``: the row in that many consecutive equal parts, each
+    divided by its own rms."""
     _need_cuda(x, y, weight, out)
     if x.dtype != torch.float32 or x.dim() != 2 or x.stride(1) != 1:
         raise KernelError("residual_add_norm: the stream is float32 [rows, n] with unit inner stride")
@@ -706,7 +707,7 @@ def residual_add_norm(x: torch.Tensor, y: Optional[torch.Tensor], mult: float, w
     _check(library().mu_residual_add_norm(_ptr(x), x.stride(0), _ptr(y), y.stride(0) if y is not None else 0, float(mult),
                                           _ptr(weight), float(eps), x.shape[0], x.shape[1], _ptr(out),
                                           out.stride(0) if out is not None else 0,
-                                          _is_bf16(out) if out is not None else 0, _stream()),
+                                          _is_bf16(out) if out is not None else 0, _stream(), int(groups)),
            ("residual_add_norm(n={})", x.shape[1]))
     return out
 

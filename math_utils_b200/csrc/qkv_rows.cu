@@ -122,8 +122,10 @@ residual_add_norm_kernel(float* __restrict__ x, long long ldx, const float* __re
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
-    float* xs = x + (long long)t * ldx;
-    const float* ys = y ? y + (long long)t * ldy : nullptr;
+    const long long part0 = (long long)blockIdx.y * width;   // rows normed in parts: this block's part
+    float* xs = x + (long long)t * ldx + part0;
+    const float* ys = y ? y + (long long)t * ldy + part0 : nullptr;
+    weight = weight ? weight + part0 : nullptr;
     float kept[RA_KEEP];
     float sq = 0.0f;
 #pragma unroll
@@ -143,7 +145,7 @@ residual_add_norm_kernel(float* __restrict__ x, long long ldx, const float* __re
     }
     if (!weight) return;
     const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)width + eps);
-    TE* hs = h + (long long)t * ldh;
+    TE* hs = h + (long long)t * ldh + part0;
 #pragma unroll
     for (int i = 0; i < RA_KEEP; ++i) {
         const int d = threadIdx.x + i * blockDim.x;
@@ -151,6 +153,55 @@ residual_add_norm_kernel(float* __restrict__ x, long long ldx, const float* __re
     }
     for (int d = threadIdx.x + RA_KEEP * blockDim.x; d < width; d += blockDim.x)
         hs[d] = from_float<TE>(xs[d] * inv * weight[d]);      // written by this very thread above
+}
+
+__device__ __forceinline__ void ra_store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void ra_store(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 packed;
+    packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+    packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = packed;
+}
+
+// The same for rows normed in parts of up to 1,024 entries in whole, aligned 16-byte pieces: a warp a part, no barrier.
+template <typename TE>
+__global__ void __launch_bounds__(128)
+residual_add_norm_parts_kernel(float* __restrict__ x, long long ldx, const float* __restrict__ y, long long ldy, float mult,
+                               const float* __restrict__ weight, float eps, int width, int parts, long long n_parts,
+                               TE* __restrict__ h, long long ldh) {
+    pdl_trigger();
+    pdl_wait();
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= n_parts) return;
+    const int lane = threadIdx.x & 31, part = (int)(item % parts);
+    const long long t = item / parts, at0 = (long long)part * width;
+    float* xs = x + t * ldx + at0;
+    const float* ys = y ? y + t * ldy + at0 : nullptr;
+    float4 v[8];
+    float sq = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int d = 4 * (lane + 32 * i);
+        v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (d < width) {
+            v[i] = *reinterpret_cast<const float4*>(xs + d);
+            if (ys) {
+                const float4 u = *reinterpret_cast<const float4*>(ys + d);
+                v[i] = make_float4(fmaf(mult, u.x, v[i].x), fmaf(mult, u.y, v[i].y), fmaf(mult, u.z, v[i].z), fmaf(mult, u.w, v[i].w));
+                *reinterpret_cast<float4*>(xs + d) = v[i];
+            }
+        }
+        sq += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int d = 4 * (lane + 32 * i);
+        if (d >= width) continue;
+        const float4 g = *reinterpret_cast<const float4*>(weight + at0 + d);
+        ra_store(h + t * ldh + at0 + d, make_float4(v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w));
+    }
 }
 
 }  // namespace mu
@@ -180,16 +231,30 @@ MU_EXPORT int mu_qkv_norm_rows(void* q, long long ldq, const void* k, long long 
                           first, first_mode, lambda, tok_pos, tok_seq, block_table, max_pages, page_tokens, (float*)rows);
 }
 
+// groups: the row is normed in that many equal parts, each by itself (the weight is the whole row's).
 MU_EXPORT int mu_residual_add_norm(float* x, long long ldx, const float* y, long long ldy, float mult, const float* weight,
-                                   float eps, int n_rows, int width, void* h, long long ldh, int is_bf16, void* stream) {
+                                   float eps, int n_rows, int width, void* h, long long ldh, int is_bf16, void* stream,
+                                   int groups) {
     if (n_rows <= 0 || width <= 0) return MU_OK;
-    if (!x || (weight && !h) || (!weight && !y)) return MU_ERR_BAD_ARGUMENT;
+    if (!x || (weight && !h) || (!weight && !y) || groups < 1 || groups > 65535 || width % groups) return MU_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid(n_rows), block(width > 1024 ? 256 : 128);
     typedef __nv_bfloat16 bf;
+    const int part = width / groups;
+    if (weight && groups > 1 && part % 4 == 0 && part <= 1024 && ldx % 4 == 0 && ldy % 4 == 0 && ldh % 4 == 0 &&
+        (((uintptr_t)x | (uintptr_t)y | (uintptr_t)weight) & 15) == 0 && ((uintptr_t)h & (is_bf16 ? 7 : 15)) == 0) {
+        const long long n_parts = (long long)n_rows * groups;
+        const int warps = n_parts >= 2048 ? 4 : 1;           // a few parts: a block each, spread over the SMs
+        const dim3 grid((unsigned)((n_parts + warps - 1) / warps)), block(32 * warps);
+        if (is_bf16)
+            return mu::launch_pdl(mu::residual_add_norm_parts_kernel<bf>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight,
+                                  eps, part, groups, n_parts, (bf*)h, ldh);
+        return mu::launch_pdl(mu::residual_add_norm_parts_kernel<float>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight,
+                              eps, part, groups, n_parts, (float*)h, ldh);
+    }
+    const dim3 grid(n_rows, groups), block(part > 1024 ? 256 : 128);
     if (is_bf16)
         return mu::launch_pdl(mu::residual_add_norm_kernel<bf>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight, eps,
-                              width, (bf*)h, ldh);
+                              part, (bf*)h, ldh);
     return mu::launch_pdl(mu::residual_add_norm_kernel<float>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight, eps,
-                          width, (float*)h, ldh);
+                          part, (float*)h, ldh);
 }

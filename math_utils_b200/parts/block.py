@@ -27,6 +27,9 @@ norm of their own.  Both norms are made before either sublayer adds into the str
 by one launch: one pass over x, one statistic, two weights); then the mixer and the feed-forward add into the
 float32 stream in their last launches.  A layer without a feed-forward is x += mixer(norm1(x)).  With the parameter
 ``shared_norm`` there is one norm, and both sublayers read its output: x += mixer(norm1(x)) + feed_forward(norm1(x)).
+In steps of a few tokens (single-token steps above all) the feed-forward then runs on a stream of its own beside the
+mixer, into a buffer that the next norm's launch adds to the stream: both are chains of short dependent launches, and
+side by side the layer's chain is as long as the longer of the two.
 """
 from __future__ import annotations
 
@@ -201,7 +204,7 @@ class ScaledPreNormBlock(Arrangement):
     @staticmethod
     def _norm(norm, x, ctx):
         """The normed stream, with what is still to be added to the stream added by the same launch."""
-        if isinstance(norm, RmsNorm) and norm.offset == 0.0 and norm.scale == 1.0 and norm.groups == 1 and x.stride(1) == 1:
+        if isinstance(norm, RmsNorm) and norm.offset == 0.0 and norm.scale == 1.0 and x.stride(1) == 1:
             pending, ctx.pending_join = ctx.pending_join, None
             if pending is not None and pending[0] is not x:
                 ctx.pending_join = pending
@@ -209,7 +212,7 @@ class ScaledPreNormBlock(Arrangement):
                 pending = None
             out = ctx.buffer("stream.normed", tuple(x.shape), norm.runtime.dtype)
             y, mult = (pending[1], pending[2]) if pending is not None else (None, 0.0)
-            return norm.runtime.ops.residual_add_norm(x, y, mult, norm.weight, norm.eps, out)
+            return norm.runtime.ops.residual_add_norm(x, y, mult, norm.weight, norm.eps, out, groups=norm.groups)
         ctx.flush_join()
         return norm.forward(x)
 
@@ -218,16 +221,36 @@ class ParallelPreNormBlock(Arrangement):
     def __init__(self, spec):
         super().__init__(spec)
         self.shared_norm = bool(self.param("shared_norm", False))
+        self.joins_pending = self.shared_norm
+        self._side = None
+
+    # Steps of up to this many tokens run the two sublayers side by side.  (At this size every product is a kernel that
+    # keeps no workspace in device memory that two launches could share.)
+    SIDE_BY_SIDE_TOKENS = 32
+
+    def _side_by_side(self, x, h, layer, ctx, cache, owns_cache: bool) -> None:
+        y = ctx.buffer("sublayer.out", tuple(x.shape), torch.float32)
+        main = torch.cuda.current_stream()
+        if self._side is None:
+            self._side = torch.cuda.Stream(device=h.device)
+            self._fork, self._join = torch.cuda.Event(), torch.cuda.Event()
+        self._fork.record(main)
+        self._side.wait_event(self._fork)                     # the input is ready
+        with torch.cuda.stream(self._side):
+            layer.feed_forward.forward(h, y, ctx, accumulate=False)
+            self._join.record(self._side)
+        layer.mixer.forward(h, x, ctx, cache, owns_cache)
+        main.wait_event(self._join)
+        ctx.pending_join = (x, y, 1.0)
 
     def forward(self, x, layer, ctx, cache, owns_cache: bool) -> None:
         n1, n2 = layer.norm1, layer.norm2
         alone = isinstance(layer.feed_forward, NoFeedForward)
         if self.shared_norm:
-            if type(n1) is RmsNorm:
-                h1 = n1.forward(x, out=ctx.buffer("stream.normed", tuple(x.shape), n1.runtime.dtype))
-            else:
-                h1 = n1.forward(x)
-            h2 = h1
+            h1 = h2 = ScaledPreNormBlock._norm(n1, x, ctx)
+            if (not alone and layer.feed_forward.can_overwrite and ctx.trace is None and h1.is_cuda
+                    and ctx.n_tokens <= self.SIDE_BY_SIDE_TOKENS):
+                return self._side_by_side(x, h1, layer, ctx, cache, owns_cache)
         elif (not alone and type(n1) is RmsNorm and type(n2) is RmsNorm and n1.eps == n2.eps and x.stride(1) == 1
                 and n1.offset == n2.offset == 0.0 and n1.scale == n2.scale == 1.0 and n1.groups == n2.groups == 1):
             dt = n1.runtime.dtype

@@ -6,6 +6,8 @@ configuration gives the rank: it is a ``FreeSize`` that the weight file fixes.
 """
 from __future__ import annotations
 
+import torch
+
 from .base import FreeSize, TensorSpec
 
 
@@ -22,7 +24,12 @@ class LowRank:
         return (TensorSpec(self.down_name, (self.free, self.hidden_size)), TensorSpec(self.up_name, (self.n, self.free)))
 
     def bind(self, tensors) -> None:
+        """The inner size is padded with zeros to a multiple of 16: whole pieces for the tensor cores."""
         self.down, self.up = tensors[self.down_name], tensors[self.up_name]
+        pad = -self.down.shape[0] % 16
+        if pad:
+            self.down = torch.nn.functional.pad(self.down, (0, 0, 0, pad))
+            self.up = torch.nn.functional.pad(self.up, (0, pad)).contiguous()
         self.rank = self.down.shape[0]
 
     def part(self, ops, col: int, out, **what):
