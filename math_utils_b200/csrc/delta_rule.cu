@@ -9,12 +9,14 @@
 // mu_delta_prepare   per token: every kv head's q and k become unit vectors, x / sqrt(sum x^2 + 1e-6), q also times
 //                    q_scale, in place; kq = q . k of the finished vectors; per head beta = sigmoid(b_raw) and
 //                    decay = exp(-exp(A_log) * softplus(a_raw + dt_bias)).  Everything float32.
-// mu_delta_scan      per (sequence, head, 16 columns of S), the step's tokens in order:
+// mu_delta_scan      per (sequence, head, a few columns of S), the step's tokens in order:
 //                        S <- decay S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
-//                    A column of S (one value entry) lives in the registers of 8 lanes.  The two sums a token needs
-//                    are made together and of the state as the token found it: (decay S)^T k = decay (S^T k), and
-//                    the read-out of the written state is decay (S^T q) + u (k . q).  So a token costs one exchange
-//                    between the lanes, not two, and the decay is off the path that waits for it.
+//                    Two columns of S (two value entries) live in the registers of up to 16 lanes, two entries to a
+//                    64-bit register; a key and a query read from shared memory serve both columns.  A token waits for
+//                    one exchange between the lanes only, that of S^T k, made of the state as the token found it:
+//                    (decay S)^T k = decay (S^T k).  The read-out of the written state is decay (S^T q) + u (k . q);
+//                    nothing waits for it, so the lanes keep their shares of it for as many (token, column) pairs as
+//                    there are lanes and add them crosswise.
 //                    q, k, v, beta, decay and k . q of 16 tokens at a time are copied to shared memory
 //                    asynchronously, the next 16 while these are worked on.
 //                    The order of every sum is fixed by the column alone: a token's result does not depend on how
@@ -68,57 +70,63 @@ delta_prepare_kernel(float* __restrict__ qkv, int channels, const TE* __restrict
     }
 }
 
-constexpr int DL_COLS = 16;       // columns a block takes
+constexpr int DL_THREADS = 128;
+constexpr int DL_PER = 2;         // columns of S whose entries a lane holds
 constexpr int DL_CHUNK = 16;      // tokens staged at a time
 constexpr int DL_MAX_DK = 256;    // the longest column
 
+// Columns a block takes: LANES lanes share two columns.
+__host__ __device__ constexpr int dl_columns(int lanes) { return DL_PER * DL_THREADS / lanes; }
 // Floats of one staged chunk: keys, queries (and the channels' decays) padded to DKP entries, the block's values,
 // (beta, decay, k . q, -).
-__host__ __device__ constexpr int dl_chunk_floats(int dkp, bool per_channel) {
-    return DL_CHUNK * ((per_channel ? 3 : 2) * dkp + DL_COLS + 4);
+__host__ __device__ constexpr int dl_chunk_floats(int dkp, int cols, bool per_channel) {
+    return DL_CHUNK * ((per_channel ? 3 : 2) * dkp + cols + 4);
 }
 
-// LANES: lanes that share a column of S; R: entries of the column a lane holds (a multiple of 4); dk <= LANES * R.
-// The column is dealt to the lanes four entries at a time: lane l holds entries 4 (l + LANES i) .. 4 (l + LANES i) + 3,
-// i < R / 4, so that 8 neighbouring lanes read 128 consecutive bytes of a staged key at once.  (Measured at dk = 128:
-// 8 lanes with 16 entries each beat 16 lanes with 8 and one more exchange.)  LANES and R follow from dk alone, so the
-// order of the sums does too.
+// LANES lanes hold two columns of S, R entries of each a lane (a multiple of 4; dk <= LANES R).  The columns are dealt
+// to the lanes four entries at a time: lane l holds entries 4 (l + LANES i) .. 4 (l + LANES i) + 3, i < R / 4, so that
+// neighbouring lanes read consecutive bytes of a staged key, and what a lane reads serves both of its columns.  LANES
+// and R follow from dk alone, so the order of the sums does too.
 // VEC: dk, dv, the row length and the state's offset and stride are all multiples of 4, so keys, queries, values and
 // the state move 16 bytes at a time.  PER_CHANNEL: `decay` is [T][n_heads * dk] (else [T][n_heads]).
 template <int R, int LANES, bool VEC, bool PER_CHANNEL>
-__global__ void __launch_bounds__(LANES * DL_COLS)
+__global__ void __launch_bounds__(DL_THREADS, R > 8 ? 2 : 4)
 delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __restrict__ kq,
                   const float* __restrict__ beta, const float* __restrict__ decay, int n_heads, int n_kv_heads, int dk,
                   int dv, const int* __restrict__ seq_first, const int* __restrict__ seq_slots,
                   float* __restrict__ state, long long state_stride, long long state_offset, float* __restrict__ out) {
-    constexpr int DL_LANES = LANES, DL_THREADS = LANES * DL_COLS;
-    constexpr int DKP = DL_LANES * R, Q = R / 4, BUF = dl_chunk_floats(DKP, PER_CHANNEL);
+    constexpr int DKP = LANES * R, Q = R / 4, COLS = dl_columns(LANES), BUF = dl_chunk_floats(DKP, COLS, PER_CHANNEL);
+    constexpr int GROUP = LANES / DL_PER;                    // tokens whose read-outs are summed together
     extern __shared__ __align__(16) float dl_smem[];
-    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DL_COLS;
-    const int tid = threadIdx.x, c = tid / DL_LANES, l = tid % DL_LANES;
+    const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
+    const int tid = threadIdx.x, c0 = DL_PER * (tid / LANES), l = tid % LANES;
     const int g = h / (n_heads / n_kv_heads);
-    const int j = col0 + c;
-    const bool live = j < dv;
+    const int n_live = min(DL_PER, dv - col0 - c0);          // (may be negative)
     for (int i = tid; i < 2 * BUF; i += DL_THREADS) dl_smem[i] = 0.0f;   // the padding past dk and dv stays zero
     pdl_wait();
     const int first = seq_first[s], count = seq_first[s + 1] - first;
-    float* mine = state + (long long)seq_slots[s] * state_stride + state_offset + ((long long)h * dv + j) * dk;
-    float2x S[2 * Q];                                        // the lane's entries in pairs
+    float* const mine = state + (long long)seq_slots[s] * state_stride + state_offset + ((long long)h * dv + col0 + c0) * dk;
+    float2x S[DL_PER][2 * Q];                                // the lane's entries in pairs
 #pragma unroll
-    for (int i = 0; i < Q; ++i) {
-        const int d = 4 * (l + DL_LANES * i);
-        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (VEC) {
-            if (live && d < dk) x = *reinterpret_cast<const float4*>(mine + d);
-        } else if (live) {
-            if (d < dk) x.x = mine[d];
-            if (d + 1 < dk) x.y = mine[d + 1];
-            if (d + 2 < dk) x.z = mine[d + 2];
-            if (d + 3 < dk) x.w = mine[d + 3];
+    for (int c = 0; c < DL_PER; ++c)
+#pragma unroll
+        for (int i = 0; i < Q; ++i) {
+            const int d = 4 * (l + LANES * i);
+            const float* col = mine + (long long)c * dk;
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (c < n_live) {
+                if (VEC) {
+                    if (d < dk) x = *reinterpret_cast<const float4*>(col + d);
+                } else {
+                    if (d < dk) x.x = col[d];
+                    if (d + 1 < dk) x.y = col[d + 1];
+                    if (d + 2 < dk) x.z = col[d + 2];
+                    if (d + 3 < dk) x.w = col[d + 3];
+                }
+            }
+            S[c][2 * i] = pair_of_floats(x.x, x.y);
+            S[c][2 * i + 1] = pair_of_floats(x.z, x.w);
         }
-        S[2 * i] = pair_of_floats(x.x, x.y);
-        S[2 * i + 1] = pair_of_floats(x.z, x.w);
-    }
     const long long q_off = (long long)g * dk, k_off = (long long)(n_kv_heads + g) * dk;
     const long long v_off = (long long)2 * n_kv_heads * dk + (long long)h * dv + col0;
     // stages the chunk that starts at the sequence's li0-th token of this step into buffer `b`
@@ -127,7 +135,7 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
         float* qs = ks + DL_CHUNK * DKP;
         float* gs = qs + DL_CHUNK * DKP;
         float* vs = gs + (PER_CHANNEL ? DL_CHUNK * DKP : 0);
-        float* sc = vs + DL_CHUNK * DL_COLS;
+        float* sc = vs + DL_CHUNK * COLS;
         const int n = min(DL_CHUNK, count - li0);
         if (VEC) {
             const int per = dk / 4;
@@ -138,10 +146,10 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
                 copy_async16(qs + tok * DKP + d, row + q_off + d);
                 if (PER_CHANNEL) copy_async16(gs + tok * DKP + d, decay + ((long long)(first + li0 + tok) * n_heads + h) * dk + d);
             }
-            for (int i = tid; i < n * (DL_COLS / 4); i += DL_THREADS) {
-                const int tok = i / (DL_COLS / 4), cc = 4 * (i % (DL_COLS / 4));
+            for (int i = tid; i < n * (COLS / 4); i += DL_THREADS) {
+                const int tok = i / (COLS / 4), cc = 4 * (i % (COLS / 4));
                 if (col0 + cc < dv)
-                    copy_async16(vs + tok * DL_COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
+                    copy_async16(vs + tok * COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
             }
         } else {
             for (int i = tid; i < n * dk; i += DL_THREADS) {
@@ -151,10 +159,10 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
                 copy_async4(qs + tok * DKP + d, row + q_off + d);
                 if (PER_CHANNEL) copy_async4(gs + tok * DKP + d, decay + ((long long)(first + li0 + tok) * n_heads + h) * dk + d);
             }
-            for (int i = tid; i < n * DL_COLS; i += DL_THREADS) {
-                const int tok = i / DL_COLS, cc = i % DL_COLS;
+            for (int i = tid; i < n * COLS; i += DL_THREADS) {
+                const int tok = i / COLS, cc = i % COLS;
                 if (col0 + cc < dv)
-                    copy_async4(vs + tok * DL_COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
+                    copy_async4(vs + tok * COLS + cc, qkv + (long long)(first + li0 + tok) * channels + v_off + cc);
             }
         }
         for (int tok = tid; tok < n; tok += DL_THREADS) {
@@ -181,60 +189,86 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
         const float* qs = ks + DL_CHUNK * DKP;
         const float* gs = qs + DL_CHUNK * DKP;
         const float* vs = gs + (PER_CHANNEL ? DL_CHUNK * DKP : 0);
-        const float* sc = vs + DL_CHUNK * DL_COLS;
-        // A token's keys, queries, decays, value and scalars are read into registers while the token before it is
-        // still waiting for its sums to come round the lanes.
-        ulonglong2 kr[Q], qr[Q], gr[PER_CHANNEL ? Q : 1];
-        float4 par = *reinterpret_cast<const float4*>(sc);                           // beta, decay, k . q
-        float v = vs[c];
-#pragma unroll
-        for (int i = 0; i < Q; ++i) {
-            kr[i] = *reinterpret_cast<const ulonglong2*>(ks + 4 * (l + DL_LANES * i));
-            qr[i] = *reinterpret_cast<const ulonglong2*>(qs + 4 * (l + DL_LANES * i));
-            if (PER_CHANNEL) gr[i] = *reinterpret_cast<const ulonglong2*>(gs + 4 * (l + DL_LANES * i));
-        }
-        for (int tok = 0; tok < n; ++tok) {
-            float2x k1 = 0, k2 = 0, q1 = 0, q2 = 0;                                  // (two zeros each)
+        const float* sc = vs + DL_CHUNK * COLS;
+        // One token.  S^T k has to come round the lanes before the state can move on; the read-out need not: the lane's
+        // share of it goes to `sum`, u (k . q) into lane 0's.
+        auto step = [&](int tok, float* sum) {
+            const float4 par = *reinterpret_cast<const float4*>(sc + tok * 4);           // beta, decay, k . q
+            const float2 v = *reinterpret_cast<const float2*>(vs + tok * COLS + c0);
+            ulonglong2 kr[Q];
+            float2x a[DL_PER] = {0, 0}, o[DL_PER] = {0, 0};                              // (two zeros each)
 #pragma unroll
             for (int i = 0; i < Q; ++i) {
-                if (PER_CHANNEL) {
-                    S[2 * i] = pair_mul(gr[i].x, S[2 * i]);
-                    S[2 * i + 1] = pair_mul(gr[i].y, S[2 * i + 1]);
+                const int at = tok * DKP + 4 * (l + LANES * i);
+                kr[i] = *reinterpret_cast<const ulonglong2*>(ks + at);
+                const ulonglong2 qr = *reinterpret_cast<const ulonglong2*>(qs + at);
+                ulonglong2 gr = make_ulonglong2(0, 0);
+                if (PER_CHANNEL) gr = *reinterpret_cast<const ulonglong2*>(gs + at);
+#pragma unroll
+                for (int c = 0; c < DL_PER; ++c) {
+                    if (PER_CHANNEL) {
+                        S[c][2 * i] = pair_mul(gr.x, S[c][2 * i]);
+                        S[c][2 * i + 1] = pair_mul(gr.y, S[c][2 * i + 1]);
+                    }
+                    a[c] = pair_fma(S[c][2 * i], kr[i].x, a[c]);
+                    a[c] = pair_fma(S[c][2 * i + 1], kr[i].y, a[c]);
+                    o[c] = pair_fma(S[c][2 * i], qr.x, o[c]);
+                    o[c] = pair_fma(S[c][2 * i + 1], qr.y, o[c]);
                 }
-                k1 = pair_fma(S[2 * i], kr[i].x, k1), q1 = pair_fma(S[2 * i], qr[i].x, q1);
-                k2 = pair_fma(S[2 * i + 1], kr[i].y, k2), q2 = pair_fma(S[2 * i + 1], qr[i].y, q2);
             }
-            const float2 ka = floats_of_pair(k1), kb = floats_of_pair(k2), qa = floats_of_pair(q1), qb = floats_of_pair(q2);
-            float sk = (ka.x + ka.y) + (kb.x + kb.y), sq = (qa.x + qa.y) + (qb.x + qb.y);
-            const int nxt = min(tok + 1, DL_CHUNK - 1);                              // the last one reads itself again
-            ulonglong2 nk[Q];
+            float sk[DL_PER];
 #pragma unroll
-            for (int i = 0; i < Q; ++i) {
-                nk[i] = *reinterpret_cast<const ulonglong2*>(ks + nxt * DKP + 4 * (l + DL_LANES * i));
-                qr[i] = *reinterpret_cast<const ulonglong2*>(qs + nxt * DKP + 4 * (l + DL_LANES * i));
-                if (PER_CHANNEL) gr[i] = *reinterpret_cast<const ulonglong2*>(gs + nxt * DKP + 4 * (l + DL_LANES * i));
+            for (int c = 0; c < DL_PER; ++c) {
+                const float2 x = floats_of_pair(a[c]);
+                sk[c] = x.x + x.y;
             }
-            const float4 npar = *reinterpret_cast<const float4*>(sc + nxt * 4);
-            const float nv = vs[nxt * DL_COLS + c];
 #pragma unroll
-            for (int o = DL_LANES / 2; o > 0; o >>= 1) {
-                sk += __shfl_xor_sync(0xffffffffu, sk, o);
-                sq += __shfl_xor_sync(0xffffffffu, sq, o);
-            }
-            // (one decay for the head: the sums are of the state before it, (decay S)^T k = decay (S^T k))
-            const float u = par.x * (v - (PER_CHANNEL ? sk : par.y * sk));
-            const float2x u2 = pair_of_floats(u, u), dec2 = pair_of_floats(par.y, par.y);
+            for (int w = LANES / 2; w > 0; w >>= 1)
 #pragma unroll
-            for (int i = 0; i < Q; ++i) {
-                S[2 * i] = pair_fma(kr[i].x, u2, PER_CHANNEL ? S[2 * i] : pair_mul(dec2, S[2 * i]));
-                S[2 * i + 1] = pair_fma(kr[i].y, u2, PER_CHANNEL ? S[2 * i + 1] : pair_mul(dec2, S[2 * i + 1]));
-                kr[i] = nk[i];
+                for (int c = 0; c < DL_PER; ++c) sk[c] += __shfl_xor_sync(0xffffffffu, sk[c], w);
+            const float2x dec2 = pair_of_floats(par.y, par.y);
+#pragma unroll
+            for (int c = 0; c < DL_PER; ++c) {
+                // (one decay for the head: the sums are of the state before it, (decay S)^T k = decay (S^T k))
+                const float u = par.x * ((c ? v.y : v.x) - (PER_CHANNEL ? sk[c] : par.y * sk[c]));
+                const float2x u2 = pair_of_floats(u, u);
+#pragma unroll
+                for (int i = 0; i < Q; ++i) {
+                    S[c][2 * i] = pair_fma(kr[i].x, u2, PER_CHANNEL ? S[c][2 * i] : pair_mul(dec2, S[c][2 * i]));
+                    S[c][2 * i + 1] = pair_fma(kr[i].y, u2, PER_CHANNEL ? S[c][2 * i + 1] : pair_mul(dec2, S[c][2 * i + 1]));
+                }
+                const float2 x = floats_of_pair(o[c]);
+                const float share = PER_CHANNEL ? x.x + x.y : par.y * (x.x + x.y);
+                sum[c] = l == 0 ? fmaf(u, par.z, share) : share;
             }
-            if (l == 0 && live)
-                out[(long long)(first + li0 + tok) * n_heads * dv + (long long)h * dv + j] =
-                    fmaf(u, par.z, PER_CHANNEL ? sq : par.y * sq);
-            par = npar;
-            v = nv;
+        };
+        for (int t0 = 0; t0 < n; t0 += GROUP) {
+            float acc[LANES];                                // token t0 + i, column c at [2 i + c]
+            const int left = n - t0;
+            if (left >= GROUP) {                             // a whole group: no branch between the tokens
+#pragma unroll
+                for (int i = 0; i < GROUP; ++i) step(t0 + i, acc + DL_PER * i);
+            } else {
+#pragma unroll
+                for (int i = 0; i < GROUP; ++i) {
+#pragma unroll
+                    for (int c = 0; c < DL_PER; ++c) acc[DL_PER * i + c] = 0.0f;
+                    if (i < left) step(t0 + i, acc + DL_PER * i);
+                }
+            }
+#pragma unroll
+            for (int width = LANES / 2; width >= 1; width >>= 1) {
+#pragma unroll
+                for (int i = 0; i < width; ++i) {
+                    const bool upper = (l & width) != 0;
+                    const float send = upper ? acc[i] : acc[i + width];
+                    const float keep = upper ? acc[i + width] : acc[i];
+                    acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, width);
+                }
+            }
+            const int tok = l / DL_PER, c = l % DL_PER;      // what this lane's sum is of
+            if (tok < left && c < n_live)
+                out[((long long)(first + li0 + t0 + tok) * n_heads + h) * dv + col0 + c0 + c] = acc[0];
         }
         __syncthreads();                                     // this buffer is free for the chunk after the next
     }
@@ -242,19 +276,22 @@ delta_scan_kernel(const float* __restrict__ qkv, int channels, const float* __re
     // here has one warp a scheduler, which every waiting warp there slows down.
     pdl_trigger();
 #pragma unroll
-    for (int i = 0; i < Q; ++i) {
-        const int d = 4 * (l + DL_LANES * i);
-        const float2 lo = floats_of_pair(S[2 * i]), hi = floats_of_pair(S[2 * i + 1]);
-        if (!live) continue;
-        if (VEC) {
-            if (d < dk) *reinterpret_cast<float4*>(mine + d) = make_float4(lo.x, lo.y, hi.x, hi.y);
-        } else {
-            if (d < dk) mine[d] = lo.x;
-            if (d + 1 < dk) mine[d + 1] = lo.y;
-            if (d + 2 < dk) mine[d + 2] = hi.x;
-            if (d + 3 < dk) mine[d + 3] = hi.y;
+    for (int c = 0; c < DL_PER; ++c)
+#pragma unroll
+        for (int i = 0; i < Q; ++i) {
+            const int d = 4 * (l + LANES * i);
+            const float2 lo = floats_of_pair(S[c][2 * i]), hi = floats_of_pair(S[c][2 * i + 1]);
+            if (c >= n_live) continue;
+            float* col = mine + (long long)c * dk;
+            if (VEC) {
+                if (d < dk) *reinterpret_cast<float4*>(col + d) = make_float4(lo.x, lo.y, hi.x, hi.y);
+            } else {
+                if (d < dk) col[d] = lo.x;
+                if (d + 1 < dk) col[d + 1] = lo.y;
+                if (d + 2 < dk) col[d + 2] = hi.x;
+                if (d + 3 < dk) col[d + 3] = hi.y;
+            }
         }
-    }
 }
 
 }  // namespace mu
@@ -294,7 +331,6 @@ MU_EXPORT int mu_delta_scan(const float* qkv, int channels, const float* kq, con
         return MU_ERR_BAD_ARGUMENT;
     if (dk > mu::DL_MAX_DK) return MU_ERR_UNSUPPORTED_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid(n_seqs, n_heads, (dv + mu::DL_COLS - 1) / mu::DL_COLS);
     const bool vec = dk % 4 == 0 && dv % 4 == 0 && channels % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0 &&
                      (reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(state) |
                       (per_channel ? reinterpret_cast<uintptr_t>(decay) : 0)) % 16 == 0;
@@ -304,11 +340,12 @@ MU_EXPORT int mu_delta_scan(const float* qkv, int channels, const float* kq, con
     // memory as shared memory several blocks fit, and the state is read once, so the L1 is no loss
 #define MU_DELTA_SCAN_V(R, LANES, V, PC)                                                                              \
     do {                                                                                                              \
-        const size_t smem = 2 * sizeof(float) * mu::dl_chunk_floats(LANES * R, PC);                                   \
+        const size_t smem = 2 * sizeof(float) * mu::dl_chunk_floats(LANES * R, mu::dl_columns(LANES), PC);            \
+        const dim3 grid(n_seqs, n_heads, (dv + mu::dl_columns(LANES) - 1) / mu::dl_columns(LANES));                   \
         auto kernel = mu::delta_scan_kernel<R, LANES, V, PC>;                                                         \
         if (!mu::allow_shared((const void*)kernel, smem)) return MU_ERR_LAUNCH;                                       \
         mu::prefer_shared_memory((const void*)kernel);                                                                \
-        const dim3 block(LANES * mu::DL_COLS);                                                                        \
+        const dim3 block(mu::DL_THREADS);                                                                             \
         if (long_steps)                                                                                               \
             return mu::launch_after(kernel, grid, block, smem, s, qkv, channels, kq, beta, decay, n_heads,            \
                                     n_kv_heads, dk, dv, seq_first, seq_slots, state, state_stride, state_offset, out); \
@@ -323,9 +360,9 @@ MU_EXPORT int mu_delta_scan(const float* qkv, int channels, const float* kq, con
         MU_DELTA_SCAN_V(R, LANES, false, false);                                                                      \
     } while (0)
     if (dk <= 32) MU_DELTA_SCAN(4, 8);
-    if (dk <= 64) MU_DELTA_SCAN(8, 8);
-    if (dk <= 128) MU_DELTA_SCAN(16, 8);
-    MU_DELTA_SCAN(32, 8);
+    if (dk <= 64) MU_DELTA_SCAN(4, 16);
+    if (dk <= 128) MU_DELTA_SCAN(8, 16);
+    MU_DELTA_SCAN(16, 16);
 #undef MU_DELTA_SCAN_V
 #undef MU_DELTA_SCAN
 }

@@ -372,10 +372,10 @@ low_rank_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowR
     }
 }
 
-// The same on tensor cores for steps of many tokens with bfloat16 weights: a block takes 64 tokens x 64 channels of one
-// part, a warp 16 tokens.  The tokens' rows enter as two bfloat16 terms (rounded, and what the rounding left), so a
+// The same on tensor cores for steps of many tokens with bfloat16 weights: a block takes 64 tokens x 128 channels of one
+// part, a warp 16 tokens x 64 channels.  The tokens' rows enter as two bfloat16 terms (rounded, and what the rounding left), so a
 // product keeps 16 bits of the row and all of the weight; float32 accumulators.  rank: a multiple of 16.
-constexpr int LM_TOK = 64, LM_CH = 64, LM_PAD = 8;
+constexpr int LM_TOK = 64, LM_CH = 128, LM_PAD = 8, LM_THREADS = 256;
 
 __device__ __forceinline__ void lm_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -387,9 +387,9 @@ __device__ __forceinline__ void lm_ldmatrix(uint32_t (&r)[4], const __nv_bfloat1
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
 }
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(LM_THREADS)
 low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowRankPart p0, LowRankPart p1, int blocks0) {
-    extern __shared__ __align__(16) unsigned char lm_raw[];  // weights [64][pitch], rows' two terms [64][pitch] each
+    extern __shared__ __align__(16) unsigned char lm_raw[];  // weights [128][pitch], rows' two terms [64][pitch] each
     pdl_trigger();
     const bool second = (int)blockIdx.y >= blocks0;
     const LowRankPart p = second ? p1 : p0;
@@ -398,19 +398,23 @@ low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, 
     __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(lm_raw);
     __nv_bfloat16* hi = ws + LM_CH * pitch;
     __nv_bfloat16* lo = hi + LM_TOK * pitch;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
-    for (int i = tid; i < LM_CH * pieces; i += 128) {        // (the weights: nothing in flight writes them)
+    const int tid = threadIdx.x, warp = (tid >> 5) & 3, half0 = (tid >> 7) * (LM_CH / 2);
+    const int lane = tid & 31, gid = lane >> 2, tig = lane & 3;
+#pragma unroll 4
+    for (int i = tid; i < LM_CH * pieces; i += LM_THREADS) {        // (the weights: nothing in flight writes them)
         const int r = i / pieces, c = 8 * (i % pieces);
         const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.w) + (long long)min(c0 + r, p.n - 1) * p.ldw + c;
         *reinterpret_cast<uint4*>(ws + r * pitch + c) = *reinterpret_cast<const uint4*>(src);
     }
     pdl_wait();
-    for (int i = tid; i < LM_TOK * (p.rank / 4); i += 128) {
+    const bool wide = ldl % 4 == 0 && p.col % 4 == 0 && ((uintptr_t)low & 15) == 0;
+#pragma unroll 4
+    for (int i = tid; i < LM_TOK * (p.rank / 4); i += LM_THREADS) {
         const int r = i / (p.rank / 4), c = 4 * (i % (p.rank / 4));
         float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (t0 + r < n_tokens) {
             const float* src = low + (long long)(t0 + r) * ldl + p.col + c;
-            x = make_float4(src[0], src[1], src[2], src[3]);
+            x = wide ? *reinterpret_cast<const float4*>(src) : make_float4(src[0], src[1], src[2], src[3]);
         }
         const __nv_bfloat162 h0 = __floats2bfloat162_rn(x.x, x.y), h1 = __floats2bfloat162_rn(x.z, x.w);
         __nv_bfloat162* hp = reinterpret_cast<__nv_bfloat162*>(hi + r * pitch + c);
@@ -420,15 +424,15 @@ low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, 
         lp[1] = __floats2bfloat162_rn(x.z - __low2float(h1), x.w - __high2float(h1));
     }
     __syncthreads();
-    float acc[LM_CH / 8][4] = {};
+    float acc[LM_CH / 16][4] = {};
     for (int kk = 0; kk < p.rank; kk += 16) {
         uint32_t ah[4], al[4], bf[4];
         const int arow = (warp * 16 + (lane & 15)) * pitch + kk + (lane >> 4) * 8;
         lm_ldmatrix(ah, hi + arow);
         lm_ldmatrix(al, lo + arow);
 #pragma unroll
-        for (int j = 0; j < LM_CH / 8; j += 2) {
-            lm_ldmatrix(bf, ws + (j * 8 + (lane & 7) + (lane >> 4) * 8) * pitch + kk + ((lane >> 3) & 1) * 8);
+        for (int j = 0; j < LM_CH / 16; j += 2) {
+            lm_ldmatrix(bf, ws + (half0 + j * 8 + (lane & 7) + (lane >> 4) * 8) * pitch + kk + ((lane >> 3) & 1) * 8);
             lm_mma(acc[j], ah, bf[0], bf[1]);
             lm_mma(acc[j], al, bf[0], bf[1]);
             lm_mma(acc[j + 1], ah, bf[2], bf[3]);
@@ -436,19 +440,28 @@ low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, 
         }
     }
 #pragma unroll
-    for (int j = 0; j < LM_CH / 8; ++j)
+    for (int j = 0; j < LM_CH / 16; ++j) {
+        const int c = c0 + half0 + j * 8 + tig * 2;          // this thread's two channels
+        if (c >= p.n) continue;
+        const bool two = c + 1 < p.n;
+        const int d = two ? c + 1 : c;
+        const float bias0 = p.bias ? p.bias[c] : 0.0f, bias1 = p.bias ? p.bias[d] : 0.0f;
+        const float rate0 = p.fn == 2 ? expf(p.a_log[c / p.per_head]) : 0.0f;
+        const float rate1 = p.fn == 2 ? expf(p.a_log[d / p.per_head]) : 0.0f;
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int c = c0 + j * 8 + tig * 2 + e;
-            if (c >= p.n) continue;
-            const float bias = p.bias ? p.bias[c] : 0.0f;
-            const float rate = p.fn == 2 ? expf(p.a_log[c / p.per_head]) : 0.0f;
-#pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int t = t0 + warp * 16 + gid + 8 * half;
-                if (t < n_tokens) p.out[(long long)t * p.n + c] = low_rank_fn(acc[j][2 * half + e] + bias, p, rate);
+        for (int half = 0; half < 2; ++half) {
+            const int t = t0 + warp * 16 + gid + 8 * half;
+            if (t >= n_tokens) continue;
+            const float y0 = low_rank_fn(acc[j][2 * half] + bias0, p, rate0), y1 = low_rank_fn(acc[j][2 * half + 1] + bias1, p, rate1);
+            float* dst = p.out + (long long)t * p.n + c;
+            if (two && p.n % 2 == 0) {
+                *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
+            } else {
+                dst[0] = y0;
+                if (two) dst[1] = y1;
             }
         }
+    }
 }
 
 }  // namespace mu
@@ -537,13 +550,14 @@ MU_EXPORT int mu_low_rank(const float* low, long long ldl, int n_tokens, const m
     // steps of many tokens with weights in whole 16-byte pieces: tensor cores
     bool tc = w_bf16 && n_tokens >= 64;
     for (int i = 0; i < n_parts; ++i)
-        tc = tc && parts[i].rank % 16 == 0 && parts[i].rank <= 512 && parts[i].ldw % 8 == 0 && ((uintptr_t)parts[i].w & 15) == 0;
+        tc = tc && parts[i].rank % 16 == 0 && parts[i].rank <= 384 && parts[i].ldw % 8 == 0 && ((uintptr_t)parts[i].w & 15) == 0;
     if (tc) {
         int by[2] = {0, 0};
         for (int i = 0; i < n_parts; ++i) by[i] = (parts[i].n + mu::LM_CH - 1) / mu::LM_CH;
         const size_t bytes = (size_t)(mu::LM_CH + 2 * mu::LM_TOK) * (rank + mu::LM_PAD) * sizeof(__nv_bfloat16);
         if (!mu::allow_shared((const void*)mu::low_rank_mma_kernel, 220 * 1024)) return MU_ERR_LAUNCH;
-        return mu::launch_pdl(mu::low_rank_mma_kernel, dim3((n_tokens + mu::LM_TOK - 1) / mu::LM_TOK, by[0] + by[1]), dim3(128),
+        return mu::launch_pdl(mu::low_rank_mma_kernel, dim3((n_tokens + mu::LM_TOK - 1) / mu::LM_TOK, by[0] + by[1]),
+                              dim3(mu::LM_THREADS),
                               bytes, s, 1, low, ldl, n_tokens, p0, p1, by[0]);
     }
     const int tok = n_tokens >= 256 ? 16 : n_tokens >= 8 ? 4 : 1;
