@@ -21,7 +21,8 @@
 //                  maximum is kept changes no result; it is found for 256 tokens at a time by a scan.
 // mu_low_rank      out[t][c] = fn( sum_r W[c][r] low[t][r] + bias[c] ): the second of a projection's two matrices, for
 //                  one or two such projections in one launch, with what follows it:
-//                  (bfloat16 weights and many tokens: tensor cores, else one running sum per output over r.)
+//                  (bfloat16 weights and many tokens: tensor cores; few tokens: eight lanes an output; else one
+//                  running sum per output over r.)
 //                  fn 0: nothing;  1: sigmoid(z)^power;  2: exp(-exp(A_log[c / per_head]) softplus(z)).
 #include "common.cuh"
 
@@ -282,7 +283,7 @@ exp_gates_kernel(const float* __restrict__ i_raw, const float* __restrict__ f_ra
     if (tid == 0) *kept = carry;
 }
 
-constexpr int LR_CHANNELS = 128, LR_THREADS = 64;            // a thread takes two channels
+constexpr int LR_CHANNELS = 128, LR_THREADS = 64, LR_TOK = 16;           // a thread takes two channels
 struct LowRankPart {
     const void* w;            // [n][ldw], the first `rank` entries of a row
     const float* bias;        // [n] or null
@@ -304,30 +305,30 @@ template <int N, typename T> __device__ __forceinline__ void load_weights(float 
     for (int i = 0; i < N; ++i) x[i] = i < n ? to_float(p[i]) : 0.0f;
 }
 
-// A block: TOK tokens x 128 channels of one of the parts.  The tokens' low-rank rows are staged in shared memory; a
+// A block: 16 tokens x 128 channels of one of the parts.  The tokens' low-rank rows are staged in shared memory; a
 // thread keeps eight weights of each of its two channels and runs over the tokens.  One running sum per output over r
 // in order, whatever shares its block.
-template <typename TW, int TOK>
+template <typename TW>
 __global__ void __launch_bounds__(LR_THREADS)
 low_rank_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowRankPart p0, LowRankPart p1, int blocks0) {
-    extern __shared__ __align__(16) float lr_smem[];         // [TOK][rank padded to 8]
+    extern __shared__ __align__(16) float lr_smem[];         // [LR_TOK][rank padded to 8]
     pdl_trigger();
     const bool second = (int)blockIdx.y >= blocks0;
     const LowRankPart p = second ? p1 : p0;
     const int c0 = ((int)blockIdx.y - (second ? blocks0 : 0)) * LR_CHANNELS + threadIdx.x, c1 = c0 + LR_THREADS;
-    const int t0 = blockIdx.x * TOK, nt = min(TOK, n_tokens - t0);
+    const int t0 = blockIdx.x * LR_TOK, nt = min(LR_TOK, n_tokens - t0);
     const int rp = (p.rank + 7) & ~7;
     pdl_wait();
-    for (int i = threadIdx.x; i < TOK * rp; i += LR_THREADS) {
+    for (int i = threadIdx.x; i < LR_TOK * rp; i += LR_THREADS) {
         const int t = i / rp, r = i % rp;
         lr_smem[i] = t < nt && r < p.rank ? low[(long long)(t0 + t) * ldl + p.col + r] : 0.0f;
     }
     __syncthreads();
     const TW* w0 = reinterpret_cast<const TW*>(p.w) + (long long)min(c0, p.n - 1) * p.ldw;
     const TW* w1 = reinterpret_cast<const TW*>(p.w) + (long long)min(c1, p.n - 1) * p.ldw;
-    float a0[TOK], a1[TOK];
+    float a0[LR_TOK], a1[LR_TOK];
 #pragma unroll
-    for (int t = 0; t < TOK; ++t) a0[t] = a1[t] = 0.0f;
+    for (int t = 0; t < LR_TOK; ++t) a0[t] = a1[t] = 0.0f;
     const bool vec = sizeof(TW) == 2 && p.ldw % 8 == 0 && ((uintptr_t)p.w & 15) == 0;
     for (int r = 0; r < p.rank; r += 8) {
         float x0[8], x1[8];
@@ -345,7 +346,7 @@ low_rank_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowR
             load_weights<8>(x1, w1 + r, p.rank - r);
         }
 #pragma unroll
-        for (int t = 0; t < TOK; ++t) {
+        for (int t = 0; t < LR_TOK; ++t) {
             const float4 y = *reinterpret_cast<const float4*>(lr_smem + t * rp + r);
             const float4 z = *reinterpret_cast<const float4*>(lr_smem + t * rp + r + 4);
             a0[t] = fmaf(x0[0], y.x, a0[t]), a1[t] = fmaf(x1[0], y.x, a1[t]);
@@ -365,16 +366,88 @@ low_rank_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowR
         const float bias = p.bias ? p.bias[c] : 0.0f;
         const float rate = p.fn == 2 ? expf(p.a_log[c / p.per_head]) : 0.0f;
 #pragma unroll
-        for (int t = 0; t < TOK; ++t) {
+        for (int t = 0; t < LR_TOK; ++t) {
             if (t >= nt) break;
             p.out[(long long)(t0 + t) * p.n + c] = low_rank_fn((half ? a1[t] : a0[t]) + bias, p, rate);
         }
     }
 }
 
+// The same for a few tokens (single-token steps above all): eight lanes share a channel and take its weights eight
+// entries at a time in turn, so that a row's weights are on their way at once; the lanes' sums meet by shuffles, and
+// lane i finishes token i of the block's four.
+constexpr int LF_TOK = 4, LF_THREADS = 128, LF_CHANNELS = LF_THREADS / 8;
+
+template <typename TW>
+__global__ void __launch_bounds__(LF_THREADS)
+low_rank_few_kernel(const float* __restrict__ low, long long ldl, int n_tokens, LowRankPart p0, LowRankPart p1, int blocks0) {
+    pdl_trigger();
+    const bool second = (int)blockIdx.y >= blocks0;
+    const LowRankPart p = second ? p1 : p0;
+    const int lane = threadIdx.x & 7, c = ((int)blockIdx.y - (second ? blocks0 : 0)) * LF_CHANNELS + (threadIdx.x >> 3);
+    const int t0 = blockIdx.x * LF_TOK, nt = min(LF_TOK, n_tokens - t0);
+    const TW* w = reinterpret_cast<const TW*>(p.w) + (long long)min(c, p.n - 1) * p.ldw;
+    const bool vec = sizeof(TW) == 2 && p.ldw % 8 == 0 && ((uintptr_t)p.w & 15) == 0;
+    const bool wide = ldl % 4 == 0 && p.col % 4 == 0 && ((uintptr_t)low & 15) == 0;
+    float acc[LF_TOK] = {};
+    bool ready = false;
+#pragma unroll 2
+    for (int r = 8 * lane; r < p.rank; r += 64) {
+        float x[8];
+        if (vec && r + 8 <= p.rank) {
+            const uint4 u = *reinterpret_cast<const uint4*>(w + r);
+            const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 f = __bfloat1622float2(b[i]);
+                x[2 * i] = f.x, x[2 * i + 1] = f.y;
+            }
+        } else {
+            load_weights<8>(x, w + r, p.rank - r);
+        }
+        if (!ready) {                                        // the weights are asked for before the rows are there
+            pdl_wait();
+            ready = true;
+        }
+#pragma unroll
+        for (int t = 0; t < LF_TOK; ++t) {
+            if (t >= nt) break;
+            const float* y = low + (long long)(t0 + t) * ldl + p.col + r;
+            if (wide && r + 8 <= p.rank) {
+                const float4 a = *reinterpret_cast<const float4*>(y), b = *reinterpret_cast<const float4*>(y + 4);
+                acc[t] = fmaf(x[0], a.x, fmaf(x[1], a.y, fmaf(x[2], a.z, fmaf(x[3], a.w, acc[t]))));
+                acc[t] = fmaf(x[4], b.x, fmaf(x[5], b.y, fmaf(x[6], b.z, fmaf(x[7], b.w, acc[t]))));
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                    if (r + i < p.rank) acc[t] = fmaf(x[i], y[i], acc[t]);
+            }
+        }
+    }
+    if (!ready) pdl_wait();
+#pragma unroll
+    for (int t = 0; t < LF_TOK; ++t)
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) acc[t] += __shfl_xor_sync(0xffffffffu, acc[t], o);
+    const float z = lane == 0 ? acc[0] : lane == 1 ? acc[1] : lane == 2 ? acc[2] : acc[3];
+    if (lane >= nt || c >= p.n) return;
+    const float rate = p.fn == 2 ? expf(p.a_log[c / p.per_head]) : 0.0f;
+    p.out[(long long)(t0 + lane) * p.n + c] = low_rank_fn(z + (p.bias ? p.bias[c] : 0.0f), p, rate);
+}
+
 // The same on tensor cores for steps of many tokens with bfloat16 weights: a block takes 64 tokens x 128 channels of one
 // part, a warp 16 tokens x 64 channels.  The tokens' rows enter as two bfloat16 terms (rounded, and what the rounding left), so a
 // product keeps 16 bits of the row and all of the weight; float32 accumulators.  rank: a multiple of 16.
+// The decays for the tensor-core kernel (bfloat16 models): softplus with the fast exponential and logarithm, a series
+// where e^-|z| is small (its next term is 3e-9), so that a decay is off by a few of its own roundings; the exact
+// functions cost several times the product.
+__device__ __forceinline__ float low_rank_fn_fast(float z, const LowRankPart& p, float rate) {
+    if (p.fn == 0) return z;
+    const float y = p.fn == 1 ? -z : z, e = __expf(-fabsf(y));
+    const float tail = e < 0.01f ? e * fmaf(e, fmaf(e, 1.0f / 3.0f, -0.5f), 1.0f) : __logf(1.0f + e);
+    return __expf(-(p.fn == 1 ? p.power : rate) * (fmaxf(y, 0.0f) + tail));
+}
+
 constexpr int LM_TOK = 64, LM_CH = 128, LM_PAD = 8, LM_THREADS = 256;
 
 __device__ __forceinline__ void lm_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -394,34 +467,38 @@ low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, 
     const bool second = (int)blockIdx.y >= blocks0;
     const LowRankPart p = second ? p1 : p0;
     const int c0 = ((int)blockIdx.y - (second ? blocks0 : 0)) * LM_CH, t0 = blockIdx.x * LM_TOK;
-    const int pitch = p.rank + LM_PAD, pieces = p.rank / 8;
+    const int pitch = p.rank + LM_PAD;
     __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(lm_raw);
     __nv_bfloat16* hi = ws + LM_CH * pitch;
     __nv_bfloat16* lo = hi + LM_TOK * pitch;
     const int tid = threadIdx.x, warp = (tid >> 5) & 3, half0 = (tid >> 7) * (LM_CH / 2);
     const int lane = tid & 31, gid = lane >> 2, tig = lane & 3;
-#pragma unroll 4
-    for (int i = tid; i < LM_CH * pieces; i += LM_THREADS) {        // (the weights: nothing in flight writes them)
-        const int r = i / pieces, c = 8 * (i % pieces);
-        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.w) + (long long)min(c0 + r, p.n - 1) * p.ldw + c;
-        *reinterpret_cast<uint4*>(ws + r * pitch + c) = *reinterpret_cast<const uint4*>(src);
+    // sixteen threads a row, sixteen rows at a time
+    const int row0 = tid >> 4, piece0 = tid & 15;
+    for (int c = 8 * piece0; c < p.rank; c += 128) {         // (the weights: nothing in flight writes them)
+#pragma unroll
+        for (int r = row0; r < LM_CH; r += LM_THREADS / 16) {
+            const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.w) + (long long)min(c0 + r, p.n - 1) * p.ldw + c;
+            *reinterpret_cast<uint4*>(ws + r * pitch + c) = *reinterpret_cast<const uint4*>(src);
+        }
     }
     pdl_wait();
     const bool wide = ldl % 4 == 0 && p.col % 4 == 0 && ((uintptr_t)low & 15) == 0;
-#pragma unroll 4
-    for (int i = tid; i < LM_TOK * (p.rank / 4); i += LM_THREADS) {
-        const int r = i / (p.rank / 4), c = 4 * (i % (p.rank / 4));
-        float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (t0 + r < n_tokens) {
-            const float* src = low + (long long)(t0 + r) * ldl + p.col + c;
-            x = wide ? *reinterpret_cast<const float4*>(src) : make_float4(src[0], src[1], src[2], src[3]);
+    for (int c = 4 * piece0; c < p.rank; c += 64) {
+#pragma unroll
+        for (int r = row0; r < LM_TOK; r += LM_THREADS / 16) {
+            float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (t0 + r < n_tokens) {
+                const float* src = low + (long long)(t0 + r) * ldl + p.col + c;
+                x = wide ? *reinterpret_cast<const float4*>(src) : make_float4(src[0], src[1], src[2], src[3]);
+            }
+            const __nv_bfloat162 h0 = __floats2bfloat162_rn(x.x, x.y), h1 = __floats2bfloat162_rn(x.z, x.w);
+            __nv_bfloat162* hp = reinterpret_cast<__nv_bfloat162*>(hi + r * pitch + c);
+            __nv_bfloat162* lp = reinterpret_cast<__nv_bfloat162*>(lo + r * pitch + c);
+            hp[0] = h0, hp[1] = h1;
+            lp[0] = __floats2bfloat162_rn(x.x - __low2float(h0), x.y - __high2float(h0));
+            lp[1] = __floats2bfloat162_rn(x.z - __low2float(h1), x.w - __high2float(h1));
         }
-        const __nv_bfloat162 h0 = __floats2bfloat162_rn(x.x, x.y), h1 = __floats2bfloat162_rn(x.z, x.w);
-        __nv_bfloat162* hp = reinterpret_cast<__nv_bfloat162*>(hi + r * pitch + c);
-        __nv_bfloat162* lp = reinterpret_cast<__nv_bfloat162*>(lo + r * pitch + c);
-        hp[0] = h0, hp[1] = h1;
-        lp[0] = __floats2bfloat162_rn(x.x - __low2float(h0), x.y - __high2float(h0));
-        lp[1] = __floats2bfloat162_rn(x.z - __low2float(h1), x.w - __high2float(h1));
     }
     __syncthreads();
     float acc[LM_CH / 16][4] = {};
@@ -452,7 +529,8 @@ low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, 
         for (int half = 0; half < 2; ++half) {
             const int t = t0 + warp * 16 + gid + 8 * half;
             if (t >= n_tokens) continue;
-            const float y0 = low_rank_fn(acc[j][2 * half] + bias0, p, rate0), y1 = low_rank_fn(acc[j][2 * half + 1] + bias1, p, rate1);
+            const float y0 = low_rank_fn_fast(acc[j][2 * half] + bias0, p, rate0);
+            const float y1 = low_rank_fn_fast(acc[j][2 * half + 1] + bias1, p, rate1);
             float* dst = p.out + (long long)t * p.n + c;
             if (two && p.n % 2 == 0) {
                 *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
@@ -560,19 +638,20 @@ MU_EXPORT int mu_low_rank(const float* low, long long ldl, int n_tokens, const m
                               dim3(mu::LM_THREADS),
                               bytes, s, 1, low, ldl, n_tokens, p0, p1, by[0]);
     }
-    const int tok = n_tokens >= 256 ? 16 : n_tokens >= 8 ? 4 : 1;
-    const size_t smem = (size_t)tok * ((rank + 7) / 8 * 8) * sizeof(float);
-    if (smem > 48 * 1024) return MU_ERR_UNSUPPORTED_SIZE;
-    const dim3 grid((n_tokens + tok - 1) / tok, blocks[0] + blocks[1]), block(mu::LR_THREADS);
-#define MU_LOW_RANK(T, TOK)                                                                                           \
-    return mu::launch_pdl(mu::low_rank_kernel<T, TOK>, grid, block, smem, s, 1, low, ldl, n_tokens, p0, p1, blocks[0])
-    if (w_bf16) {
-        if (tok == 16) MU_LOW_RANK(__nv_bfloat16, 16);
-        if (tok == 4) MU_LOW_RANK(__nv_bfloat16, 4);
-        MU_LOW_RANK(__nv_bfloat16, 1);
+    if (n_tokens < 64) {
+        int by[2] = {0, 0};
+        for (int i = 0; i < n_parts; ++i) by[i] = (parts[i].n + mu::LF_CHANNELS - 1) / mu::LF_CHANNELS;
+        const dim3 few((n_tokens + mu::LF_TOK - 1) / mu::LF_TOK, by[0] + by[1]), threads(mu::LF_THREADS);
+        if (w_bf16)
+            return mu::launch_pdl(mu::low_rank_few_kernel<__nv_bfloat16>, few, threads, 0, s, 1, low, ldl, n_tokens, p0, p1, by[0]);
+        return mu::launch_pdl(mu::low_rank_few_kernel<float>, few, threads, 0, s, 1, low, ldl, n_tokens, p0, p1, by[0]);
     }
-    if (tok == 16) MU_LOW_RANK(float, 16);
-    if (tok == 4) MU_LOW_RANK(float, 4);
-    MU_LOW_RANK(float, 1);
+    const size_t smem = (size_t)mu::LR_TOK * ((rank + 7) / 8 * 8) * sizeof(float);
+    if (smem > 48 * 1024) return MU_ERR_UNSUPPORTED_SIZE;
+    const dim3 grid((n_tokens + mu::LR_TOK - 1) / mu::LR_TOK, blocks[0] + blocks[1]), block(mu::LR_THREADS);
+#define MU_LOW_RANK(T)                                                                                                \
+    return mu::launch_pdl(mu::low_rank_kernel<T>, grid, block, smem, s, 1, low, ldl, n_tokens, p0, p1, blocks[0])
+    if (w_bf16) MU_LOW_RANK(__nv_bfloat16);
+    MU_LOW_RANK(float);
 #undef MU_LOW_RANK
 }

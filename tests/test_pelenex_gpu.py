@@ -567,6 +567,21 @@ def test_low_rank_kernel(dtype, T):
         assert np.abs(host(outs[2]) - plain.sigmoid(za) ** 0.125).max() < 2e-5
 
 
+def test_decays_near_one_keep_their_distance_from_it():
+    """Slow channels: one minus the decay is what matters over hundreds of tokens, in both forms of the kernel."""
+    ops = _ops()
+    z = np.linspace(-12.0, 12.0, 256)
+    for T, dtype in ((3, torch.bfloat16), (128, torch.bfloat16), (128, torch.float32)):
+        out, bias, zero = torch.zeros((T, 256), device="cuda"), dev(z), dev(np.zeros((256, 16)), dtype)
+        low, a_log = torch.zeros((T, 16), device="cuda"), dev(np.array([-3.0, 0.5]))
+        for fn, more, want in (("exp_softplus", {"a_log": a_log}, -np.repeat(np.exp([-3.0, 0.5]), 128) * plain.softplus(z)),
+                               ("sigmoid_power", {"power": 1.0 / 16}, -plain.softplus(-z) / 16)):
+            ops.low_rank(low, dtype, ops.low_rank_part(zero, 0, out, bias=bias, fn=fn, **more))
+            assert np.abs(host(out)[-1] - np.exp(want)).max() < 4e-7, fn
+            near = want > -1e-2
+            assert np.abs((host(out)[-1] - 1.0 - np.expm1(want))[near]).max() < 1.5e-7, fn
+
+
 # Cuts of two sequences into shared steps: portions of 1, 2 and many, one sequence ending before the other.
 CUTS = [[(0, 2), (2, 3), (3, 20), (20, 21), (21, 22), (22, 300)], [(0, 1), (1, 3), (3, 20), (20, 21), (21, 21), (21, 21)]]
 
