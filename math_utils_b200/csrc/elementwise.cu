@@ -47,7 +47,7 @@ __global__ void embed_pair_kernel(const int* __restrict__ ids, const int* __rest
                                   const int* __restrict__ seq_slots, int* __restrict__ last_token,
                                   const TW* __restrict__ table, const TW* __restrict__ pair_table, float* __restrict__ x,
                                   __nv_bfloat16* __restrict__ copy, int hidden, int buckets, long long mul_prev,
-                                  long long mul_cur, int remember) {
+                                  long long mul_cur, int remember, float scale) {
     __shared__ long long pair_row;
     pdl_trigger();
     pdl_wait();
@@ -70,7 +70,7 @@ __global__ void embed_pair_kernel(const int* __restrict__ ids, const int* __rest
     float* dst = x + (long long)t * hidden;
 #pragma unroll 4
     for (int d = threadIdx.x; d < hidden; d += blockDim.x) {
-        const float v = to_float(src[d]) + to_float(psrc[d]);
+        const float v = fmaf(to_float(src[d]), scale, to_float(psrc[d]));
         dst[d] = v;
         if (copy) copy[(long long)t * hidden + d] = __float2bfloat16_rn(v);    // the first sublayer's input
     }
@@ -213,12 +213,12 @@ MU_EXPORT int mu_embed(const int* ids, const int* pos, const void* table, const 
                           (const float*)table, (const float*)pos_table, x, hidden, scale, turns);
 }
 
-// Token rows plus hashed rows of (token before, token); single_tokens: every sequence brings one token.
+// Token rows times `scale` plus hashed rows of (token before, token); single_tokens: every sequence brings one token.
 // copy (optional, bfloat16 [n_tokens][hidden]): the same rows rounded, for a first sublayer that reads the stream itself.
 MU_EXPORT int mu_embed_pair(const int* ids, const int* pos, const int* tok_seq, const int* seq_first, const int* seq_slots,
                             int* last_token, const void* table, const void* pair_table, float* x, void* copy, int n_tokens, int n_seqs,
                             int hidden, int buckets, long long mul_prev, long long mul_cur, int table_bf16,
-                            int single_tokens, void* stream) {
+                            int single_tokens, void* stream, float scale) {
     if (n_tokens <= 0) return MU_OK;
     if (hidden <= 0 || buckets <= 0 || !ids || !pos || !tok_seq || !seq_first || !seq_slots || !last_token || !table ||
         !pair_table || !x)
@@ -229,10 +229,10 @@ MU_EXPORT int mu_embed_pair(const int* ids, const int* pos, const int* tok_seq, 
         table_bf16 ? mu::launch_pdl(mu::embed_pair_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, s, 1, ids, pos,
                                     tok_seq, seq_slots, last_token, (const __nv_bfloat16*)table,
                                     (const __nv_bfloat16*)pair_table, x, (__nv_bfloat16*)copy, hidden, buckets, mul_prev,
-                                    mul_cur, single_tokens)
+                                    mul_cur, single_tokens, scale)
                    : mu::launch_pdl(mu::embed_pair_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, 1, ids, pos, tok_seq,
                                     seq_slots, last_token, (const float*)table, (const float*)pair_table, x,
-                                    (__nv_bfloat16*)copy, hidden, buckets, mul_prev, mul_cur, single_tokens);
+                                    (__nv_bfloat16*)copy, hidden, buckets, mul_prev, mul_cur, single_tokens, scale);
     if (code != MU_OK || single_tokens) return code;
     return mu::launch_pdl(mu::remember_tokens_kernel, dim3((n_seqs + 127) / 128), dim3(128), 0, s, 1, ids, seq_first,
                           seq_slots, last_token, n_seqs);

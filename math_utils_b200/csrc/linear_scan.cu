@@ -5,7 +5,9 @@
 // mu_linear_scan   per (sequence, head, a few columns of S), the step's tokens in order.  The decay is one number per
 //                  head (with a `take` beside it) or one per head and key channel (gated linear attention).  With a
 //                  normalizer the state has one more column, n <- decay n + take k, whose read-out n . q goes to an
-//                  array of its own (the matrix memory of xLSTM).  State of a slot, from state_offset on:
+//                  array of its own (the matrix memory of xLSTM).  Gates that are the same for every token (lightning
+//                  attention's constant decays) are read with a token stride of zero; with `silu_rows` keys, queries and
+//                  values pass silu once they are staged.  State of a slot, from state_offset on:
 //                  [ S: heads x dv x dk (a head's S column after column) | n: heads x dk ].
 //                  Four columns live in the registers of up to 32 lanes, two entries to a 64-bit register; a key, a
 //                  query and a decay read from shared memory serve four columns.  Nothing waits for a token's
@@ -23,7 +25,7 @@
 //                  one or two such projections in one launch, with what follows it:
 //                  (bfloat16 weights and many tokens: tensor cores; few tokens: eight lanes an output; else one
 //                  running sum per output over r.)
-//                  fn 0: nothing;  1: sigmoid(z)^power;  2: exp(-exp(A_log[c / per_head]) softplus(z)).
+//                  fn 0: nothing;  1: sigmoid(z)^power;  2: exp(-exp(A_log[c / per_head]) softplus(z));  3: softplus(z).
 #include "common.cuh"
 
 #include <math.h>
@@ -42,6 +44,8 @@ __host__ __device__ constexpr int ls_chunk_floats(int dkp, int cols, bool per_ch
     return LS_CHUNK * ((per_channel ? 3 : 2) * dkp + cols + 4);
 }
 
+__device__ __forceinline__ float ls_silu(float z) { return z / (1.0f + expf(-z)); }
+
 // LANES lanes hold four columns of S, R entries of each a lane (a multiple of 4; dk <= LANES R), dealt to the lanes
 // four entries at a time: what a lane reads of a staged key, query and decay serves its four columns.  LANES and R
 // follow from dk alone.  VEC: every row, slice and state column starts on a 16-byte boundary.
@@ -51,7 +55,7 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
                    const float* __restrict__ decay, int n_heads, int dk, int dv, float scale,
                    const int* __restrict__ seq_first, const int* __restrict__ seq_slots, float* __restrict__ state,
                    long long state_stride, long long state_offset, float* __restrict__ out, long long ldo,
-                   float* __restrict__ norm_out) {
+                   float* __restrict__ norm_out, long long gate_stride, int silu_rows) {
     constexpr int DKP = LANES * R, Q = R / 4, COLS = ls_columns(LANES), BUF = ls_chunk_floats(DKP, COLS, PER_CHANNEL);
     constexpr int GROUP = LANES / LS_PER;                    // tokens whose read-outs are summed together
     extern __shared__ __align__(16) float ls_smem[];
@@ -125,7 +129,7 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
             }
         }
         if (!PER_CHANNEL)
-            for (int tok = tid; tok < n; tok += LS_THREADS) copy_async16(sc + tok * 4, decay + 4 * ((t0 + tok) * n_heads + h));
+            for (int tok = tid; tok < n; tok += LS_THREADS) copy_async16(sc + tok * 4, decay + (t0 + tok) * gate_stride + 4 * h);
         copy_async_commit();
     };
     __syncthreads();                                         // the zeros are down before the first copies land
@@ -140,6 +144,16 @@ linear_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, con
             copy_async_wait<0>();
         }
         __syncthreads();
+        if (silu_rows) {                                     // (zeros stay zeros)
+            float* rows = ls_smem + b * BUF;
+            for (int i = tid; i < n * DKP; i += LS_THREADS) {
+                rows[i] = ls_silu(rows[i]);
+                rows[LS_CHUNK * DKP + i] = ls_silu(rows[LS_CHUNK * DKP + i]);
+            }
+            float* values = rows + (PER_CHANNEL ? 3 : 2) * LS_CHUNK * DKP;
+            for (int i = tid; i < n * COLS; i += LS_THREADS) values[i] = ls_silu(values[i]);
+            __syncthreads();
+        }
         const float* ks = ls_smem + b * BUF;
         const float* qs = ks + LS_CHUNK * DKP;
         const float* gs = qs + LS_CHUNK * DKP;
@@ -297,6 +311,7 @@ struct LowRankPart {
 __device__ __forceinline__ float low_rank_fn(float z, const LowRankPart& p, float rate) {
     if (p.fn == 1) return expf(-p.power * softplus(-z));
     if (p.fn == 2) return expf(-rate * softplus(z));
+    if (p.fn == 3) return softplus(z);
     return z;
 }
 
@@ -445,6 +460,7 @@ __device__ __forceinline__ float low_rank_fn_fast(float z, const LowRankPart& p,
     if (p.fn == 0) return z;
     const float y = p.fn == 1 ? -z : z, e = __expf(-fabsf(y));
     const float tail = e < 0.01f ? e * fmaf(e, fmaf(e, 1.0f / 3.0f, -0.5f), 1.0f) : __logf(1.0f + e);
+    if (p.fn == 3) return fmaxf(y, 0.0f) + tail;
     return __expf(-(p.fn == 1 ? p.power : rate) * (fmaxf(y, 0.0f) + tail));
 }
 
@@ -548,18 +564,18 @@ low_rank_mma_kernel(const float* __restrict__ low, long long ldl, int n_tokens, 
 MU_EXPORT int mu_linear_scan_max_dk() { return mu::LS_MAX_DK; }
 
 // q, k [T][heads * dk], v [T][heads * dv]: float32 slices of rows `ld` apart.  per_channel: decay is [T][heads * dk];
-// else [T][heads][4] = (decay, take, -, -).  norm_out (may be null; not with per_channel): [T][heads].  long_steps:
+// else [T][heads][4] = (decay, take, -, -), a token's gates `gate_stride` floats after the one's before (0: the same for all).  norm_out (may be null; not with per_channel): [T][heads].  long_steps:
 // many tokens a sequence; the launch then waits for an empty device.
 MU_EXPORT int mu_linear_scan(const float* q, const float* k, const float* v, long long ld, const float* decay,
                              int per_channel, int n_seqs, int n_heads, int dk, int dv, float scale,
                              const int* seq_first, const int* seq_slots, float* state, long long state_stride,
                              long long state_offset, float* out, long long ldo, float* norm_out, int long_steps,
-                             void* stream) {
+                             void* stream, long long gate_stride, int silu_rows) {
     if (n_seqs <= 0) return MU_OK;
     if (!q || !k || !v || !decay || !seq_first || !seq_slots || !state || !out || n_heads <= 0 || dk <= 0 || dv <= 0)
         return MU_ERR_BAD_ARGUMENT;
     if (dk > mu::LS_MAX_DK) return MU_ERR_UNSUPPORTED_SIZE;
-    if (!per_channel && ((uintptr_t)decay & 15)) return MU_ERR_ALIGNMENT;
+    if (!per_channel && (((uintptr_t)decay & 15) || gate_stride % 4)) return MU_ERR_ALIGNMENT;
     cudaStream_t s = (cudaStream_t)stream;
     const int cols = dv + (norm_out ? 1 : 0);
     const bool vec = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0 &&
@@ -574,9 +590,11 @@ MU_EXPORT int mu_linear_scan(const float* q, const float* k, const float* v, lon
         mu::prefer_shared_memory((const void*)kernel);                                                                \
         if (long_steps)                                                                                               \
             return mu::launch_after(kernel, grid, block, smem, s, q, k, v, ld, decay, n_heads, dk, dv, scale,         \
-                                    seq_first, seq_slots, state, state_stride, state_offset, out, ldo, norm_out);     \
+                                    seq_first, seq_slots, state, state_stride, state_offset, out, ldo, norm_out,      \
+                                    gate_stride, silu_rows);                                                          \
         return mu::launch_pdl(kernel, grid, block, smem, s, 1, q, k, v, ld, decay, n_heads, dk, dv, scale, seq_first, \
-                              seq_slots, state, state_stride, state_offset, out, ldo, norm_out);                      \
+                              seq_slots, state, state_stride, state_offset, out, ldo, norm_out, gate_stride,          \
+                              silu_rows);                                                                             \
     } while (0)
 #define MU_LINEAR_SCAN(R, LANES)                                                                                      \
     do {                                                                                                              \
@@ -617,7 +635,7 @@ MU_EXPORT int mu_low_rank(const float* low, long long ldl, int n_tokens, const m
     int blocks[2] = {0, 0}, rank = 0;
     for (int i = 0; i < n_parts; ++i) {
         const mu::LowRankPart& p = parts[i];
-        if (!p.w || !p.out || p.rank <= 0 || p.n <= 0 || p.col < 0 || p.ldw < p.rank || p.fn < 0 || p.fn > 2 ||
+        if (!p.w || !p.out || p.rank <= 0 || p.n <= 0 || p.col < 0 || p.ldw < p.rank || p.fn < 0 || p.fn > 3 ||
             (p.fn == 2 && (!p.a_log || p.per_head <= 0)))
             return MU_ERR_BAD_ARGUMENT;
         blocks[i] = (p.n + mu::LR_CHANNELS - 1) / mu::LR_CHANNELS;

@@ -11,8 +11,10 @@
 //                      i + rot_dims / 2 by the angle position * freq[i]; cos and sin times a magnitude);
 //                      queries are written back in place, keys and values go to the token's cache row.
 //                      Statistics, angles, cos and sin are float32 whatever the storage type.
-//                      Options for other designs: a null weight leaves the slices as they are (no norm);
-//                      `pairs` rotates entry 2i with entry 2i + 1 instead of entry i with entry i + rot_dims / 2.
+//                      Options for other designs: a null weight leaves the slices as they are (no norm; without a
+//                      rotation the queries are then not touched);
+//                      `pairs` rotates entry 2i with entry 2i + 1 instead of entry i with entry i + rot_dims / 2;
+//                      `shared` keeps rows of keys alone, for attention whose values are the cached keys themselves.
 // mu_mapped_attention  per (token, head): softmax attention of each map over the keys the token sees
 //                      (positions max(0, p - window + 1) .. p; window 0: all of 0 .. p), both maps over the
 //                      same values.  With two maps the result is a1 - lambda * a2, brought to unit rms over
@@ -26,7 +28,10 @@
 //                      position p sees the positions p - p % c .. p only, chunks counted from position 0 of the
 //                      sequence; it replaces the window), `slopes` (one float per head: the score of a key at
 //                      distance n loses slopes[h] * n), `keep` (with a window: the sequence's first `keep`
-//                      positions stay in sight of every later token, at their true distances).
+//                      positions stay in sight of every later token, at their true distances), `softcap` (c > 0: the
+//                      scaled score s becomes c tanh(s / c), before any slope), `gate_each` (the gate has one entry per
+//                      value entry, [T, heads * vdim]), `shared` (the values are the cached keys: a row holds the keys
+//                      alone, one map, vdim = dim).
 #include "common.cuh"
 
 #include <math.h>
@@ -44,7 +49,7 @@ qk_prepare_kernel(TE* __restrict__ q, long long ldq, const TE* __restrict__ k, l
                   int rot_dims, float eps, int n_heads, int n_kv_heads, int maps, int dim, int vdim,
                   const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                   const int* __restrict__ block_table, int max_pages, int page_tokens, TE* __restrict__ rows,
-                  int pairs) {
+                  int pairs, int shared) {
     extern __shared__ float staged[];                       // [warps][dim] | cos [rot_dims / 2] | sin [rot_dims / 2]
     pdl_trigger();
     pdl_wait();
@@ -61,8 +66,8 @@ qk_prepare_kernel(TE* __restrict__ q, long long ldq, const TE* __restrict__ k, l
         sn_tab[i] = sn * magnitude;
     }
     __syncthreads();
-    const int n_q = n_heads * maps, n_k = k ? n_kv_heads * maps : 0;
-    const long long width = (long long)n_kv_heads * (maps * dim + vdim);
+    const int n_q = q_weight || rot_dims ? n_heads * maps : 0, n_k = k ? n_kv_heads * maps : 0;
+    const long long width = (long long)n_kv_heads * (maps * dim + (shared ? 0 : vdim));
     TE* row = nullptr;
     if (k) {
         const long long page = block_table[(long long)tok_seq[t] * max_pages + pos / page_tokens];
@@ -106,6 +111,14 @@ qk_prepare_kernel(TE* __restrict__ q, long long ldq, const TE* __restrict__ k, l
         const TE* vsrc = v + (long long)t * ldv;
         for (int d = threadIdx.x; d < n_kv_heads * vdim; d += blockDim.x) vdst[d] = vsrc[d];
     }
+}
+
+__device__ __forceinline__ float capped_score(float s, float softcap) {
+    return softcap > 0.0f ? softcap * tanhf(s / softcap) : s;
+}
+template <typename TE>
+__device__ __forceinline__ float entry_gate(const TE* gate, long long ldg, int t, int at) {
+    return 1.0f / (1.0f + expf(-to_float(gate[(long long)t * ldg + at])));
 }
 
 template <typename TE>
@@ -159,7 +172,7 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
                         int n_kv_heads, int dim, int vdim, float scale, int window, float lambda, float out_scale,
                         float eps, int unit_rms, int vec, TE* __restrict__ out, long long ldo,
                         const float* __restrict__ head_scale, int sink, const TE* __restrict__ gate, long long ldg,
-                        int chunk, const float* __restrict__ slopes, int keep) {
+                        int chunk, const float* __restrict__ slopes, int keep, float softcap, int gate_each, int shared) {
     extern __shared__ float smem[];
     float* qs = smem;                                        // [MAPS][dim]
     float* part_acc = qs + MAPS * dim;                       // [warps][MAPS][vdim]
@@ -172,8 +185,9 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
     const int pos = tok_pos[t];
     if (head_scale) scale *= head_scale[h];
     const int* pages = block_table + (long long)tok_seq[t] * max_pages;
-    const long long width = (long long)n_kv_heads * (MAPS * dim + vdim);
-    const long long key_off = (long long)g * MAPS * dim, val_off = (long long)n_kv_heads * MAPS * dim + (long long)g * vdim;
+    const long long width = (long long)n_kv_heads * (MAPS * dim + (shared ? 0 : vdim));
+    const long long key_off = (long long)g * MAPS * dim;
+    const long long val_off = shared ? key_off : (long long)n_kv_heads * MAPS * dim + (long long)g * vdim;
     for (int d = threadIdx.x; d < MAPS * dim; d += blockDim.x)
         qs[d] = to_float(q[(long long)t * ldq + (long long)h * MAPS * dim + d]);
     __syncthreads();
@@ -199,7 +213,9 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
         if (live) {
             row = rows + ((long long)pages[j / page_tokens] * page_tokens + j % page_tokens) * width;
 #pragma unroll
-            for (int a = 0; a < MAPS; ++a) s[a] = dot_key<TE>(qs + a * dim, row + key_off + a * dim, dim, vec != 0) * scale - slope * (float)(pos - j);
+            for (int a = 0; a < MAPS; ++a)
+                s[a] = capped_score(dot_key<TE>(qs + a * dim, row + key_off + a * dim, dim, vec != 0) * scale, softcap) -
+                       slope * (float)(pos - j);
         }
         float p[MAPS];
 #pragma unroll
@@ -266,10 +282,11 @@ mapped_attention_kernel(const TE* __restrict__ q, long long ldq, const TE* __res
     }
     float mult = out_scale;
     if (unit_rms) mult *= 1.0f / sqrtf(block_sum(sq, scratch) / (float)vdim + eps);
-    if (gate) mult *= 1.0f / (1.0f + expf(-to_float(gate[(long long)t * ldg + h])));
+    if (gate && !gate_each) mult *= 1.0f / (1.0f + expf(-to_float(gate[(long long)t * ldg + h])));
     __syncthreads();
     for (int d = threadIdx.x; d < vdim; d += blockDim.x)
-        out[(long long)t * ldo + (long long)h * vdim + d] = from_float<TE>(part_acc[d] * mult);
+        out[(long long)t * ldo + (long long)h * vdim + d] =
+            from_float<TE>(part_acc[d] * mult * (gate_each ? entry_gate(gate, ldg, t, h * vdim + d) : 1.0f));
 }
 
 // Single-token steps.  A block takes one (token, kv head) and every MD_SPLITS-th page of what the token sees
@@ -286,9 +303,11 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
                      const int* __restrict__ block_table, int max_pages, const int* __restrict__ tok_pos,
                      const int* __restrict__ tok_seq, int n_heads, int n_kv_heads, int dim, int vdim, float scale,
                      int window, int vec, float* __restrict__ part_acc, float* __restrict__ part_ml,
-                     const float* __restrict__ head_scale, int chunk, const float* __restrict__ slopes, int keep) {
+                     const float* __restrict__ head_scale, int chunk, const float* __restrict__ slopes, int keep,
+                     float softcap, int shared) {
     extern __shared__ __align__(16) unsigned char md_raw[];
-    const int kw = MAPS * dim, rw = kw + vdim;                 // the kv head's entries of a row
+    const int vw = shared ? 0 : vdim, val_at = shared ? 0 : MAPS * dim;
+    const int kw = MAPS * dim, rw = kw + vw;                   // the kv head's entries of a row
     const int pitch = rw + (vec ? 16 / (int)sizeof(TE) : 1);   // rows start in different banks
     TE* tile = reinterpret_cast<TE*>(md_raw);                  // [MD_KEYS][pitch]: keys (both maps), then values
     float* qs = reinterpret_cast<float*>(md_raw + (((size_t)MD_KEYS * pitch * sizeof(TE) + 15) / 16) * 16);   // [group][kw]
@@ -302,7 +321,7 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
     const int page_lo = first / MD_KEYS, page_hi = pos / MD_KEYS;
     const int* pages = block_table + (long long)tok_seq[t] * max_pages;
     const long long width = (long long)n_kv_heads * rw;
-    const long long key_off = (long long)g * kw, val_off = (long long)n_kv_heads * kw + (long long)g * vdim;
+    const long long key_off = (long long)g * kw, val_off = (long long)n_kv_heads * kw + (long long)g * vw;
     for (int i = tid; i < group * kw; i += blockDim.x)
         qs[i] = to_float(q[(long long)t * ldq + (long long)g * group * kw + i]);
     // heads of the group this warp takes: warp, warp + warps, ... (at most MD_HEADS of them)
@@ -327,7 +346,7 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
         const TE* src = rows + (long long)pages[pg] * MD_KEYS * width;
         if (vec) {
             constexpr int E = 16 / (int)sizeof(TE);
-            const int kc = kw / E, vc = vdim / E;
+            const int kc = kw / E, vc = vw / E;
             for (int i = tid; i < MD_KEYS * (kc + vc); i += blockDim.x) {
                 const int r = i / (kc + vc), c = i % (kc + vc);
                 const TE* from = c < kc ? src + r * width + key_off + c * E : src + r * width + val_off + (c - kc) * E;
@@ -355,7 +374,8 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
                 float p[MAPS];
 #pragma unroll
                 for (int a = 0; a < MAPS; ++a) {
-                    const float sc = live ? dot_key<TE>(qs + hg * kw + a * dim, tile + jl * pitch + a * dim, dim, vec != 0) * scale_h -
+                    const float sc = live ? capped_score(dot_key<TE>(qs + hg * kw + a * dim, tile + jl * pitch + a * dim, dim,
+                                                                     vec != 0) * scale_h, softcap) -
                                                 slope * (float)(pos - j)
                                           : -INFINITY;
                     const float m_new = fmaxf(m_run[u][a], warp_max(sc));
@@ -370,7 +390,7 @@ mapped_decode_kernel(const TE* __restrict__ q, long long ldq, const TE* __restri
                     float pj[MAPS];
 #pragma unroll
                     for (int a = 0; a < MAPS; ++a) pj[a] = __shfl_sync(0xffffffffu, p[a], jj);
-                    const TE* vrow = tile + (half * 32 + jj) * pitch + kw;
+                    const TE* vrow = tile + (half * 32 + jj) * pitch + val_at;
 #pragma unroll
                     for (int i = 0; i < MA_VPL; ++i) {
                         const int d = lane + 32 * i;
@@ -409,7 +429,7 @@ template <typename TE, int MAPS>
 __global__ void __launch_bounds__(128)
 mapped_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, int n_heads, int vdim,
                     float lambda, float out_scale, float eps, int unit_rms, TE* __restrict__ out, long long ldo,
-                    int sink, const TE* __restrict__ gate, long long ldg) {
+                    int sink, const TE* __restrict__ gate, long long ldg, int gate_each) {
     extern __shared__ float merged[];                        // [vdim]
     __shared__ float scratch[32];
     __shared__ float factor[MAPS][MD_SPLITS];
@@ -447,10 +467,11 @@ mapped_merge_kernel(const float* __restrict__ part_acc, const float* __restrict_
     }
     float mult = out_scale;
     if (unit_rms) mult *= 1.0f / sqrtf(block_sum(sq, scratch) / (float)vdim + eps);
-    if (gate) mult *= 1.0f / (1.0f + expf(-to_float(gate[(long long)t * ldg + h])));
+    if (gate && !gate_each) mult *= 1.0f / (1.0f + expf(-to_float(gate[(long long)t * ldg + h])));
     __syncthreads();
     for (int d = threadIdx.x; d < vdim; d += blockDim.x)
-        out[(long long)t * ldo + (long long)h * vdim + d] = from_float<TE>(merged[d] * mult);
+        out[(long long)t * ldo + (long long)h * vdim + d] =
+            from_float<TE>(merged[d] * mult * (gate_each ? entry_gate(gate, ldg, t, h * vdim + d) : 1.0f));
 }
 
 }  // namespace mu
@@ -461,10 +482,11 @@ MU_EXPORT int mu_qk_prepare(void* q, long long ldq, const void* k, long long ldk
                             const float* q_weight, const float* k_weight, const float* freqs, float magnitude,
                             int rot_dims, float eps, int n_tokens, int n_heads, int n_kv_heads, int maps, int dim,
                             int vdim, const int* tok_pos, const int* tok_seq, const int* block_table, int max_pages,
-                            int page_tokens, void* rows, int is_bf16, void* stream, int pairs) {
+                            int page_tokens, void* rows, int is_bf16, void* stream, int pairs, int shared) {
     if (n_tokens <= 0) return MU_OK;
     if (!q || !tok_pos || dim <= 0 || maps < 1 || maps > 2 || rot_dims < 0 || rot_dims % 2 ||
-        rot_dims > dim || (rot_dims > 0 && !freqs) || (k != nullptr) != (v != nullptr))
+        rot_dims > dim || (rot_dims > 0 && !freqs) || (k != nullptr && !shared) != (v != nullptr) ||
+        (shared && (maps != 1 || vdim != dim)))
         return MU_ERR_BAD_ARGUMENT;
     if (k && ((k_weight != nullptr) != (q_weight != nullptr) || !tok_seq || !block_table || !rows || page_tokens <= 0))
         return MU_ERR_BAD_ARGUMENT;
@@ -473,7 +495,9 @@ MU_EXPORT int mu_qk_prepare(void* q, long long ldq, const void* k, long long ldk
     const int threads = 128;
     const size_t smem = ((size_t)(threads / 32) * dim + rot_dims) * sizeof(float);
     // a token's slices are spread over several blocks, a warp a slice
-    const int items = (n_heads + (k ? n_kv_heads : 0)) * maps;
+    const bool queries = q_weight || rot_dims;
+    const int items = ((queries ? n_heads : 0) + (k ? n_kv_heads : 0)) * maps;
+    if (items == 0) return MU_OK;                            // queries as they are and no keys to keep
     const int shares = (items + 3) / 4;
     const dim3 grid(n_tokens, shares);
     typedef __nv_bfloat16 bf;
@@ -481,11 +505,11 @@ MU_EXPORT int mu_qk_prepare(void* q, long long ldq, const void* k, long long ldk
         return mu::launch_pdl(mu::qk_prepare_kernel<bf>, grid, dim3(threads), smem, s, 1, (bf*)q, ldq,
                               (const bf*)k, ldk, (const bf*)v, ldv, q_weight, k_weight, freqs, magnitude, rot_dims, eps,
                               n_heads, n_kv_heads, maps, dim, vdim, tok_pos, tok_seq, block_table, max_pages,
-                              page_tokens, (bf*)rows, pairs);
+                              page_tokens, (bf*)rows, pairs, shared);
     return mu::launch_pdl(mu::qk_prepare_kernel<float>, grid, dim3(threads), smem, s, 1, (float*)q, ldq,
                           (const float*)k, ldk, (const float*)v, ldv, q_weight, k_weight, freqs, magnitude, rot_dims,
                           eps, n_heads, n_kv_heads, maps, dim, vdim, tok_pos, tok_seq, block_table, max_pages,
-                          page_tokens, (float*)rows, pairs);
+                          page_tokens, (float*)rows, pairs, shared);
 }
 
 MU_EXPORT int mu_mapped_attention(const void* q, long long ldq, const void* rows, const int* block_table,
@@ -493,9 +517,10 @@ MU_EXPORT int mu_mapped_attention(const void* q, long long ldq, const void* rows
                                   int n_tokens, int n_heads, int n_kv_heads, int maps, int dim, int vdim, float scale,
                                   int window, float lambda, float out_scale, float eps, int unit_rms, void* out,
                                   long long ldo, int is_bf16, void* stream, const float* head_scale, int sink,
-                                  const void* gate, long long ldg, int chunk, const float* slopes, int keep) {
+                                  const void* gate, long long ldg, int chunk, const float* slopes, int keep,
+                                  float softcap, int gate_each, int shared) {
     if (n_tokens <= 0) return MU_OK;
-    if (keep < 0) return MU_ERR_BAD_ARGUMENT;
+    if (keep < 0 || (gate_each && !gate) || (shared && (maps != 1 || vdim != dim))) return MU_ERR_BAD_ARGUMENT;
     if (!q || !rows || !block_table || !tok_pos || !tok_seq || !out || n_heads <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || maps < 1 || maps > 2 || dim <= 0 || vdim <= 0 || page_tokens <= 0 || window < 0 ||
         chunk < 0)
@@ -505,7 +530,7 @@ MU_EXPORT int mu_mapped_attention(const void* q, long long ldq, const void* rows
     if (smem > 48 * 1024) return MU_ERR_UNSUPPORTED_SIZE;
     // 16-byte pieces of a key: every slice of a row must start on such a boundary
     const int per = is_bf16 ? 8 : 4;
-    const int vec = dim % per == 0 && (n_kv_heads * vdim) % per == 0 && ((uintptr_t)rows & 15) == 0;
+    const int vec = dim % per == 0 && (shared || (n_kv_heads * vdim) % per == 0) && ((uintptr_t)rows & 15) == 0;
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid(n_tokens, n_heads), block(mu::MA_WARPS * 32);
     typedef __nv_bfloat16 bf;
@@ -513,7 +538,7 @@ MU_EXPORT int mu_mapped_attention(const void* q, long long ldq, const void* rows
     return mu::launch_pdl(mu::mapped_attention_kernel<TE, M>, grid, block, smem, s, 1, (const TE*)q, ldq,             \
                           (const TE*)rows, block_table, max_pages, page_tokens, tok_pos, tok_seq, n_heads, n_kv_heads, \
                           dim, vdim, scale, window, lambda, out_scale, eps, unit_rms, vec, (TE*)out, ldo, head_scale,  \
-                          sink, (const TE*)gate, ldg, chunk, slopes, keep)
+                          sink, (const TE*)gate, ldg, chunk, slopes, keep, softcap, gate_each, shared)
     if (is_bf16) {
         if (maps == 2) MU_MAPPED(bf, 2);
         MU_MAPPED(bf, 1);
@@ -544,9 +569,9 @@ MU_EXPORT int mu_mapped_attention_decode(const void* q, long long ldq, const voi
                                          float scale, int window, float lambda, float out_scale, float eps, int unit_rms,
                                          float* scratch, void* out, long long ldo, int is_bf16, void* stream,
                                          const float* head_scale, int sink, const void* gate, long long ldg, int chunk,
-                                         const float* slopes, int keep) {
+                                         const float* slopes, int keep, float softcap, int gate_each, int shared) {
     if (n_tokens <= 0) return MU_OK;
-    if (keep < 0) return MU_ERR_BAD_ARGUMENT;
+    if (keep < 0 || (gate_each && !gate) || (shared && (maps != 1 || vdim != dim))) return MU_ERR_BAD_ARGUMENT;
     if (!q || !rows || !block_table || !tok_pos || !tok_seq || !out || !scratch || n_heads <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || maps < 1 || maps > 2 || dim <= 0 || vdim <= 0 || window < 0 || chunk < 0)
         return MU_ERR_BAD_ARGUMENT;
@@ -554,7 +579,7 @@ MU_EXPORT int mu_mapped_attention_decode(const void* q, long long ldq, const voi
     if (page_tokens != mu::MD_KEYS || vdim > 32 * mu::MA_VPL || group > 16) return MU_ERR_UNSUPPORTED_SIZE;
     const int esize = is_bf16 ? 2 : 4, per = 16 / esize;
     const int vec = dim % per == 0 && vdim % per == 0 && ((uintptr_t)rows & 15) == 0;
-    const int rw = maps * dim + vdim, pitch = rw + (vec ? per : 1);
+    const int rw = maps * dim + (shared ? 0 : vdim), pitch = rw + (vec ? per : 1);
     const size_t smem = (((size_t)mu::MD_KEYS * pitch * esize + 15) / 16) * 16 + (size_t)group * maps * dim * sizeof(float);
     if (smem > 200 * 1024) return MU_ERR_UNSUPPORTED_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
@@ -572,11 +597,12 @@ MU_EXPORT int mu_mapped_attention_decode(const void* q, long long ldq, const voi
             return MU_ERR_LAUNCH;                                                                                      \
         const int code = mu::launch_pdl(kernel, grid, block, smem, s, 1, (const TE*)q, ldq, (const TE*)rows,           \
                                         block_table, max_pages, tok_pos, tok_seq, n_heads, n_kv_heads, dim, vdim,      \
-                                        scale, window, vec, part_acc, part_ml, head_scale, chunk, slopes, keep);       \
+                                        scale, window, vec, part_acc, part_ml, head_scale, chunk, slopes, keep,        \
+                                        softcap, shared);                                                              \
         if (code != MU_OK) return code;                                                                                \
         return mu::launch_pdl(mu::mapped_merge_kernel<TE, M>, mgrid, mblock, (size_t)vdim * sizeof(float), s, 1,       \
                               (const float*)part_acc, (const float*)part_ml, n_heads, vdim, lambda, out_scale, eps,    \
-                              unit_rms, (TE*)out, ldo, sink, (const TE*)gate, ldg);                                    \
+                              unit_rms, (TE*)out, ldo, sink, (const TE*)gate, ldg, gate_each);                         \
     } while (0)
     if (is_bf16) {
         if (maps == 2) MU_MAPPED_DECODE(bf, 2);

@@ -6,7 +6,8 @@
 // P enter that product as two bfloat16 terms (the rounded weight and what the rounding left), so they act with
 // some 16 bits of mantissa instead of 8.  At the end a1 - lambda a2, the head's unit rms and the output scale, and
 // the options of mapped_attention.cu (a multiplier per head on the scores, a sink in the denominator, a gate per head,
-// chunks of positions instead of a window, a distance bias per head, kept first positions beside a window).
+// chunks of positions instead of a window, a distance bias per head, kept first positions beside a window, a soft cap on
+// the scores, a gate per value entry, rows of keys that are the values too: then one staged page serves both products).
 //
 // Sizes: page of 64 positions; dim a multiple of 16 up to 256 per map; vdim a multiple of 16 up to 128; the cache
 // row a multiple of 8 entries.  Anything else takes the CUDA-core kernel.
@@ -43,6 +44,15 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
                  : "memory");
 }
 
+// cap * tanh(s / cap): the series near zero (five terms, to 0.3, where the next one is 5e-8 of the sum), beyond it
+// 1 - 2 / (e^(2y) + 1) with the fast exponential, where the result is no smaller than 0.29.
+__device__ __forceinline__ float softcap_fast(float s, float cap, float inv_cap) {
+    const float y = s * inv_cap, a = fabsf(y), y2 = y * y;
+    const float near = y * fmaf(y2, fmaf(y2, fmaf(y2, fmaf(y2, 62.0f / 2835.0f, -17.0f / 315.0f), 2.0f / 15.0f), -1.0f / 3.0f), 1.0f);
+    const float far = copysignf(1.0f - __fdividef(2.0f, __expf(2.0f * fminf(a, 40.0f)) + 1.0f), y);
+    return cap * (a < 0.3f ? near : far);
+}
+
 // VD: the head's value entries rounded up to 32, 64 or 128 (columns past vdim are zeros in shared memory).
 template <int MAPS, int VD>
 __global__ void __launch_bounds__(128, 1)
@@ -52,13 +62,15 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
                             int dim, int vdim, float scale, int window, float lambda, float out_scale, float eps,
                             int unit_rms, __nv_bfloat16* __restrict__ out, long long ldo,
                             const float* __restrict__ head_scale, int sink, const __nv_bfloat16* __restrict__ gate,
-                            long long ldg, int chunk, const float* __restrict__ slopes, int keep) {
+                            long long ldg, int chunk, const float* __restrict__ slopes, int keep, float softcap,
+                            int gate_each, int shared) {
     extern __shared__ __align__(16) unsigned char raw[];
     const int kw = MAPS * dim;                               // key entries of one kv head
-    const int kp = kw + MM_PAD, vp = VD + MM_PAD;            // row pitches in shared memory
+    // row pitches in shared memory (a shared row is as wide as either product reads it)
+    const int kp = (shared ? max(kw, VD) : kw) + MM_PAD, vp = shared ? kp : VD + MM_PAD;
     __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(raw);                 // [64][kp]
     __nv_bfloat16* ks = qs + MM_TILE * kp;                                     // [2][64][kp]
-    __nv_bfloat16* vs = ks + 2 * MM_TILE * kp;                                 // [2][64][vp]
+    __nv_bfloat16* vs = shared ? ks : ks + 2 * MM_TILE * kp;                   // [2][64][vp]
     pdl_trigger();
     pdl_wait();
     const int flat0 = tiles[2 * blockIdx.x], count = min(tiles[2 * blockIdx.x + 1], MM_TILE);
@@ -67,8 +79,9 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
     const int pos0 = tok_pos[flat0];
     if (head_scale) scale *= head_scale[h];
     const int* pages = block_table + (long long)tok_seq[flat0] * max_pages;
-    const long long width = (long long)n_kv_heads * (kw + vdim);
+    const long long width = (long long)n_kv_heads * (kw + (shared ? 0 : vdim));
     const long long key_off = (long long)g * kw, val_off = (long long)n_kv_heads * kw + (long long)g * vdim;
+    const float inv_cap = softcap > 0.0f ? 1.0f / softcap : 0.0f;
     const int last_key = pos0 + count - 1;
     // (with chunks: the first query's chunk starts first; a tile may reach into the next chunk)
     const int first_key = chunk > 0 ? pos0 - pos0 % chunk : window > 0 ? max(0, pos0 - window + 1) : 0;
@@ -89,7 +102,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
     }
     __syncthreads();                                         // the zeros are in place before any copy lands on them
 
-    const int vchunks = vdim / 8;
+    const int vchunks = shared ? 0 : vdim / 8;
     auto load_page = [&](int page_index, int stage) {
         const __nv_bfloat16* src = rows + (long long)pages[page_index] * MM_TILE * width;
         __nv_bfloat16* kd = ks + stage * MM_TILE * kp;
@@ -160,7 +173,9 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
                         const bool seen = real[r] && kj <= qpos[r] &&
                                           (chunk > 0 ? kj >= qpos[r] - qpos[r] % chunk
                                                      : window == 0 || qpos[r] - kj < window || kj < keep);
-                        s[j][e] = seen ? s[j][e] * scale - slope * (float)(qpos[r] - kj) : -INFINITY;
+                        float sc = s[j][e] * scale;
+                        if (softcap > 0.0f) sc = softcap_fast(sc, softcap, inv_cap);
+                        s[j][e] = seen ? sc - slope * (float)(qpos[r] - kj) : -INFINITY;
                         top[r] = fmaxf(top[r], s[j][e]);
                     }
                 float corr[2];
@@ -251,7 +266,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
             mult[r] *= 1.0f / sqrtf(sq[r] / (float)vdim + eps);
         }
     }
-    if (gate) {
+    if (gate && !gate_each) {
 #pragma unroll
         for (int r = 0; r < 2; ++r)
             if (real[r]) mult[r] *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(long long)(flat0 + row0 + 8 * r) * ldg + h])));
@@ -264,8 +279,14 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
             for (int r = 0; r < 2; ++r)
                 if (real[r]) {
                     __nv_bfloat16* dst = out + (long long)(flat0 + row0 + 8 * r) * ldo + (long long)h * vdim + col;
-                    *reinterpret_cast<__nv_bfloat162*>(dst) =
-                        __floats2bfloat162_rn(o[0][j][2 * r] * mult[r], o[0][j][2 * r + 1] * mult[r]);
+                    float y0 = o[0][j][2 * r] * mult[r], y1 = o[0][j][2 * r + 1] * mult[r];
+                    if (gate_each) {
+                        const __nv_bfloat162 z = *reinterpret_cast<const __nv_bfloat162*>(
+                            gate + (long long)(flat0 + row0 + 8 * r) * ldg + (long long)h * vdim + col);
+                        y0 = __fdividef(y0, 1.0f + __expf(-__low2float(z)));
+                        y1 = __fdividef(y1, 1.0f + __expf(-__high2float(z)));
+                    }
+                    *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(y0, y1);
                 }
         }
     }
@@ -274,8 +295,8 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
 }  // namespace mu
 
 // Whether the tensor-core kernel takes these sizes (page of 64 positions assumed by the caller's check).
-MU_EXPORT int mu_mapped_attention_mma_fits(int n_kv_heads, int maps, int dim, int vdim, int page_tokens) {
-    const long long width = (long long)n_kv_heads * (maps * dim + vdim);
+MU_EXPORT int mu_mapped_attention_mma_fits(int n_kv_heads, int maps, int dim, int vdim, int page_tokens, int shared) {
+    const long long width = (long long)n_kv_heads * (maps * dim + (shared ? 0 : vdim));
     return page_tokens == mu::MM_TILE && (maps == 1 || maps == 2) && dim % 16 == 0 && dim > 0 && dim <= 256 &&
            vdim % 16 == 0 && vdim > 0 && vdim <= 128 && width % 8 == 0;
 }
@@ -285,17 +306,20 @@ MU_EXPORT int mu_mapped_attention_mma(const void* q, long long ldq, const void* 
                                       const int* tiles, int n_tiles, int n_heads, int n_kv_heads, int maps, int dim,
                                       int vdim, float scale, int window, float lambda, float out_scale, float eps,
                                       int unit_rms, void* out, long long ldo, void* stream, const float* head_scale,
-                                      int sink, const void* gate, long long ldg, int chunk, const float* slopes, int keep) {
+                                      int sink, const void* gate, long long ldg, int chunk, const float* slopes, int keep,
+                                      float softcap, int gate_each, int shared) {
     if (n_tiles <= 0) return MU_OK;
-    if (keep < 0) return MU_ERR_BAD_ARGUMENT;
+    if (keep < 0 || (gate_each && !gate) || (shared && (maps != 1 || vdim != dim))) return MU_ERR_BAD_ARGUMENT;
+    if (gate_each && (ldg % 2 || ((uintptr_t)gate & 3))) return MU_ERR_ALIGNMENT;
     if (!q || !rows || !block_table || !tok_pos || !tok_seq || !tiles || !out || n_heads <= 0 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || window < 0 || chunk < 0)
         return MU_ERR_BAD_ARGUMENT;
-    if (!mu_mapped_attention_mma_fits(n_kv_heads, maps, dim, vdim, page_tokens)) return MU_ERR_UNSUPPORTED_SIZE;
+    if (!mu_mapped_attention_mma_fits(n_kv_heads, maps, dim, vdim, page_tokens, shared)) return MU_ERR_UNSUPPORTED_SIZE;
     if (((uintptr_t)q & 15) || ((uintptr_t)rows & 15) || ((uintptr_t)out & 3) || ldq % 8 || ldo % 2)
         return MU_ERR_ALIGNMENT;
     const int vd = vdim <= 32 ? 32 : vdim <= 64 ? 64 : 128;
-    const size_t smem = ((size_t)3 * mu::MM_TILE * (maps * dim + mu::MM_PAD) + (size_t)2 * mu::MM_TILE * (vd + mu::MM_PAD)) *
+    const int kw = maps * dim, kp = (shared && vd > kw ? vd : kw) + mu::MM_PAD;
+    const size_t smem = ((size_t)3 * mu::MM_TILE * kp + (shared ? 0 : (size_t)2 * mu::MM_TILE * (vd + mu::MM_PAD))) *
                         sizeof(__nv_bfloat16);
     if (smem > 220 * 1024) return MU_ERR_UNSUPPORTED_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
@@ -310,7 +334,7 @@ MU_EXPORT int mu_mapped_attention_mma(const void* q, long long ldq, const void* 
         return mu::launch_pdl(kernel, grid, block, smem, s, 1, (const bf*)q, ldq, (const bf*)rows, block_table,        \
                               max_pages, tok_pos, tok_seq, tiles, n_heads, n_kv_heads, dim, vdim, scale, window,       \
                               lambda, out_scale, eps, unit_rms, (bf*)out, ldo, head_scale, sink, (const bf*)gate, ldg, \
-                              chunk, slopes, keep);                                                                    \
+                              chunk, slopes, keep, softcap, gate_each, shared);                                        \
     } while (0)
     if (maps == 2) {
         if (vd == 32) MU_MAPPED_MMA(2, 32);

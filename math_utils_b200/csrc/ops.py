@@ -86,7 +86,7 @@ _SIGNATURES = {
     "mu_attention_decode_tc": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_int, _c_int,
                                _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_p, _c_p],
     "mu_embed_pair": [_c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_ll,
-                      _c_ll, _c_int, _c_int, _c_p],
+                      _c_ll, _c_int, _c_int, _c_p, _c_f],
     "mu_rms_norm_out": [_c_p, _c_ll, _c_p, _c_ll, _c_f, _c_f, _c_p, _c_p, _c_f, _c_f, _c_f, _c_p, _c_ll, _c_int, _c_int,
                         _c_p, _c_ll, _c_int, _c_int, _c_p, _c_int],
     "mu_rms_norm_sum": [_c_p, _c_ll, _c_f, _c_p, _c_p, _c_ll, _c_f, _c_p, _c_f, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p],
@@ -94,22 +94,23 @@ _SIGNATURES = {
     "mu_scaled_sum": [_c_p, _c_ll, _c_f, _c_p, _c_ll, _c_f, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p],
     "mu_cast_rows": [_c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_p],
     "mu_qk_prepare": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_f, _c_int, _c_f, _c_int, _c_int, _c_int,
-                      _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_p, _c_int],
+                      _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_p, _c_int, _c_int],
     "mu_mapped_attention": [_c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                             _c_int, _c_f, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_ll, _c_int, _c_p,
-                            _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
+                            _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int, _c_f, _c_int, _c_int],
     "mu_mapped_decode_fits": [_c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int],
     "mu_mapped_decode_scratch": [_c_int, _c_int, _c_int, _c_int],
     "mu_mapped_attention_decode": [_c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                                    _c_int, _c_f, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_p, _c_ll, _c_int, _c_p,
-                                   _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
-    "mu_mapped_attention_mma_fits": [_c_int, _c_int, _c_int, _c_int, _c_int],
+                                   _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int, _c_f, _c_int, _c_int],
+    "mu_mapped_attention_mma_fits": [_c_int, _c_int, _c_int, _c_int, _c_int, _c_int],
     "mu_mapped_attention_mma": [_c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
                                 _c_int, _c_int, _c_f, _c_int, _c_f, _c_f, _c_f, _c_int, _c_p, _c_ll, _c_p,
-                                _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
+                                _c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int, _c_f, _c_int, _c_int],
     "mu_qkv_norm_rows": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_f, _c_int, _c_int, _c_int, _c_int, _c_int,
                          _c_int, _c_p, _c_int, _c_f, _c_p, _c_p, _c_p, _c_int, _c_int, _c_p, _c_int, _c_p],
-    "mu_residual_add_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_f, _c_p, _c_f, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int],
+    "mu_residual_add_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_f, _c_p, _c_f, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_int,
+                             _c_p, _c_ll, _c_f, _c_p],
     "mu_delta_prepare": [_c_p, _c_int, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_f,
                          _c_p, _c_p, _c_p, _c_int, _c_p],
     "mu_delta_scan_max_dk": [],
@@ -117,13 +118,16 @@ _SIGNATURES = {
                       _c_ll, _c_p, _c_int, _c_p, _c_int],
     "mu_linear_scan_max_dk": [],
     "mu_linear_scan": [_c_p, _c_p, _c_p, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_p, _c_p, _c_p,
-                       _c_ll, _c_ll, _c_p, _c_ll, _c_p, _c_int, _c_p],
+                       _c_ll, _c_ll, _c_p, _c_ll, _c_p, _c_int, _c_p, _c_ll, _c_int],
     "mu_exp_gates": [_c_p, _c_p, _c_ll, _c_p, _c_p, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_ll, _c_ll, _c_p,
                      _c_p],
     "mu_low_rank": [_c_p, _c_ll, _c_int, _c_p, _c_int, _c_int, _c_p],
     "mu_xielu": [_c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p],
     "mu_ssd_conv": [_c_p, _c_ll, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_p, _c_ll,
-                    _c_int, _c_p, _c_p],
+                    _c_int, _c_p, _c_p, _c_int],
+    "mu_selective_scan_max_state": [],
+    "mu_selective_scan": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_p, _c_p, _c_int, _c_int, _c_int,
+                          _c_p, _c_p, _c_p, _c_ll, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_p],
     "mu_ssd_scan": [_c_p, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p,
                     _c_p, _c_p, _c_ll, _c_ll, _c_p, _c_int, _c_p],
     "mu_gated_group_norm": [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p, _c_ll, _c_int, _c_p, _c_int, _c_int, _c_p, _c_p, _c_int],
@@ -457,8 +461,8 @@ def scaled_sum(p: torch.Tensor, a: float, q: torch.Tensor, b: float, out: torch.
 def embed_pair(ids: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tensor, seq_first: torch.Tensor,
                seq_slots: torch.Tensor, last_token: torch.Tensor, table: torch.Tensor, pair_table: torch.Tensor,
                mul_prev: int, mul_cur: int, single_tokens: bool, out: Optional[torch.Tensor] = None,
-               copy: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[t] = table[ids[t]] + pair_table[(previous * mul_prev + ids[t] * mul_cur) mod buckets] as float32, with
+               copy: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
+    """out[t] = scale * table[ids[t]] + pair_table[(previous * mul_prev + ids[t] * mul_cur) mod buckets] as float32, with
     buckets = pair_table's rows - 1 and that last row for a sequence's first token.  The token before the step's
     first token of a sequence is ``last_token[slot]``, which is then set to the sequence's last token of the step.
     ``copy`` (contiguous bfloat16 [T, hidden]) receives the same rows rounded."""
@@ -478,7 +482,7 @@ def embed_pair(ids: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tensor
     _check(library().mu_embed_pair(_ptr(ids), _ptr(positions), _ptr(tok_seq), _ptr(seq_first), _ptr(seq_slots),
                                    _ptr(last_token), _ptr(table), _ptr(pair_table), _ptr(out), _ptr(copy), n, seq_slots.numel(),
                                    hidden, pair_table.shape[0] - 1, int(mul_prev), int(mul_cur), _is_bf16(table),
-                                   int(single_tokens), _stream()), "embed_pair", launches=1 if single_tokens else 2)
+                                   int(single_tokens), _stream(), float(scale)), "embed_pair", launches=1 if single_tokens else 2)
     return out
 
 
@@ -487,20 +491,21 @@ def qk_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Ten
                k_weight: Optional[torch.Tensor], freqs: torch.Tensor, magnitude: float, rot_dims: int, eps: float,
                n_heads: int, n_kv_heads: int, maps: int, dim: int, vdim: int, tok_pos, tok_seq,
                block_table: Optional[torch.Tensor], page_tokens: int, rows: Optional[torch.Tensor],
-               pairs: bool = False) -> None:
+               pairs: bool = False, shared: bool = False) -> None:
     """Unit rms times a weight, then the rotation, for every (head, map) slice of the queries (in place) and of the
     keys (into the token's cache row, with the values behind them).  ``k`` and ``v`` None: queries only.
     Without weights (both None) the slices are not normed.  ``pairs``: entry 2i turns with entry 2i + 1 instead of
-    entry i with entry i + rot_dims / 2."""
+    entry i with entry i + rot_dims / 2.  ``shared`` (``v`` None): the rows hold keys alone, which are the values too."""
     _need_cuda(q, k, v, q_weight, k_weight, freqs, tok_pos, tok_seq, block_table, rows)
     for t, name in ((tok_pos, "tok_pos"), (tok_seq, "tok_seq"), (block_table, "block_table")):
         _i32(t, name)
     if q.stride(1) != 1 or q.shape[1] != n_heads * maps * dim:
         raise KernelError("qk_prepare: queries are [T, heads * maps * dim] with unit inner stride")
     if k is not None:
-        if (k.dtype != q.dtype or v.dtype != q.dtype or rows.dtype != q.dtype or k.stride(1) != 1 or v.stride(1) != 1
-                or k.shape[1] != n_kv_heads * maps * dim or v.shape[1] != n_kv_heads * vdim or not rows.is_contiguous()
-                or rows.shape[1] != page_tokens or rows.shape[2] != n_kv_heads * (maps * dim + vdim)):
+        if (k.dtype != q.dtype or rows.dtype != q.dtype or k.stride(1) != 1 or k.shape[1] != n_kv_heads * maps * dim
+                or (v is None) != shared or not rows.is_contiguous() or rows.shape[1] != page_tokens
+                or rows.shape[2] != n_kv_heads * (maps * dim + (0 if shared else vdim))
+                or (v is not None and (v.dtype != q.dtype or v.stride(1) != 1 or v.shape[1] != n_kv_heads * vdim))):
             raise KernelError("qk_prepare: keys, values and cache rows do not fit the sizes given")
     for w in (q_weight, k_weight, freqs):
         if w is not None and (w.dtype != torch.float32 or not w.is_contiguous()):
@@ -510,7 +515,7 @@ def qk_prepare(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Ten
                                    float(magnitude), int(rot_dims), float(eps), q.shape[0], int(n_heads),
                                    int(n_kv_heads), int(maps), int(dim), int(vdim), _ptr(tok_pos), _ptr(tok_seq),
                                    _ptr(block_table), block_table.shape[1] if block_table is not None else 0,
-                                   int(page_tokens), _ptr(rows), _is_bf16(q), _stream(), int(pairs)),
+                                   int(page_tokens), _ptr(rows), _is_bf16(q), _stream(), int(pairs), int(shared)),
            ("qk_prepare(dim={}, maps={})", dim, maps))
 
 
@@ -521,7 +526,7 @@ def mapped_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
                      tensor_cores: Optional[bool] = None, single_tokens: bool = False,
                      head_scale: Optional[torch.Tensor] = None, sink: bool = False,
                      gate: Optional[torch.Tensor] = None, chunk: int = 0, slopes: Optional[torch.Tensor] = None,
-                     keep: int = 0) -> torch.Tensor:
+                     keep: int = 0, softcap: float = 0.0, shared: bool = False) -> torch.Tensor:
     """Softmax attention of every (token, head) over the cached rows it sees (``window`` 0: all up to its own
     position), one result per score map over the same values; with two maps a1 - lam * a2.  ``unit_rms`` brings
     each head's result to unit rms (eps inside the root); ``out_scale`` multiplies it.
@@ -533,9 +538,10 @@ def mapped_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
 
     ``head_scale`` (float32, one per head) multiplies the head's scores besides ``scale``; ``sink`` adds to the
     softmax's denominator one key of score zero that has no value; ``gate`` ([T, heads] view in the compute dtype)
-    multiplies each head's result by sigmoid(gate[t, h]); ``chunk`` c > 0 replaces the window: position p sees
+    multiplies each head's result by sigmoid(gate[t, h]), or as [T, heads * vdim] entry by entry; ``chunk`` c > 0 replaces the window: position p sees
     p - p % c .. p; ``slopes`` (float32, one per head): a key at distance n loses slopes[h] * n of its score;
-    ``keep`` (with a window): the sequence's first ``keep`` positions stay in sight."""
+    ``keep`` (with a window): the sequence's first ``keep`` positions stay in sight; ``softcap`` c > 0 makes a scaled score s
+    c * tanh(s / c) before anything is taken off it; ``shared``: the rows hold keys alone, which are the values too."""
     _need_cuda(q, rows, block_table, tok_pos, tok_seq, out, head_scale, gate, slopes)
     if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != n_heads or not slopes.is_contiguous()):
         raise KernelError("mapped_attention: slopes are one contiguous float32 per head")
@@ -544,15 +550,18 @@ def mapped_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
     if head_scale is not None and (head_scale.dtype != torch.float32 or head_scale.numel() != n_heads
                                    or not head_scale.is_contiguous()):
         raise KernelError("mapped_attention: head_scale is one contiguous float32 per head")
-    if gate is not None and (gate.dtype != rows.dtype or gate.dim() != 2 or gate.shape != (q.shape[0], n_heads)
-                             or gate.stride(1) != 1):
-        raise KernelError("mapped_attention: the gate is [T, heads] in the compute dtype with unit inner stride")
+    if gate is not None and (gate.dtype != rows.dtype or gate.dim() != 2 or gate.shape[0] != q.shape[0]
+                             or gate.shape[1] not in (n_heads, n_heads * vdim) or gate.stride(1) != 1):
+        raise KernelError("mapped_attention: the gate is [T, heads] or [T, heads * vdim] in the compute dtype with unit inner stride")
+    if shared and (maps != 1 or vdim != dim):
+        raise KernelError("mapped_attention: keys that are the values have one map and the values' size")
+    gate_each = gate is not None and gate.shape[1] != n_heads
     extras = (_ptr(head_scale), int(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, int(chunk),
-              _ptr(slopes), int(keep))
+              _ptr(slopes), int(keep), float(softcap), int(gate_each), int(shared))
     for t, name in ((tok_pos, "tok_pos"), (tok_seq, "tok_seq"), (block_table, "block_table")):
         _i32(t, name)
     if (q.dtype != rows.dtype or out.dtype != rows.dtype or q.stride(1) != 1 or out.stride(1) != 1
-            or not rows.is_contiguous() or rows.shape[2] != n_kv_heads * (maps * dim + vdim)
+            or not rows.is_contiguous() or rows.shape[2] != n_kv_heads * (maps * dim + (0 if shared else vdim))
             or q.shape[1] != n_heads * maps * dim or out.shape[1] != n_heads * vdim):
         raise KernelError("mapped_attention: queries, rows and output do not fit the sizes given")
     if single_tokens and library().mu_mapped_decode_fits(int(n_heads), int(n_kv_heads), int(maps), int(dim), int(vdim),
@@ -572,7 +581,9 @@ def mapped_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
         tensor_cores = MAPPED_TC
     if (tensor_cores and tiles is not None and rows.dtype == torch.bfloat16 and q.stride(0) % 8 == 0
             and out.stride(0) % 2 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 4 == 0
-            and library().mu_mapped_attention_mma_fits(int(n_kv_heads), int(maps), int(dim), int(vdim), int(page_tokens))):
+            and not (gate_each and (gate.stride(0) % 2 or gate.data_ptr() % 4))
+            and library().mu_mapped_attention_mma_fits(int(n_kv_heads), int(maps), int(dim), int(vdim), int(page_tokens),
+                                                       int(shared))):
         _need_cuda(tiles)
         _i32(tiles, "tiles")
         _check(library().mu_mapped_attention_mma(
@@ -593,19 +604,19 @@ def mapped_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
 # ------------------------------------------------------------------ state-space mixer
 def ssd_conv(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], tok_seq, seq_first, seq_slots,
              state: torch.Tensor, single_tokens: bool, out: torch.Tensor) -> torch.Tensor:
-    """silu of the short causal convolution of the channels ``u`` [T, channels] per sequence, float32 ``out``; the
-    inputs before a sequence's first token of the step come from the head of ``state[slot]``, which is moved on."""
+    """silu of the short causal convolution of the channels ``u`` [T, channels] per sequence, ``out`` float32 or ``u``'s dtype;
+    the inputs before a sequence's first token of the step come from the head of ``state[slot]``, which is moved on."""
     _need_cuda(u, weight, bias, tok_seq, seq_first, seq_slots, state, out)
     for t, name in ((tok_seq, "tok_seq"), (seq_first, "seq_first"), (seq_slots, "seq_slots")):
         _i32(t, name)
     channels, taps = weight.shape
     if (u.stride(1) != 1 or u.shape[1] != channels or weight.dtype != torch.float32 or not weight.is_contiguous()
-            or out.dtype != torch.float32 or not out.is_contiguous() or out.shape != (u.shape[0], channels)
+            or out.dtype not in (torch.float32, u.dtype) or not out.is_contiguous() or out.shape != (u.shape[0], channels)
             or state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < (taps - 1) * channels):
         raise KernelError("ssd_conv: inputs, weight, state or output do not fit")
     _check(library().mu_ssd_conv(_ptr(u), u.stride(0), _is_bf16(u), _ptr(weight), _ptr(bias), channels, taps, u.shape[0],
                                  seq_slots.numel(), _ptr(tok_seq), _ptr(seq_first), _ptr(seq_slots), _ptr(state),
-                                 state.stride(0), int(single_tokens), _ptr(out), _stream()), "ssd_conv",
+                                 state.stride(0), int(single_tokens), _ptr(out), _stream(), _is_bf16(out)), "ssd_conv",
            launches=1 if single_tokens or taps == 1 else 2)
     return out
 
@@ -629,6 +640,39 @@ def ssd_scan(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias, a_log, skip, n_he
                                  int(groups), _ptr(seq_first), _ptr(seq_slots), _ptr(state), state.stride(0),
                                  int(state_offset), _ptr(out), int(xbc.shape[0] > 4 * seq_slots.numel()), _stream()),
            ("ssd_scan(heads={}, P={}, N={})", n_heads, head_dim, n_state))
+    return out
+
+
+def selective_scan_max_state() -> int:
+    return int(library().mu_selective_scan_max_state())
+
+
+def selective_scan(x: torch.Tensor, z: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_at: int, c_at: int,
+                   rates: torch.Tensor, skip: torch.Tensor, seq_first, seq_slots, state: torch.Tensor, state_offset: int,
+                   out: torch.Tensor) -> torch.Tensor:
+    """The recurrence S[c, n] = 2^(dt_c rates[c, n]) S[c, n] + dt_c x_c B_n, out_c = (sum_n S[c, n] C_n + skip_c x_c) silu(z_c)
+    over the step's tokens of each sequence, from and to ``state[slot][state_offset:]`` (channels x N float32).  ``x``, ``z``
+    and ``out`` [T, channels] in the compute dtype, ``dt`` float32; B and C are the columns of the float32 rows ``bc`` from
+    ``b_at`` and ``c_at`` on, each followed by filling up to a multiple of four."""
+    _need_cuda(x, z, dt, bc, rates, skip, seq_first, seq_slots, state, out)
+    _i32(seq_first, "seq_first"); _i32(seq_slots, "seq_slots")
+    T, inner = x.shape
+    N = rates.shape[1]
+    n4 = -(-N // 4) * 4
+    for t in (x, z, out):
+        if t.dtype != x.dtype or tuple(t.shape) != (T, inner) or t.stride(1) != 1:
+            raise KernelError("selective_scan: x, z and the output are [T, channels] of one dtype with unit inner stride")
+    if (dt.dtype != torch.float32 or tuple(dt.shape) != (T, inner) or dt.stride(1) != 1 or bc.dtype != torch.float32
+            or bc.stride(1) != 1 or bc.shape[0] != T or max(b_at, c_at) + n4 > bc.shape[1] or rates.dtype != torch.float32
+            or rates.shape[0] != inner or not rates.is_contiguous() or skip.dtype != torch.float32 or skip.numel() != inner
+            or not skip.is_contiguous() or state.dtype != torch.float32 or state.stride(1) != 1
+            or state.shape[1] < state_offset + inner * N):
+        raise KernelError("selective_scan: step sizes, B and C, rates or state do not fit")
+    _check(library().mu_selective_scan(_ptr(x), x.stride(0), _ptr(z), z.stride(0), _ptr(dt), dt.stride(0), _ptr(bc), bc.stride(0),
+                                       int(b_at), int(c_at), _ptr(rates), _ptr(skip), seq_slots.numel(), inner, N,
+                                       _ptr(seq_first), _ptr(seq_slots), _ptr(state), state.stride(0), int(state_offset),
+                                       _ptr(out), out.stride(0), _is_bf16(out), int(T > 4 * seq_slots.numel()), _stream()),
+           ("selective_scan(channels={}, N={})", inner, N))
     return out
 
 
@@ -692,22 +736,29 @@ def qkv_norm_rows(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.
 
 
 def residual_add_norm(x: torch.Tensor, y: Optional[torch.Tensor], mult: float, weight: Optional[torch.Tensor],
-                      eps: float, out: Optional[torch.Tensor], groups: int = 1) -> Optional[torch.Tensor]:
-    """x += mult * y on the float32 stream (``y`` None: nothing is added), then out = x / rms(x) * weight in
+                      eps: float, out: Optional[torch.Tensor], groups: int = 1, y2: Optional[torch.Tensor] = None,
+                      mult2: float = 0.0, scale: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """x += (mult * y + mult2 * y2) * scale on the float32 stream (``y`` None: nothing is added; ``y2`` None: one branch;
+    ``scale`` None: ones, else one float32 per entry of the row), then out = x / rms(x) * weight in
     ``out``'s dtype (``weight`` None: the addition only).  ``groups``: the row in that many consecutive equal parts, each
     divided by its own rms."""
-    _need_cuda(x, y, weight, out)
+    _need_cuda(x, y, weight, out, y2, scale)
     if x.dtype != torch.float32 or x.dim() != 2 or x.stride(1) != 1:
         raise KernelError("residual_add_norm: the stream is float32 [rows, n] with unit inner stride")
-    if y is not None and (y.dtype != torch.float32 or y.shape != x.shape or y.stride(1) != 1):
-        raise KernelError("residual_add_norm: the sublayer's output is float32 and shaped like the stream")
+    for t in (y, y2):
+        if t is not None and (t.dtype != torch.float32 or t.shape != x.shape or t.stride(1) != 1):
+            raise KernelError("residual_add_norm: the sublayer's output is float32 and shaped like the stream")
+    if y2 is not None and y is None or scale is not None and (scale.dtype != torch.float32 or scale.numel() != x.shape[1]
+                                                              or not scale.is_contiguous()):
+        raise KernelError("residual_add_norm: a second branch goes with a first, a scale is one contiguous float32 per entry")
     if weight is not None and (weight.dtype != torch.float32 or weight.numel() != x.shape[1] or not weight.is_contiguous()
                                or out is None or out.shape != x.shape or out.stride(1) != 1):
         raise KernelError("residual_add_norm: a float32 weight of n values and an output shaped like the stream")
     _check(library().mu_residual_add_norm(_ptr(x), x.stride(0), _ptr(y), y.stride(0) if y is not None else 0, float(mult),
                                           _ptr(weight), float(eps), x.shape[0], x.shape[1], _ptr(out),
                                           out.stride(0) if out is not None else 0,
-                                          _is_bf16(out) if out is not None else 0, _stream(), int(groups)),
+                                          _is_bf16(out) if out is not None else 0, _stream(), int(groups), _ptr(y2),
+                                          y2.stride(0) if y2 is not None else 0, float(mult2), _ptr(scale)),
            ("residual_add_norm(n={})", x.shape[1]))
     return out
 
@@ -785,20 +836,22 @@ def linear_scan_max_dk() -> int:
 
 def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, n_heads: int, dk: int, dv: int,
                 scale: float, seq_first, seq_slots, state: torch.Tensor, state_offset: int, out: torch.Tensor,
-                norm_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                norm_out: Optional[torch.Tensor] = None, silu_rows: bool = False) -> torch.Tensor:
     """The recurrence S = decay S + take k v^T, o = scale S^T q per (sequence, head) over the step's tokens, from and
     to ``state[slot][state_offset:]`` (heads x dv x dk float32).  ``q``, ``k``, ``v``: float32 column blocks of one
-    buffer.  ``decay`` [T, heads * dk]: one per key channel, take 1; [T, heads, 4]: (decay, take, -, -) per head.
+    buffer.  ``decay`` [T, heads * dk]: one per key channel, take 1; [T, heads, 4]: (decay, take, -, -) per head, or
+    [1, heads, 4] of them for every token.  ``silu_rows``: queries, keys and values pass silu first.
     ``norm_out`` [T, heads] (with [T, heads, 4] gates): the read-out of a normalizer n = decay n + take k, whose
     heads x dk values follow S in the state."""
     _need_cuda(q, k, v, decay, seq_first, seq_slots, state, out, norm_out)
     _i32(seq_first, "seq_first"); _i32(seq_slots, "seq_slots")
     T = q.shape[0]
     per_channel = decay.dim() == 2
+    constant = not per_channel and decay.shape[0] == 1
     for t, n in ((q, n_heads * dk), (k, n_heads * dk), (v, n_heads * dv)):
         if t.dtype != torch.float32 or tuple(t.shape) != (T, n) or t.stride(1) != 1 or t.stride(0) != q.stride(0):
             raise KernelError("linear_scan: queries, keys and values are float32 column blocks of one buffer")
-    wanted = (T, n_heads * dk) if per_channel else (T, n_heads, 4)
+    wanted = (T, n_heads * dk) if per_channel else (1, n_heads, 4) if constant else (T, n_heads, 4)
     values = n_heads * dk * (dv + (1 if norm_out is not None else 0))
     if (tuple(decay.shape) != wanted or decay.dtype != torch.float32 or not decay.is_contiguous()
             or out.dtype != torch.float32 or out.stride(1) != 1 or tuple(out.shape) != (T, n_heads * dv)
@@ -810,7 +863,8 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
     _check(library().mu_linear_scan(_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), int(per_channel),
                                     seq_slots.numel(), int(n_heads), int(dk), int(dv), float(scale), _ptr(seq_first),
                                     _ptr(seq_slots), _ptr(state), state.stride(0), int(state_offset), _ptr(out),
-                                    out.stride(0), _ptr(norm_out), int(T > 4 * seq_slots.numel()), _stream()),
+                                    out.stride(0), _ptr(norm_out), int(T > 4 * seq_slots.numel()), _stream(),
+                                    0 if constant else 4 * n_heads, int(silu_rows)),
            ("linear_scan(heads={}, dk={}, dv={})", n_heads, dk, dv))
     return out
 
@@ -842,13 +896,13 @@ class LowRankPart(ctypes.Structure):
                 ("rank", _c_int), ("n", _c_int), ("fn", _c_int), ("per_head", _c_int), ("power", _c_f)]
 
 
-LOW_RANK_FNS = {None: 0, "sigmoid_power": 1, "exp_softplus": 2}
+LOW_RANK_FNS = {None: 0, "sigmoid_power": 1, "exp_softplus": 2, "softplus": 3}
 
 
 def low_rank_part(weight: torch.Tensor, col: int, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
                   fn: Optional[str] = None, power: float = 1.0, a_log: Optional[torch.Tensor] = None) -> LowRankPart:
     """``out`` [T, n] float32 = fn(weight [n, rank] @ low[:, col: col + rank] + bias); ``fn``: None, ``sigmoid_power``
-    (sigmoid(z)^power) or ``exp_softplus`` (exp(-exp(a_log[head]) softplus(z)), n / heads channels a head)."""
+    (sigmoid(z)^power), ``exp_softplus`` (exp(-exp(a_log[head]) softplus(z)), n / heads channels a head) or ``softplus``."""
     _need_cuda(weight, out, bias, a_log)
     n, rank = weight.shape
     if weight.stride(1) != 1 or out.dtype != torch.float32 or not out.is_contiguous() or out.shape[1] != n:

@@ -114,17 +114,47 @@ qkv_norm_rows_kernel(TE* q, long long ldq, const TE* __restrict__ k, long long l
 
 constexpr int RA_KEEP = 8;        // entries of the row a thread keeps between the sum and the output
 
+// What a sublayer adds to the stream: (mult * y [+ mult2 * y2]) [* scale, entry by entry].
+struct Addend {
+    const float* y;           // [rows][ldy], or null: nothing is added
+    long long ldy;
+    float mult;
+    const float* y2;          // a second branch, or null
+    long long ldy2;
+    float mult2;
+    const float* scale;       // [width] or null
+};
+
+__device__ __forceinline__ float ra_added(float x, const Addend& a, long long t, long long d) {
+    const float y = a.y[t * a.ldy + d];
+    if (!a.y2 && !a.scale) return fmaf(a.mult, y, x);
+    const float v = a.y2 ? fmaf(a.mult, y, a.mult2 * a.y2[t * a.ldy2 + d]) : a.mult * y;
+    return a.scale ? fmaf(v, a.scale[d], x) : x + v;
+}
+__device__ __forceinline__ float4 ra_added4(float4 x, const Addend& a, long long t, long long d) {
+    const float4 y = *reinterpret_cast<const float4*>(a.y + t * a.ldy + d);
+    float4 v = make_float4(a.mult * y.x, a.mult * y.y, a.mult * y.z, a.mult * y.w);
+    if (a.y2) {
+        const float4 u = *reinterpret_cast<const float4*>(a.y2 + t * a.ldy2 + d);
+        v = make_float4(fmaf(a.mult2, u.x, v.x), fmaf(a.mult2, u.y, v.y), fmaf(a.mult2, u.z, v.z), fmaf(a.mult2, u.w, v.w));
+    }
+    if (a.scale) {
+        const float4 g = *reinterpret_cast<const float4*>(a.scale + d);
+        return make_float4(fmaf(v.x, g.x, x.x), fmaf(v.y, g.y, x.y), fmaf(v.z, g.z, x.z), fmaf(v.w, g.w, x.w));
+    }
+    return make_float4(x.x + v.x, x.y + v.y, x.z + v.z, x.w + v.w);
+}
+
 template <typename TE>
 __global__ void __launch_bounds__(256)
-residual_add_norm_kernel(float* __restrict__ x, long long ldx, const float* __restrict__ y, long long ldy, float mult,
-                         const float* __restrict__ weight, float eps, int width, TE* __restrict__ h, long long ldh) {
+residual_add_norm_kernel(float* __restrict__ x, long long ldx, const Addend add, const float* __restrict__ weight, float eps,
+                         int width, TE* __restrict__ h, long long ldh) {
     __shared__ float scratch[32];
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
     const long long part0 = (long long)blockIdx.y * width;   // rows normed in parts: this block's part
     float* xs = x + (long long)t * ldx + part0;
-    const float* ys = y ? y + (long long)t * ldy + part0 : nullptr;
     weight = weight ? weight + part0 : nullptr;
     float kept[RA_KEEP];
     float sq = 0.0f;
@@ -133,14 +163,14 @@ residual_add_norm_kernel(float* __restrict__ x, long long ldx, const float* __re
         const int d = threadIdx.x + i * blockDim.x;
         kept[i] = 0.0f;
         if (d < width) {
-            kept[i] = ys ? fmaf(mult, ys[d], xs[d]) : xs[d];
-            if (ys) xs[d] = kept[i];
+            kept[i] = add.y ? ra_added(xs[d], add, t, part0 + d) : xs[d];
+            if (add.y) xs[d] = kept[i];
         }
         sq += kept[i] * kept[i];
     }
     for (int d = threadIdx.x + RA_KEEP * blockDim.x; d < width; d += blockDim.x) {
-        const float v = ys ? fmaf(mult, ys[d], xs[d]) : xs[d];
-        if (ys) xs[d] = v;
+        const float v = add.y ? ra_added(xs[d], add, t, part0 + d) : xs[d];
+        if (add.y) xs[d] = v;
         sq += v * v;
     }
     if (!weight) return;
@@ -164,12 +194,50 @@ __device__ __forceinline__ void ra_store(__nv_bfloat16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = packed;
 }
 
-// The same for rows normed in parts of up to 1,024 entries in whole, aligned 16-byte pieces: a warp a part, no barrier.
+// The same for whole rows of up to 4,096 entries in whole, aligned 16-byte pieces: a block of 256 threads a row, four
+// entries a load, everything a thread needs on its way at once.
+template <typename TE>
+__global__ void __launch_bounds__(256)
+residual_add_norm_vec_kernel(float* __restrict__ x, long long ldx, const Addend add, const float* __restrict__ weight,
+                             float eps, int width, TE* __restrict__ h, long long ldh) {
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const long long t = blockIdx.x;
+    float* xs = x + t * ldx;
+    float4 v[4];
+    float sq = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int d = 4 * (threadIdx.x + 256 * i);
+        v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (d < width) v[i] = *reinterpret_cast<const float4*>(xs + d);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int d = 4 * (threadIdx.x + 256 * i);
+        if (add.y && d < width) {
+            v[i] = ra_added4(v[i], add, t, d);
+            *reinterpret_cast<float4*>(xs + d) = v[i];
+        }
+        sq += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+    }
+    if (!weight) return;
+    const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int d = 4 * (threadIdx.x + 256 * i);
+        if (d >= width) continue;
+        const float4 g = *reinterpret_cast<const float4*>(weight + d);
+        ra_store(h + t * ldh + d, make_float4(v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w));
+    }
+}
+
+// Rows normed in parts of up to 1,024 entries in whole, aligned 16-byte pieces: a warp a part, no barrier.
 template <typename TE>
 __global__ void __launch_bounds__(128)
-residual_add_norm_parts_kernel(float* __restrict__ x, long long ldx, const float* __restrict__ y, long long ldy, float mult,
-                               const float* __restrict__ weight, float eps, int width, int parts, long long n_parts,
-                               TE* __restrict__ h, long long ldh) {
+residual_add_norm_parts_kernel(float* __restrict__ x, long long ldx, const Addend add, const float* __restrict__ weight,
+                               float eps, int width, int parts, long long n_parts, TE* __restrict__ h, long long ldh) {
     pdl_trigger();
     pdl_wait();
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -177,7 +245,6 @@ residual_add_norm_parts_kernel(float* __restrict__ x, long long ldx, const float
     const int lane = threadIdx.x & 31, part = (int)(item % parts);
     const long long t = item / parts, at0 = (long long)part * width;
     float* xs = x + t * ldx + at0;
-    const float* ys = y ? y + t * ldy + at0 : nullptr;
     float4 v[8];
     float sq = 0.0f;
 #pragma unroll
@@ -186,9 +253,8 @@ residual_add_norm_parts_kernel(float* __restrict__ x, long long ldx, const float
         v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (d < width) {
             v[i] = *reinterpret_cast<const float4*>(xs + d);
-            if (ys) {
-                const float4 u = *reinterpret_cast<const float4*>(ys + d);
-                v[i] = make_float4(fmaf(mult, u.x, v[i].x), fmaf(mult, u.y, v[i].y), fmaf(mult, u.z, v[i].z), fmaf(mult, u.w, v[i].w));
+            if (add.y) {
+                v[i] = ra_added4(v[i], add, t, at0 + d);
                 *reinterpret_cast<float4*>(xs + d) = v[i];
             }
         }
@@ -232,29 +298,40 @@ MU_EXPORT int mu_qkv_norm_rows(void* q, long long ldq, const void* k, long long 
 }
 
 // groups: the row is normed in that many equal parts, each by itself (the weight is the whole row's).
+// What is added: (mult * y + mult2 * y2) * scale, y2 (a second branch) and scale (one number per entry) optional.
 MU_EXPORT int mu_residual_add_norm(float* x, long long ldx, const float* y, long long ldy, float mult, const float* weight,
                                    float eps, int n_rows, int width, void* h, long long ldh, int is_bf16, void* stream,
-                                   int groups) {
+                                   int groups, const float* y2, long long ldy2, float mult2, const float* scale) {
     if (n_rows <= 0 || width <= 0) return MU_OK;
-    if (!x || (weight && !h) || (!weight && !y) || groups < 1 || groups > 65535 || width % groups) return MU_ERR_BAD_ARGUMENT;
+    if (!x || (weight && !h) || (!weight && !y) || groups < 1 || groups > 65535 || width % groups || (y2 && !y))
+        return MU_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
     const int part = width / groups;
-    if (weight && groups > 1 && part % 4 == 0 && part <= 1024 && ldx % 4 == 0 && ldy % 4 == 0 && ldh % 4 == 0 &&
-        (((uintptr_t)x | (uintptr_t)y | (uintptr_t)weight) & 15) == 0 && ((uintptr_t)h & (is_bf16 ? 7 : 15)) == 0) {
+    const mu::Addend add = {y, ldy, mult, y2, ldy2, mult2, scale};
+    const bool pieces = part % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && ldy2 % 4 == 0 && ldh % 4 == 0 &&
+                        (((uintptr_t)x | (uintptr_t)y | (uintptr_t)y2 | (uintptr_t)scale | (uintptr_t)weight) & 15) == 0 &&
+                        ((uintptr_t)h & (is_bf16 ? 7 : 15)) == 0;
+    if (weight && groups > 1 && pieces && part <= 1024) {
         const long long n_parts = (long long)n_rows * groups;
         const int warps = n_parts >= 2048 ? 4 : 1;           // a few parts: a block each, spread over the SMs
         const dim3 grid((unsigned)((n_parts + warps - 1) / warps)), block(32 * warps);
         if (is_bf16)
-            return mu::launch_pdl(mu::residual_add_norm_parts_kernel<bf>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight,
-                                  eps, part, groups, n_parts, (bf*)h, ldh);
-        return mu::launch_pdl(mu::residual_add_norm_parts_kernel<float>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight,
-                              eps, part, groups, n_parts, (float*)h, ldh);
+            return mu::launch_pdl(mu::residual_add_norm_parts_kernel<bf>, grid, block, 0, s, 1, x, ldx, add, weight, eps, part,
+                                  groups, n_parts, (bf*)h, ldh);
+        return mu::launch_pdl(mu::residual_add_norm_parts_kernel<float>, grid, block, 0, s, 1, x, ldx, add, weight, eps, part,
+                              groups, n_parts, (float*)h, ldh);
+    }
+    if (groups == 1 && pieces && width <= 4096) {
+        const dim3 grid(n_rows), block(256);
+        if (is_bf16)
+            return mu::launch_pdl(mu::residual_add_norm_vec_kernel<bf>, grid, block, 0, s, 1, x, ldx, add, weight, eps, width,
+                                  (bf*)h, ldh);
+        return mu::launch_pdl(mu::residual_add_norm_vec_kernel<float>, grid, block, 0, s, 1, x, ldx, add, weight, eps, width,
+                              (float*)h, ldh);
     }
     const dim3 grid(n_rows, groups), block(part > 1024 ? 256 : 128);
     if (is_bf16)
-        return mu::launch_pdl(mu::residual_add_norm_kernel<bf>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight, eps,
-                              part, (bf*)h, ldh);
-    return mu::launch_pdl(mu::residual_add_norm_kernel<float>, grid, block, 0, s, 1, x, ldx, y, ldy, mult, weight, eps,
-                          part, (float*)h, ldh);
+        return mu::launch_pdl(mu::residual_add_norm_kernel<bf>, grid, block, 0, s, 1, x, ldx, add, weight, eps, part, (bf*)h, ldh);
+    return mu::launch_pdl(mu::residual_add_norm_kernel<float>, grid, block, 0, s, 1, x, ldx, add, weight, eps, part, (float*)h, ldh);
 }

@@ -5,7 +5,7 @@
 //     state[slot] = [ conv tail: (taps - 1) x channels, oldest first | S: heads x N x P ]
 // mu_ssd_conv   out[t][c] = silu(bias[c] + sum_j w[c][j] in[t - taps + 1 + j][c]) over the step's tokens of
 //               each sequence, the inputs before the step's first token taken from the tail (zeros when the
-//               sequence starts: a slot's state is cleared when it is taken); float32 out.
+//               sequence starts: a slot's state is cleared when it is taken); out in float32 or bfloat16.
 //               When every sequence brings one token the same launch moves the tail on; otherwise
 //               mu_ssd_conv_tail does, after it.
 // mu_ssd_scan   per (sequence, head, a few columns of S), the step's tokens in order:
@@ -26,12 +26,12 @@ __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z));
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 
 // seq_first[s] .. seq_first[s + 1] - 1 are the flat tokens of the step's s-th sequence.
-template <typename TE>
+template <typename TE, typename TO>
 __global__ void ssd_conv_kernel(const TE* __restrict__ u, long long ldu, const float* __restrict__ weight,
                                 const float* __restrict__ bias, int channels, int taps, int n_tokens,
                                 const int* __restrict__ tok_seq, const int* __restrict__ seq_first,
                                 const int* __restrict__ seq_slots, float* __restrict__ state, long long state_stride,
-                                int move_tail, float* __restrict__ out) {
+                                int move_tail, TO* __restrict__ out) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -46,10 +46,100 @@ __global__ void ssd_conv_kernel(const TE* __restrict__ u, long long ldu, const f
                                 : tail[(long long)(taps - 1 + li) * channels + c];
         acc = fmaf(weight[(long long)c * taps + j], x, acc);
     }
-    out[(long long)t * channels + c] = silu_f(acc);
+    out[(long long)t * channels + c] = from_float<TO>(silu_f(acc));
     if (move_tail) {                                              // one token per sequence: this thread alone touches tail[.][c]
         for (int k = 0; k + 1 < taps - 1; ++k) tail[(long long)k * channels + c] = tail[(long long)(k + 1) * channels + c];
         if (taps > 1) tail[(long long)(taps - 2) * channels + c] = to_float(u[(long long)t * ldu + c]);
+    }
+}
+
+// The same for steps of many tokens with up to four taps and rows of whole, aligned 16-byte pieces: a thread takes eight
+// channels and eight consecutive tokens, whose rows are all on their way at once; the taps' inputs stay in registers.
+constexpr int CV_CH = 8, CV_TOK = 8;
+
+__device__ __forceinline__ void cv_load(float (&v)[CV_CH], const float* p) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+}
+__device__ __forceinline__ void cv_load(float (&v)[CV_CH], const __nv_bfloat16* p) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        v[2 * i] = f.x, v[2 * i + 1] = f.y;
+    }
+}
+__device__ __forceinline__ void cv_store(float* p, const float (&v)[CV_CH]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void cv_store(__nv_bfloat16* p, const float (&v)[CV_CH]) {
+    uint4 raw;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p) = raw;
+}
+
+template <typename TE, typename TO, int TAPS>
+__global__ void __launch_bounds__(128)
+ssd_conv_vec_kernel(const TE* __restrict__ u, long long ldu, const float* __restrict__ weight, const float* __restrict__ bias,
+                    int channels, int n_tokens, const int* __restrict__ tok_seq, const int* __restrict__ seq_first,
+                    const int* __restrict__ seq_slots, const float* __restrict__ state, long long state_stride,
+                    TO* __restrict__ out) {
+    pdl_trigger();
+    const int c = CV_CH * (blockIdx.y * blockDim.x + threadIdx.x);
+    if (c >= channels) return;
+    float w[CV_CH * TAPS], b8[CV_CH];                        // channel i's taps at [i TAPS]
+#pragma unroll
+    for (int i = 0; i < 2 * TAPS; ++i) {
+        const float4 f = *reinterpret_cast<const float4*>(weight + (long long)c * TAPS + 4 * i);
+        w[4 * i] = f.x, w[4 * i + 1] = f.y, w[4 * i + 2] = f.z, w[4 * i + 3] = f.w;
+    }
+#pragma unroll
+    for (int i = 0; i < CV_CH; ++i) b8[i] = bias ? bias[c + i] : 0.0f;
+    pdl_wait();
+    const int t0 = blockIdx.x * CV_TOK, nt = min(CV_TOK, n_tokens - t0);
+    float rows[CV_TOK + TAPS - 1][CV_CH];                    // the inputs before the tile, then the tile's
+#pragma unroll
+    for (int i = 0; i < CV_TOK; ++i)
+        if (i < nt) cv_load(rows[TAPS - 1 + i], u + (long long)(t0 + i) * ldu + c);
+    int s = tok_seq[t0], first = seq_first[s], end = seq_first[s + 1];
+    const float* tail = state + (long long)seq_slots[s] * state_stride + c;
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+        const int li = t0 - first - (TAPS - 1) + j;
+        if (li >= 0) cv_load(rows[j], u + (long long)(first + li) * ldu + c);
+        else
+#pragma unroll
+            for (int i = 0; i < CV_CH; ++i) rows[j][i] = tail[(long long)(TAPS - 1 + li) * channels + i];
+    }
+#pragma unroll
+    for (int k = 0; k < CV_TOK; ++k) {
+        if (k >= nt) break;
+        const int t = t0 + k;
+        if (t >= end) {                                      // another sequence begins
+            s = tok_seq[t], first = seq_first[s], end = seq_first[s + 1];
+            tail = state + (long long)seq_slots[s] * state_stride + c;
+        }
+        float acc[CV_CH];
+#pragma unroll
+        for (int i = 0; i < CV_CH; ++i) acc[i] = b8[i];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const int li = t - first - (TAPS - 1) + j;
+            // (the rows in front of the tile are the first sequence's already; a later one's begin inside the tile)
+            const bool from_tail = li < 0 && first > t0;
+#pragma unroll
+            for (int i = 0; i < CV_CH; ++i) {
+                const float v = from_tail ? tail[(long long)(TAPS - 1 + li) * channels + i] : rows[k + j][i];
+                acc[i] = fmaf(w[i * TAPS + j], v, acc[i]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < CV_CH; ++i) acc[i] = silu_f(acc[i]);
+        cv_store(out + (long long)t * channels + c, acc);
     }
 }
 
@@ -402,31 +492,59 @@ gated_group_norm_warp_kernel(const float* __restrict__ y, long long ldy, const T
 
 }  // namespace mu
 
+namespace mu {
+
+template <typename TE, typename TO>
+int ssd_conv_launch(const TE* u, long long ldu, const float* weight, const float* bias, int channels, int taps, int n_tokens,
+                    int n_seqs, const int* tok_seq, const int* seq_first, const int* seq_slots, float* state,
+                    long long state_stride, int single_tokens, TO* out, cudaStream_t s) {
+    const bool pieces = channels % 8 == 0 && (ldu * sizeof(TE)) % 16 == 0 &&
+                        (((uintptr_t)u | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    int code = MU_OK;
+    if (!single_tokens && n_tokens >= 64 && taps >= 2 && taps <= 4 && pieces) {
+        const int threads = channels / CV_CH >= 128 ? 128 : 64;
+        const dim3 grid((n_tokens + CV_TOK - 1) / CV_TOK, (channels / CV_CH + threads - 1) / threads), block(threads);
+#define MU_CONV_VEC(TAPS)                                                                                              \
+    code = launch_pdl(ssd_conv_vec_kernel<TE, TO, TAPS>, grid, block, 0, s, 1, u, ldu, weight, bias, channels, n_tokens, \
+                      tok_seq, seq_first, seq_slots, (const float*)state, state_stride, out)
+        if (taps == 2) MU_CONV_VEC(2);
+        else if (taps == 3) MU_CONV_VEC(3);
+        else MU_CONV_VEC(4);
+#undef MU_CONV_VEC
+    } else {
+        const dim3 grid(n_tokens, (channels + 255) / 256), block(256);
+        code = launch_pdl(ssd_conv_kernel<TE, TO>, grid, block, 0, s, 1, u, ldu, weight, bias, channels, taps, n_tokens,
+                          tok_seq, seq_first, seq_slots, state, state_stride, single_tokens, out);
+    }
+    if (code != MU_OK || single_tokens || taps == 1) return code;
+    const long long cells = (long long)n_seqs * channels;
+    return launch_pdl(ssd_conv_tail_kernel<TE>, dim3((unsigned)((cells + 255) / 256)), dim3(256), 0, s, 1, u, ldu, channels,
+                      taps, n_seqs, seq_first, seq_slots, state, state_stride);
+}
+
+}  // namespace mu
+
 // u: the convolution's input channels of the step's tokens ([T, channels] view of the projection, compute dtype).
 // single_tokens: every sequence of the step brings exactly one token (the tail is moved on by the same launch).
+// out: contiguous [T, channels], float32, or with out_bf16 (and bfloat16 inputs) bfloat16.
 MU_EXPORT int mu_ssd_conv(const void* u, long long ldu, int u_bf16, const float* weight, const float* bias, int channels,
                           int taps, int n_tokens, int n_seqs, const int* tok_seq, const int* seq_first,
-                          const int* seq_slots, float* state, long long state_stride, int single_tokens, float* out,
-                          void* stream) {
+                          const int* seq_slots, float* state, long long state_stride, int single_tokens, void* out,
+                          void* stream, int out_bf16) {
     if (n_tokens <= 0) return MU_OK;
-    if (!u || !weight || !tok_seq || !seq_first || !seq_slots || !state || !out || channels <= 0 || taps < 1)
+    if (!u || !weight || !tok_seq || !seq_first || !seq_slots || !state || !out || channels <= 0 || taps < 1 ||
+        (out_bf16 && !u_bf16))
         return MU_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
-    const dim3 grid(n_tokens, (channels + 255) / 256), block(256);
-    int code = u_bf16 ? mu::launch_pdl(mu::ssd_conv_kernel<bf>, grid, block, 0, s, 1, (const bf*)u, ldu, weight, bias,
-                                       channels, taps, n_tokens, tok_seq, seq_first, seq_slots, state, state_stride,
-                                       single_tokens, out)
-                      : mu::launch_pdl(mu::ssd_conv_kernel<float>, grid, block, 0, s, 1, (const float*)u, ldu, weight,
-                                       bias, channels, taps, n_tokens, tok_seq, seq_first, seq_slots, state,
-                                       state_stride, single_tokens, out);
-    if (code != MU_OK || single_tokens || taps == 1) return code;
-    const long long cells = (long long)n_seqs * channels;
-    const dim3 tail_grid((unsigned)((cells + 255) / 256));
-    return u_bf16 ? mu::launch_pdl(mu::ssd_conv_tail_kernel<bf>, tail_grid, block, 0, s, 1, (const bf*)u, ldu, channels,
-                                   taps, n_seqs, seq_first, seq_slots, state, state_stride)
-                  : mu::launch_pdl(mu::ssd_conv_tail_kernel<float>, tail_grid, block, 0, s, 1, (const float*)u, ldu,
-                                   channels, taps, n_seqs, seq_first, seq_slots, state, state_stride);
+    if (out_bf16)
+        return mu::ssd_conv_launch((const bf*)u, ldu, weight, bias, channels, taps, n_tokens, n_seqs, tok_seq, seq_first,
+                                   seq_slots, state, state_stride, single_tokens, (bf*)out, s);
+    if (u_bf16)
+        return mu::ssd_conv_launch((const bf*)u, ldu, weight, bias, channels, taps, n_tokens, n_seqs, tok_seq, seq_first,
+                                   seq_slots, state, state_stride, single_tokens, (float*)out, s);
+    return mu::ssd_conv_launch((const float*)u, ldu, weight, bias, channels, taps, n_tokens, n_seqs, tok_seq, seq_first,
+                               seq_slots, state, state_stride, single_tokens, (float*)out, s);
 }
 
 MU_EXPORT int mu_ssd_scan(const float* xbc, int channels, const void* dt_raw, long long lddt, int dt_bf16,

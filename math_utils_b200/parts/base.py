@@ -2,7 +2,8 @@
 
 A model is put together from five kinds of parts: ``embedding``, ``position``
 (position encoding), ``norm``, ``mixer`` (attention, or anything else that
-mixes tokens of a sequence), ``feed_forward``, ``head``; and an
+mixes tokens of a sequence), ``feed_forward``, ``head``; a ``scale`` (numbers
+that multiply a sublayer's result) where an arrangement wants one; and an
 ``arrangement`` that wires one layer's norms, mixer and feed-forward around
 the residual stream.  A part is built from its ``PartSpec`` alone: it never
 learns which model or architecture it is in.
@@ -25,7 +26,7 @@ from typing import Any, Callable, Dict, Mapping, Optional, Sequence, Tuple
 
 from ..config.base import ConfigError, PartSpec
 
-PART_ROLES = ("embedding", "position", "norm", "mixer", "feed_forward", "head", "arrangement")
+PART_ROLES = ("embedding", "position", "norm", "mixer", "feed_forward", "head", "arrangement", "scale")
 
 
 @dataclass(frozen=True)
@@ -259,6 +260,31 @@ class Head(Part):
         raise NotImplementedError
 
 
+class LayerScale(Part):
+    """One number per entry of the row that multiplies what a sublayer adds to the stream (parameter ``size``, tensor
+    ``weight``); the arrangement that has it as an extra part hands it to the launch that makes the addition."""
+
+    def tensor_specs(self):
+        return (TensorSpec(self.tensor_name("weight"), (int(self.param("size")),), role="vector",
+                           init=self.param("init", "norm_weight")),)
+
+    def bind(self, tensors, runtime):
+        super().bind(tensors, runtime)
+        self.weight = tensors[self.tensor_name("weight")]
+
+
+@dataclass
+class PendingJoin:
+    """What an arrangement left for the next norm's launch to add to the stream ``x``:
+    (mult * y + mult2 * y2) * scale, ``y2`` (a second branch) and ``scale`` (one float32 per entry) where given."""
+    x: Any
+    y: Any
+    mult: float = 1.0
+    y2: Any = None
+    mult2: float = 0.0
+    scale: Any = None
+
+
 class Arrangement(Part):
     """Wires one layer.  ``forward(x, layer, ctx, cache, owns_cache)`` updates
     the float32 residual stream ``x`` in place; ``layer`` has ``norm1``,
@@ -286,6 +312,9 @@ def build_part(role: str, spec: PartSpec) -> Part:
         known = sorted(k for r, k in _PARTS if r == role)
         raise ConfigError(f"no {role} of kind '{spec.kind}'; known: {', '.join(known)}") from None
     return factory(spec)
+
+
+register_part("scale", "layer_scale", LayerScale, replace=True)
 
 
 def known_parts(role: Optional[str] = None):

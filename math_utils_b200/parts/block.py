@@ -20,7 +20,9 @@ layer without a feed-forward (kind ``none``) stops after the mixer.
 (parameter ``residual_mult``) on what the sublayers add.  A sublayer writes its result to a float32
 buffer; the addition to the stream is made by the launch of the NEXT norm (``ops.residual_add_norm``:
 x += m * y, then the normed row), also across layers (``StepContext.pending_join``), so the stream is
-read and written once per sublayer.
+read and written once per sublayer.  Extra parts ``scale1`` and ``scale2`` (role ``scale``) multiply the mixer's and
+the feed-forward's result entry by entry, in the same launch; so is the weighted sum of two mixers side by side made
+there (``forward_pair``).
 
 ``parallel_pre_norm``: x += mixer(norm1(x)) + feed_forward(norm2(x)), both sublayers reading the SAME x through a
 norm of their own.  Both norms are made before either sublayer adds into the stream (two RMS norms with one eps
@@ -36,7 +38,7 @@ from __future__ import annotations
 import torch
 
 from .attention import CausalSelfAttention
-from .base import Arrangement, PositionEncoding, register_part
+from .base import Arrangement, PendingJoin, PositionEncoding, register_part
 from .feedforward import DenseFeedForward, NoFeedForward
 from .norm import IdentityNorm, LayerNorm, RmsNorm
 
@@ -187,8 +189,15 @@ class ScaledPreNormBlock(Arrangement):
         y = ctx.buffer("sublayer.out", tuple(x.shape), torch.float32)
         h = self._norm(layer.norm1, x, ctx)
         ctx.note("ln1", h)
-        SandwichNormBlock._sublayer(layer.mixer, y, h, y, ctx, cache, owns_cache)
-        ctx.pending_join = (x, y, self.mult)
+        pair = getattr(layer.mixer, "forward_pair", None)
+        if pair is not None:
+            # two mixers side by side: their weighted sum is made where it joins the stream
+            first, second = pair(h, ctx, cache, owns_cache)
+            a, b = layer.mixer.scales
+            ctx.pending_join = PendingJoin(x, first, self.mult * a, second, self.mult * b, self._scale(layer, "scale1"))
+        else:
+            SandwichNormBlock._sublayer(layer.mixer, y, h, y, ctx, cache, owns_cache)
+            ctx.pending_join = PendingJoin(x, y, self.mult, scale=self._scale(layer, "scale1"))
         if ctx.trace is not None:
             ctx.flush_join()
             ctx.note("res1", x)
@@ -196,23 +205,29 @@ class ScaledPreNormBlock(Arrangement):
             h = self._norm(layer.norm2, x, ctx)
             ctx.note("ln2", h)
             SandwichNormBlock._sublayer(layer.feed_forward, y, h, y, ctx)
-            ctx.pending_join = (x, y, self.mult)
+            ctx.pending_join = PendingJoin(x, y, self.mult, scale=self._scale(layer, "scale2"))
         if ctx.trace is not None:
             ctx.flush_join()
             ctx.note("res2", x)
+
+    @staticmethod
+    def _scale(layer, name):
+        part = layer.extra.get(name)
+        return None if part is None else part.weight
 
     @staticmethod
     def _norm(norm, x, ctx):
         """The normed stream, with what is still to be added to the stream added by the same launch."""
         if isinstance(norm, RmsNorm) and norm.offset == 0.0 and norm.scale == 1.0 and x.stride(1) == 1:
             pending, ctx.pending_join = ctx.pending_join, None
-            if pending is not None and pending[0] is not x:
+            if pending is not None and pending.x is not x:
                 ctx.pending_join = pending
                 ctx.flush_join()
                 pending = None
             out = ctx.buffer("stream.normed", tuple(x.shape), norm.runtime.dtype)
-            y, mult = (pending[1], pending[2]) if pending is not None else (None, 0.0)
-            return norm.runtime.ops.residual_add_norm(x, y, mult, norm.weight, norm.eps, out, groups=norm.groups)
+            p = pending if pending is not None else PendingJoin(x, None)
+            return norm.runtime.ops.residual_add_norm(x, p.y, p.mult, norm.weight, norm.eps, out, groups=norm.groups, y2=p.y2,
+                                                      mult2=p.mult2, scale=p.scale)
         ctx.flush_join()
         return norm.forward(x)
 
@@ -241,7 +256,7 @@ class ParallelPreNormBlock(Arrangement):
             self._join.record(self._side)
         layer.mixer.forward(h, x, ctx, cache, owns_cache)
         main.wait_event(self._join)
-        ctx.pending_join = (x, y, 1.0)
+        ctx.pending_join = PendingJoin(x, y)
 
     def forward(self, x, layer, ctx, cache, owns_cache: bool) -> None:
         n1, n2 = layer.norm1, layer.norm2

@@ -32,7 +32,7 @@ class TokenEmbedding(Embedding):
 
 
 class TokenPairEmbedding(Embedding):
-    """A row per token plus a row of a second table chosen by the token and the one before it:
+    """A row per token (times the parameter ``scale``, 1 if absent) plus a row of a second table chosen by the token and the one before it:
     row (previous * mul_prev + token * mul_cur) mod buckets, and row ``buckets`` (the table's last) for the first
     token of a sequence.  The token before the first token of a step is the sequence's state: the cache keeps
     it per slot (``StepContext.last_tokens``), and the kernel moves it on."""
@@ -44,6 +44,7 @@ class TokenPairEmbedding(Embedding):
         self.hidden_size = int(self.param("hidden_size"))
         self.buckets = int(self.param("buckets"))
         self.mul_prev, self.mul_cur = int(self.param("mul_prev")), int(self.param("mul_cur"))
+        self.scale = float(self.param("scale", 1.0))
 
     def tensor_specs(self):
         return (TensorSpec(self.tensor_name("weight"), (self.vocab_size, self.hidden_size), role="table"),
@@ -68,7 +69,7 @@ class TokenPairEmbedding(Embedding):
                 if self.runtime.dtype == torch.bfloat16 else None)
         x = self.runtime.ops.embed_pair(ctx.token_ids, ctx.tok_pos, ctx.tok_seq, ctx.seq_first, ctx.seq_slots,
                                         ctx.last_tokens, self.weight, self.pair_weight, self.mul_prev, self.mul_cur,
-                                        ctx.is_decode, copy=copy)
+                                        ctx.is_decode, copy=copy, scale=self.scale)
         ctx.stream_copy = copy
         return x
 

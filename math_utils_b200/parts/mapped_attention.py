@@ -24,7 +24,11 @@ bias), before the output projection; ``qk_norm`` ``"unit"`` norms queries and ke
 rotates nothing; ``key_values`` makes the projected keys, as they are before their norm, the values too (no ``v``
 tensor; vdim equals dim); ``slopes``: ``"geometric"`` takes slope_h * distance off every score,
 slope_h = 2^(-8 (h + 1) / n_heads); ``keep`` n > 0, with a window, leaves the sequence's first n positions in sight of
-every later token (the cache keeps them).
+every later token (the cache keeps them); ``softcap`` c > 0 makes a scaled score s into c tanh(s / c); ``sink`` counts one
+more key of score zero, without a value, in the softmax's denominator; ``entry_gate`` multiplies the heads side by side by
+sigmoid(G x) entry by entry (tensor ``gate`` [heads * vdim, hidden], no bias) before the output projection.  Where the
+keys are the values and go to the cache as they are (``key_values`` without norm and rotation) a cached row holds them
+once.  ``cache_window`` beside ``chunk``: the cache gives back pages that no later token's chunk can reach.
 """
 from __future__ import annotations
 
@@ -55,6 +59,8 @@ class MappedAttention(Mixer):
         self.key_values = bool(p("key_values", False))
         self.slopes = p("slopes", None)
         self.keep = int(p("keep", 0))
+        self.softcap, self.sink = float(p("softcap", 0.0) or 0.0), bool(p("sink", False))
+        self.entry_gate = bool(p("entry_gate", False))
         if self.qk_norm not in (True, False, "unit"):
             raise ConfigError(f"mapped attention: qk_norm '{self.qk_norm}' is not true, false or 'unit'")
         if self.key_values and (self.dim != self.vdim or self.maps != 1 or not self.own_kv):
@@ -74,6 +80,10 @@ class MappedAttention(Mixer):
             raise ConfigError(f"mapped attention has one or two score maps, got {self.maps}")
         if self.n_heads % self.n_kv_heads:
             raise ConfigError(f"mapped attention: {self.n_heads} heads do not split over {self.n_kv_heads} kv heads")
+        if self.chunk and self.cache_window and self.cache_window < self.chunk:
+            raise ConfigError("mapped attention: the cache keeps fewer positions than a chunk has")
+        if self.head_gate and self.entry_gate:
+            raise ConfigError("mapped attention: a gate per head and one per entry exclude one another")
         if self.window and self.cache_window and self.cache_window < self.window:
             raise ConfigError("mapped attention: the cache keeps fewer positions than the window sees")
         rot = p("rot") or {"dims": 0, "base": 1.0}
@@ -84,6 +94,9 @@ class MappedAttention(Mixer):
         self.q_width = self.n_heads * self.maps * self.dim
         self.k_width = self.n_kv_heads * self.maps * self.dim
         self.v_width = self.n_kv_heads * self.vdim
+        # cached keys that are the very values are kept once
+        self.shared_rows = self.key_values and self.qk_norm is False and self.rot_dims == 0
+        self.gate_width = self.n_heads * (1 if self.head_gate else self.vdim if self.entry_gate else 0)
 
     def tensor_specs(self):
         D, name = self.hidden_size, self.tensor_name
@@ -98,8 +111,8 @@ class MappedAttention(Mixer):
             if self.qk_norm is True:
                 specs.append(TensorSpec(name("k_norm"), (self.dim,), role="vector", init="norm_weight"))
             widths += [("k_bias", self.k_width)] + ([] if self.key_values else [("v_bias", self.v_width)])
-        if self.head_gate:
-            specs.append(TensorSpec(name("gate"), (self.n_heads, D)))
+        if self.gate_width:
+            specs.append(TensorSpec(name("gate"), (self.gate_width, D)))
         specs.append(TensorSpec(name("out"), (D, self.n_heads * self.vdim), init="residual_projection"))
         widths.append(("out_bias", D))
         if self.bias:
@@ -109,7 +122,7 @@ class MappedAttention(Mixer):
         return specs
 
     def cache_spec(self):
-        return RowCacheSpec(self.k_width + self.v_width, self.cache_window, self.keep)
+        return RowCacheSpec(self.k_width + (0 if self.shared_rows else self.v_width), self.cache_window, self.keep)
 
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
@@ -118,16 +131,16 @@ class MappedAttention(Mixer):
         mats = [t(r) for r in roles]
         biases = [t(r + "_bias") for r in roles] if self.bias else None
         self.gate_at = None
-        if self.head_gate:
+        if self.gate_width:
             # the gates ride in the same product, after q | k | v; rows of zeros keep the stacked row a whole
             # number of 16-byte pieces
             self.gate_at = len(mats) + 1
-            pad = -(sum(m.shape[0] for m in mats) + self.n_heads) % 8
+            pad = -(sum(m.shape[0] for m in mats) + self.gate_width) % 8
             mats.append(t("gate"))
             if pad:
                 mats.append(torch.zeros((pad, self.hidden_size), dtype=mats[0].dtype, device=mats[0].device))
             if biases is not None:
-                biases.append(torch.zeros(self.n_heads + pad, dtype=torch.float32, device=biases[0].device))
+                biases.append(torch.zeros(self.gate_width + pad, dtype=torch.float32, device=biases[0].device))
         weight = torch.cat(mats, dim=0).contiguous() if len(mats) > 1 else mats[0]
         bias = torch.cat(biases).contiguous() if biases is not None else None
         self.widths = tuple(m.shape[0] for m in mats)
@@ -160,19 +173,22 @@ class MappedAttention(Mixer):
         self.proj(h, out=views[0])
         q = views[1]
         k, v = (views[2], views[2 if self.key_values else 3]) if owns_cache else (None, None)
+        if self.shared_rows:
+            v = None
         gate = views[self.gate_at] if self.gate_at is not None else None
         table = ctx.block_tables[cache.group]
         ops.qk_prepare(q, k, v, self.q_norm, self.k_norm, self.freq_table, self.magnitude, self.rot_dims, self.eps,
                        self.n_heads, self.n_kv_heads, self.maps, self.dim, self.vdim, ctx.tok_pos, ctx.tok_seq,
                        table if owns_cache else None, cache.page_tokens, cache.pages if owns_cache else None,
-                       pairs=self.rot_layout == "pairs")
+                       pairs=self.rot_layout == "pairs", shared=self.shared_rows and owns_cache)
         ctx.note("q", q)
         heads = ctx.buffer("mapped.heads", (T, self.n_heads * self.vdim), dt)
         ops.mapped_attention(q, cache.pages, table, cache.page_tokens, ctx.tok_pos, ctx.tok_seq, self.n_heads,
                              self.n_kv_heads, self.maps, self.dim, self.vdim, self.scale, self.window, heads,
                              lam=self.lam, out_scale=self.out_scale, eps=self.eps, unit_rms=self.maps == 2,
                              tiles=None if ctx.is_decode else ctx.q_tiles, single_tokens=ctx.is_decode,
-                             gate=gate, chunk=self.chunk, slopes=self.slope_table, keep=self.keep)
+                             gate=gate, chunk=self.chunk, slopes=self.slope_table, keep=self.keep,
+                             sink=self.sink, softcap=self.softcap, shared=self.shared_rows)
         ctx.note("attn", heads)
         self.out(heads, residual=residual if accumulate else None, out=residual)
 

@@ -10,7 +10,7 @@ mean, no variance, no eps.  Tensors ``weight``, ``bias``, ``alpha`` (a scalar).
 ``weight_offset`` (0 unless given; 1 for a weight stored around zero) and ``scale`` (1 unless given:
 the multiplier with which a normed sublayer output joins the residual stream) are parameters, and so is
 ``groups`` (1 unless given): the row in that many consecutive equal parts, each divided by its own rms, times one
-weight for the whole row."""
+weight for the whole row; ``one_number``: the weight is a single number for all entries (a tensor of shape [])."""
 from __future__ import annotations
 
 from ..config.base import ConfigError, PartSpec
@@ -78,12 +78,14 @@ class RmsNorm(Norm):
             raise ConfigError(f"rms_norm: {self.size} entries do not split into {self.groups} equal groups")
 
     def tensor_specs(self):
-        return (TensorSpec(self.tensor_name("weight"), (self.size,), role="vector",
-                           init=self.param("init", "norm_weight")),)
+        shape = () if self.param("one_number", False) else (self.size,)
+        return (TensorSpec(self.tensor_name("weight"), shape, role="vector", init=self.param("init", "norm_weight")),)
 
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
         self.weight = tensors[self.tensor_name("weight")]
+        if self.param("one_number", False):
+            self.weight = self.weight.reshape(1).expand(self.size).contiguous()
 
     def forward(self, x, rows=None, out=None):
         return self.runtime.ops.rms_norm_out(x, self.weight, self.eps, self.offset, self.scale, out=out,
