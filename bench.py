@@ -9,6 +9,7 @@
     python bench.py --family seledra [--size s|m] [--batch B] [--steps K]   # Seledra beside Lusalorn at equal size
     python bench.py --family tibopel [--size s|m] [--batch B] [--steps K]   # Tibopel beside Forisun at equal size
     python bench.py --family pelenex [--size s|m] [--batch B] [--steps K]   # Pelenex beside Seledra, Lusalorn and Tibopel
+    python bench.py --family tokolorn [--size s|m] [--batch B] [--steps K]  # Tokolorn beside Pelenex, Lusalorn and Tibopel
 
 A "step" is one decode step of the whole batch.  The default run has the layer
 sizes of GPT-2 small (BASELINE.json's third configuration) with seeded random
@@ -601,6 +602,35 @@ def pelenex_config(size):
     return ours, seledra_config(size)[0], lusalorn_config(size)[0], tibopel_config(size)[0]
 
 
+TOKOLORN_SIZES = {
+    # width, chunked attention (heads, kv heads, dim, chunk), lightning attention (heads, dim, vdim), windowed attention
+    # (heads, kv heads, dim, vdim, window, rotated), selective scan (channels, state, dt rank, taps), dense ff
+    "s": (1024, (8, 2, 128, 512), (8, 128, 128), (8, 2, 128, 128, 512, 128), (2048, 16, 64, 4), 4096),
+    "m": (2048, (16, 4, 128, 512), (16, 128, 128), (16, 4, 128, 128, 512, 128), (4096, 16, 128, 4), 8192),
+}
+
+
+def tokolorn_config(size):
+    """A Tokolorn configuration with layer sizes of a real model's order (random weights): chunked attention, lightning
+    attention, windowed attention beside a selective scan, lightning attention; and beside it the designs its layers are
+    like, each at its own configuration of this size (equal width, layer count and vocabulary): Pelenex (linear
+    recurrences, attention beside a recurrence), Lusalorn (a state-space mixer beside attention, a gated feed-forward, the
+    token-pair embedding), Tibopel (chunked attention)."""
+    D, (H, G, d, chunk), (lh, ld, lv), (wh, wg, wd, wv, window, rot), (inner, state, rank, taps), ff = TOKOLORN_SIZES[size]
+    dense = {"kind": "dense", "ff": ff}
+    fading = {"type": "lightning", "mlp": dense, "mixer": {"heads": lh, "dim": ld, "vdim": lv, "decay": [
+        round(1.0 - 2.0 ** (-1.0 - 7.0 * h / max(lh - 1, 1)), 6) for h in range(lh)]}}
+    both = {"left": {"heads": wh, "kv_heads": wg, "dim": wd, "vdim": wv, "scale": wd ** -0.5, "softcap": 30.0,
+                     "mask": {"size": window}, "rot": {"base": 10000.0, "dims": rot}},
+            "right": {"inner": inner, "state": state, "dt_rank": rank, "conv": taps}, "left_scale": 0.7, "right_scale": 0.4}
+    layers = [{"type": "attention", "mlp": dense, "mixer": {"heads": H, "kv_heads": G, "dim": d, "scale": d ** -0.5,
+                                                            "mask": {"size": chunk}}},
+              fading, {"type": "parallel", "mlp": dense, "mixer": both}, fading]
+    ours = {"architecture": "Tokolorn", "vocab": FAMILY_VOCAB, "width": D, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+            "embedding": {"scale": 8.0, "bigram": {"buckets": 4093, "mul_prev": 17, "mul_cur": 5}}, "layers": layers}
+    return ours, pelenex_config(size)[0], lusalorn_config(size)[0], tibopel_config(size)[0]
+
+
 def stage_times(model, prompts, single_steps=8):
     """Device milliseconds per stage of one eager prompt step and of eager single-token steps (their mean)."""
     import torch
@@ -624,18 +654,19 @@ def stage_times(model, prompts, single_steps=8):
 
 
 def run_family(args):
-    """``--family forisun | lusalorn | seledra | tibopel | pelenex``: prompt and single-token throughput of that design at
+    """``--family forisun | lusalorn | seledra | tibopel | pelenex | tokolorn``: prompt and single-token throughput of that design at
     sizes of a real model's order beside GPT-2 (Seledra: beside Lusalorn; Tibopel: beside Forisun; Pelenex: beside the
-    three it is like) at equal size, the same workload shape as the default run (2 x 1,024-token prompts; a batch from
+    three it is like; Tokolorn too) at equal size, the same workload shape as the default run (2 x 1,024-token prompts; a batch from
     512-token prompts towards 1,024).  Prints one JSON line; the default run and its line are not touched."""
     import numpy as np
     from math_utils_b200.sampling import SamplingParams
     pk = peaks()
     rng = np.random.default_rng(0)
     configs = {"forisun": forisun_config, "lusalorn": lusalorn_config, "seledra": seledra_config,
-               "tibopel": tibopel_config, "pelenex": pelenex_config}[args.family](args.size)
+               "tibopel": tibopel_config, "pelenex": pelenex_config, "tokolorn": tokolorn_config}[args.family](args.size)
     others = {"seledra": ("lusalorn_twin",), "tibopel": ("forisun_twin",),
-              "pelenex": ("seledra_twin", "lusalorn_twin", "tibopel_twin")}.get(args.family, ("gpt2_twin",))
+              "pelenex": ("seledra_twin", "lusalorn_twin", "tibopel_twin"),
+              "tokolorn": ("pelenex_twin", "lusalorn_twin", "tibopel_twin")}.get(args.family, ("gpt2_twin",))
     record = {"family": args.family, "size": args.size, "batch": args.batch, "steps": args.steps, "dtype": "bfloat16",
               "data": "synthetic: random weights, random tokens", "peaks": pk, "models": {}}
     for name, cfg in zip((args.family,) + others, configs):
@@ -822,9 +853,10 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="with --only decode: tokens per prompt")
     ap.add_argument("--reference-dir", default="", help="with --impl reference: a checkout other than baseline/_ref")
     ap.add_argument("--tokens", type=int, default=0, help="with --config: fewer tokens per request than fill the context")
-    ap.add_argument("--family", default="", choices=["", "forisun", "lusalorn", "seledra", "tibopel", "pelenex"],
+    ap.add_argument("--family", default="", choices=["", "forisun", "lusalorn", "seledra", "tibopel", "pelenex", "tokolorn"],
                     help="that design at sizes of a real model's order beside GPT-2 (seledra: beside Lusalorn; tibopel: "
-                         "beside Forisun; pelenex: beside Seledra, Lusalorn and Tibopel) at equal size")
+                         "beside Forisun; pelenex: beside Seledra, Lusalorn and Tibopel; tokolorn: beside Pelenex, Lusalorn "
+                         "and Tibopel) at equal size")
     ap.add_argument("--size", default="s", choices=sorted(FORISUN_SIZES), help="with --family: which sizes")
     args = ap.parse_args()
     if args.gpus != 1:

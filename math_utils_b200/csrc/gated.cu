@@ -18,6 +18,11 @@ __device__ __forceinline__ float gate_act(float z, int act) {
     return apply_act(z, act);
 }
 
+__device__ __forceinline__ float gate_act_bf16(float z, int act) {       // for a product that is rounded to bfloat16
+    if (act == ACT_SILU) return __fdividef(z, 1.0f + __expf(-z));
+    return apply_act_bf16(z, act);
+}
+
 template <typename T>
 __global__ void gated_act_kernel(const T* __restrict__ a, long long lda, T* __restrict__ out, long long ldo, int n_rows,
                                  int width, int act) {
@@ -51,7 +56,7 @@ __global__ void gated_act_vec_kernel(const __nv_bfloat16* __restrict__ a, long l
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
             const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
-            o2[k] = __floats2bfloat162_rn(gate_act(g.x, act) * u.x, gate_act(g.y, act) * u.y);
+            o2[k] = __floats2bfloat162_rn(gate_act_bf16(g.x, act) * u.x, gate_act_bf16(g.y, act) * u.y);
         }
         *reinterpret_cast<uint4*>(out + r * ldo + c) = packed;
     }

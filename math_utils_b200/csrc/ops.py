@@ -119,6 +119,10 @@ _SIGNATURES = {
     "mu_linear_scan_max_dk": [],
     "mu_linear_scan": [_c_p, _c_p, _c_p, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_f, _c_p, _c_p, _c_p,
                        _c_ll, _c_ll, _c_p, _c_ll, _c_p, _c_int, _c_p, _c_ll, _c_int],
+    "mu_lightning_prompt_fits": [_c_int, _c_int],
+    "mu_lightning_prompt_scratch": [_c_int, _c_int, _c_int, _c_int, _c_int],
+    "mu_lightning_prompt": [_c_p, _c_p, _c_p, _c_ll, _c_p, _c_int, _c_p, _c_int, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_p,
+                            _c_p, _c_ll, _c_ll, _c_p, _c_ll, _c_p],
     "mu_exp_gates": [_c_p, _c_p, _c_ll, _c_p, _c_p, _c_f, _c_int, _c_int, _c_int, _c_p, _c_p, _c_p, _c_ll, _c_ll, _c_p,
                      _c_p],
     "mu_low_rank": [_c_p, _c_ll, _c_int, _c_p, _c_int, _c_int, _c_p],
@@ -866,6 +870,38 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
                                     out.stride(0), _ptr(norm_out), int(T > 4 * seq_slots.numel()), _stream(),
                                     0 if constant else 4 * n_heads, int(silu_rows)),
            ("linear_scan(heads={}, dk={}, dv={})", n_heads, dk, dv))
+    return out
+
+
+def lightning_prompt_ok(dk: int, dv: int) -> bool:
+    return bool(library().mu_lightning_prompt_fits(int(dk), int(dv)))
+
+
+def lightning_prompt(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, powers: torch.Tensor, n_heads: int, dk: int, dv: int,
+                     tiles: torch.Tensor, tok_seq, seq_first, seq_slots, state: torch.Tensor, state_offset: int,
+                     out: torch.Tensor) -> torch.Tensor:
+    """``linear_scan`` with one constant decay per head, no scale and silu on its rows, for steps of many tokens on
+    tensor cores: ``q``, ``k``, ``v`` bfloat16 column blocks of one buffer, ``tiles`` the step's query tiles (int32 [n, 2]),
+    ``powers`` float32 [heads, 65] = decay^0 .. decay^64, ``out`` float32 [T, heads * dv]."""
+    _need_cuda(q, k, v, powers, tiles, tok_seq, seq_first, seq_slots, state, out)
+    for t, name in ((tiles, "tiles"), (tok_seq, "tok_seq"), (seq_first, "seq_first"), (seq_slots, "seq_slots")):
+        _i32(t, name)
+    T = q.shape[0]
+    for t, n in ((q, n_heads * dk), (k, n_heads * dk), (v, n_heads * dv)):
+        if t.dtype != torch.bfloat16 or tuple(t.shape) != (T, n) or t.stride(1) != 1 or t.stride(0) != q.stride(0):
+            raise KernelError("lightning_prompt: queries, keys and values are bfloat16 column blocks of one buffer")
+    if (powers.dtype != torch.float32 or tuple(powers.shape) != (n_heads, 65) or not powers.is_contiguous()
+            or out.dtype != torch.float32 or out.stride(1) != 1 or tuple(out.shape) != (T, n_heads * dv)
+            or state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < state_offset + n_heads * dk * dv):
+        raise KernelError("lightning_prompt: powers, state or output do not fit")
+    lib = library()
+    lib.mu_lightning_prompt_scratch.restype = _c_ll
+    n_seqs = seq_slots.numel()
+    room = scratch("lightning_prompt", q.device, int(lib.mu_lightning_prompt_scratch(T, n_seqs, n_heads, dk, dv)), torch.float32)
+    _check(lib.mu_lightning_prompt(_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(tiles), tiles.shape[0], _ptr(tok_seq), n_seqs,
+                                   _ptr(seq_first), _ptr(seq_slots), _ptr(powers), int(n_heads), int(dk), int(dv), _ptr(room),
+                                   _ptr(state), state.stride(0), int(state_offset), _ptr(out), out.stride(0), _stream()),
+           ("lightning_prompt(heads={}, dk={}, dv={})", n_heads, dk, dv), launches=3)
     return out
 
 

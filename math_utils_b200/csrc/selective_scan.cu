@@ -27,6 +27,11 @@ __device__ __forceinline__ float exp2_fast(float x) {        // results below 2^
 }
 
 // VEC: every channel's state starts on a 16-byte boundary and N is a multiple of four.
+template <typename TE> __device__ __forceinline__ float gated(float v, float z) { return v * z / (1.0f + expf(-z)); }
+template <> __device__ __forceinline__ float gated<__nv_bfloat16>(float v, float z) {      // rounded right after
+    return __fdividef(v * z, 1.0f + __expf(-z));
+}
+
 // SS_CHUNK: tokens staged at a time.
 template <typename TE, int LPC, int NS, bool VEC, int SS_CHUNK>
 __global__ void __launch_bounds__(SS_THREADS)
@@ -90,34 +95,34 @@ selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restr
         }
         copy_async_commit();
     };
-    float xr[PER], dr[PER], zr[PER], gate_x[PER], gate_z[PER];
+    // (read as they are, from places that always exist: nothing may wait for a load before all are on their way)
+    TE xr[PER], zr[PER];
+    float dr[PER], gate_x[PER], gate_z[PER];
     auto read_rows = [&](int li0) {
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const int i = tid + SS_THREADS * k, tok = i / COLS, col = c0 + i % COLS;
-            xr[k] = dr[k] = zr[k] = 0.0f;
-            if (i < SS_CHUNK * COLS && li0 + tok < count && col < inner) {
-                const long long t = first + li0 + tok;
-                xr[k] = to_float(x[t * ldx + col]);
-                dr[k] = dt[t * lddt + col];
-                zr[k] = to_float(z[t * ldz + col]);
-            }
+            const int i = tid + SS_THREADS * k, col = min(c0 + i % COLS, inner - 1);
+            const long long t = first + min(li0 + i / COLS, count - 1);
+            xr[k] = x[t * ldx + col];
+            dr[k] = dt[t * lddt + col];
+            zr[k] = z[t * ldz + col];
         }
     };
-    auto stage_rows = [&](int b) {
+    auto stage_rows = [&](int li0, int b) {
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
             const int i = tid + SS_THREADS * k;
-            if (i < SS_CHUNK * COLS) ds[b][i / COLS][i % COLS] = make_float2(dr[k], dr[k] * xr[k]);
-            gate_x[k] = xr[k];
-            gate_z[k] = zr[k];
+            const float step = li0 + i / COLS < count ? dr[k] : 0.0f;
+            gate_x[k] = to_float(xr[k]);
+            gate_z[k] = to_float(zr[k]);
+            if (i < SS_CHUNK * COLS) ds[b][i / COLS][i % COLS] = make_float2(step, step * gate_x[k]);
         }
     };
     __syncthreads();                                         // the zeros are down before the first copies land
     if (count > 0) {
         copy_bc(0, 0);
         read_rows(0);
-        stage_rows(0);
+        stage_rows(0, 0);
     }
     int b = 0;
     for (int li0 = 0; li0 < count; li0 += SS_CHUNK, b ^= 1) {
@@ -174,10 +179,10 @@ selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restr
             const int i = tid + SS_THREADS * k, tok = i / COLS, col = c0 + i % COLS;
             if (i < SS_CHUNK * COLS && tok < n && col < inner) {
                 const float v = fmaf(skip[col], gate_x[k], ys[tok][i % COLS]), zz = gate_z[k];
-                y[(long long)(first + li0 + tok) * ldy + col] = from_float<TE>(v * zz / (1.0f + expf(-zz)));
+                y[(long long)(first + li0 + tok) * ldy + col] = from_float<TE>(gated<TE>(v, zz));
             }
         }
-        if (more) stage_rows(b ^ 1);
+        if (more) stage_rows(li0 + SS_CHUNK, b ^ 1);
     }
     pdl_trigger();
     if (!live) return;

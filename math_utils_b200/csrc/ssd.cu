@@ -57,19 +57,25 @@ __global__ void ssd_conv_kernel(const TE* __restrict__ u, long long ldu, const f
 // channels and eight consecutive tokens, whose rows are all on their way at once; the taps' inputs stay in registers.
 constexpr int CV_CH = 8, CV_TOK = 8;
 
-__device__ __forceinline__ void cv_load(float (&v)[CV_CH], const float* p) {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+// A row's eight inputs as they lie in memory, and as numbers: all rows are on their way before the first is used.
+struct CvRaw32 { float4 a, b; };
+__device__ __forceinline__ CvRaw32 cv_raw(const float* p) {
+    return {*reinterpret_cast<const float4*>(p), *reinterpret_cast<const float4*>(p + 4)};
 }
-__device__ __forceinline__ void cv_load(float (&v)[CV_CH], const __nv_bfloat16* p) {
-    const uint4 raw = *reinterpret_cast<const uint4*>(p);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+__device__ __forceinline__ uint4 cv_raw(const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); }
+__device__ __forceinline__ void cv_numbers(float (&v)[CV_CH], const CvRaw32& r) {
+    v[0] = r.a.x, v[1] = r.a.y, v[2] = r.a.z, v[3] = r.a.w, v[4] = r.b.x, v[5] = r.b.y, v[6] = r.b.z, v[7] = r.b.w;
+}
+__device__ __forceinline__ void cv_numbers(float (&v)[CV_CH], const uint4& r) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&r);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const float2 f = __bfloat1622float2(h[i]);
         v[2 * i] = f.x, v[2 * i + 1] = f.y;
     }
 }
+__device__ __forceinline__ float cv_silu(float z, float) { return silu_f(z); }
+__device__ __forceinline__ float cv_silu(float z, __nv_bfloat16) { return __fdividef(z, 1.0f + __expf(-z)); }   // rounded right after
 __device__ __forceinline__ void cv_store(float* p, const float (&v)[CV_CH]) {
     *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
     *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
@@ -101,19 +107,22 @@ ssd_conv_vec_kernel(const TE* __restrict__ u, long long ldu, const float* __rest
     for (int i = 0; i < CV_CH; ++i) b8[i] = bias ? bias[c + i] : 0.0f;
     pdl_wait();
     const int t0 = blockIdx.x * CV_TOK, nt = min(CV_TOK, n_tokens - t0);
-    float rows[CV_TOK + TAPS - 1][CV_CH];                    // the inputs before the tile, then the tile's
+    decltype(cv_raw(u)) raw[CV_TOK + TAPS - 1];              // the rows before the tile, then the tile's
 #pragma unroll
-    for (int i = 0; i < CV_TOK; ++i)
-        if (i < nt) cv_load(rows[TAPS - 1 + i], u + (long long)(t0 + i) * ldu + c);
+    for (int i = 0; i < CV_TOK + TAPS - 1; ++i)
+        raw[i] = cv_raw(u + (long long)min(max(t0 + i - (TAPS - 1), 0), n_tokens - 1) * ldu + c);
     int s = tok_seq[t0], first = seq_first[s], end = seq_first[s + 1];
-    const float* tail = state + (long long)seq_slots[s] * state_stride + c;
+    float rows[TAPS][CV_CH];                                 // the inputs of the taps, oldest first
+    auto from_tail = [&](int j, int back) {                  // rows[j] = the input `back` places before the step's first token
+        const float* tail = state + (long long)seq_slots[s] * state_stride + (long long)(TAPS - 1 - back) * channels + c;
+#pragma unroll
+        for (int i = 0; i < CV_CH; ++i) rows[j][i] = tail[i];
+    };
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j) {
-        const int li = t0 - first - (TAPS - 1) + j;
-        if (li >= 0) cv_load(rows[j], u + (long long)(first + li) * ldu + c);
-        else
-#pragma unroll
-            for (int i = 0; i < CV_CH; ++i) rows[j][i] = tail[(long long)(TAPS - 1 + li) * channels + i];
+        const int back = (TAPS - 1) - j - (t0 - first);
+        if (back > 0) from_tail(j, back);
+        else cv_numbers(rows[j], raw[j]);
     }
 #pragma unroll
     for (int k = 0; k < CV_TOK; ++k) {
@@ -121,25 +130,23 @@ ssd_conv_vec_kernel(const TE* __restrict__ u, long long ldu, const float* __rest
         const int t = t0 + k;
         if (t >= end) {                                      // another sequence begins
             s = tok_seq[t], first = seq_first[s], end = seq_first[s + 1];
-            tail = state + (long long)seq_slots[s] * state_stride + c;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) from_tail(j, TAPS - 1 - j);
         }
+        cv_numbers(rows[TAPS - 1], raw[TAPS - 1 + k]);
         float acc[CV_CH];
 #pragma unroll
-        for (int i = 0; i < CV_CH; ++i) acc[i] = b8[i];
+        for (int i = 0; i < CV_CH; ++i) {
+            acc[i] = b8[i];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) {
-            const int li = t - first - (TAPS - 1) + j;
-            // (the rows in front of the tile are the first sequence's already; a later one's begin inside the tile)
-            const bool from_tail = li < 0 && first > t0;
-#pragma unroll
-            for (int i = 0; i < CV_CH; ++i) {
-                const float v = from_tail ? tail[(long long)(TAPS - 1 + li) * channels + i] : rows[k + j][i];
-                acc[i] = fmaf(w[i * TAPS + j], v, acc[i]);
-            }
+            for (int j = 0; j < TAPS; ++j) acc[i] = fmaf(w[i * TAPS + j], rows[j][i], acc[i]);
+            acc[i] = cv_silu(acc[i], TO());
         }
-#pragma unroll
-        for (int i = 0; i < CV_CH; ++i) acc[i] = silu_f(acc[i]);
         cv_store(out + (long long)t * channels + c, acc);
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+            for (int i = 0; i < CV_CH; ++i) rows[j][i] = rows[j + 1][i];
     }
 }
 

@@ -7,8 +7,9 @@ From the mixer's input x: q = silu(Q x), k = silu(K x) (n_heads x dim), v = silu
 The heads' o, side by side, is brought to unit rms over all of them, multiplied by a weight of that size and by
 sigmoid(G x), and goes through the output matrix.  The state is float32 and lives in the sequence's cache slot.
 
-Single tokens, short runs and the 32-bit path go token by token through the linear scan (``ops.linear_scan``), which
-applies silu to the rows it has staged.
+Prompt steps in bfloat16 go chunk by chunk over tensor cores (``ops.lightning_prompt``), all chunks at once but for the
+states between them; single tokens, short runs and the 32-bit path go token by token through the linear scan
+(``ops.linear_scan``, float32 rows).  Both apply silu to the rows as they stage them.
 """
 from __future__ import annotations
 
@@ -57,17 +58,28 @@ class LightningAttention(Mixer):
         self.out = Linear(t("out"), None, runtime)
         self.norm_weight = t("norm")
         # (decay, take, -, -) per head, the same for every token
+        self.chunked = runtime.dtype == torch.bfloat16 and runtime.ops.lightning_prompt_ok(self.dim, self.vdim)
+        exponents = torch.arange(65, dtype=torch.float64)
+        self.powers = (torch.tensor(self.decay, dtype=torch.float64)[:, None] ** exponents).float().contiguous().to(runtime.device)
         self.gates = torch.tensor([[[d, 1.0, 0.0, 0.0] for d in self.decay]], dtype=torch.float32, device=runtime.device)
+
+    CHUNKED_TOKENS = 24              # tokens a sequence brings on average from which on the chunked form pays
 
     def forward(self, h, residual, ctx, cache, owns_cache: bool, accumulate: bool = True) -> None:
         ops, T, H = self.runtime.ops, ctx.n_tokens, self.n_heads
         if not owns_cache:
             raise ConfigError("lightning attention keeps its own state: it cannot read another layer's")
-        u, q, k, v, gate = ctx.buffer("lightning.proj", (T, sum(self.columns)), torch.float32, columns=self.columns)[:5]
+        chunked = self.chunked and ctx.q_tiles is not None and T >= self.CHUNKED_TOKENS * ctx.n_seqs
+        u, q, k, v, gate = ctx.buffer("lightning.proj", (T, sum(self.columns)),
+                                      self.runtime.dtype if chunked else torch.float32, columns=self.columns)[:5]
         self.proj(h, out=u)
         o = ctx.buffer("lightning.o", (T, self.inner), torch.float32)
-        ops.linear_scan(q, k, v, self.gates, H, self.dim, self.vdim, 1.0, ctx.seq_first, ctx.seq_slots, cache.values, 0, o,
-                        silu_rows=True)
+        if chunked:
+            ops.lightning_prompt(q, k, v, self.powers, H, self.dim, self.vdim, ctx.q_tiles, ctx.tok_seq, ctx.seq_first,
+                                 ctx.seq_slots, cache.values, 0, o)
+        else:
+            ops.linear_scan(q, k, v, self.gates, H, self.dim, self.vdim, 1.0, ctx.seq_first, ctx.seq_slots, cache.values, 0, o,
+                            silu_rows=True)
         ctx.note("scan", o)
         gated = ctx.buffer("lightning.gated", (T, self.inner), self.runtime.dtype)
         ops.gated_group_norm(o, gate, self.norm_weight, 1, self.eps, gated, gate_after=True, sigmoid=True)

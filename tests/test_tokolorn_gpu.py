@@ -1,0 +1,838 @@
+"""Tokolorn through the engine against the plain NumPy statement of the design (plain_tokolorn.py):
+each mechanism alone, whole prompts, token-by-token decoding, prompts in portions, unequal batches,
+slots, pages and states used again, keys far away, at page borders and just inside and outside every window and chunk,
+looped layers, long decoding, odd sizes, and greedy generation through the library's own entry point."""
+import functools
+import json
+import math
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import helpers
+import plain_tokolorn as plain
+from helpers import run_batch, run_tail_one_by_one, run_whole
+from math_utils_b200 import DecoderModel, LLM, StepEntry
+from math_utils_b200.weights.safetensors import write_safetensors
+
+pytestmark = pytest.mark.gpu
+
+BF16_ROW = 0.03          # rms of a bfloat16 row's errors over its spread: layers that run again add their rounding again
+
+
+def check_logits(got, want, dtype, what=""):
+    helpers.check_logits(got, want, dtype, what, bf16_rms=BF16_ROW)
+
+
+def chunked(heads, kv_heads, dim, scale, chunk, ff=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "scale": scale}
+    if chunk:
+        m["mask"] = {"size": chunk}
+    return {"type": "attention", "mixer": m, "mlp": dense(ff)}
+
+
+def fading(dim, vdim, decay, ff=None):
+    return {"type": "lightning", "mixer": {"heads": len(decay), "dim": dim, "vdim": vdim, "decay": decay}, "mlp": dense(ff)}
+
+
+def both(heads, kv_heads, dim, vdim, scale, window, rot, softcap, inner, state, rank, conv, scales, ff=None):
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+    if window:
+        left["mask"] = {"size": window}
+    if rot:
+        left["rot"] = {"base": rot[0], "dims": rot[1]}
+    if softcap:
+        left["softcap"] = softcap
+    return {"type": "parallel", "mlp": dense(ff),
+            "mixer": {"left": left, "right": {"inner": inner, "state": state, "dt_rank": rank, "conv": conv},
+                      "left_scale": scales[0], "right_scale": scales[1]}}
+
+
+def dense(ff):
+    return None if ff is None else {"kind": "dense", "ff": ff}
+
+
+def config(vocab, width, eps, scale, bigram, logit_scale, loop, layers):
+    out = {"architecture": "Tokolorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "logit_scale": logit_scale,
+           "embedding": {"scale": scale}, "layers": layers}
+    if bigram:
+        out["embedding"]["bigram"] = dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))
+    if loop:
+        out["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return out
+
+
+# a chunk and a window that are no whole pages; a layer without a feed-forward; a loop over inner layers, three times
+CFG_A = config(300, 64, 1e-6, 4.0, (97, 13, 3), 0.6, (1, 3, 3), [
+    chunked(4, 2, 16, 0.4, 40, 96), fading(16, 8, [0.5, 0.93, 0.995]),
+    both(4, 1, 16, 24, 0.3, 33, (5000.0, 12), 6.0, 48, 6, 5, 4, (0.8, 0.3), 80), fading(8, 24, [0.9, 0.2], 72)])
+# nothing a multiple of 8; as many kv heads as heads and one; a window and a chunk of one; no mask, no rotation, no cap;
+# one tap and two, a rank of one; no bigram, no loop; a large eps; scales of one and below zero
+CFG_B = config(131, 50, 1e-3, 1.0, None, 1.0, None, [
+    chunked(3, 3, 7, 0.7, None, 33), both(5, 5, 6, 9, 0.5, 1, (100.0, 6), None, 21, 3, 1, 1, (1.0, 1.0), 21),
+    chunked(6, 1, 5, 0.6, 1), fading(5, 7, [0.8], 17), both(2, 1, 9, 5, 0.4, None, None, 2.5, 19, 17, 7, 2, (-0.6, 1.2)),
+    fading(33, 3, [0.999, 0.05, 1.0], 40)])
+# sizes the tensor-core kernels take; a window and a chunk of a page; the whole model twice
+CFG_C = config(384, 128, 2e-5, 7.0, (251, 1000003, 11), 0.4, (0, 5, 2), [
+    chunked(8, 2, 32, 0.25, 64, 256), fading(64, 32, [0.6, 0.9, 0.97, 0.999], 256),
+    both(8, 2, 32, 64, 0.2, 64, (20000.0, 32), 15.0, 256, 16, 8, 4, (0.5, 0.7), 192), chunked(4, 4, 64, 0.2, 130),
+    both(4, 1, 64, 128, 0.15, 100, (10000.0, 16), 30.0, 64, 24, 40, 3, (0.7, 0.4), 128), fading(128, 64, [0.98, 0.85], 128)])
+CONFIGS = {"a": CFG_A, "b": CFG_B, "c": CFG_C}
+CASES = [(n, d) for n in CONFIGS for d in ("float32", "bfloat16")]
+
+
+@functools.lru_cache(maxsize=None)
+def weights_of(name):
+    return plain.random_weights(CONFIGS[name], seed=sum(map(ord, name)) + 31)
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    out = {}
+    for name, cfg in CONFIGS.items():
+        d = str(tmp_path_factory.mktemp(f"tokolorn_{name}"))
+        with open(os.path.join(d, "config.json"), "w") as f:
+            json.dump(cfg, f)
+        write_safetensors(os.path.join(d, "model.safetensors"),
+                          {k: torch.from_numpy(np.array(v)).to(torch.bfloat16) for k, v in weights_of(name).items()})
+        out[name] = d
+    return out
+
+
+_models = {}
+
+
+def engine(folders, name, dtype):
+    if (name, dtype) not in _models:
+        model = DecoderModel.from_dir(folders[name], dtype=dtype)
+        _models[name, dtype] = (model, model.new_cache(max_tokens=64 * 24, n_slots=8))
+    return _models[name, dtype]
+
+
+def tokens_for(name, n, seed=0):
+    return np.random.default_rng(7000 + seed).integers(0, CONFIGS[name]["vocab"], size=n).tolist()
+
+
+_plain_cache = {}
+
+
+def plain_logits(name, tokens):
+    key = (name, tuple(tokens))
+    if key not in _plain_cache:
+        _plain_cache[key] = plain.forward(CONFIGS[name], weights_of(name), list(tokens))
+    return _plain_cache[key]
+
+
+# ------------------------------------------------------------------ whole models
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_whole_prompt_and_every_layer(folders, name, dtype):
+    model, cache = engine(folders, name, dtype)
+    toks = tokens_for(name, 150)
+    layers = []
+    want = plain.forward(CONFIGS[name], weights_of(name), toks, layers)
+    slot = cache.acquire()
+    trace = {}
+    got = model.step(cache, [StepEntry(slot, toks, list(range(len(toks))))], trace=trace).cpu().numpy()
+    cache.release(slot)
+    if dtype == "float32":
+        for i, x in enumerate(layers):                   # every pass of a looped layer counts
+            assert np.abs(trace[f"h.{i}.res2"] - x).max() < 2e-4, f"residual stream after layer run {i}"
+    check_logits(got, want, dtype, f"tokolorn {name} whole prompt")
+    check_logits(run_whole(model, cache, toks), want, dtype, f"tokolorn {name} whole prompt, no trace")
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_prompt_then_token_by_token(folders, name, dtype):
+    model, cache = engine(folders, name, dtype)
+    toks = tokens_for(name, 150, seed=1)                 # the tail crosses page and chunk borders and moves out of every window
+    got = run_tail_one_by_one(model, cache, toks, tail=120)
+    check_logits(got, plain_logits(name, toks), dtype, f"tokolorn {name} tail one by one")
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+@pytest.mark.parametrize("portions", [(2, 3, 59, 1, 64, 21), (64, 64, 22), (127, 2, 2, 19), (1, 1, 1, 147), (2,) * 12 + (126,)])
+def test_prompt_in_portions(folders, name, dtype, portions):
+    model, cache = engine(folders, name, dtype)
+    toks = tokens_for(name, 150, seed=2)[:sum(portions)]
+    slot = cache.acquire()
+    rows, at = [], 0
+    for n in portions:
+        rows.append(model.step(cache, [StepEntry(slot, toks[at:at + n], list(range(n)))]).cpu().numpy())
+        at += n
+    cache.release(slot)
+    check_logits(np.concatenate(rows), plain_logits(name, toks), dtype, f"tokolorn {name} portions {portions}")
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_unequal_batch_against_each_alone(folders, name, dtype):
+    model, cache = engine(folders, name, dtype)
+    lens, prompts = (140, 5, 66, 131), (129, 1, 33, 64)
+    requests = [tokens_for(name, n, seed=10 + i) for i, n in enumerate(lens)]
+    got = run_batch(model, cache, requests, prompts)
+    for i, r in enumerate(requests):
+        check_logits(got[i], plain_logits(name, r), dtype, f"tokolorn {name} batch request {i}")
+        if dtype == "float32":
+            alone = run_tail_one_by_one(model, cache, r, tail=lens[i] - prompts[i])
+            assert np.abs(alone - got[i]).max() < 4e-5, "a request's logits depend on its batch"
+
+
+@pytest.mark.parametrize("name,dtype", [("a", "float32"), ("b", "bfloat16"), ("c", "float32"), ("a", "bfloat16")])
+def test_slots_pages_and_state_used_again(folders, name, dtype):
+    model, cache = engine(folders, name, dtype)
+    free = [cache.free_pages(g.index) for g in cache.kv_groups]
+    first, second = tokens_for(name, 200, seed=20), tokens_for(name, 90, seed=21)
+    a = run_whole(model, cache, first)
+    slot = cache.acquire()                               # the slot, the pages and the state the first request held
+    model.step(cache, [StepEntry(slot, second[:70], [])])
+    b = [model.step(cache, [StepEntry(slot, [t], [0])]).cpu().numpy() for t in second[70:]]
+    cache.release(slot)
+    assert [cache.free_pages(g.index) for g in cache.kv_groups] == free
+    check_logits(a, plain_logits(name, first), dtype, f"tokolorn {name} first holder")
+    check_logits(np.concatenate(b), plain_logits(name, second)[70:], dtype, f"tokolorn {name} second holder of the slot")
+
+
+@pytest.mark.parametrize("name,dtype", [("a", "float32"), ("b", "float32"), ("c", "bfloat16")])
+@pytest.mark.parametrize("n", [1, 2, 3, 4, 23, 24, 39, 40, 41, 63, 64, 65, 127, 128, 129, 193])
+def test_first_tokens_and_lengths_around_borders(folders, name, dtype, n):
+    model, cache = engine(folders, name, dtype)
+    toks = tokens_for(name, 193, seed=30)
+    slot = cache.acquire()
+    got = model.step(cache, [StepEntry(slot, toks[:n], [0, n - 1])]).cpu().numpy()
+    cache.release(slot)
+    want = plain_logits(name, toks)                                    # causal: a prefix's logits are the long prompt's
+    check_logits(got, want[[0, n - 1]], dtype, f"tokolorn {name} prompt of {n}")
+
+
+@pytest.mark.parametrize("name,dtype", [("a", "float32"), ("b", "float32"), ("c", "bfloat16"), ("c", "float32")])
+def test_long_decoding(folders, name, dtype):
+    model, cache = engine(folders, name, dtype)
+    toks = tokens_for(name, 300, seed=40)
+    free = [cache.free_pages(g.index) for g in cache.kv_groups]
+    got = run_tail_one_by_one(model, cache, toks, tail=297)            # three tokens, then one by one over five pages
+    check_logits(got, plain_logits(name, toks), dtype, f"tokolorn {name} long decoding")
+    assert [cache.free_pages(g.index) for g in cache.kv_groups] == free
+
+
+def test_pages_go_back_when_a_chunk_or_window_is_left(folders):
+    model, cache = engine(folders, "a", "float32")                     # a chunk of 40, a window of 33
+    slot = cache.acquire()
+    model.step(cache, [StepEntry(slot, tokens_for("a", 250), [])])
+    for t in tokens_for("a", 90, seed=3):
+        model.step(cache, [StepEntry(slot, [t], [])])
+        assert all(g.pages_held(slot) <= 2 for g in cache.kv_groups)
+    cache.release(slot)
+
+
+@pytest.mark.parametrize("name", ["a", "b", "c"])
+def test_greedy_generation_through_the_library(folders, name):
+    llm = LLM(folders[name], dtype="float32", temperature=0.0, max_tokens=24, context=512)
+    assert llm.model.graph_safe                                            # single-token steps replay from a graph
+    prompts = [tokens_for(name, n, seed=50 + n) for n in (70, 3, 129)]
+    outs = llm.generate(prompts)
+    for p, out in zip(prompts, outs):
+        assert len(out) == 24
+        rows = plain.forward(CONFIGS[name], weights_of(name), list(p) + out)       # causal: one pass gives every step's row
+        for i, tok in enumerate(out):
+            row = rows[len(p) + i - 1]
+            best = int(np.argmax(row))
+            assert tok == best or row[best] - row[tok] < 1e-4, f"greedy token {i} of a prompt of {len(p)}"
+    alone = llm.generate([prompts[2]])[0]
+    assert alone == outs[2], "a request generates other tokens alone than in a batch"
+    from math_utils_b200 import SamplingParams
+    from math_utils_b200.engine.generate import generate
+    eager = generate(llm.model, [prompts[0]], 24, SamplingParams(0.0, 1, 0), context=512, use_graph=False)[0]
+    assert eager == outs[0], "eager steps and replayed steps generate different tokens"
+
+
+def test_requests_that_end_early_leave_the_others_alone(folders):
+    llm = LLM(folders["a"], dtype="float32", temperature=0.0, max_tokens=30, context=512)
+    prompts = [tokens_for("a", n, seed=70 + n) for n in (40, 9, 66, 3, 21)]
+    free = llm.generate(prompts, stop_ids=[])
+    stop = free[0][5]
+    want = [out[:out.index(stop)] if stop in out else out for out in free]
+    assert llm.generate(prompts, stop_ids=[stop]) == want
+    assert llm.generate(prompts[1:], stop_ids=[stop]) == want[1:]
+
+
+def test_conversation_on_a_kept_slot(folders):
+    """Two turns through ``LLM.prompt``: the slot keeps keys, the last token, and the recurrences' states of every pass."""
+    llm = LLM(folders["a"], dtype="float32", temperature=0.0, max_tokens=9, context=512)
+    first, second = tokens_for("a", 45, seed=60), tokens_for("a", 30, seed=61)
+    out1 = llm.prompt(first)
+    out2 = llm.prompt(second)
+    seq = list(first) + out1 + list(second)
+    assert len(out1) == 9 and len(out2) == 9
+    rows = plain.forward(CONFIGS["a"], weights_of("a"), seq + out2)
+    for i, tok in enumerate(out2):
+        row = rows[len(seq) + i - 1]
+        best = int(np.argmax(row))
+        assert tok == best or row[best] - row[tok] < 1e-4
+
+
+@pytest.mark.parametrize("name,dtype", [("a", "float32"), ("b", "bfloat16")])
+def test_replay_of_steps_through_the_program(folders, name, dtype, tmp_path):
+    """``bin/trace_run``: a batch of unequal prompts decoded together, requests that end early, then a second batch
+    that takes over the freed slots, pages and states; every position's logits against the plain model."""
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    lens = {"p": 97, "q": 12, "r": 70, "s": 3, "t": 131}
+    reqs = {rid: tokens_for(name, n, seed=80 + i) for i, (rid, n) in enumerate(lens.items())}
+    steps, rows = [], {rid: [] for rid in reqs}                   # rows[rid]: (step, index in the step's file) per position
+    for ids, cuts in ((("p", "q", "r"), (64, 10, 1)), (("s", "t"), (2, 129))):
+        pos = dict(zip(ids, cuts))
+        entries = [{"id": i, "tokens": reqs[i][:pos[i]], "want": list(range(pos[i]))} for i in ids]
+        live = list(ids)
+        while live:
+            step, at = len(steps), 0
+            for e in entries:
+                rows[e["id"]] += [(step, at + k) for k in e["want"]]
+                at += len(e["want"])
+            ends = [i for i in live if pos[i] >= lens[i]]
+            steps.append({"step": step, "entries": entries, "end": ends})
+            live = [i for i in live if i not in ends]
+            entries = [{"id": i, "tokens": [reqs[i][pos[i]]], "want": [0]} for i in live]
+            for i in live:
+                pos[i] += 1
+    out_dir = str(tmp_path / "out")
+    proc = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", folders[name], "--dtype",
+                           dtype, "--out", out_dir, "--max-tokens", "320"],
+                          input="".join(json.dumps(st) + "\n" for st in steps), capture_output=True, text=True, timeout=900)
+    assert proc.returncode == 0, proc.stderr[-3000:]
+    assert [l for l in proc.stdout.splitlines() if l.startswith("done")] == [f"done {st['step']}" for st in steps]
+    vocab = CONFIGS[name]["vocab"]
+    files = {}
+    for rid, r in reqs.items():
+        got = []
+        for step, k in rows[rid]:
+            if step not in files:
+                files[step] = np.fromfile(os.path.join(out_dir, f"{step}.f32"), dtype="<f4").reshape(-1, vocab)
+            got.append(files[step][k])
+        assert len(got) == lens[rid]
+        check_logits(np.stack(got), plain_logits(name, r), dtype, f"tokolorn {name} replayed request {rid}")
+
+
+# ------------------------------------------------------------------ mechanisms alone
+def _ops():
+    from math_utils_b200.csrc import ops
+    return ops
+
+
+def dev(a, dtype=torch.float32):
+    return torch.from_numpy(np.ascontiguousarray(a)).to(device="cuda", dtype=dtype)
+
+
+def ints(a):
+    return dev(np.asarray(a), torch.int32)
+
+
+def host(t):
+    return t.float().cpu().numpy().astype(np.float64)
+
+
+@pytest.mark.parametrize("n,groups", [(44, 1), (45, 1), (3000, 1), (4096, 1), (5000, 1), (45, 9), (2560, 4)])
+def test_join_with_scale_and_second_branch_kernel(n, groups):
+    """What the stream becomes and its normed row, with and without a second branch and a scale per entry."""
+    ops, rng = _ops(), np.random.default_rng(1)
+    x, y, z = (rng.normal(0, s, (5, n)) for s in (2.0, 1.0, 3.0))
+    w, g, eps = rng.normal(1, 0.2, n), rng.normal(0.3, 0.5, n), 1e-2
+    for second in (False, True):
+        for scale in (False, True):
+            stream = x + (0.7 * y + (-0.4 * z if second else 0.0)) * (g if scale else 1.0)
+            want = plain.unit_rms(stream.reshape(5, groups, -1), eps).reshape(5, n) * w
+            kw = dict(y2=dev(z) if second else None, mult2=-0.4, scale=dev(g) if scale else None)
+            for dtype, tol in ((torch.float32, 1e-5), (torch.bfloat16, 4e-2)):
+                xs, out = dev(x), torch.zeros((5, n), device="cuda", dtype=dtype)
+                ops.residual_add_norm(xs, dev(y), 0.7, dev(w), eps, out, groups=groups, **kw)
+                assert np.abs(host(xs) - stream).max() < 1e-5 and np.abs(host(out) - want).max() < tol
+            xs = dev(x)
+            ops.residual_add_norm(xs, dev(y), 0.7, None, 0.0, None, **kw)          # the addition alone
+            assert np.abs(host(xs) - stream).max() < 1e-5
+
+
+def test_norm_with_one_number():
+    from math_utils_b200.config import PartSpec
+    from math_utils_b200.engine.runtime import Runtime
+    from math_utils_b200.parts.base import build_part
+    rng = np.random.default_rng(2)
+    part = build_part("norm", PartSpec("rms_norm", {"size": 44, "eps": 0.3, "one_number": True, "scale": 1.7}, {"weight": "g"}))
+    assert [tuple(s.shape) for s in part.tensor_specs()] == [()]
+    part.bind({"g": torch.tensor(-1.3, device="cuda")}, Runtime.create("float32"))
+    x = rng.normal(0, 2, (6, 44))
+    want = 1.7 * plain.scalar_rms_norm(x, -1.3, 0.3)
+    assert np.abs(host(part.forward(dev(x))) - want).max() < 1e-5
+    assert np.abs(host(part.forward(dev(x), rows=ints([4, 0]))) - want[[4, 0]]).max() < 1e-5
+
+
+def test_scaled_token_pair_embedding_kernel():
+    ops, rng = _ops(), np.random.default_rng(3)
+    V, D, buckets, mp, mc, scale = 50, 20, 13, 1000003, 7, 5.5
+    w = {"embed": rng.normal(0, 1, (V, D)), "bigram": rng.normal(0, 1, (buckets + 1, D))}
+    cfg = {"embedding": {"scale": scale, "bigram": {"buckets": buckets, "mul_prev": mp, "mul_cur": mc}}}
+    seqs = [rng.integers(0, V, n).tolist() for n in (5, 1, 9)]
+    last = torch.full((6,), -7, dtype=torch.int32, device="cuda")
+    slots = [4, 0, 2]
+    for step in [[(0, 0, 3), (1, 0, 1), (2, 0, 4)], [(0, 3, 4), (2, 4, 6)], [(0, 4, 5), (2, 6, 7)], [(2, 7, 8)], [(2, 8, 9)]]:
+        ids = np.concatenate([seqs[s][a:b] for s, a, b in step])
+        pos = np.concatenate([np.arange(a, b) for s, a, b in step])
+        seq = np.concatenate([[i] * (b - a) for i, (s, a, b) in enumerate(step)])
+        first = np.cumsum([0] + [b - a for s, a, b in step])
+        got = ops.embed_pair(ints(ids), ints(pos), ints(seq), ints(first), ints([slots[s] for s, a, b in step]), last,
+                             dev(w["embed"]), dev(w["bigram"]), mp, mc, all(b - a == 1 for s, a, b in step), scale=scale)
+        want = np.concatenate([plain.embedding(cfg, seqs[s], w)[a:b] for s, a, b in step])
+        assert np.abs(host(got) - want).max() < 2e-6, f"step {step}"
+
+
+def test_gated_activation_kernel():
+    ops, rng = _ops(), np.random.default_rng(4)
+    for width in (24, 13):
+        a = rng.normal(0, 3, (7, 2 * width))
+        a[0, :6] = (-40.0, -6.0, -1e-3, 1e-3, 6.0, 40.0)
+        for dtype, tol in ((torch.float32, 2e-6), (torch.bfloat16, 1e-2)):
+            x = host(dev(a, dtype))
+            out = torch.zeros((7, width), device="cuda", dtype=dtype)
+            ops.gated_act(dev(a, dtype), out, "gelu_new")
+            want = plain.gelu_tanh(x[:, :width]) * x[:, width:]
+            assert (np.abs(host(out) - want) <= tol * np.maximum(1.0, np.abs(want))).all()
+
+
+# ------------------------------------------------------------------ attention
+def _paged(rng, lens, width, page=64):
+    """Rows of several sequences in pages handed out in a scrambled order."""
+    n_pages = sum(-(-n // page) for n in lens) + 3
+    order = rng.permutation(n_pages)
+    pages, table, seqs, at = np.zeros((n_pages, page, width)), np.zeros((len(lens), 24), dtype=np.int32), [], 0
+    for s, n in enumerate(lens):
+        rows = rng.normal(0, 1, (n, width))
+        seqs.append(rows)
+        for i in range(-(-n // page)):
+            table[s, i] = order[at]
+            chunk = rows[i * page:(i + 1) * page]
+            pages[order[at], :len(chunk)] = chunk
+            at += 1
+    return seqs, pages, table
+
+
+class Case:
+    """Attention of single tokens over paged rows: keys alone (``shared``: they are the values) or keys and values, a
+    window or chunks, with or without cap, sink and gate."""
+
+    def __init__(self, H, G, dim, vdim, window=0, chunk=0, shared=False, softcap=0.0, sink=False, gate=False, scale=0.37):
+        self.__dict__.update(locals())
+        self.width = G * (dim + (0 if shared else vdim))
+
+    def sees(self, i, j):
+        return plain.in_chunk(i, j, self.chunk) if self.chunk else plain.in_window(i, j, self.window or None)
+
+    def keys(self, rows, g):
+        return rows[:, g * self.dim:(g + 1) * self.dim]
+
+    def values(self, rows, g):
+        return self.keys(rows, g) if self.shared else rows[:, self.G * self.dim + g * self.vdim:][:, :self.vdim]
+
+    def token(self, q, rows, pos, gate=None):
+        """One token's heads [H, vdim], through the plain function on the one query."""
+        js = np.array([j for j in range(pos + 1) if self.sees(pos, j)])
+        out = np.zeros((self.H, self.vdim))
+        for a in range(self.H):
+            g = a // (self.H // self.G)
+            n = len(js)
+            queries = np.zeros((n, self.dim))
+            queries[-1] = q[a]
+            out[a] = plain.masked_attention(queries, self.keys(rows, g)[js], self.values(rows, g)[js], self.scale,
+                                            lambda i, j: j <= i and i == n - 1 or i == j, softcap=self.softcap or None,
+                                            sink=self.sink)[-1]
+        return out if gate is None else out * plain.sigmoid(gate.reshape(self.H, self.vdim))
+
+    def edges(self, n):
+        """(position, key pointed at): just inside and outside the window or chunk, the ends, page borders."""
+        size, picks = self.window or self.chunk or n, set()
+        for p in {n - 1, min(n - 1, size), min(n - 1, size - 1), min(n - 1, 2 * size), min(n - 1, 64), min(n - 1, 63), n // 2}:
+            lo = p - p % size if self.chunk else p - size + 1
+            picks |= {(p, j) for j in (0, lo - 1, lo, p, p // 2, 63, 64) if 0 <= j <= p}
+        return sorted(picks)
+
+    def point(self, q, rows, j):
+        """Makes every head's query point at key j so that its score stands out (also under the cap)."""
+        for a in range(self.H):
+            k = self.keys(rows, a // (self.H // self.G))[j]
+            q[a] = k * 24.0 / self.scale / (k ** 2).sum()
+
+
+KINDS = [Case(4, 2, 16, 24, window=70, softcap=30.0, gate=True), Case(3, 3, 6, 5, window=7, softcap=12.0, gate=True),
+         Case(6, 1, 64, 128, window=64, softcap=50.0, gate=True), Case(8, 1, 8, 200, window=33), Case(2, 1, 10, 12, softcap=9.0, gate=True),
+         Case(4, 2, 16, 16, chunk=70, shared=True, sink=True), Case(3, 3, 7, 7, chunk=5, shared=True, sink=True),
+         Case(8, 4, 48, 48, chunk=64, shared=True, sink=True), Case(17, 1, 24, 24, chunk=1, shared=True, sink=True),
+         Case(5, 5, 128, 128, chunk=100, shared=True, sink=True), Case(4, 1, 32, 32, shared=True),
+         Case(4, 2, 40, 40, window=100, shared=True, sink=True, softcap=20.0, gate=True)]
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("case", KINDS, ids=range(len(KINDS)))
+def test_attention_of_single_tokens(dtype, case):
+    """Both CUDA-core kernels; pages that no token of the case sees hold values that would show (not a number)."""
+    ops, rng = _ops(), np.random.default_rng(5)
+    lens = [1, 5, 64, 130, 700]
+    seqs, pages, table = _paged(rng, lens, case.width)
+    if dtype == torch.bfloat16:
+        pages = host(dev(pages, dtype))
+        seqs = [np.concatenate([pages[table[s, i]] for i in range(-(-n // 64))])[:n] for s, n in enumerate(lens)]
+    picks = [(s, p, j) for s, n in enumerate(lens) for p, j in case.edges(n)]
+    H, dim, vdim = case.H, case.dim, case.vdim
+    q = rng.normal(0, 1, (len(picks), H, dim)) / math.sqrt(dim)
+    for i, (s, p, j) in enumerate(picks):
+        case.point(q[i], seqs[s], j)
+    gate = rng.normal(0, 2, (len(picks), H * vdim))
+    if dtype == torch.bfloat16:
+        q, gate = host(dev(q, dtype)), host(dev(gate, dtype))
+    want = np.stack([case.token(q[i], seqs[s], p, gate[i] if case.gate else None) for i, (s, p, j) in enumerate(picks)])
+    tol = 3e-4 if dtype == torch.float32 else 6e-2
+    for sel in ([i for i, (s, p, j) in enumerate(picks) if s < 4], [i for i, (s, p, j) in enumerate(picks) if s == 4 and p == 699]):
+        poisoned = pages.copy()
+        if picks[sel[0]][0] == 4:                                     # only the last token of the longest: most pages are unseen
+            seen = {j // 64 for j in range(700) if case.sees(699, j)}
+            for i in range(11):
+                if i not in seen:
+                    poisoned[table[4, i]] = np.nan
+        for single in (False, True):
+            out = torch.zeros((len(sel), H * vdim), device="cuda", dtype=dtype)
+            ops.mapped_attention(dev(q[sel].reshape(len(sel), -1), dtype), dev(poisoned, dtype), ints(table), 64,
+                                 ints([picks[i][1] for i in sel]), ints([picks[i][0] for i in sel]), H, case.G, 1, dim, vdim,
+                                 case.scale, case.window, out, single_tokens=single, chunk=case.chunk, sink=case.sink,
+                                 softcap=case.softcap, shared=case.shared, gate=dev(gate[sel], dtype) if case.gate else None)
+            err = np.abs(host(out).reshape(len(sel), H, vdim) - want[sel]).max(axis=(1, 2))
+            bad = int(np.argmax(~(err < tol)))
+            assert (err < tol).all(), f"single {single}: (sequence, position, key) {picks[sel[bad]]}: {err[bad]}"
+
+
+TC_KINDS = [Case(4, 2, 16, 16, window=70, softcap=30.0, gate=True), Case(8, 2, 64, 128, window=64, softcap=50.0, gate=True),
+            Case(3, 3, 32, 48, window=7, softcap=14.0), Case(2, 1, 80, 112, softcap=40.0, gate=True),
+            Case(4, 2, 16, 16, chunk=70, shared=True, sink=True), Case(8, 4, 48, 48, chunk=64, shared=True, sink=True),
+            Case(6, 2, 128, 128, chunk=100, shared=True, sink=True), Case(4, 1, 32, 32, chunk=3, shared=True, sink=True),
+            Case(4, 2, 80, 80, window=90, shared=True, sink=True, softcap=25.0, gate=True)]
+
+
+@pytest.mark.parametrize("case", TC_KINDS, ids=range(len(TC_KINDS)))
+def test_attention_of_prompt_tiles_on_tensor_cores(case):
+    """Several sequences' tokens in one step as tiles of up to 64; some sequences bring only their last tokens."""
+    ops, rng = _ops(), np.random.default_rng(8)
+    lens, new = [130, 1, 64, 65, 7, 500], [130, 1, 64, 3, 7, 70]
+    seqs, pages, table = _paged(rng, lens, case.width)
+    pages = host(dev(pages, torch.bfloat16))
+    seqs = [np.concatenate([pages[table[s, i]] for i in range(-(-n // 64))])[:n] for s, n in enumerate(lens)]
+    tok_seq = np.repeat(np.arange(len(lens)), new)
+    tok_pos = np.concatenate([np.arange(n - k, n) for n, k in zip(lens, new)])
+    T, H, dim, vdim = len(tok_seq), case.H, case.dim, case.vdim
+    size = case.window or case.chunk or 1000
+    q = rng.normal(0, 1, (T, H, dim)) / math.sqrt(dim)
+    for t in range(T):                                                # each token points at one key around an edge, in turn
+        p = tok_pos[t]
+        lo = p - p % size if case.chunk else p - size + 1
+        j = [0, lo - 1, lo, p, p // 2, None][t % 6]                   # (and some at none: many small scores, the sink)
+        if j is not None and 0 <= j <= p:
+            case.point(q[t], seqs[tok_seq[t]], j)
+    q, gate = host(dev(q, torch.bfloat16)), host(dev(rng.normal(0, 2, (T, H * vdim)), torch.bfloat16))
+    tiles, at = [], 0
+    for k in new:
+        tiles += [(at + o, min(64, k - o)) for o in range(0, k, 64)]
+        at += k
+    want = np.stack([case.token(q[t], seqs[tok_seq[t]], tok_pos[t], gate[t] if case.gate else None) for t in range(T)])
+    for tc in (True, False):
+        out = torch.zeros((T, H * vdim), device="cuda", dtype=torch.bfloat16)
+        ops.mapped_attention(dev(q.reshape(T, -1), torch.bfloat16), dev(pages, torch.bfloat16), ints(table), 64, ints(tok_pos),
+                             ints(tok_seq), H, case.G, 1, dim, vdim, case.scale, case.window, out, tiles=ints(np.array(tiles)),
+                             tensor_cores=tc, chunk=case.chunk, sink=case.sink, softcap=case.softcap, shared=case.shared,
+                             gate=dev(gate, torch.bfloat16) if case.gate else None)
+        err = np.abs(host(out).reshape(T, H, vdim) - want).max(axis=(1, 2))
+        bad = int(np.argmax(err > 6e-2))
+        assert err.max() < 6e-2, f"tensor cores {tc}: first wrong token {bad} (sequence {tok_seq[bad]}, position {tok_pos[bad]})"
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_rows_of_keys_alone(dtype):
+    """No norm, no rotation: the queries stay as they are, and the projected keys go to the cache once."""
+    ops, rng = _ops(), np.random.default_rng(9)
+    H, G, dim = 4, 2, 24
+    proj = dev(rng.normal(0, 2, (3, (H + G) * dim)), dtype)
+    x = host(proj)
+    rows = torch.full((4, 64, G * dim), 5.0, device="cuda", dtype=dtype)
+    q, k = proj[:, :H * dim], proj[:, H * dim:]
+    ops.qk_prepare(q, k, None, None, None, torch.zeros(1, device="cuda"), 1.0, 0, 0.0, H, G, 1, dim, dim, ints([0, 63, 70]),
+                   ints([0, 0, 1]), ints([[2, 0], [0, 3]]), 64, rows, shared=True)
+    assert np.array_equal(host(proj), x)
+    assert np.array_equal(host(torch.stack([rows[2, 0], rows[2, 63], rows[3, 6]])), x[:, H * dim:])
+    assert (rows == 5.0).sum() == rows.numel() - 3 * G * dim              # nothing else is written
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("dim,vdim,dims,base", [(16, 24, 12, 5000.0), (6, 5, 6, 100.0), (64, 128, 64, 20000.0), (10, 3, 2, 7.0), (9, 5, 0, 9.0)])
+def test_rotation_of_pairs(dtype, dim, vdim, dims, base):
+    ops, rng = _ops(), np.random.default_rng(10)
+    H, G, pos = 3, 1, [0, 1, 63, 64, 900]
+    x = dev(rng.normal(0, 1, (len(pos), H * dim + G * (dim + vdim))), dtype)
+    raw = host(x)
+    rows = torch.zeros((16, 64, G * (dim + vdim)), device="cuda", dtype=dtype)
+    freqs = dev(np.array([base ** (-2.0 * i / dims) for i in range(dims // 2)] or [0.0]))
+    q, k, v = x[:, :H * dim], x[:, H * dim:(H + G) * dim], x[:, (H + G) * dim:]
+    ops.qk_prepare(q, k, v, None, None, freqs, 1.0, dims, 0.0, H, G, 1, dim, vdim, ints(pos), ints([0] * len(pos)),
+                   ints([list(range(16))]), 64, rows, pairs=True)
+
+    def turned(cols):                                    # the plain rotation, taken at each token's position
+        y = np.zeros((901, 1, dim))
+        y[pos, 0] = cols
+        return plain.rotate_pairs(y, base, dims)[pos, 0]
+
+    tol = 1e-4 if dtype == torch.float32 else 3e-2
+    for h in range(H):
+        assert np.abs(host(q)[:, h * dim:(h + 1) * dim] - turned(raw[:, h * dim:(h + 1) * dim])).max() < tol
+    got = host(torch.stack([rows[p // 64, p % 64] for p in pos]))
+    assert np.abs(got[:, :dim] - turned(raw[:, H * dim:(H + 1) * dim])).max() < tol
+    assert np.array_equal(got[:, dim:], raw[:, (H + G) * dim:])
+
+
+# ------------------------------------------------------------------ recurrences
+# Cuts of two sequences into shared steps: portions of 1, 2 and many, one sequence ending before the other.
+CUTS = [[(0, 2), (2, 3), (3, 20), (20, 21), (21, 22), (22, 300)], [(0, 1), (1, 3), (3, 20), (20, 21), (21, 21), (21, 21)]]
+LONG = [[(0, 64), (64, 66), (66, 193), (193, 194), (194, 300)], [(0, 100), (100, 101), (101, 170), (170, 170), (170, 171)]]
+
+
+def _in_steps(us, slots, run, cuts=CUTS):
+    """Runs two sequences' rows through ``run(rows, seq, first, slots, single)`` in the steps of ``cuts``; each one's rows."""
+    got = [[], []]
+    for step in range(len(cuts[0])):
+        live = [s for s in range(2) if cuts[s][step][1] > cuts[s][step][0]]
+        u = torch.cat([us[s][cuts[s][step][0]:cuts[s][step][1]] for s in live])
+        counts = [cuts[s][step][1] - cuts[s][step][0] for s in live]
+        out = run(u, ints(np.repeat(np.arange(len(live)), counts)), ints(np.cumsum([0] + counts)), ints([slots[s] for s in live]),
+                  counts)
+        at = 0
+        for s, c in zip(live, counts):
+            got[s].append(host(out[at:at + c]))
+            at += c
+    return [np.concatenate(g) for g in got]
+
+
+def _check_steps(got, want, tol):
+    for s in range(2):
+        err = np.abs(got[s] - want[s]).max(axis=1)
+        bound = tol * max(1.0, np.abs(want[s]).max())
+        assert err.max() < bound, f"sequence {s}: first wrong token {int(np.argmax(err > bound))} of {len(err)}, {err.max():.2e}"
+
+
+@pytest.mark.parametrize("H,dk,dv,decay", [(2, 16, 24, (0.9, 0.999)), (3, 7, 5, (0.1, 1.0, 0.97)), (1, 33, 9, (0.5,)),
+                                           (2, 128, 64, (0.99, 0.6)), (2, 200, 16, (0.95, 0.3)), (1, 1, 2, (0.8,)), (4, 1, 3, (0.9,) * 4)])
+def test_lightning_attention_token_by_token(H, dk, dv, decay):
+    """Activations, recurrence and gated norm against the plain mixer with identity matrices around them: a prompt cut into
+    steps of several sizes for two sequences that share the steps (also steps of as many tokens as there are heads)."""
+    ops, rng = _ops(), np.random.default_rng(11)
+    qk, inner, eps = H * dk, H * dv, 1e-3
+    wide = 2 * qk + 2 * inner
+    wide += -wide % 4
+    eye = np.eye(wide)
+    at = np.cumsum([0, qk, qk, inner, inner])
+    m = {"heads": H, "dim": dk, "vdim": dv, "decay": list(decay)}
+    w = {n: eye[a:b] for n, a, b in zip(("q", "k", "v", "g"), at, at[1:])}
+    w.update({"o": np.eye(inner), "norm": rng.normal(1, 0.2, inner)})
+    us = [dev(rng.normal(0, 1.5, (n, wide))) for n in (300, 21)]
+    want = [plain.lightning_mixer(host(u), m, w, "", eps) for u in us]
+    state = torch.full((5, inner * dk), 9.0, device="cuda")
+    slots = [3, 1]
+    state[slots] = 0.0                                                   # what taking a slot does
+    gates, norm = dev([[[d, 1.0, 0.0, 0.0] for d in decay]]), dev(w["norm"])
+
+    def run(u, seq, first, sl, counts):
+        col = lambda n: u[:, at[n]:at[n + 1]]
+        o, out = torch.zeros((u.shape[0], inner), device="cuda"), torch.zeros((u.shape[0], inner), device="cuda")
+        ops.linear_scan(col(0), col(1), col(2), gates, H, dk, dv, 1.0, first, sl, state, 0, o, silu_rows=True)
+        return ops.gated_group_norm(o, col(3), norm, 1, eps, out, gate_after=True, sigmoid=True)
+
+    _check_steps(_in_steps(us, slots, run), want, 1e-4)
+    assert (state[[0, 2, 4]] == 9.0).all()                              # other slots' state is left alone
+
+
+def _tiles(counts):
+    tiles, at = [], 0
+    for k in counts:
+        tiles += [(at + o, min(64, k - o)) for o in range(0, k, 64)]
+        at += k
+    return ints(np.array(sorted(tiles, key=lambda t: -t[1])))           # in any order
+
+
+@pytest.mark.parametrize("H,dk,dv,decay", [(2, 16, 24, (0.9, 0.999)), (1, 8, 8, (1.0,)), (3, 40, 72, (0.1, 0.97, 0.99)), (2, 128, 128, (0.99, 0.6)),
+                                           (1, 256, 136, (0.95,)), (4, 64, 64, (0.5, 0.75, 0.9, 0.9999))])
+def test_lightning_attention_in_chunks(H, dk, dv, decay):
+    """The tensor-core form against the recurrence on the same rounded rows, steps of 1 to 127 tokens; the two forms take
+    over each other's states."""
+    ops, rng = _ops(), np.random.default_rng(12)
+    qk, inner = H * dk, H * dv
+    us = [dev(rng.normal(0, 1.5, (n, 2 * qk + inner)), torch.bfloat16) for n in (300, 171)]
+    want = []
+    for u in us:
+        r = plain.to_bf16(plain.silu(host(u)))
+        q, k, v = r[:, :qk].reshape(-1, H, dk), r[:, qk:2 * qk].reshape(-1, H, dk), r[:, 2 * qk:].reshape(-1, H, dv)
+        want.append(np.stack([plain.fading_recurrence(q[:, a], k[:, a], v[:, a], decay[a]) for a in range(H)], axis=1).reshape(-1, inner))
+    powers = dev(np.array(decay)[:, None] ** np.arange(65))
+    gates = dev([[[d, 1.0, 0.0, 0.0] for d in decay]])
+    for mixed in (False, True):
+        state = torch.full((5, inner * dk), 9.0, device="cuda")
+        slots = [3, 1]
+        state[slots] = 0.0
+
+        def run(u, seq, first, sl, counts):
+            o = torch.full((u.shape[0], inner), 7.0, device="cuda")
+            if mixed and max(counts) <= 2:
+                r = plain.to_bf16(plain.silu(host(u)))                  # the same rows, rounded as the other form rounds them
+                f = dev(r)
+                return ops.linear_scan(f[:, :qk], f[:, qk:2 * qk], f[:, 2 * qk:], gates, H, dk, dv, 1.0, first, sl, state, 0, o)
+            return ops.lightning_prompt(u[:, :qk], u[:, qk:2 * qk], u[:, 2 * qk:], powers, H, dk, dv, _tiles(counts), seq, first, sl,
+                                        state, 0, o)
+
+        # (a rounding that falls the other way now and then moves one term by 2^-9)
+        _check_steps(_in_steps(us, slots, run, LONG), want, 1e-3)
+        assert (state[[0, 2, 4]] == 9.0).all()
+
+
+def test_lightning_attention_keeps_a_value_over_hundreds_of_tokens():
+    """One key written early and asked for hundreds of tokens later, across steps and chunks; a head that fades at once has
+    forgotten it."""
+    ops = _ops()
+    H, dk, dv, T = 2, 16, 8, 700
+    u = np.full((T, H * (2 * dk + dv)), -200.0)                         # silu of that is nothing
+    q, k, v = u[:, :H * dk], u[:, H * dk:2 * H * dk], u[:, 2 * H * dk:]
+    for a in range(H):
+        k[np.arange(T), a * dk + np.arange(T) % 15] = 4.0
+        v[:, a * dv:(a + 1) * dv] = 1.0
+        k[5, a * dk:(a + 1) * dk] = -200.0
+        k[5, a * dk + 15], q[T - 1, a * dk + 15] = 4.0, 4.0             # (the one key of its kind)
+        v[5, a * dv:(a + 1) * dv] = np.arange(2.0, 2.0 + dv)
+    s4 = plain.silu(4.0)
+    want = plain.silu(np.arange(2.0, 2.0 + dv)) * s4 * s4 * 0.999 ** (T - 6)
+    decay = (0.999, 0.5)
+    powers, gates = dev(np.array(decay)[:, None] ** np.arange(65)), dev([[[d, 1.0, 0.0, 0.0] for d in decay]])
+    for form in ("chunks", "tokens"):
+        for cuts in ([0, T], [0, 300, 301, T - 1, T]):
+            state = torch.zeros((1, H * dk * dv), device="cuda")
+            for a, b in zip(cuts, cuts[1:]):
+                o = torch.zeros((b - a, H * dv), device="cuda")
+                x = dev(u[a:b], torch.bfloat16 if form == "chunks" else torch.float32)
+                parts = (x[:, :H * dk], x[:, H * dk:2 * H * dk], x[:, 2 * H * dk:])
+                where = (ints([0, b - a]), ints([0]), state, 0, o)
+                if form == "chunks":
+                    ops.lightning_prompt(*parts, powers, H, dk, dv, _tiles([b - a]), ints([0] * (b - a)), *where)
+                else:
+                    ops.linear_scan(*parts, gates, H, dk, dv, 1.0, *where, silu_rows=True)
+            got = host(o)[-1].reshape(H, dv)
+            assert np.abs(got[0] / want - 1.0).max() < (1e-2 if form == "chunks" else 1e-4), form
+            assert np.abs(got[1]).max() < 1e-20, form
+
+
+@pytest.mark.parametrize("channels,taps", [(16, 4), (24, 3), (8, 2), (40, 1), (10, 4), (64, 6), (1032, 4)])
+@pytest.mark.parametrize("u_dtype,out_dtype", [(torch.float32, torch.float32), (torch.bfloat16, torch.float32), (torch.bfloat16, torch.bfloat16)])
+def test_short_convolution_kernel(channels, taps, u_dtype, out_dtype):
+    """Steps of many tokens whose sequences begin inside a tile of eight, and single tokens; inputs are a view."""
+    ops, rng = _ops(), np.random.default_rng(13)
+    lens = (200, 3, 1, 90, 11)
+    w, b = rng.normal(0, 0.6, (channels, taps)), rng.normal(0, 0.3, channels)
+    us = [dev(rng.normal(0, 1.5, (n, channels + 8)), u_dtype) for n in lens]
+    want = [plain.silu(plain.short_convolution(host(u)[:, 8:], w, b)) for u in us]
+    state = torch.full((7, (taps - 1) * channels + 4), 9.0, device="cuda")
+    slots = [3, 1, 6, 0, 4]
+    state[slots] = 0.0
+    got, pos = [[] for _ in lens], [0] * len(lens)
+    for counts in ((77, 1, 1, 2, 9), (2, 2, 0, 83, 0), (1, 0, 0, 1, 1), (120, 0, 0, 4, 1)):
+        live = [s for s, c in enumerate(counts) if c]
+        u = torch.cat([us[s][pos[s]:pos[s] + counts[s]] for s in live])
+        n = [counts[s] for s in live]
+        out = torch.full((u.shape[0], channels), 7.0, device="cuda", dtype=out_dtype)
+        ops.ssd_conv(u[:, 8:], dev(w), dev(b), ints(np.repeat(np.arange(len(live)), n)), ints(np.cumsum([0] + n)),
+                     ints([slots[s] for s in live]), state, all(c == 1 for c in n), out)
+        at = 0
+        for s, c in zip(live, n):
+            got[s].append(host(out[at:at + c]))
+            pos[s] += c
+            at += c
+    assert pos == list(lens)
+    tol = 1e-5 if out_dtype == torch.float32 else 3e-2
+    for s in range(len(lens)):
+        err = np.abs(np.concatenate(got[s]) - want[s]).max(axis=1)
+        assert err.max() < tol, f"sequence {s}: first wrong token {int(np.argmax(err > tol))}"
+    assert (state[[2, 5]] == 9.0).all() and (state[:, (taps - 1) * channels:][slots] == 0.0).all()
+
+
+@pytest.mark.parametrize("dtype,T", [(torch.float32, 3), (torch.float32, 70), (torch.bfloat16, 3), (torch.bfloat16, 200)])
+def test_step_sizes(dtype, T):
+    """softplus of a low-rank projection and a bias, from far below zero (where its relative accuracy counts) to far above."""
+    ops, rng = _ops(), np.random.default_rng(14)
+    n, rank = 130, 16
+    low, w, bias = rng.normal(0, 1, (T, rank + 8)), host(dev(rng.normal(0, 0.2, (n, rank)), dtype)), np.linspace(-30.0, 30.0, n)
+    out = torch.zeros((T, n), device="cuda")
+    keep = dev(w, dtype), dev(bias), dev(low)
+    ops.low_rank(keep[2], dtype, ops.low_rank_part(keep[0], 8, out, bias=keep[1], fn="softplus"))
+    want = plain.softplus(low[:, 8:] @ w.T + bias)
+    assert np.abs(host(out) / want - 1.0).max() < 5e-5 if dtype == torch.bfloat16 else 1e-5
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("c,N", [(24, 16), (5, 1), (130, 3), (40, 8), (33, 17), (70, 24), (9, 40), (16, 64), (6, 100), (12, 128), (7, 200), (4, 256)])
+def test_selective_scan_kernel(dtype, c, N):
+    """Two sequences in shared steps of 1 to 278 tokens; channels that forget at once and channels that keep all."""
+    ops, rng = _ops(), np.random.default_rng(15)
+    n4 = -(-N // 4) * 4
+    A_log = rng.uniform(-4.0, 3.0, (c, N))
+    D = rng.normal(0.5, 0.5, c)
+    data, want = [], []
+    for n in (300, 21):
+        x, z = (host(dev(rng.normal(0, 1.5, (n, c)), dtype)) for _ in range(2))
+        dt, bc = plain.softplus(rng.uniform(-6.0, 1.0, (n, c))), rng.normal(0, 1, (n, 4 + 2 * n4))
+        bc[:, 4 + N:4 + n4] = bc[:, 4 + n4 + N:] = 0.0                   # the filling
+        data.append(dev(np.concatenate([x, z, dt, bc], axis=1)))
+        y = plain.selective_scan(x, dt, -np.exp(A_log), bc[:, 4:4 + N], bc[:, 4 + n4:4 + n4 + N], D)
+        want.append(y * plain.silu(z))
+    tail = 5 if c == 5 else 8
+    state = torch.full((5, tail + c * N), 9.0, device="cuda")
+    slots = [3, 1]
+    state[slots] = 0.0
+    rates, skip = dev(-np.exp(A_log) / math.log(2.0)), dev(D)
+
+    def run(u, seq, first, sl, counts):
+        x, z, dt, bc = (u[:, a:b] for a, b in ((0, c), (c, 2 * c), (2 * c, 3 * c), (3 * c, u.shape[1])))
+        out = torch.full((u.shape[0], c), 7.0, device="cuda", dtype=dtype)
+        return ops.selective_scan(x.to(dtype), z.to(dtype), dt, bc.contiguous(), 4, 4 + n4, rates, skip, first, sl, state, tail, out)
+
+    _check_steps(_in_steps(data, slots, run), want, 1e-4 if dtype == torch.float32 else 1e-2)
+    assert (state[[0, 2, 4]] == 9.0).all() and (state[slots][:, :tail] == 0.0).all()
+
+
+def test_selective_scan_keeps_a_value_over_hundreds_of_tokens():
+    """What one token wrote into an entry that hardly fades comes back 600 tokens later, across steps; an entry that fades
+    at once has lost it."""
+    ops = _ops()
+    T, c = 640, 3
+    x, dt, B, C = np.zeros((T, c)), np.full((T, c), 0.1), np.zeros((T, 4)), np.zeros((T, 4))
+    x[7] = (1.0, -2.0, 3.0)
+    B[7], C[T - 1] = (1.0, 1.0, 0.0, 0.0), (1.0, 1.0, 1.0, 1.0)
+    A = np.tile([-1e-3, -50.0, -1.0, -1.0], (c, 1))
+    state, z = torch.zeros((1, 4 * c), device="cuda"), np.full((T, c), 30.0)                  # silu(30) = 30
+    for a, b in ((0, 7), (7, 8), (8, 300), (300, T - 1), (T - 1, T)):
+        out = torch.zeros((b - a, c), device="cuda")
+        ops.selective_scan(dev(x[a:b]), dev(z[a:b]), dev(dt[a:b]), dev(np.concatenate([B, C], axis=1)[a:b]), 0, 4,
+                           dev(A / math.log(2.0)), dev(np.zeros(c)), ints([0, b - a]), ints([0]), state, 0, out)
+    want = 30.0 * 0.1 * x[7] * math.exp(-1e-3 * 0.1 * (T - 8))
+    assert np.abs(host(out)[-1] / want - 1.0).max() < 1e-4
+
+
+def test_mixers_refuse_what_their_kernels_do_not_take():
+    """More state entries than the scan's, keys larger than the recurrence's: a clear error at load."""
+    from math_utils_b200.config import ConfigError, PartSpec
+    from math_utils_b200.engine.runtime import Runtime
+    from math_utils_b200.parts.base import build_part
+    rt = Runtime.create("float32")
+    for kind, params in (("selective_scan", {"hidden_size": 8, "inner": 8, "state": 300, "dt_rank": 1, "conv": 2}),
+                         ("lightning_attention", {"hidden_size": 8, "n_heads": 1, "dim": 300, "vdim": 8, "decay": [0.9], "eps": 0.0})):
+        names = {r: r for r in ("in", "conv", "conv_bias", "x", "dt", "dt_bias", "A_log", "D", "out", "q", "k", "v", "gate", "norm")}
+        part = build_part("mixer", PartSpec(kind, params, names))
+        tensors = {s.name: torch.zeros(s.shape, device="cuda") for s in part.tensor_specs()}
+        with pytest.raises(ConfigError, match="300"):
+            part.bind(tensors, rt)
