@@ -20,24 +20,26 @@
 
 namespace mu {
 
-constexpr int LP_TOK = 64, LP_COLS = 64, LP_PAD = 8, LP_THREADS = 128;
+constexpr int LP_TOK = 64, LP_COLS = 64, LP_PAD = 8, LP_SUM_THREADS = 128, LP_OUT_THREADS = 256;
 
 __device__ __forceinline__ float lp_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 
 // Rows flat0 .. flat0 + count - 1 (zeros up to 64), `width` entries each (zeros up to `padded`), silu applied, into
 // `hi` [64][pitch]; with `power`, row r is multiplied by power[count - 1 - r] and goes to `hi` and `lo` in two terms.
+template <int THREADS>
 __device__ __forceinline__ void lp_stage(__nv_bfloat16* hi, __nv_bfloat16* lo, int pitch, const __nv_bfloat16* src,
                                          long long ld, long long flat0, int count, int width, int padded, const float* power) {
+    constexpr int STEP = THREADS / 16, N = LP_TOK / STEP;    // sixteen threads a row
     const int row0 = threadIdx.x >> 4, piece0 = threadIdx.x & 15;
     for (int c = 8 * piece0; c < padded; c += 128) {
-        uint4 raw[8];
+        uint4 raw[N];
         const int from = min(c, width - 8);
 #pragma unroll
-        for (int i = 0; i < 8; ++i)
-            raw[i] = *reinterpret_cast<const uint4*>(src + (flat0 + min(row0 + 8 * i, count - 1)) * ld + from);
+        for (int i = 0; i < N; ++i)
+            raw[i] = *reinterpret_cast<const uint4*>(src + (flat0 + min(row0 + STEP * i, count - 1)) * ld + from);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int r = row0 + 8 * i;
+        for (int i = 0; i < N; ++i) {
+            const int r = row0 + STEP * i;
             const bool in = r < count && c < width;
             const float f = power && r < count ? power[count - 1 - r] : 1.0f;
             const __nv_bfloat162* z = reinterpret_cast<const __nv_bfloat162*>(&raw[i]);
@@ -57,7 +59,7 @@ __device__ __forceinline__ void lp_stage(__nv_bfloat16* hi, __nv_bfloat16* lo, i
 
 __device__ __forceinline__ long long lp_place(int flat0, int s, int first) { return first / LP_TOK + s + (flat0 - first) / LP_TOK; }
 
-__global__ void __launch_bounds__(LP_THREADS)
+__global__ void __launch_bounds__(LP_SUM_THREADS)
 lightning_sums_kernel(const __nv_bfloat16* __restrict__ k, const __nv_bfloat16* __restrict__ v, long long ld,
                       const int* __restrict__ tiles, const int* __restrict__ tok_seq, const int* __restrict__ seq_first,
                       const float* __restrict__ powers, int n_heads, int dk, int dkp, int dv, float* __restrict__ sums) {
@@ -72,8 +74,8 @@ lightning_sums_kernel(const __nv_bfloat16* __restrict__ k, const __nv_bfloat16* 
     const int h = blockIdx.y, col0 = blockIdx.z * LP_COLS, cols = min(LP_COLS, dv - col0);
     const int s = tok_seq[flat0];
     float* dst = sums + (lp_place(flat0, s, seq_first[s]) * n_heads + h) * (long long)dv * dk;
-    lp_stage(kh, kl, pitch, k + (long long)h * dk, ld, flat0, count, dk, dkp, powers + h * (LP_TOK + 1));
-    lp_stage(vs, nullptr, vp, v + (long long)h * dv + col0, ld, flat0, count, cols, LP_COLS, nullptr);
+    lp_stage<LP_SUM_THREADS>(kh, kl, pitch, k + (long long)h * dk, ld, flat0, count, dk, dkp, powers + h * (LP_TOK + 1));
+    lp_stage<LP_SUM_THREADS>(vs, nullptr, vp, v + (long long)h * dv + col0, ld, flat0, count, cols, LP_COLS, nullptr);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     // this warp's 16 value columns, as rows of the product: V^T [16 x 64 tokens]
@@ -142,7 +144,7 @@ lightning_states_kernel(float* __restrict__ sums, const int* __restrict__ seq_fi
     *kept = S;
 }
 
-__global__ void __launch_bounds__(LP_THREADS)
+__global__ void __launch_bounds__(LP_OUT_THREADS, 2)
 lightning_outputs_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k,
                          const __nv_bfloat16* __restrict__ v, long long ld, const int* __restrict__ tiles,
                          const int* __restrict__ tok_seq, const int* __restrict__ seq_first, const float* __restrict__ powers,
@@ -163,23 +165,24 @@ lightning_outputs_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     const int s = tok_seq[flat0];
     const float* S = sums + (lp_place(flat0, s, seq_first[s]) * n_heads + h) * (long long)dv * dk + (long long)col0 * dk;
     if (threadIdx.x <= LP_TOK) power[threadIdx.x] = powers[h * (LP_TOK + 1) + threadIdx.x];
-    lp_stage(qs, nullptr, pitch, q + (long long)h * dk, ld, flat0, count, dk, dkp, nullptr);
-    lp_stage(ks, nullptr, pitch, k + (long long)h * dk, ld, flat0, count, dk, dkp, nullptr);
-    lp_stage(vs, nullptr, vp, v + (long long)h * dv + col0, ld, flat0, count, cols, LP_COLS, nullptr);
+    lp_stage<LP_OUT_THREADS>(qs, nullptr, pitch, q + (long long)h * dk, ld, flat0, count, dk, dkp, nullptr);
+    lp_stage<LP_OUT_THREADS>(ks, nullptr, pitch, k + (long long)h * dk, ld, flat0, count, dk, dkp, nullptr);
+    lp_stage<LP_OUT_THREADS>(vs, nullptr, vp, v + (long long)h * dv + col0, ld, flat0, count, cols, LP_COLS, nullptr);
     {
+        constexpr int STEP = LP_OUT_THREADS / 16, N = LP_COLS / STEP;
         const int row0 = threadIdx.x >> 4, piece0 = threadIdx.x & 15;
         for (int c = 8 * piece0; c < dkp; c += 128) {
-            float4 raw[8][2];
+            float4 raw[N][2];
             const int from = min(c, dk - 8);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                const float* src = S + (long long)min(row0 + 8 * i, cols - 1) * dk + from;
+            for (int i = 0; i < N; ++i) {
+                const float* src = S + (long long)min(row0 + STEP * i, cols - 1) * dk + from;
                 raw[i][0] = *reinterpret_cast<const float4*>(src);
                 raw[i][1] = *reinterpret_cast<const float4*>(src + 4);
             }
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                const int r = row0 + 8 * i;
+            for (int i = 0; i < N; ++i) {
+                const int r = row0 + STEP * i;
                 const float f = r < cols && c < dk ? 1.0f : 0.0f;
                 uint32_t hw[4], lw[4];
 #pragma unroll
@@ -193,20 +196,23 @@ lightning_outputs_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         }
     }
     __syncthreads();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
-    if (warp * 16 >= count) return;
+    // a warp 16 tokens and 32 of the columns
+    constexpr int WCOLS = LP_COLS / 2;
+    const int warp = (threadIdx.x >> 5) & 3, half0 = (threadIdx.x >> 7) * WCOLS;
+    const int lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+    if (warp * 16 >= count || half0 >= cols) return;
     const int t0 = warp * 16 + gid;                          // this thread's two tokens: t0 and t0 + 8
-    float o[LP_COLS / 8][4] = {}, w[LP_TOK / 8][4] = {};
+    float o[WCOLS / 8][4] = {}, w[LP_TOK / 8][4] = {};
     const int steps = warp + 1;                              // runs of 16 keys that this warp's tokens see
     for (int kk = 0; kk < dkp / 16; ++kk) {
         uint32_t a[4];
         ldsm_x4(a, qs + (warp * 16 + (lane & 15)) * pitch + kk * 16 + (lane >> 4) * 8);
         const int at = ((lane & 7) + (lane >> 4) * 8) * pitch + kk * 16 + ((lane >> 3) & 1) * 8;
 #pragma unroll
-        for (int j = 0; j < LP_COLS / 16; ++j) {
+        for (int j = 0; j < WCOLS / 16; ++j) {
             uint32_t bh[4], bl[4];
-            ldsm_x4(bh, sh + j * 16 * pitch + at);
-            ldsm_x4(bl, sl + j * 16 * pitch + at);
+            ldsm_x4(bh, sh + (half0 + j * 16) * pitch + at);
+            ldsm_x4(bl, sl + (half0 + j * 16) * pitch + at);
             mma_bf16(o[2 * j], a, bh[0], bh[1]);
             mma_bf16(o[2 * j + 1], a, bh[2], bh[3]);
             mma_bf16(o[2 * j], a, bl[0], bl[1]);
@@ -223,7 +229,7 @@ lightning_outputs_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     }
     const float f0 = power[t0 + 1], f1 = power[min(t0 + 9, LP_TOK)];
 #pragma unroll
-    for (int j = 0; j < LP_COLS / 8; ++j) {
+    for (int j = 0; j < WCOLS / 8; ++j) {
         o[j][0] *= f0, o[j][1] *= f0;
         o[j][2] *= f1, o[j][3] *= f1;
     }
@@ -241,9 +247,9 @@ lightning_outputs_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                 split_bf16(p0, p1, ph[2 * half + r], pl[2 * half + r]);
             }
 #pragma unroll
-        for (int j = 0; j < LP_COLS / 16; ++j) {
+        for (int j = 0; j < WCOLS / 16; ++j) {
             uint32_t b[4];
-            ldsm_x4_trans(b, vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vp + j * 16 + (lane >> 4) * 8);
+            ldsm_x4_trans(b, vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vp + half0 + j * 16 + (lane >> 4) * 8);
             mma_bf16(o[2 * j], ph, b[0], b[1]);
             mma_bf16(o[2 * j + 1], ph, b[2], b[3]);
             mma_bf16(o[2 * j], pl, b[0], b[1]);
@@ -251,8 +257,8 @@ lightning_outputs_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         }
     }
 #pragma unroll
-    for (int j = 0; j < LP_COLS / 8; ++j) {
-        const int col = 8 * j + 2 * tig;
+    for (int j = 0; j < WCOLS / 8; ++j) {
+        const int col = half0 + 8 * j + 2 * tig;
         if (col >= cols) continue;
 #pragma unroll
         for (int r = 0; r < 2; ++r)
@@ -289,7 +295,7 @@ MU_EXPORT int mu_lightning_prompt(const void* q, const void* k, const void* v, l
     typedef __nv_bfloat16 bf;
     cudaStream_t s = (cudaStream_t)stream;
     const int dkp = (dk + 15) / 16 * 16, pitch = dkp + mu::LP_PAD, vp = mu::LP_COLS + mu::LP_PAD;
-    const dim3 grid(n_tiles, n_heads, (dv + mu::LP_COLS - 1) / mu::LP_COLS), block(mu::LP_THREADS);
+    const dim3 grid(n_tiles, n_heads, (dv + mu::LP_COLS - 1) / mu::LP_COLS);
     const size_t smem1 = ((size_t)2 * mu::LP_TOK * pitch + mu::LP_TOK * vp) * sizeof(bf);
     const size_t smem3 = ((size_t)(2 * mu::LP_TOK + 2 * mu::LP_COLS) * pitch + mu::LP_TOK * vp) * sizeof(bf);
     if (!mu::allow_shared((const void*)mu::lightning_sums_kernel, 100 * 1024) ||
@@ -297,13 +303,13 @@ MU_EXPORT int mu_lightning_prompt(const void* q, const void* k, const void* v, l
         return MU_ERR_LAUNCH;
     mu::prefer_shared_memory((const void*)mu::lightning_sums_kernel);
     mu::prefer_shared_memory((const void*)mu::lightning_outputs_kernel);
-    int code = mu::launch_pdl(mu::lightning_sums_kernel, grid, block, smem1, s, 1, (const bf*)k, (const bf*)v, ld, tiles, tok_seq,
+    int code = mu::launch_pdl(mu::lightning_sums_kernel, grid, dim3(mu::LP_SUM_THREADS), smem1, s, 1, (const bf*)k, (const bf*)v, ld, tiles, tok_seq,
                               seq_first, powers, n_heads, dk, dkp, dv, scratch);
     if (code != MU_OK) return code;
     const int entries = dk * dv;
     code = mu::launch_pdl(mu::lightning_states_kernel, dim3((entries / 4 + 127) / 128, n_heads, n_seqs), dim3(128), 0, s, 1, scratch,
                           seq_first, seq_slots, powers, n_heads, entries, state, state_stride, state_offset);
     if (code != MU_OK) return code;
-    return mu::launch_pdl(mu::lightning_outputs_kernel, grid, block, smem3, s, 1, (const bf*)q, (const bf*)k, (const bf*)v, ld, tiles,
-                          tok_seq, seq_first, powers, n_heads, dk, dkp, dv, (const float*)scratch, out, ldo);
+    return mu::launch_pdl(mu::lightning_outputs_kernel, grid, dim3(mu::LP_OUT_THREADS), smem3, s, 1, (const bf*)q, (const bf*)k,
+                          (const bf*)v, ld, tiles, tok_seq, seq_first, powers, n_heads, dk, dkp, dv, (const float*)scratch, out, ldo);
 }

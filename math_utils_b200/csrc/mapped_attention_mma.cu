@@ -4,7 +4,7 @@
 // stages; per map S = Q K^T is mma.sync.m16n8k16 with float32 accumulators, the softmax runs in float32 on the
 // accumulators (running maximum and sum per row), and P V follows with the SAME values for both maps.  The weights
 // P enter that product as two bfloat16 terms (the rounded weight and what the rounding left), so they act with
-// some 16 bits of mantissa instead of 8.  At the end a1 - lambda a2, the head's unit rms and the output scale, and
+// some 16 bits of mantissa instead of 8 (for which the fast exponential is exact enough).  At the end a1 - lambda a2, the head's unit rms and the output scale, and
 // the options of mapped_attention.cu (a multiplier per head on the scores, a sink in the denominator, a gate per head,
 // chunks of positions instead of a window, a distance bias per head, kept first positions beside a window, a soft cap on
 // the scores, a gate per value entry, rows of keys that are the values too: then one staged page serves both products).
@@ -70,8 +70,8 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
     // the value columns past vdim stay zero; the queries of the tile (rows past count are zeros)
     for (int i = tid; i < 2 * MM_TILE * vp; i += blockDim.x) vs[i] = __float2bfloat16_rn(0.0f);
     const int qchunks = kw / 8;
-    for (int i = tid; i < MM_TILE * qchunks; i += blockDim.x) {
-        const int r = i / qchunks, c = (i % qchunks) * 8;
+    for (int r = warp; r < MM_TILE; r += 4)
+      for (int c = lane * 8; c < kw; c += 32 * 8) {
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
         if (r < count) v = *reinterpret_cast<const uint4*>(q + (long long)(flat0 + r) * ldq + (long long)h * kw + c);
         *reinterpret_cast<uint4*>(qs + r * kp + c) = v;
@@ -83,8 +83,8 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
         const __nv_bfloat16* src = rows + (long long)pages[page_index] * MM_TILE * width;
         __nv_bfloat16* kd = ks + stage * MM_TILE * kp;
         __nv_bfloat16* vd = vs + stage * MM_TILE * vp;
-        for (int i = tid; i < MM_TILE * (qchunks + vchunks); i += blockDim.x) {
-            const int r = i / (qchunks + vchunks), c = i % (qchunks + vchunks);
+        for (int r = warp; r < MM_TILE; r += 4)              // a warp a row, a lane a piece
+          for (int c = lane; c < qchunks + vchunks; c += 32) {
             if (c < qchunks) cp_async16(kd + r * kp + c * 8, src + r * width + key_off + c * 8);
             else cp_async16(vd + r * vp + (c - qchunks) * 8, src + r * width + val_off + (c - qchunks) * 8);
         }
@@ -103,6 +103,12 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
     const int row0 = warp * 16 + gid;                        // this thread's two rows of the tile: row0 and row0 + 8
     const int qpos[2] = {pos0 + row0, pos0 + row0 + 8};
     const bool real[2] = {row0 < count, row0 + 8 < count};
+    int lo[2], hi[2];                                        // the positions each row sees: lo .. hi, and those before `keep`
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        hi[r] = real[r] ? qpos[r] : -1;
+        lo[r] = chunk > 0 ? qpos[r] - qpos[r] % chunk : window > 0 ? qpos[r] - window + 1 : 0;
+    }
 
     load_page(page_at(0), 0);
     for (int turn = 0; turn < n_pages; ++turn) {
@@ -128,6 +134,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
                 float s[8][4];
 #pragma unroll
                 for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
+#pragma unroll 4
                 for (int kk = 0; kk < dim / 16; ++kk) {
                     uint32_t af[4];
                     ldsm_x4(af, qs + (warp * 16 + (lane & 15)) * kp + a * dim + kk * 16 + (lane >> 4) * 8);
@@ -146,9 +153,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const int r = e >> 1, kj = key0 + j * 8 + tig * 2 + (e & 1);
-                        const bool seen = real[r] && kj <= qpos[r] &&
-                                          (chunk > 0 ? kj >= qpos[r] - qpos[r] % chunk
-                                                     : window == 0 || qpos[r] - kj < window || kj < keep);
+                        const bool seen = kj <= hi[r] && (kj >= lo[r] || kj < keep);
                         float sc = s[j][e] * scale;
                         if (softcap > 0.0f) sc = softcap_fast(sc, softcap, inv_cap);
                         s[j][e] = seen ? sc - slope * (float)(qpos[r] - kj) : -INFINITY;
@@ -160,7 +165,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
                     top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 1));
                     top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 2));
                     const float m_new = fmaxf(m_run[a][r], top[r]);
-                    corr[r] = m_new == -INFINITY ? 1.0f : expf(m_run[a][r] - m_new);
+                    corr[r] = m_new == -INFINITY ? 1.0f : __expf(m_run[a][r] - m_new);
                     m_run[a][r] = m_new;
                     l_run[a][r] *= corr[r];
                 }
@@ -176,7 +181,7 @@ mapped_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long ldq, 
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const int r = e >> 1;
-                        p[e] = s[j][e] == -INFINITY ? 0.0f : expf(s[j][e] - m_run[a][r]);
+                        p[e] = s[j][e] == -INFINITY ? 0.0f : __expf(s[j][e] - m_run[a][r]);
                         l_run[a][r] += p[e];
                     }
                     const uint32_t h01 = pack_bf16(p[0], p[1]), h23 = pack_bf16(p[2], p[3]);

@@ -3,12 +3,13 @@
 //     S[c][n] <- exp(dt_c A[c][n]) S[c][n] + dt_c x_c B_n,    y_c = (sum_n S[c][n] C_n + D_c x_c) * silu(z_c).
 // The state, decays, step sizes, B, C and all sums are float32; x, z and y are in the compute dtype.
 //
-// A channel's N state entries live in the registers of LPC lanes, NS entries each (multiples of four; N <= LPC NS),
-// with their rates A log2(e), so a token costs a lane NS exponentials (the hardware's 2^x), NS multiply-adds of the
-// state and NS of the read-out, two entries to a 64-bit register.  Nothing waits for a token's read-out: a lane keeps
-// its partial sums of GROUP tokens, which are then added crosswise, after which lane i holds token i's sum.  The step's tokens
-// come 16 (for large states 8) at a time: B and C by asynchronous copies in two stages, x, dt and z through registers (read ahead while the
-// ones before are worked on), which also carry x and z to the gate.  Tokens past a sequence's end are staged with
+// A channel's N state entries live in the registers of LPC lanes, NS entries each (pairs dealt to the lanes in turn;
+// N <= LPC NS), with their rates A log2(e), so a token costs a lane NS exponentials (the hardware's 2^x), NS multiply-adds
+// of the state and NS of the read-out, two entries to a 64-bit register.  Few entries a lane make many warps: a lone
+// warp a scheduler would wait for its own exponentials.  Nothing waits for a token's read-out: a lane keeps its partial sums of
+// GROUP tokens, which are then added crosswise, after which lane i holds token i's sum.  The step's tokens come 16 (for
+// large states 8) at a time: B and C by asynchronous copies in two stages, x, dt and z through registers (read ahead while
+// the ones before are worked on), which also carry x and z to the gate.  Tokens past a sequence's end are staged with
 // dt = 0, which leaves the state as it is.  The order of every sum is fixed by N alone: a token's result does not depend on
 // how the sequence was cut into steps or on the batch.
 #include "common.cuh"
@@ -26,13 +27,12 @@ __device__ __forceinline__ float exp2_fast(float x) {        // results below 2^
     return y;
 }
 
-// VEC: every channel's state starts on a 16-byte boundary and N is a multiple of four.
 template <typename TE> __device__ __forceinline__ float gated(float v, float z) { return v * z / (1.0f + expf(-z)); }
 template <> __device__ __forceinline__ float gated<__nv_bfloat16>(float v, float z) {      // rounded right after
     return __fdividef(v * z, 1.0f + __expf(-z));
 }
 
-// SS_CHUNK: tokens staged at a time.
+// SS_CHUNK: tokens staged at a time.  VEC: every pair of a channel's state starts on an 8-byte boundary.
 template <typename TE, int LPC, int NS, bool VEC, int SS_CHUNK>
 __global__ void __launch_bounds__(SS_THREADS)
 selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restrict__ z, long long ldz,
@@ -40,8 +40,10 @@ selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restr
                       int c_at, const float* __restrict__ rates, const float* __restrict__ skip, int inner, int N,
                       const int* __restrict__ seq_first, const int* __restrict__ seq_slots, float* __restrict__ state,
                       long long state_stride, long long state_offset, TE* __restrict__ y, long long ldy) {
-    constexpr int NPAD = LPC * NS, Q = NS / 4, COLS = ss_channels(LPC), GROUP = LPC < SS_CHUNK ? LPC : SS_CHUNK;
-    constexpr int PER = (SS_CHUNK * COLS + SS_THREADS - 1) / SS_THREADS;     // (token, channel) pairs of a chunk a thread stages
+    constexpr int NPAD = LPC * NS, Q = NS / 2, COLS = ss_channels(LPC), GROUP = LPC < SS_CHUNK ? LPC : SS_CHUNK;
+    constexpr int ROWS = SS_THREADS / COLS;                  // tokens of a chunk that are staged at once, a channel a thread
+    constexpr int PER = (SS_CHUNK + ROWS - 1) / ROWS;
+    constexpr int PIECES = NPAD / 4, COPIES = (SS_CHUNK * PIECES + SS_THREADS - 1) / SS_THREADS;
     __shared__ __align__(16) float Bs[2][SS_CHUNK][NPAD], Cs[2][SS_CHUNK][NPAD];
     __shared__ __align__(16) float2 ds[2][SS_CHUNK][COLS];                   // (dt, dt x)
     __shared__ float ys[SS_CHUNK][COLS];
@@ -53,69 +55,73 @@ selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restr
         (&Cs[0][0][0])[i] = 0.0f;
     }
     // the rates do not depend on the launches before this one
-    float2x A[2 * Q], S[2 * Q];
+    float2x A[Q], S[Q];
     const bool live = c < inner;
 #pragma unroll
     for (int q = 0; q < Q; ++q) {
-        const int n = 4 * (l + LPC * q);
-        float a[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-            if (live && n + e < N) a[e] = rates[(long long)c * N + n + e];
-        A[2 * q] = pair_of_floats(a[0], a[1]);
-        A[2 * q + 1] = pair_of_floats(a[2], a[3]);
+        const int n = 2 * (l + LPC * q);
+        const float a0 = live && n < N ? rates[(long long)c * N + n] : 0.0f;
+        const float a1 = live && n + 1 < N ? rates[(long long)c * N + n + 1] : 0.0f;
+        A[q] = pair_of_floats(a0, a1);
     }
+    // staging: this thread's channel and first token of a chunk
+    const int col = c0 + tid % COLS, row = tid / COLS;
+    const bool real = col < inner;
+    const float d_skip = real ? skip[col] : 0.0f;
     pdl_wait();
     const int first = seq_first[s], count = seq_first[s + 1] - first;
     float* const mine = state + (long long)seq_slots[s] * state_stride + state_offset + (long long)c * N;
 #pragma unroll
     for (int q = 0; q < Q; ++q) {
-        const int n = 4 * (l + LPC * q);
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const int n = 2 * (l + LPC * q);
+        float2 v = make_float2(0.0f, 0.0f);
         if (live) {
             if (VEC) {
-                if (n < N) v = *reinterpret_cast<const float4*>(mine + n);
+                if (n < N) v = *reinterpret_cast<const float2*>(mine + n);
             } else {
                 if (n < N) v.x = mine[n];
                 if (n + 1 < N) v.y = mine[n + 1];
-                if (n + 2 < N) v.z = mine[n + 2];
-                if (n + 3 < N) v.w = mine[n + 3];
             }
         }
-        S[2 * q] = pair_of_floats(v.x, v.y);
-        S[2 * q + 1] = pair_of_floats(v.z, v.w);
+        S[q] = pair_of_floats(v.x, v.y);
     }
+    const long long at = first + row, place = real ? col : inner - 1;
+    const TE* xp = x + at * ldx + place;
+    const TE* zp = z + at * ldz + place;
+    const float* dp = dt + at * lddt + place;
+    TE* yp = y + at * ldy + place;
     auto copy_bc = [&](int li0, int b) {
-        const int pieces = n4 / 4, left = min(SS_CHUNK, count - li0);
-        for (int i = tid; i < left * pieces; i += SS_THREADS) {
-            const int tok = i / pieces, n = 4 * (i % pieces);
-            const float* row = bc + (long long)(first + li0 + tok) * ldbc;
-            copy_async16(&Bs[b][tok][n], row + b_at + n);
-            copy_async16(&Cs[b][tok][n], row + c_at + n);
+        const float* from = bc + (long long)(first + li0) * ldbc;
+#pragma unroll
+        for (int k = 0; k < COPIES; ++k) {
+            const int i = tid + SS_THREADS * k, tok = i / PIECES, n = 4 * (i % PIECES);
+            if (tok < SS_CHUNK && li0 + tok < count && n < n4) {
+                copy_async16(&Bs[b][tok][n], from + tok * ldbc + b_at + n);
+                copy_async16(&Cs[b][tok][n], from + tok * ldbc + c_at + n);
+            }
         }
         copy_async_commit();
     };
-    // (read as they are, from places that always exist: nothing may wait for a load before all are on their way)
+    // (rows are read as they are, from places that always exist: nothing may wait for a load before all are on their way)
     TE xr[PER], zr[PER];
     float dr[PER], gate_x[PER], gate_z[PER];
     auto read_rows = [&](int li0) {
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const int i = tid + SS_THREADS * k, col = min(c0 + i % COLS, inner - 1);
-            const long long t = first + min(li0 + i / COLS, count - 1);
-            xr[k] = x[t * ldx + col];
-            dr[k] = dt[t * lddt + col];
-            zr[k] = z[t * ldz + col];
+            const int li = min(li0 + row + ROWS * k, count - 1) - row;           // (pointers stand at the step's row-th token)
+            xr[k] = xp[li * ldx];
+            dr[k] = dp[li * lddt];
+            zr[k] = zp[li * ldz];
         }
     };
     auto stage_rows = [&](int li0, int b) {
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const int i = tid + SS_THREADS * k;
-            const float step = li0 + i / COLS < count ? dr[k] : 0.0f;
+            const int tok = row + ROWS * k;
+            const float step = li0 + tok < count ? dr[k] : 0.0f;
             gate_x[k] = to_float(xr[k]);
             gate_z[k] = to_float(zr[k]);
-            if (i < SS_CHUNK * COLS) ds[b][i / COLS][i % COLS] = make_float2(step, step * gate_x[k]);
+            if (tok < SS_CHUNK) ds[b][tok][tid % COLS] = make_float2(step, step * gate_x[k]);
         }
     };
     __syncthreads();                                         // the zeros are down before the first copies land
@@ -142,19 +148,17 @@ selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restr
             for (int i = 0; i < GROUP; ++i) {
                 const float2 d = ds[b][t0 + i][ch];
                 const float2x d2 = pair_of_floats(d.x, d.x), x2 = pair_of_floats(d.y, d.y);
-                float2x a0 = 0, a1 = 0;                      // (two zeros each)
+                float2x a = 0;                               // (two zeros)
 #pragma unroll
                 for (int q = 0; q < Q; ++q) {
-                    const ulonglong2 bb = *reinterpret_cast<const ulonglong2*>(&Bs[b][t0 + i][4 * (l + LPC * q)]);
-                    const ulonglong2 cc = *reinterpret_cast<const ulonglong2*>(&Cs[b][t0 + i][4 * (l + LPC * q)]);
-                    const float2 e0 = floats_of_pair(pair_mul(d2, A[2 * q])), e1 = floats_of_pair(pair_mul(d2, A[2 * q + 1]));
-                    S[2 * q] = pair_fma(pair_of_floats(exp2_fast(e0.x), exp2_fast(e0.y)), S[2 * q], pair_mul(x2, bb.x));
-                    S[2 * q + 1] = pair_fma(pair_of_floats(exp2_fast(e1.x), exp2_fast(e1.y)), S[2 * q + 1], pair_mul(x2, bb.y));
-                    a0 = pair_fma(S[2 * q], cc.x, a0);
-                    a1 = pair_fma(S[2 * q + 1], cc.y, a1);
+                    const float2x bb = *reinterpret_cast<const float2x*>(&Bs[b][t0 + i][2 * (l + LPC * q)]);
+                    const float2x cc = *reinterpret_cast<const float2x*>(&Cs[b][t0 + i][2 * (l + LPC * q)]);
+                    const float2 e = floats_of_pair(pair_mul(d2, A[q]));
+                    S[q] = pair_fma(pair_of_floats(exp2_fast(e.x), exp2_fast(e.y)), S[q], pair_mul(x2, bb));
+                    a = pair_fma(S[q], cc, a);
                 }
-                const float2 s0 = floats_of_pair(a0), s1 = floats_of_pair(a1);
-                acc[i] = (s0.x + s0.y) + (s1.x + s1.y);
+                const float2 sum = floats_of_pair(a);
+                acc[i] = sum.x + sum.y;
             }
 #pragma unroll
             for (int width = LPC / 2; width >= GROUP; width >>= 1) {
@@ -176,11 +180,9 @@ selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restr
         __syncthreads();
 #pragma unroll
         for (int k = 0; k < PER; ++k) {
-            const int i = tid + SS_THREADS * k, tok = i / COLS, col = c0 + i % COLS;
-            if (i < SS_CHUNK * COLS && tok < n && col < inner) {
-                const float v = fmaf(skip[col], gate_x[k], ys[tok][i % COLS]), zz = gate_z[k];
-                y[(long long)(first + li0 + tok) * ldy + col] = from_float<TE>(gated<TE>(v, zz));
-            }
+            const int tok = row + ROWS * k;
+            if (tok < n && real)
+                yp[(li0 + ROWS * k) * ldy] = from_float<TE>(gated<TE>(fmaf(d_skip, gate_x[k], ys[tok][tid % COLS]), gate_z[k]));
         }
         if (more) stage_rows(li0 + SS_CHUNK, b ^ 1);
     }
@@ -188,15 +190,13 @@ selective_scan_kernel(const TE* __restrict__ x, long long ldx, const TE* __restr
     if (!live) return;
 #pragma unroll
     for (int q = 0; q < Q; ++q) {
-        const int n = 4 * (l + LPC * q);
-        const float2 lo = floats_of_pair(S[2 * q]), hi = floats_of_pair(S[2 * q + 1]);
+        const int n = 2 * (l + LPC * q);
+        const float2 v = floats_of_pair(S[q]);
         if (VEC) {
-            if (n < N) *reinterpret_cast<float4*>(mine + n) = make_float4(lo.x, lo.y, hi.x, hi.y);
+            if (n < N) *reinterpret_cast<float2*>(mine + n) = v;
         } else {
-            if (n < N) mine[n] = lo.x;
-            if (n + 1 < N) mine[n + 1] = lo.y;
-            if (n + 2 < N) mine[n + 2] = hi.x;
-            if (n + 3 < N) mine[n + 3] = hi.y;
+            if (n < N) mine[n] = v.x;
+            if (n + 1 < N) mine[n + 1] = v.y;
         }
     }
 }
@@ -222,11 +222,11 @@ MU_EXPORT int mu_selective_scan(const void* x, long long ldx, const void* z, lon
     if (b_at % 4 || c_at % 4 || ldbc % 4 || ((uintptr_t)bc & 15)) return MU_ERR_ALIGNMENT;
     cudaStream_t s = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
-    const bool vec = N % 4 == 0 && state_stride % 4 == 0 && state_offset % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    const bool vec = N % 2 == 0 && state_stride % 2 == 0 && state_offset % 2 == 0 && ((uintptr_t)state & 7) == 0;
 #define MU_SELECTIVE_V(TE, LPC, NS, V)                                                                                 \
     do {                                                                                                               \
         const dim3 grid(n_seqs, (inner + mu::ss_channels(LPC) - 1) / mu::ss_channels(LPC)), block(mu::SS_THREADS);     \
-        auto kernel = mu::selective_scan_kernel<TE, LPC, NS, V, NS == 4 ? 16 : 8>;                                                       \
+        auto kernel = mu::selective_scan_kernel<TE, LPC, NS, V, NS <= 4 ? 16 : 8>;                                                       \
         if (long_steps)                                                                                                \
             return mu::launch_after(kernel, grid, block, 0, s, (const TE*)x, ldx, (const TE*)z, ldz, dt, lddt, bc,     \
                                     ldbc, b_at, c_at, rates, skip, inner, N, seq_first, seq_slots, state,              \
@@ -242,10 +242,10 @@ MU_EXPORT int mu_selective_scan(const void* x, long long ldx, const void* z, lon
         if (vec) MU_SELECTIVE_V(float, LPC, NS, true);                                                                 \
         MU_SELECTIVE_V(float, LPC, NS, false);                                                                         \
     } while (0)
-    if (N <= 8) MU_SELECTIVE(2, 4);
-    if (N <= 16) MU_SELECTIVE(4, 4);
-    if (N <= 32) MU_SELECTIVE(8, 4);
-    if (N <= 64) MU_SELECTIVE(16, 4);
+    if (N <= 8) MU_SELECTIVE(4, 2);
+    if (N <= 16) MU_SELECTIVE(8, 2);
+    if (N <= 32) MU_SELECTIVE(16, 2);
+    if (N <= 64) MU_SELECTIVE(32, 2);
     if (N <= 128) MU_SELECTIVE(32, 4);
     MU_SELECTIVE(32, 8);
 #undef MU_SELECTIVE

@@ -21,11 +21,23 @@ from math_utils_b200.weights.safetensors import write_safetensors
 
 pytestmark = pytest.mark.gpu
 
-BF16_ROW = 0.03          # rms of a bfloat16 row's errors over its spread: layers that run again add their rounding again
+# Rows in bfloat16.  Rounding the plain statement's normed rows, activations, queries, keys, values and heads to bfloat16
+# moves the median row of these models by 0.005 to 0.012 of its spread and single rows by up to 0.043 (layers that run again
+# add their rounding again).  So the median row gets a narrow bound, all but one row in fifty a wider one, and the few
+# others one that only a fault passes.  The float32 runs hold every row to FP32_ABS.
+BF16_MEDIAN, BF16_ROW, BF16_ANY = 0.02, 0.05, 0.12
 
 
 def check_logits(got, want, dtype, what=""):
-    helpers.check_logits(got, want, dtype, what, bf16_rms=BF16_ROW)
+    if dtype == "float32":
+        return helpers.check_logits(got, want, dtype, what)
+    got = np.asarray(got, dtype=np.float64)
+    assert got.shape == want.shape and np.isfinite(got).all(), what
+    rms = np.sqrt(((got - want) ** 2).mean(axis=-1)) / want.std(axis=-1)
+    over = np.flatnonzero(rms > BF16_ROW)
+    note = f"{what}: rows {over[:5]} of {len(rms)} are off by {rms[over][:5]} of their spread, the median row by {np.median(rms):.4f}"
+    assert len(over) <= max(1, len(rms) // 50) and rms.max() < BF16_ANY, note
+    assert len(rms) < 16 or np.median(rms) < BF16_MEDIAN, note
 
 
 def chunked(heads, kv_heads, dim, scale, chunk, ff=None):
@@ -754,9 +766,9 @@ def test_short_convolution_kernel(channels, taps, u_dtype, out_dtype):
             pos[s] += c
             at += c
     assert pos == list(lens)
-    tol = 1e-5 if out_dtype == torch.float32 else 3e-2
+    tol = 1e-5 if out_dtype == torch.float32 else 5e-3
     for s in range(len(lens)):
-        err = np.abs(np.concatenate(got[s]) - want[s]).max(axis=1)
+        err = (np.abs(np.concatenate(got[s]) - want[s]) / np.maximum(1.0, np.abs(want[s]))).max(axis=1)
         assert err.max() < tol, f"sequence {s}: first wrong token {int(np.argmax(err > tol))}"
     assert (state[[2, 5]] == 9.0).all() and (state[:, (taps - 1) * channels:][slots] == 0.0).all()
 
@@ -771,7 +783,7 @@ def test_step_sizes(dtype, T):
     keep = dev(w, dtype), dev(bias), dev(low)
     ops.low_rank(keep[2], dtype, ops.low_rank_part(keep[0], 8, out, bias=keep[1], fn="softplus"))
     want = plain.softplus(low[:, 8:] @ w.T + bias)
-    assert np.abs(host(out) / want - 1.0).max() < 5e-5 if dtype == torch.bfloat16 else 1e-5
+    assert np.abs(host(out) / want - 1.0).max() < (5e-5 if dtype == torch.bfloat16 else 1e-5)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -799,7 +811,7 @@ def test_selective_scan_kernel(dtype, c, N):
     def run(u, seq, first, sl, counts):
         x, z, dt, bc = (u[:, a:b] for a, b in ((0, c), (c, 2 * c), (2 * c, 3 * c), (3 * c, u.shape[1])))
         out = torch.full((u.shape[0], c), 7.0, device="cuda", dtype=dtype)
-        return ops.selective_scan(x.to(dtype), z.to(dtype), dt, bc.contiguous(), 4, 4 + n4, rates, skip, first, sl, state, tail, out)
+        return ops.selective_scan(x.to(dtype), z.to(dtype), dt, bc.reshape(-1).clone().view(bc.shape), 4, 4 + n4, rates, skip, first, sl, state, tail, out)
 
     _check_steps(_in_steps(data, slots, run), want, 1e-4 if dtype == torch.float32 else 1e-2)
     assert (state[[0, 2, 4]] == 9.0).all() and (state[slots][:, :tail] == 0.0).all()
